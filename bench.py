@@ -214,13 +214,8 @@ def attention_flops(runner, T):
 
 def cache_bytes_per_step(runner, batch, context):
     """Keys and values of the live requests (read once) plus their fixed-size state (read and written)."""
-    from kappai_b200.cache.storage import StateView
-
     kv = sum(runner.storage.bytes_per_token(g) for g in runner.storage.pools) * context * batch
-    st = 0
-    for v in runner.storage.views:
-        if isinstance(v, StateView) and v.writes:
-            st += 2 * v.tensor[0].numel() * v.tensor.element_size() * batch
+    st = sum(2 * t[0].numel() * t.element_size() * batch for t in runner.storage.state_tensors())
     return kv + st
 
 

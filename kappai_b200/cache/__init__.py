@@ -1,5 +1,5 @@
-from .spec import PagedKVSpec, StateSpec
+from .spec import CompositeSpec, PagedKVSpec, StateSpec, leaf_specs
 from .manager import (CacheManager, PagePool, SlotPool, CacheError, OutOfPages, OutOfSlots, RELEASED)
 
-__all__ = ["PagedKVSpec", "StateSpec", "CacheManager", "PagePool", "SlotPool", "CacheError", "OutOfPages",
+__all__ = ["PagedKVSpec", "StateSpec", "CompositeSpec", "leaf_specs", "CacheManager", "PagePool", "SlotPool", "CacheError", "OutOfPages",
            "OutOfSlots", "RELEASED"]

@@ -10,11 +10,14 @@ recurrent/conv state of fixed size per layer):
   own.  A windowed group may keep the first ``keep_first`` keys of every
   sequence readable: the pages that hold them are never given back early.
 * :class:`StateSpec` — a fixed-size tensor per request; kept in a slot.
+
+A mixer that needs several of these at once (keys and values beside the last
+inputs of a convolution; two mixers in one) asks for a :class:`CompositeSpec`.
 """
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional, Tuple
+from typing import Iterator, Optional, Tuple
 
 
 @dataclass(frozen=True)
@@ -39,3 +42,19 @@ class PagedKVSpec:
 class StateSpec:
     shape: Tuple[int, ...]            # per request
     dtype: str = "float32"
+
+
+@dataclass(frozen=True)
+class CompositeSpec:
+    """Several memories of one mixer, in the mixer's own order (they may be composite again)."""
+
+    parts: Tuple[object, ...]
+
+
+def leaf_specs(spec) -> Iterator[object]:
+    """The paged and state specs that ``spec`` is made of (nothing for None)."""
+    if isinstance(spec, CompositeSpec):
+        for p in spec.parts:
+            yield from leaf_specs(p)
+    elif spec is not None:
+        yield spec

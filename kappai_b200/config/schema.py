@@ -136,7 +136,8 @@ class LayerSpec:
     layer by layer.  ``side`` (category ``side``): something that changes the
     residual at the layer's end, behind the feed-forward.  ``mixer_post_norm``
     / ``ffn_post_norm``: norms of a sublayer's output before it joins the
-    residual, for arrangements that norm on both sides."""
+    residual, for arrangements that norm on both sides.  ``block_prefix`` /
+    ``block_rename``: where an arrangement with tensors of its own finds them."""
 
     mixer: PartSpec
     ffn: Optional[PartSpec]
@@ -147,6 +148,8 @@ class LayerSpec:
     side: Optional[PartSpec] = None
     mixer_post_norm: Optional[PartSpec] = None
     ffn_post_norm: Optional[PartSpec] = None
+    block_prefix: str = ""
+    block_rename: Dict[str, str] = field(default_factory=dict)
 
 
 @dataclass
@@ -176,6 +179,7 @@ class ModelSpec:
     head: PartSpec
     eos_token_id: Optional[int] = None
     entry: Optional[PartSpec] = None           # category ``entry``: runs in front of schedule entries marked ``enter``
+    residual: Optional[PartSpec] = None        # category ``residual``: how a row's residual is kept between the layers (None: one float32 row)
     token_table: Optional[PartSpec] = None     # a second table by token id that the layers' ``side`` parts read
     ignored_tensors: List[str] = field(default_factory=list)   # names a weight file may hold although nothing reads them
 

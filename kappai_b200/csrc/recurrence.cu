@@ -1,0 +1,1001 @@
+// Linear recurrences with data-dependent decays.  A head keeps a float32 state S [D, P] a request and follows, row after
+// row,
+//
+//   S <- diag(g) S ;   u = v                       ("gated": gated linear attention)
+//                  or  u = beta (v - S^T k)        ("delta": the gated delta rule: what S holds for k is taken off v first)
+//   S <- S + k u^T ;   o = S^T q ,
+//
+// g one factor in (0, 1] a head, or one a key channel (a row of S), given by its logarithm.  Several heads may share a
+// query and key (head h reads q/k head h / (H / G)).
+//
+// Everything here is float32: decays and their logarithms, step sizes, unit norms, the state, products and sums; the
+// storage type holds projections only.
+//
+// Kernels: what stands between the projections and a delta recurrence (convolutions over time with silu, unit norms of
+// q and k, step sizes, logarithms of decays) in one launch; the logarithms of decays alone for a gated recurrence; the
+// scan (row after row, the state in registers, every sum in an order fixed by the sizes alone, so a row's bits do not
+// depend on how the sequence was cut); and the chunked form for prompt portions in 16-bit mode (below).
+#include "common.cuh"
+#include "chanconv.cuh"
+
+// ------------------------------------------------------------------------------------------------ in front of the scan
+
+// The logarithm of a decay from its projection z: kind 0, exp(-A softplus(z + bias)): -A softplus(z + bias), A = exp(A_log);
+// kind 1, sigmoid(z)^(1/tau): -softplus(-z) / tau.
+__device__ __forceinline__ float rc_log_decay_step(float z, float bias, float neg_a) { return neg_a * ss_softplus(z + bias); }
+__device__ __forceinline__ float rc_log_decay_sigmoid(float z, float inv_tau) { return -ss_softplus(-z) * inv_tau; }
+
+// Entry e of a row's H step sizes and its decays (H of them, or H D in place in lg): e < H is beta_e, the rest decays.
+template <typename T>
+__device__ __forceinline__ void rc_gate_entry(const T* __restrict__ prow, int b_col, int a_col, const float* __restrict__ neg_a,
+                                              const float* __restrict__ dt_bias, float* __restrict__ beta, float* __restrict__ lg,
+                                              int r, int e, int H, int D, int per_channel) {
+    if (e < H) {
+        beta[(size_t)r * H + e] = 1.0f / (1.0f + expf(-to_f32(prow[b_col + e])));
+        return;
+    }
+    e -= H;
+    if (per_channel) {
+        float* z = lg + (size_t)r * H * D + e;
+        *z = rc_log_decay_step(*z, dt_bias[e], neg_a[e / D]);
+    } else {
+        lg[(size_t)r * H + e] = rc_log_decay_step(to_f32(prow[a_col + e]), dt_bias[e], neg_a[e]);
+    }
+}
+
+// p: rows [n, ld] in the storage type with the channels [q: G heads of D | k: G heads of D | v: H heads of P] side by side
+// from conv_col.  out: [n, C] float32, the same channels behind convolution and silu, q and k as unit vectors a head
+// (x / sqrt(sum x^2 + 1e-6)), q times q_scale.  A warp takes one q or k head, or 128 channels of v, or 128 gate entries, of
+// one row.  single_rows: every segment has one row, and the lane that read a channel's kept inputs writes the new ones.
+#define RP_UNIT_EPS 1e-6f
+template <typename T>
+__global__ void __launch_bounds__(128)
+delta_prep_kernel(const T* __restrict__ p, int ld, int conv_col, int b_col, int a_col, const float* __restrict__ taps,
+                  const float* __restrict__ neg_a, const float* __restrict__ dt_bias, float* __restrict__ kept, size_t slot_stride,
+                  const int* __restrict__ row_seg, const int* __restrict__ cu_rows, const int* __restrict__ seg_pos,
+                  const int* __restrict__ seg_slot, float* __restrict__ out, float* __restrict__ beta, float* __restrict__ lg,
+                  int H, int G, int D, int P, int K, float q_scale, int per_channel, int single_rows) {
+    kp_pdl_begin();
+    const int lane = threadIdx.x & 31;
+    int it = blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int r = blockIdx.y;
+    const int qk = 2 * G, vb = (H * P + 127) / 128, C = 2 * G * D + H * P;
+    if (it >= qk + vb) {
+        const int e0 = (it - qk - vb) * 128, n_e = H + (per_channel ? H * D : H);
+        for (int e = e0 + lane; e < min(e0 + 128, n_e); e += 32)
+            rc_gate_entry<T>(p + (size_t)r * ld, b_col, a_col, neg_a, dt_bias, beta, lg, r, e, H, D, per_channel);
+        return;
+    }
+    const int base = it < qk ? it * D : 2 * G * D + (it - qk) * 128;
+    const int count = it < qk ? D : min(128, C - base);
+    const int seg = row_seg[r], row0 = cu_rows[seg];
+    const bool fresh = seg_pos[seg] == 0;
+    float* kp = kept + (size_t)seg_slot[seg] * slot_stride;
+    float y[8];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+        y[j] = 0.f;
+        const int c = base + lane + 32 * j;
+        if (lane + 32 * j >= count) continue;
+        float acc = 0.f;
+        for (int m = 0; m < K; m++) {
+            const int rr = r - (K - 1) + m;
+            float v;
+            if (rr >= row0) v = to_f32(p[(size_t)rr * ld + conv_col + c]);
+            else v = fresh ? 0.f : kp[(size_t)(rr - row0 + K - 1) * C + c];
+            // (tap m's input becomes the kept input m - 1 of the next row, written behind its read)
+            if (single_rows && m > 0) kp[(size_t)(m - 1) * C + c] = v;
+            acc = fmaf(taps[(size_t)c * K + m], v, acc);
+        }
+        y[j] = ss_silu(acc);
+        ss = fmaf(y[j], y[j], ss);
+    }
+    float scale = 1.f;
+    if (it < qk) {
+        ss = warp_sum(ss);
+        scale = 1.0f / sqrtf(ss + RP_UNIT_EPS);
+        if (it < G) scale *= q_scale;
+    }
+    float* dst = out + (size_t)r * C + base;
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+        if (lane + 32 * j < count) dst[lane + 32 * j] = y[j] * scale;
+}
+
+// The same for steps of several rows where heads are multiples of 4 wide and rows start on 8 (16) bytes: a lane takes four
+// channels (eight where D > 128: QL = 2) of RP_ROWS consecutive rows and fetches every row of p once for all of them; heads
+// of 4, 8, .. 64 channels share a warp.  The blocks from conv_blocks on compute the gate entries of the tile's rows.
+#define RP_ROWS 4
+__device__ __forceinline__ float4 rp_load4(const float* s) { return __ldg(reinterpret_cast<const float4*>(s)); }
+__device__ __forceinline__ float4 rp_load4(const bf16* s) {
+    const uint2 raw = __ldg(reinterpret_cast<const uint2*>(s));
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void rp_fma4(float4& acc, const float4 w, const float4 v) {
+    acc.x = fmaf(w.x, v.x, acc.x); acc.y = fmaf(w.y, v.y, acc.y); acc.z = fmaf(w.z, v.z, acc.z); acc.w = fmaf(w.w, v.w, acc.w);
+}
+
+template <typename T, int K, int QL>
+__global__ void __launch_bounds__(128)
+delta_prep_vec_kernel(const T* __restrict__ p, int ld, int conv_col, int b_col, int a_col, const float* __restrict__ taps,
+                      const float* __restrict__ neg_a, const float* __restrict__ dt_bias, const float* __restrict__ kept,
+                      size_t slot_stride, const int* __restrict__ row_seg, const int* __restrict__ cu_rows,
+                      const int* __restrict__ seg_pos, const int* __restrict__ seg_slot, float* __restrict__ out,
+                      float* __restrict__ beta, float* __restrict__ lg, int n, int H, int G, int D, int P, float q_scale,
+                      int per_channel, int conv_blocks, int team) {
+    kp_pdl_begin();
+    const int r0 = blockIdx.y * RP_ROWS;
+    if ((int)blockIdx.x >= conv_blocks) {
+        const int n_e = H + (per_channel ? H * D : H);
+        for (int i = 0; i < RP_ROWS && r0 + i < n; i++)
+            for (int e = (blockIdx.x - conv_blocks) * blockDim.x + threadIdx.x; e < n_e; e += (gridDim.x - conv_blocks) * blockDim.x)
+                rc_gate_entry<T>(p + (size_t)(r0 + i) * ld, b_col, a_col, neg_a, dt_bias, beta, lg, r0 + i, e, H, D, per_channel);
+        return;
+    }
+    const int lane = threadIdx.x & 31, it = blockIdx.x * 4 + (threadIdx.x >> 5);
+    const int C = 2 * G * D + H * P;
+    const int per_warp = 32 / team;                                  // heads a warp takes (team lanes a head)
+    const int qk = (2 * G + per_warp - 1) / per_warp;                // items that are q and k heads
+    int c[QL];                                                       // this lane's channels (-1: none)
+    int head = -1;
+    if (it < qk) {
+        head = it * per_warp + lane / team;
+        if (head >= 2 * G) head = -1;
+#pragma unroll
+        for (int q = 0; q < QL; q++) {
+            const int d = (lane % team + 32 * q) * 4;
+            c[q] = head >= 0 && d < D ? head * D + d : -1;
+        }
+    } else {
+#pragma unroll
+        for (int q = 0; q < QL; q++) {
+            c[q] = 2 * G * D + (it - qk) * 128 * QL + (lane + 32 * q) * 4;
+            if (c[q] >= C) c[q] = -1;
+        }
+    }
+    float4 y[RP_ROWS][QL];
+#pragma unroll
+    for (int q = 0; q < QL; q++) {
+        if (c[q] < 0) {
+#pragma unroll
+            for (int i = 0; i < RP_ROWS; i++) y[i][q] = make_float4(0.f, 0.f, 0.f, 0.f);
+            continue;
+        }
+        float4 win[RP_ROWS + K - 1];
+#pragma unroll
+        for (int i = 0; i < RP_ROWS + K - 1; i++) {
+            const int rr = r0 - (K - 1) + i;
+            win[i] = rr >= 0 && rr < n ? rp_load4(p + (size_t)rr * ld + conv_col + c[q]) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        float4 tp[K];
+#pragma unroll
+        for (int m = 0; m < K; m++)
+            tp[m] = make_float4(__ldg(taps + (size_t)c[q] * K + m), __ldg(taps + (size_t)(c[q] + 1) * K + m),
+                                __ldg(taps + (size_t)(c[q] + 2) * K + m), __ldg(taps + (size_t)(c[q] + 3) * K + m));
+#pragma unroll
+        for (int i = 0; i < RP_ROWS; i++) {
+            const int r = r0 + i;
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r < n) {
+                const int seg = row_seg[r], row0 = cu_rows[seg];
+                const bool fresh = seg_pos[seg] == 0;
+                const float* kp = kept + (size_t)seg_slot[seg] * slot_stride;
+#pragma unroll
+                for (int m = 0; m < K; m++) {
+                    const int rr = r - (K - 1) + m;
+                    if (rr >= row0) rp_fma4(acc, tp[m], win[i + m]);
+                    else if (!fresh) {
+                        const float* k4 = kp + (size_t)(rr - row0 + K - 1) * C + c[q];
+                        rp_fma4(acc, tp[m], make_float4(k4[0], k4[1], k4[2], k4[3]));
+                    }
+                }
+            }
+            y[i][q] = make_float4(ss_silu(acc.x), ss_silu(acc.y), ss_silu(acc.z), ss_silu(acc.w));
+        }
+    }
+    if (it < qk) {
+#pragma unroll
+        for (int i = 0; i < RP_ROWS; i++) {
+            float ss = 0.f;
+#pragma unroll
+            for (int q = 0; q < QL; q++) {
+                ss = fmaf(y[i][q].x, y[i][q].x, ss); ss = fmaf(y[i][q].y, y[i][q].y, ss);
+                ss = fmaf(y[i][q].z, y[i][q].z, ss); ss = fmaf(y[i][q].w, y[i][q].w, ss);
+            }
+            for (int o = team >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            float scale = 1.0f / sqrtf(ss + RP_UNIT_EPS);
+            if (head < G) scale *= q_scale;
+#pragma unroll
+            for (int q = 0; q < QL; q++) { y[i][q].x *= scale; y[i][q].y *= scale; y[i][q].z *= scale; y[i][q].w *= scale; }
+        }
+    }
+#pragma unroll
+    for (int q = 0; q < QL; q++) {
+        if (c[q] < 0) continue;
+#pragma unroll
+        for (int i = 0; i < RP_ROWS; i++)
+            if (r0 + i < n) *reinterpret_cast<float4*>(out + (size_t)(r0 + i) * C + c[q]) = y[i][q];
+    }
+}
+
+// z <- -softplus(-z) / tau in place: the logarithms of the decays sigmoid(z)^(1/tau)
+__global__ void log_decay_sigmoid_kernel(float* __restrict__ z, size_t n, float inv_tau) {
+    kp_pdl_begin();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
+        z[i] = rc_log_decay_sigmoid(z[i], inv_tau);
+}
+
+// ------------------------------------------------------------------------------------------------ the scan
+#define RS_CH 8                  // rows staged at a time
+#define RS_COLS 32               // value columns of a block: 8 a warp
+#define RS_PARTS 4               // parts the state's rows are cut in: the lanes of a column
+#define RS_THREADS 128
+
+// R: state rows a thread keeps (D <= RS_PARTS R).  Lane (part q, column c) owns rows 4 (q + 4 m) + e, m < R / 4, e < 4: the
+// four parts read 64 contiguous bytes of a staged vector.  Sums over a column's rows: in a lane by m and e, then the
+// lanes by a butterfly.  The read-out is S_new^T q = (g S)^T q + (k . q) u, so that both sums over the old state run
+// side by side.
+template <typename T, int R, bool DELTA, bool CHAN>
+__global__ void __launch_bounds__(RS_THREADS)
+recur_scan_kernel(const T* __restrict__ qp, const T* __restrict__ kp, const T* __restrict__ vp, int ldi, const float* __restrict__ lg,
+                  const float* __restrict__ beta, float q_scale, float* __restrict__ state, size_t slot_stride,
+                  const int* __restrict__ cu_rows, const int* __restrict__ seg_pos, const int* __restrict__ seg_slot,
+                  float* __restrict__ out, int ldo, int H, int G, int D, int P, int write_state) {
+    kp_pdl_begin();
+    constexpr int NP = RS_PARTS * R;
+    __shared__ __align__(16) float sq[RS_CH][NP], sk[RS_CH][NP], sg[CHAN ? RS_CH : 1][CHAN ? NP : 4];
+    __shared__ float sv[RS_CH][RS_COLS], sdec[RS_CH], sbeta[RS_CH], skq[RS_CH];
+    const int head = blockIdx.y, tile = blockIdx.x, seg = blockIdx.z;
+    const int grp = head / (H / G);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int col = lane & 7, part = lane >> 3;
+    const int jl = warp * 8 + col, j = tile * RS_COLS + jl;
+    const bool jok = j < P;
+    float* st = state + (size_t)seg_slot[seg] * slot_stride + (size_t)head * D * P;
+    const bool fresh = seg_pos[seg] == 0;
+    float s[R];
+#pragma unroll
+    for (int m = 0; m < R / 4; m++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const int i = 4 * (part + 4 * m) + e;
+            s[4 * m + e] = (!fresh && jok && i < D) ? st[(size_t)i * P + j] : 0.f;
+        }
+    const int row0 = cu_rows[seg], row1 = cu_rows[seg + 1];
+    for (int t0 = row0; t0 < row1; t0 += RS_CH) {
+        const int nt = min(RS_CH, row1 - t0);
+        __syncthreads();
+        for (int t = warp; t < nt; t += RS_THREADS / 32) {
+            const size_t row = (size_t)(t0 + t) * ldi;
+            float kq = 0.f;
+            for (int i = lane; i < NP; i += 32) {
+                float qv = 0.f, kv = 0.f, gv = 1.f;
+                if (i < D) {
+                    qv = to_f32(qp[row + (size_t)grp * D + i]) * q_scale;
+                    kv = to_f32(kp[row + (size_t)grp * D + i]);
+                    if (CHAN) gv = expf(lg[((size_t)(t0 + t) * H + head) * D + i]);
+                }
+                sq[t][i] = qv;
+                sk[t][i] = kv;
+                if (CHAN) sg[t][i] = gv;
+                kq = fmaf(qv, kv, kq);
+            }
+            kq = warp_sum(kq);
+            const int jj = tile * RS_COLS + lane;
+            sv[t][lane] = jj < P ? to_f32(vp[row + (size_t)head * P + jj]) : 0.f;
+            if (lane == 0) {
+                skq[t] = kq;
+                if (!CHAN) sdec[t] = expf(lg[(size_t)(t0 + t) * H + head]);
+                if (DELTA) sbeta[t] = beta[(size_t)(t0 + t) * H + head];
+            }
+        }
+        __syncthreads();
+        for (int t = 0; t < nt; t++) {
+            const float4* k4 = reinterpret_cast<const float4*>(sk[t]);
+            const float4* q4 = reinterpret_cast<const float4*>(sq[t]);
+            const float4* g4 = reinterpret_cast<const float4*>(sg[CHAN ? t : 0]);
+            const float a = CHAN ? 0.f : sdec[t];
+            float ak = 0.f, aq = 0.f;
+#pragma unroll
+            for (int m = 0; m < R / 4; m++) {
+                const float4 kv = k4[part + 4 * m], qv = q4[part + 4 * m];
+                const float ke[4] = {kv.x, kv.y, kv.z, kv.w}, qe[4] = {qv.x, qv.y, qv.z, qv.w};
+                float ge[4] = {a, a, a, a};
+                if (CHAN) {
+                    const float4 gv = g4[part + 4 * m];
+                    ge[0] = gv.x; ge[1] = gv.y; ge[2] = gv.z; ge[3] = gv.w;
+                }
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const float x = s[4 * m + e] * ge[e];
+                    s[4 * m + e] = x;
+                    if (DELTA) ak = fmaf(x, ke[e], ak);
+                    aq = fmaf(x, qe[e], aq);
+                }
+            }
+            if (DELTA) {
+                ak += __shfl_xor_sync(0xffffffffu, ak, 8);
+                ak += __shfl_xor_sync(0xffffffffu, ak, 16);
+            }
+            aq += __shfl_xor_sync(0xffffffffu, aq, 8);
+            aq += __shfl_xor_sync(0xffffffffu, aq, 16);
+            const float u = DELTA ? sbeta[t] * (sv[t][jl] - ak) : sv[t][jl];
+#pragma unroll
+            for (int m = 0; m < R / 4; m++) {
+                const float4 kv = k4[part + 4 * m];
+                s[4 * m + 0] = fmaf(kv.x, u, s[4 * m + 0]); s[4 * m + 1] = fmaf(kv.y, u, s[4 * m + 1]);
+                s[4 * m + 2] = fmaf(kv.z, u, s[4 * m + 2]); s[4 * m + 3] = fmaf(kv.w, u, s[4 * m + 3]);
+            }
+            if (part == 0 && jok) out[(size_t)(t0 + t) * ldo + (size_t)head * P + j] = fmaf(skq[t], u, aq);
+        }
+    }
+    if (write_state && jok) {
+#pragma unroll
+        for (int m = 0; m < R / 4; m++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int i = 4 * (part + 4 * m) + e;
+                if (i < D) st[(size_t)i * P + j] = s[4 * m + e];
+            }
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ chunked
+// For prompt portions in 16-bit mode: a segment in chunks of RC_C rows.  With G_i the sum of the decays' logarithms from
+// the chunk's first row up to row i (a number, or one a key channel) and S the state at the chunk's head, the chunk's
+// written rows u_i solve the lower triangular system
+//   u_i + beta_i sum_{j < i} A_ij u_j = beta_i (v_i - (exp(G_i) k_i)^T S) ,   A_ij = sum_d k_i k_j exp(G_i - G_j) ,
+// (in the gated recurrence u = v), and
+//   o_i = (exp(G_i) q_i)^T S + sum_{j <= i} B_ij u_j ,                        B_ij = sum_d q_i k_j exp(G_i - G_j) ,
+//   S'  = exp(G_last) S + sum_j (exp(G_last - G_j) k_j) u_j^T .
+// Three passes: (0) for all chunks side by side what does not need S: A and B, the system solved for the right hand
+// sides beta v and beta exp(G) k, so that u = Wv - Wk S; (1) a serial pass a (segment, head, 32 value columns): u and S',
+// leaving every chunk's S; (2) for all chunks side by side the outputs.  Every exponent is <= 0: where a product of two
+// exponentials stands for exp(G_i - G_j) with factors a channel, its reference is the sum in front of i's 16 rows, which
+// lies between the two; inside 16 rows every pair takes its own exponential.
+//
+// The matrix products run on the tensor cores in tf32 with both operands cut into a rounded part and what it leaves
+// (three products a pair: what is dropped is 2^-22 of a term), float32 sums.
+#define RC_C 64
+#define RC_THREADS 256
+#define RC_PT 32                 // value columns of a block of pass 1
+#define RC_LDU 40                // row pitch of [.., 32] operands read by columns (40 % 32 == 8: no bank conflicts)
+#define RC_LDB 68                // row pitch of the 64 x 64 matrices
+#define RC_MAX_D 256
+#define RC_LOG2E 1.4426950408889634f
+
+__device__ __forceinline__ void rc_split(float x, uint32_t& hi, uint32_t& lo) {
+    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
+    const float rest = x - __uint_as_float(hi);
+    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(lo) : "f"(rest));
+}
+__device__ __forceinline__ void rc_mma(float* c, const uint32_t* a, const uint32_t* b) {
+    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+struct RcA { uint32_t hi[4], lo[4]; };
+struct RcB { uint32_t hi[2], lo[2]; };
+__device__ __forceinline__ void rc_mma3(float* c, const RcA& a, const RcB& b) {
+    rc_mma(c, a.lo, b.hi);
+    rc_mma(c, a.hi, b.lo);
+    rc_mma(c, a.hi, b.hi);
+}
+// A tile [16, 8] of an operand stored [row][k]: rows m0 .., columns k0 ..
+__device__ __forceinline__ void rc_load_a(RcA& f, const float* s, int ld, int m0, int k0, int g, int t) {
+    const float* p = s + (m0 + g) * ld + k0 + t;
+    rc_split(p[0], f.hi[0], f.lo[0]);
+    rc_split(p[8 * ld], f.hi[1], f.lo[1]);
+    rc_split(p[4], f.hi[2], f.lo[2]);
+    rc_split(p[8 * ld + 4], f.hi[3], f.lo[3]);
+}
+// The same of an operand stored [k][row]
+__device__ __forceinline__ void rc_load_at(RcA& f, const float* s, int ld, int m0, int k0, int g, int t) {
+    const float* p = s + (k0 + t) * ld + m0 + g;
+    rc_split(p[0], f.hi[0], f.lo[0]);
+    rc_split(p[8], f.hi[1], f.lo[1]);
+    rc_split(p[4 * ld], f.hi[2], f.lo[2]);
+    rc_split(p[4 * ld + 8], f.hi[3], f.lo[3]);
+}
+// A tile [8, 8] of a right operand stored [k][col]
+__device__ __forceinline__ void rc_load_b(RcB& f, const float* s, int ld, int k0, int n0, int g, int t) {
+    const float* p = s + (k0 + t) * ld + n0 + g;
+    rc_split(p[0], f.hi[0], f.lo[0]);
+    rc_split(p[4 * ld], f.hi[1], f.lo[1]);
+}
+// The same of one stored [col][k]
+__device__ __forceinline__ void rc_load_bt(RcB& f, const float* s, int ld, int k0, int n0, int g, int t) {
+    const float* p = s + (n0 + g) * ld + k0 + t;
+    rc_split(p[0], f.hi[0], f.lo[0]);
+    rc_split(p[4], f.hi[1], f.lo[1]);
+}
+
+// What pass 0 leaves of a (chunk, head): exp(G_last - G_j) k_j [64][D], exp(G_i) q_i [64][D], with DELTA Wk [64][D], Wv (v in
+// the gated recurrence; pass 1 puts u in its place) [64][P], B [64][64], exp(G_last) [D].  All pieces start on 16 bytes.
+struct RcRec { size_t kh, qt, wk, wv, bm, el, size; };
+__host__ __device__ inline RcRec rc_record(int D, int P, bool delta) {
+    RcRec r;
+    r.kh = 0;
+    r.qt = r.kh + (size_t)RC_C * D;
+    r.wk = r.qt + (size_t)RC_C * D;
+    r.wv = r.wk + (delta ? (size_t)RC_C * D : 0);
+    r.bm = r.wv + (size_t)RC_C * P;
+    r.el = r.bm + (size_t)RC_C * RC_C;
+    r.size = (r.el + D + 3) / 4 * 4;
+    return r;
+}
+
+// Pass 0, one block a (chunk, head).
+template <typename T, bool DELTA, bool CHAN>
+__global__ void __launch_bounds__(RC_THREADS)
+recur_chunk_prepare_kernel(const T* __restrict__ qp, const T* __restrict__ kp, const T* __restrict__ vp, int ldi,
+                           const float* __restrict__ lg, const float* __restrict__ beta, float q_scale,
+                           const int* __restrict__ cu_rows, const int* __restrict__ chunk_seg, const int* __restrict__ chunk_row0,
+                           float* __restrict__ rec, int H, int G, int D, int P) {
+    kp_pdl_begin();
+    extern __shared__ __align__(16) float rc_sm[];
+    const int Dp = (D + 31) & ~31, ld = Dp + 4;
+    float* Ks = rc_sm;                                           // [64][ld]
+    float* Qs = Ks + RC_C * ld;                                  // [64][ld]
+    float* As = Qs + RC_C * ld;                                  // [64][RC_LDB] (with DELTA)
+    float* bt = As + (DELTA ? RC_C * RC_LDB : 0);                // [64]
+    float* Gs = bt + RC_C;                                       // [64][ld], or [64]: sums of base-2 logarithms
+    const int chunk = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int grp = head / (H / G);
+    const int t0 = chunk_row0[chunk], n = min(RC_C, cu_rows[chunk_seg[chunk] + 1] - t0);
+    const RcRec R = rc_record(D, P, DELTA);
+    float* out = rec + ((size_t)chunk * H + head) * R.size;
+    for (int i = warp; i < RC_C; i += RC_THREADS / 32) {
+        const bool live = i < n;
+        const size_t row = (size_t)(t0 + i) * ldi + (size_t)grp * D;
+        for (int d = lane; d < Dp; d += 32) {
+            const bool ok = live && d < D;
+            Ks[i * ld + d] = ok ? to_f32(kp[row + d]) : 0.f;
+            Qs[i * ld + d] = ok ? to_f32(qp[row + d]) * q_scale : 0.f;
+            if (CHAN) Gs[i * ld + d] = ok ? lg[((size_t)(t0 + i) * H + head) * D + d] * RC_LOG2E : 0.f;
+        }
+    }
+    if (tid < RC_C) {
+        bt[tid] = DELTA && tid < n ? beta[(size_t)(t0 + tid) * H + head] : 0.f;
+        if (!CHAN) Gs[tid] = tid < n ? lg[(size_t)(t0 + tid) * H + head] * RC_LOG2E : 0.f;
+    }
+    __syncthreads();
+    if (CHAN) {
+        for (int d = tid; d < Dp; d += RC_THREADS) {
+            float acc = 0.f;
+#pragma unroll 8
+            for (int i = 0; i < RC_C; i++) {
+                acc += Gs[i * ld + d];
+                Gs[i * ld + d] = acc;
+            }
+        }
+    } else if (tid == 0) {
+        float acc = 0.f;
+#pragma unroll 8
+        for (int i = 0; i < RC_C; i++) {
+            acc += Gs[i];
+            Gs[i] = acc;
+        }
+    }
+    __syncthreads();
+    const int g = lane >> 2, t = lane & 3;
+    float* Bm = out + R.bm;
+    if (!CHAN) {
+        // rows 16 (warp & 3) .., four tiles of eight columns
+        const int m0 = (warp & 3) * 16, nt0 = (warp >> 2) * 4;
+        float ca[4][4], cb[4][4];
+#pragma unroll
+        for (int x = 0; x < 4; x++)
+#pragma unroll
+            for (int y = 0; y < 4; y++) { ca[x][y] = 0.f; cb[x][y] = 0.f; }
+        if (nt0 * 8 <= m0 + 15) {
+            for (int k0 = 0; k0 < D; k0 += 8) {
+                RcA fk, fq;
+                if (DELTA) rc_load_a(fk, Ks, ld, m0, k0, g, t);
+                rc_load_a(fq, Qs, ld, m0, k0, g, t);
+#pragma unroll
+                for (int x = 0; x < 4; x++) {
+                    if ((nt0 + x) * 8 > m0 + 15) continue;
+                    RcB fb;
+                    rc_load_bt(fb, Ks, ld, k0, (nt0 + x) * 8, g, t);
+                    if (DELTA) rc_mma3(ca[x], fk, fb);
+                    rc_mma3(cb[x], fq, fb);
+                }
+            }
+        }
+#pragma unroll
+        for (int x = 0; x < 4; x++)
+#pragma unroll
+            for (int y = 0; y < 4; y++) {
+                const int i = m0 + g + (y >> 1) * 8, j = (nt0 + x) * 8 + 2 * t + (y & 1);
+                const float w = j <= i ? exp2f(Gs[i] - Gs[j]) : 0.f;
+                if (DELTA) As[i * RC_LDB + j] = j < i ? bt[i] * (w * ca[x][y]) : 0.f;
+                Bm[i * RC_C + j] = w * cb[x][y];
+            }
+    } else {
+        // pairs of 16 rows and 16 earlier rows of another sixteen: both factors by the sum in front of the later sixteen
+        if (warp < 6) {
+            const int a = warp == 0 ? 1 : (warp < 3 ? 2 : 3), b = warp == 0 ? 0 : (warp < 3 ? warp - 1 : warp - 3);
+            const int m0 = 16 * a, n0 = 16 * b;
+            const float* Gr = Gs + (m0 - 1) * ld;
+            float ca[2][4], cb[2][4];
+#pragma unroll
+            for (int x = 0; x < 2; x++)
+#pragma unroll
+                for (int y = 0; y < 4; y++) { ca[x][y] = 0.f; cb[x][y] = 0.f; }
+            for (int k0 = 0; k0 < D; k0 += 8) {
+                RcA fk, fq;
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int i = m0 + g + (e & 1) * 8, d = k0 + t + (e >> 1) * 4;
+                    const float w = exp2f(Gs[i * ld + d] - Gr[d]);
+                    if (DELTA) rc_split(Ks[i * ld + d] * w, fk.hi[e], fk.lo[e]);
+                    rc_split(Qs[i * ld + d] * w, fq.hi[e], fq.lo[e]);
+                }
+#pragma unroll
+                for (int x = 0; x < 2; x++) {
+                    RcB fb;
+#pragma unroll
+                    for (int e = 0; e < 2; e++) {
+                        const int jj = n0 + x * 8 + g, d = k0 + t + e * 4;
+                        rc_split(Ks[jj * ld + d] * exp2f(Gr[d] - Gs[jj * ld + d]), fb.hi[e], fb.lo[e]);
+                    }
+                    if (DELTA) rc_mma3(ca[x], fk, fb);
+                    rc_mma3(cb[x], fq, fb);
+                }
+            }
+#pragma unroll
+            for (int x = 0; x < 2; x++)
+#pragma unroll
+                for (int y = 0; y < 4; y++) {
+                    const int i = m0 + g + (y >> 1) * 8, jj = n0 + x * 8 + 2 * t + (y & 1);
+                    if (DELTA) As[i * RC_LDB + jj] = bt[i] * ca[x][y];
+                    Bm[i * RC_C + jj] = cb[x][y];
+                }
+        }
+        // pairs inside sixteen rows: a warp a row, the lanes over the channels (two rows of every sixteen a warp, 17 pairs)
+        for (int blk = 0; blk < RC_C / 16; blk++)
+            for (int half = 0; half < 2; half++) {
+                const int i = 16 * blk + (half ? 15 - warp : warp);
+                float ki[RC_MAX_D / 32], qi[RC_MAX_D / 32], gi[RC_MAX_D / 32];
+#pragma unroll
+                for (int m = 0; m < RC_MAX_D / 32; m++) {
+                    const int d = lane + 32 * m;
+                    const bool ok = d < Dp;
+                    ki[m] = ok && DELTA ? Ks[i * ld + d] : 0.f;
+                    qi[m] = ok ? Qs[i * ld + d] : 0.f;
+                    gi[m] = ok ? Gs[i * ld + d] : 0.f;
+                }
+                for (int jj = 16 * blk; jj < 16 * blk + 16; jj++) {
+                    float sa = 0.f, sb = 0.f;
+                    if (jj <= i) {
+#pragma unroll
+                        for (int m = 0; m < RC_MAX_D / 32; m++) {
+                            const int d = lane + 32 * m;
+                            if (d < Dp) {
+                                const float x = Ks[jj * ld + d] * exp2f(gi[m] - Gs[jj * ld + d]);
+                                if (DELTA) sa = fmaf(ki[m], x, sa);
+                                sb = fmaf(qi[m], x, sb);
+                            }
+                        }
+                        if (DELTA) sa = warp_sum(sa);
+                        sb = warp_sum(sb);
+                    }
+                    if (lane == 0) {
+                        if (DELTA) As[i * RC_LDB + jj] = jj < i ? bt[i] * sa : 0.f;
+                        Bm[i * RC_C + jj] = sb;
+                    }
+                }
+            }
+    }
+    __syncthreads();
+    // the system, one right hand side a thread; the gated recurrence takes v as it is
+    for (int c = tid; c < (DELTA ? P + D : P); c += RC_THREADS) {
+        const bool is_v = c < P;
+        if (!DELTA) {
+            for (int i = 0; i < RC_C; i++)
+                out[R.wv + (size_t)i * P + c] = i < n ? to_f32(vp[(size_t)(t0 + i) * ldi + (size_t)head * P + c]) : 0.f;
+            continue;
+        }
+        const int d = c - P;
+        float w[RC_C];
+        if (is_v) {
+#pragma unroll
+            for (int i = 0; i < RC_C; i++) w[i] = i < n ? to_f32(vp[(size_t)(t0 + i) * ldi + (size_t)head * P + c]) : 0.f;
+#pragma unroll
+            for (int i = 0; i < RC_C; i++) w[i] *= bt[i];
+        } else {
+#pragma unroll
+            for (int i = 0; i < RC_C; i++) w[i] = bt[i] * (Ks[i * ld + d] * exp2f(CHAN ? Gs[i * ld + d] : Gs[i]));
+        }
+#pragma unroll
+        for (int i = 1; i < RC_C; i++) {
+            float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+            const float4* row = reinterpret_cast<const float4*>(As + i * RC_LDB);
+#pragma unroll
+            for (int q = 0; q < (i + 3) / 4; q++) {
+                const float4 r4 = row[q];
+                a0 = fmaf(r4.x, w[4 * q], a0);
+                if (4 * q + 1 < i) a1 = fmaf(r4.y, w[4 * q + 1], a1);
+                if (4 * q + 2 < i) a2 = fmaf(r4.z, w[4 * q + 2], a2);
+                if (4 * q + 3 < i) a3 = fmaf(r4.w, w[4 * q + 3], a3);
+            }
+            w[i] -= (a0 + a1) + (a2 + a3);
+        }
+        float* dst = is_v ? out + R.wv + c : out + R.wk + d;
+        const int step = is_v ? P : D;
+#pragma unroll
+        for (int i = 0; i < RC_C; i++) dst[(size_t)i * step] = w[i];
+    }
+    for (int i = warp; i < RC_C; i += RC_THREADS / 32)
+        for (int d = lane; d < D; d += 32) {
+            const float gi = CHAN ? Gs[i * ld + d] : Gs[i], gl = CHAN ? Gs[(RC_C - 1) * ld + d] : Gs[RC_C - 1];
+            out[R.kh + (size_t)i * D + d] = Ks[i * ld + d] * exp2f(gl - gi);
+            out[R.qt + (size_t)i * D + d] = Qs[i * ld + d] * exp2f(gi);
+        }
+    for (int d = tid; d < D; d += RC_THREADS) out[R.el + d] = exp2f(CHAN ? Gs[(RC_C - 1) * ld + d] : Gs[RC_C - 1]);
+}
+
+__device__ __forceinline__ void rc_cp16(float* dst, const float* src) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src) : "memory");
+}
+// rows x cols floats from global (row pitch src_ld) to shared memory (row pitch ld); vec: everything starts on 16 bytes
+__device__ __forceinline__ void rc_fetch(float* dst, int ld, const float* src, int src_ld, int rows, int cols, bool vec, int warp, int lane) {
+    for (int i = warp; i < rows; i += RC_THREADS / 32) {
+        if (vec) for (int x = lane * 4; x < cols; x += 128) rc_cp16(dst + i * ld + x, src + (size_t)i * src_ld + x);
+        else for (int x = lane; x < cols; x += 32) dst[i * ld + x] = src[(size_t)i * src_ld + x];
+    }
+}
+
+// Pass 1, one block a (32 value columns, head, segment): S[chunk] <- the state at the chunk's head; u in the place of Wv;
+// the segment's slot <- the state behind its last chunk.  stages: 2 fetches a chunk's operands while the one before runs.
+template <bool DELTA>
+__global__ void __launch_bounds__(RC_THREADS)
+recur_chunk_states_kernel(float* __restrict__ rec, float* __restrict__ heads_s, float* __restrict__ state, size_t slot_stride,
+                          const int* __restrict__ seg_pos, const int* __restrict__ seg_slot, const int* __restrict__ seg_chunk0,
+                          int H, int D, int P, int write_state, int stages, int vec) {
+    kp_pdl_begin();
+    extern __shared__ __align__(16) float rc_sm[];
+    const int Dp = (D + 31) & ~31, lda = Dp + 4, ldb = Dp + 8;
+    const int stage_floats = (DELTA ? RC_C * lda : 0) + RC_C * ldb + RC_C * RC_LDU;
+    float* Ss = rc_sm;                                           // [Dp][RC_LDU]
+    float* st0 = Ss + Dp * RC_LDU;
+    const int tile = blockIdx.x, head = blockIdx.y, seg = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = lane >> 2, t = lane & 3;
+    const int j0 = tile * RC_PT, cols = min(RC_PT, P - j0);
+    const RcRec R = rc_record(D, P, DELTA);
+    // (columns and rows behind the sizes stay zero: nothing is fetched into them)
+    for (int x = tid; x < Dp * RC_LDU + stages * stage_floats; x += RC_THREADS) rc_sm[x] = 0.f;
+    __syncthreads();
+    float* st = state + (size_t)seg_slot[seg] * slot_stride + (size_t)head * D * P;
+    if (seg_pos[seg] != 0)
+        for (int i = warp; i < D; i += RC_THREADS / 32)
+            if (lane < cols) Ss[i * RC_LDU + lane] = st[(size_t)i * P + j0 + lane];
+    const int c_begin = seg_chunk0[seg], c_end = seg_chunk0[seg + 1];
+    auto fetch = [&](int c, int s) {
+        const float* src = rec + ((size_t)c * H + head) * R.size;
+        float* wk = st0 + s * stage_floats;
+        float* kh = wk + (DELTA ? RC_C * lda : 0);
+        float* wv = kh + RC_C * ldb;
+        if (DELTA) rc_fetch(wk, lda, src + R.wk, D, RC_C, D, vec, warp, lane);
+        rc_fetch(kh, ldb, src + R.kh, D, RC_C, D, vec, warp, lane);
+        rc_fetch(wv, RC_LDU, src + R.wv + j0, P, RC_C, cols, vec, warp, lane);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (c_begin < c_end) fetch(c_begin, 0);
+    for (int c = c_begin; c < c_end; c++) {
+        const int s = stages == 2 ? (c - c_begin) & 1 : 0;
+        if (stages == 2 && c + 1 < c_end) {
+            fetch(c + 1, s ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        float* wk = st0 + s * stage_floats;
+        float* kh = wk + (DELTA ? RC_C * lda : 0);
+        float* us = kh + RC_C * ldb;
+        float* dst = heads_s + ((size_t)c * H + head) * D * P + j0;
+        for (int i = warp; i < D; i += RC_THREADS / 32)
+            if (lane < cols) dst[(size_t)i * P + lane] = Ss[i * RC_LDU + lane];
+        float* rc = rec + ((size_t)c * H + head) * R.size;
+        if (DELTA) {
+            const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 16;
+            float acc[2][4];
+#pragma unroll
+            for (int x = 0; x < 2; x++)
+#pragma unroll
+                for (int y = 0; y < 4; y++) acc[x][y] = 0.f;
+#pragma unroll 2
+            for (int k0 = 0; k0 < D; k0 += 8) {
+                RcA fa;
+                rc_load_a(fa, wk, lda, m0, k0, g, t);
+#pragma unroll
+                for (int x = 0; x < 2; x++) {
+                    RcB fb;
+                    rc_load_b(fb, Ss, RC_LDU, k0, n0 + 8 * x, g, t);
+                    rc_mma3(acc[x], fa, fb);
+                }
+            }
+#pragma unroll
+            for (int x = 0; x < 2; x++)
+#pragma unroll
+                for (int y = 0; y < 4; y++) {
+                    const int i = m0 + g + (y >> 1) * 8, j = n0 + 8 * x + 2 * t + (y & 1);
+                    const float u = us[i * RC_LDU + j] - acc[x][y];
+                    us[i * RC_LDU + j] = u;
+                    if (j < cols) rc[R.wv + (size_t)i * P + j0 + j] = u;
+                }
+        }
+        __syncthreads();
+        for (int m0 = warp * 16; m0 < D; m0 += 16 * (RC_THREADS / 32)) {
+            float acc[4][4];
+            const float e0 = m0 + g < D ? rc[R.el + m0 + g] : 0.f, e1 = m0 + g + 8 < D ? rc[R.el + m0 + g + 8] : 0.f;
+#pragma unroll
+            for (int x = 0; x < 4; x++)
+#pragma unroll
+                for (int y = 0; y < 4; y++)
+                    acc[x][y] = (y < 2 ? e0 : e1) * Ss[(m0 + g + (y >> 1) * 8) * RC_LDU + 8 * x + 2 * t + (y & 1)];
+#pragma unroll 2
+            for (int k0 = 0; k0 < RC_C; k0 += 8) {
+                RcA fa;
+                rc_load_at(fa, kh, ldb, m0, k0, g, t);
+#pragma unroll
+                for (int x = 0; x < 4; x++) {
+                    RcB fb;
+                    rc_load_b(fb, us, RC_LDU, k0, 8 * x, g, t);
+                    rc_mma3(acc[x], fa, fb);
+                }
+            }
+#pragma unroll
+            for (int x = 0; x < 4; x++)
+#pragma unroll
+                for (int y = 0; y < 4; y++)
+                    Ss[(m0 + g + (y >> 1) * 8) * RC_LDU + 8 * x + 2 * t + (y & 1)] = acc[x][y];
+        }
+        __syncthreads();
+        if (stages == 1 && c + 1 < c_end) fetch(c + 1, 0);
+    }
+    if (write_state)
+        for (int i = warp; i < D; i += RC_THREADS / 32)
+            if (lane < cols) st[(size_t)i * P + j0 + lane] = Ss[i * RC_LDU + lane];
+}
+
+// Pass 2, one block a (PT value columns, chunk, head): o = exp(G) q S + B u.
+template <int PT>
+__global__ void __launch_bounds__(RC_THREADS)
+recur_chunk_out_kernel(const float* __restrict__ rec, const float* __restrict__ heads_s, const int* __restrict__ cu_rows,
+                       const int* __restrict__ chunk_seg, const int* __restrict__ chunk_row0, float* __restrict__ out, int ldo,
+                       int H, int D, int P, int delta, int vec) {
+    kp_pdl_begin();
+    constexpr int LDP = PT + 8;                                  // (PT 32 or 64: 8 beyond a multiple of 32)
+    constexpr int NT = PT / 16;                                  // tiles of eight columns a warp
+    extern __shared__ __align__(16) float rc_sm[];
+    const int Dp = (D + 31) & ~31, lda = Dp + 4;
+    float* Qt = rc_sm;                                           // [64][lda]
+    float* Ss = Qt + RC_C * lda;                                 // [Dp][LDP]
+    float* Bs = Ss + Dp * LDP;                                   // [64][RC_LDB]
+    float* us = Bs + RC_C * RC_LDB;                              // [64][LDP]
+    const int chunk = blockIdx.y, head = blockIdx.z, tile = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = lane >> 2, t = lane & 3;
+    const int t0 = chunk_row0[chunk], n = min(RC_C, cu_rows[chunk_seg[chunk] + 1] - t0);
+    const int j0 = tile * PT, cols = min(PT, P - j0);
+    const RcRec R = rc_record(D, P, delta != 0);
+    const float* rc = rec + ((size_t)chunk * H + head) * R.size;
+    if (D < Dp || cols < PT) {                                   // zeros where nothing is fetched
+        for (int x = tid; x < RC_C * lda + Dp * LDP; x += RC_THREADS) rc_sm[x] = 0.f;
+        for (int x = tid; x < RC_C * LDP; x += RC_THREADS) us[x] = 0.f;
+        __syncthreads();
+    }
+    rc_fetch(Qt, lda, rc + R.qt, D, RC_C, D, vec, warp, lane);
+    rc_fetch(Ss, LDP, heads_s + ((size_t)chunk * H + head) * D * P + j0, P, D, cols, vec, warp, lane);
+    rc_fetch(Bs, RC_LDB, rc + R.bm, RC_C, RC_C, RC_C, true, warp, lane);
+    rc_fetch(us, LDP, rc + R.wv + j0, P, RC_C, cols, vec, warp, lane);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * (PT / 2);
+    if (m0 >= n) return;
+    float acc[NT][4];
+#pragma unroll
+    for (int x = 0; x < NT; x++)
+#pragma unroll
+        for (int y = 0; y < 4; y++) acc[x][y] = 0.f;
+#pragma unroll 2
+    for (int k0 = 0; k0 < D; k0 += 8) {
+        RcA fa;
+        rc_load_a(fa, Qt, lda, m0, k0, g, t);
+#pragma unroll
+        for (int x = 0; x < NT; x++) {
+            RcB fb;
+            rc_load_b(fb, Ss, LDP, k0, n0 + 8 * x, g, t);
+            rc_mma3(acc[x], fa, fb);
+        }
+    }
+    for (int k0 = 0; k0 < m0 + 16; k0 += 8) {
+        RcA fa;
+        rc_load_a(fa, Bs, RC_LDB, m0, k0, g, t);
+#pragma unroll
+        for (int x = 0; x < NT; x++) {
+            RcB fb;
+            rc_load_b(fb, us, LDP, k0, n0 + 8 * x, g, t);
+            rc_mma3(acc[x], fa, fb);
+        }
+    }
+#pragma unroll
+    for (int x = 0; x < NT; x++)
+#pragma unroll
+        for (int y = 0; y < 4; y++) {
+            const int i = m0 + g + (y >> 1) * 8, j = n0 + 8 * x + 2 * t + (y & 1);
+            if (i < n && j < cols) out[(size_t)(t0 + i) * ldo + (size_t)head * P + j0 + j] = acc[x][y];
+        }
+}
+
+extern "C" {
+
+// Convolutions, unit norms, step sizes and decays in front of a delta recurrence: see delta_prep_kernel.  per_channel: lg
+// holds the decays' projections [n, H D] and is changed in place; else they are columns a_col .. of p and lg [n, H] is
+// written.  taps [C][K]; neg_a [H]: -exp(A_log); dt_bias [H D] or [H].  kept: a slot's last K - 1 inputs at `kept + slot *
+// slot_stride`; renewed unless keep == 0 (single_rows: by the same launch, else by a second one).
+int kp_delta_prep(const void* p, int ld, int conv_col, int b_col, int a_col, const float* taps, const float* neg_a,
+                  const float* dt_bias, float* kept, long long slot_stride, const int* row_seg, const int* cu_rows, const int* seg_pos,
+                  const int* seg_slot, float* out, float* beta, float* lg, int n, int n_seg, int H, int G, int D, int P, int K,
+                  float q_scale, int per_channel, int single_rows, int keep, int dtype, void* stream) {
+    if (n <= 0) return 0;
+    if (H < 1 || G < 1 || H % G || D < 1 || P < 1) return KP_ERR_BAD_ARG;
+    if (D > 256 || K < 1 || K > SS_MAX_TAPS || n > 65535 || n_seg > 65535) return KP_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int C = 2 * G * D + H * P, n_e = H + (per_channel ? H * D : H);
+    const int esz = dtype == KP_DTYPE_F32 ? 4 : 2;
+    const bool vec = !single_rows && K <= 4 && n >= 2 * RP_ROWS && D % 4 == 0 && (H * P) % 4 == 0 && ld % 4 == 0 && conv_col % 4 == 0 &&
+                     (uintptr_t)p % (4 * esz) == 0 && (uintptr_t)out % 16 == 0;
+    if (vec) {
+        const int quads = D / 4, team = (quads & (quads - 1)) == 0 && quads <= 32 ? quads : 32;
+        const int ql = D > 128 ? 2 : 1, per_warp = 32 / team;
+        const int items = (2 * G + per_warp - 1) / per_warp + (H * P + 128 * ql - 1) / (128 * ql);
+        const int conv_blocks = (items + 3) / 4;
+        int gate_blocks = (n_e + 127) / 128;
+        if (gate_blocks > 32) gate_blocks = 32;
+        const dim3 grid(conv_blocks + gate_blocks, (n + RP_ROWS - 1) / RP_ROWS);
+#define RP_LAUNCH(KK, QQ)                                                                                                    \
+        KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(delta_prep_vec_kernel<T, KK, QQ>, grid, dim3(128), 0, s, (const T*)p, ld, conv_col, b_col, \
+                                                   a_col, taps, neg_a, dt_bias, (const float*)kept, (size_t)slot_stride, row_seg, cu_rows,   \
+                                                   seg_pos, seg_slot, out, beta, lg, n, H, G, D, P, q_scale, per_channel, conv_blocks, team)))
+#define RP_LAUNCH_K(QQ)                                                                                                      \
+        do { if (K == 1) RP_LAUNCH(1, QQ); else if (K == 2) RP_LAUNCH(2, QQ); else if (K == 3) RP_LAUNCH(3, QQ); else RP_LAUNCH(4, QQ); } while (0)
+        if (ql == 1) RP_LAUNCH_K(1);
+        else RP_LAUNCH_K(2);
+#undef RP_LAUNCH_K
+#undef RP_LAUNCH
+    } else {
+        const int items = 2 * G + (H * P + 127) / 128 + (n_e + 127) / 128;
+        KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(delta_prep_kernel<T>, dim3((items + 3) / 4, n), dim3(128), 0, s, (const T*)p, ld, conv_col,
+                                                   b_col, a_col, taps, neg_a, dt_bias, kept, (size_t)slot_stride, row_seg, cu_rows, seg_pos,
+                                                   seg_slot, out, beta, lg, H, G, D, P, K, q_scale, per_channel, single_rows && keep)));
+    }
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) return (int)e;
+    if (keep && !single_rows && K > 1) {
+        KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(ssm_conv_keep_kernel<T>, dim3((C + 127) / 128, n_seg), dim3(128), 0, s, (const T*)p, ld,
+                                                   conv_col, kept, (size_t)slot_stride, cu_rows, seg_pos, seg_slot, C, K)));
+    }
+    return kp_launch_status();
+}
+
+int kp_log_decay_sigmoid(float* z, long long n, float inv_tau, void* stream) {
+    if (n <= 0) return 0;
+    long long blocks = (n + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    kp_launch_pdl(log_decay_sigmoid_kernel, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, z, (size_t)n, inv_tau);
+    return kp_launch_status();
+}
+
+// q, k (G heads of D) and v (H heads of P): rows of pitch ldi, in float32 or the storage type (dtype).  lg: [n, H] or, with
+// per_channel, [n, H D] float32; beta: [n, H], or null for the gated recurrence.  state: a slot's [H][D][P] float32 at
+// `state + slot * slot_stride`.  out: [n, ldo] float32, heads side by side.
+int kp_recur_scan(const void* q, const void* k, const void* v, int ldi, const float* lg, const float* beta, float q_scale, float* state,
+                  long long slot_stride, const int* cu_rows, const int* seg_pos, const int* seg_slot, float* out, int ldo, int n_seg,
+                  int H, int G, int D, int P, int per_channel, int write_state, int dtype, void* stream) {
+    if (n_seg <= 0) return 0;
+    if (H < 1 || G < 1 || H % G || D < 1 || P < 1) return KP_ERR_BAD_ARG;
+    if (D > 256 || H > 65535 || n_seg > 65535) return KP_ERR_UNSUPPORTED;
+    const dim3 grid((P + RS_COLS - 1) / RS_COLS, H, n_seg), block(RS_THREADS);
+    cudaStream_t s = (cudaStream_t)stream;
+#define RS_LAUNCH(T, R, DL, CH)                                                                                              \
+    kp_launch_pdl(recur_scan_kernel<T, R, DL, CH>, grid, block, 0, s, (const T*)q, (const T*)k, (const T*)v, ldi, lg, beta, q_scale, state,  \
+                  (size_t)slot_stride, cu_rows, seg_pos, seg_slot, out, ldo, H, G, D, P, write_state)
+#define RS_LAUNCH_R(T, DL, CH)                                                                                               \
+    do {                                                                                                                     \
+        if (D <= 32) RS_LAUNCH(T, 8, DL, CH);                                                                                \
+        else if (D <= 64) RS_LAUNCH(T, 16, DL, CH);                                                                          \
+        else if (D <= 128) RS_LAUNCH(T, 32, DL, CH);                                                                         \
+        else RS_LAUNCH(T, 64, DL, CH);                                                                                       \
+    } while (0)
+    // (the rows a thread keeps depend on the state's size only, so a row's sums have the same order in every launch)
+    if (beta) {
+        if (dtype != KP_DTYPE_F32) return KP_ERR_UNSUPPORTED;          // (what delta_prep leaves)
+        if (per_channel) RS_LAUNCH_R(float, true, true);
+        else RS_LAUNCH_R(float, true, false);
+    } else {
+        if (!per_channel) return KP_ERR_UNSUPPORTED;
+        KP_DISPATCH_DTYPE(dtype, T, RS_LAUNCH_R(T, false, true));
+    }
+#undef RS_LAUNCH_R
+#undef RS_LAUNCH
+    return kp_launch_status();
+}
+
+int kp_recur_chunk_rows() { return RC_C; }
+// floats of scratch that kp_recur_chunks wants: the records of pass 0, then every chunk's state a head
+long long kp_recur_chunks_scratch(int n_chunks, int H, int D, int P, int delta) {
+    return (long long)n_chunks * H * ((long long)rc_record(D, P, delta != 0).size + (long long)D * P);
+}
+
+// The chunked form: the arguments of kp_recur_scan and the list of chunks (chunk_seg, chunk_row0 [n_chunks]: every chunk's
+// segment, numbered among the n_seg segments given here, and first row; seg_chunk0 [n_seg + 1]: the first chunk of every
+// segment).  scratch: kp_recur_chunks_scratch floats, 16-byte aligned.
+int kp_recur_chunks(const void* q, const void* k, const void* v, int ldi, const float* lg, const float* beta, float q_scale, float* state,
+                    long long slot_stride, const int* cu_rows, const int* seg_pos, const int* seg_slot, const int* chunk_seg,
+                    const int* chunk_row0, const int* seg_chunk0, int n_chunks, float* scratch, float* out, int ldo, int n_seg, int H,
+                    int G, int D, int P, int per_channel, int write_state, int dtype, void* stream) {
+    if (n_seg <= 0 || n_chunks <= 0) return 0;
+    if (H < 1 || G < 1 || H % G || D < 1 || P < 1 || (uintptr_t)scratch % 16) return KP_ERR_BAD_ARG;
+    if (D > RC_MAX_D || H > 65535 || n_seg > 65535 || n_chunks > 65535) return KP_ERR_UNSUPPORTED;
+    const bool delta = beta != nullptr;
+    const int Dp = (D + 31) & ~31, ld = Dp + 4;
+    const size_t sm0 = ((size_t)(per_channel ? 3 : 2) * RC_C * ld + (delta ? RC_C * RC_LDB : 0) + 2 * RC_C) * sizeof(float);
+    const size_t stage = ((delta ? (size_t)RC_C * ld : 0) + (size_t)RC_C * (Dp + 8) + (size_t)RC_C * RC_LDU) * sizeof(float);
+    const size_t keep1 = (size_t)Dp * RC_LDU * sizeof(float);
+    const int stages = keep1 + 2 * stage <= 227 * 1024 ? 2 : 1;
+    const size_t sm1 = keep1 + stages * stage;
+    const int pt = P > 32 ? 64 : 32;
+    const size_t sm2 = ((size_t)RC_C * ld + (size_t)Dp * (pt + 8) + (size_t)RC_C * RC_LDB + (size_t)RC_C * (pt + 8)) * sizeof(float);
+    const int vec = D % 4 == 0 && P % 4 == 0;
+    float* rec = scratch;
+    float* hs = scratch + (size_t)n_chunks * H * rc_record(D, P, delta).size;
+    cudaStream_t s = (cudaStream_t)stream;
+    cudaError_t e;
+#define RC_PREPARE(T, DL, CH)                                                                                                \
+    do {                                                                                                                     \
+        if ((e = cudaFuncSetAttribute(recur_chunk_prepare_kernel<T, DL, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm0)) != cudaSuccess) return (int)e; \
+        kp_launch_pdl(recur_chunk_prepare_kernel<T, DL, CH>, dim3(n_chunks, H), dim3(RC_THREADS), sm0, s, (const T*)q, (const T*)k, (const T*)v, \
+                      ldi, lg, beta, q_scale, cu_rows, chunk_seg, chunk_row0, rec, H, G, D, P);                              \
+    } while (0)
+    if (delta) {
+        if (dtype != KP_DTYPE_F32) return KP_ERR_UNSUPPORTED;
+        if (per_channel) RC_PREPARE(float, true, true);
+        else RC_PREPARE(float, true, false);
+    } else {
+        if (!per_channel) return KP_ERR_UNSUPPORTED;
+        KP_DISPATCH_DTYPE(dtype, T, RC_PREPARE(T, false, true));
+    }
+#undef RC_PREPARE
+    if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
+    const dim3 grid1((P + RC_PT - 1) / RC_PT, H, n_seg);
+    if (delta) {
+        if ((e = cudaFuncSetAttribute(recur_chunk_states_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return (int)e;
+        kp_launch_pdl(recur_chunk_states_kernel<true>, grid1, dim3(RC_THREADS), sm1, s, rec, hs, state, (size_t)slot_stride, seg_pos, seg_slot,
+                      seg_chunk0, H, D, P, write_state, stages, vec);
+    } else {
+        if ((e = cudaFuncSetAttribute(recur_chunk_states_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return (int)e;
+        kp_launch_pdl(recur_chunk_states_kernel<false>, grid1, dim3(RC_THREADS), sm1, s, rec, hs, state, (size_t)slot_stride, seg_pos, seg_slot,
+                      seg_chunk0, H, D, P, write_state, stages, vec);
+    }
+    if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
+    const dim3 grid2((P + pt - 1) / pt, n_chunks, H);
+    if (pt == 64) {
+        if ((e = cudaFuncSetAttribute(recur_chunk_out_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm2)) != cudaSuccess) return (int)e;
+        kp_launch_pdl(recur_chunk_out_kernel<64>, grid2, dim3(RC_THREADS), sm2, s, (const float*)rec, (const float*)hs, cu_rows, chunk_seg, chunk_row0,
+                      out, ldo, H, D, P, (int)delta, vec);
+    } else {
+        if ((e = cudaFuncSetAttribute(recur_chunk_out_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm2)) != cudaSuccess) return (int)e;
+        kp_launch_pdl(recur_chunk_out_kernel<32>, grid2, dim3(RC_THREADS), sm2, s, (const float*)rec, (const float*)hs, cu_rows, chunk_seg, chunk_row0,
+                      out, ldo, H, D, P, (int)delta, vec);
+    }
+    return kp_launch_status();
+}
+
+}  // extern "C"

@@ -16,11 +16,8 @@
 // alone, so a row's bits do not depend on how the sequence was cut); and the chunked form for prompt portions in 16-bit
 // mode (below).
 #include "common.cuh"
+#include "chanconv.cuh"
 
-#define SS_MAX_TAPS 16
-
-__device__ __forceinline__ float ss_silu(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float ss_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // p: rows [n, ld] in the storage type, the convolved channels at column conv_col (C of them), dt behind at dt_col (H).
 // kept: [slots][slot_stride] float32, a slot's inputs as [taps - 1][C], oldest first.  out: [n, C] in the storage type.
@@ -32,7 +29,7 @@ ssm_conv_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, const
                 const float* __restrict__ bias, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                 float* __restrict__ kept, size_t slot_stride, const int* __restrict__ row_seg, const int* __restrict__ cu_rows,
                 const int* __restrict__ seg_pos, const int* __restrict__ seg_slot, T* __restrict__ out, float* __restrict__ dt_out,
-                float* __restrict__ da_out, int C, int H, int K, int fused_state) {
+                float* __restrict__ da_out, int C, int H, int K, int fused_state, int act) {
     kp_pdl_begin();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     const int r = blockIdx.y;
@@ -47,7 +44,7 @@ ssm_conv_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, const
     const int seg = row_seg[r], row0 = cu_rows[seg];
     const bool fresh = seg_pos[seg] == 0;
     float* kp = kept + (size_t)seg_slot[seg] * slot_stride;
-    float acc = bias[c];
+    float acc = bias ? bias[c] : 0.f;
     float in[SS_MAX_TAPS];
 #pragma unroll
     for (int j = 0; j < SS_MAX_TAPS; j++) {
@@ -60,7 +57,7 @@ ssm_conv_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, const
             acc = fmaf(taps[(size_t)c * K + j], v, acc);
         }
     }
-    out[(size_t)r * C + c] = from_f32<T>(ss_silu(acc));
+    out[(size_t)r * C + c] = from_f32<T>((act ? ss_silu(acc) : acc));
     if (fused_state) {
 #pragma unroll
         for (int j = 0; j < SS_MAX_TAPS - 1; j++)
@@ -73,41 +70,13 @@ ssm_conv_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, const
 // the same chain of multiply-adds as above (bias, then the taps from the oldest), so a row's bits do not depend on
 // which form ran.  The last blocks along x compute dt and the decay's logarithm of the tile's rows.
 #define SV_ROWS 4
-template <typename T> struct SsVec;
-template <> struct SsVec<bf16> {
-    static constexpr int W = 8;
-    __device__ static void load(const bf16* src, float* v) {
-        const uint4 raw = __ldg(reinterpret_cast<const uint4*>(src));
-        const bf16* e = reinterpret_cast<const bf16*>(&raw);
-#pragma unroll
-        for (int i = 0; i < 8; i++) v[i] = __bfloat162float(e[i]);
-    }
-    __device__ static void store(bf16* dst, const float* v) {
-        uint4 o;
-        __nv_bfloat162 t;
-        t = __floats2bfloat162_rn(v[0], v[1]); o.x = *reinterpret_cast<uint32_t*>(&t);
-        t = __floats2bfloat162_rn(v[2], v[3]); o.y = *reinterpret_cast<uint32_t*>(&t);
-        t = __floats2bfloat162_rn(v[4], v[5]); o.z = *reinterpret_cast<uint32_t*>(&t);
-        t = __floats2bfloat162_rn(v[6], v[7]); o.w = *reinterpret_cast<uint32_t*>(&t);
-        *reinterpret_cast<uint4*>(dst) = o;
-    }
-};
-template <> struct SsVec<float> {
-    static constexpr int W = 4;
-    __device__ static void load(const float* src, float* v) {
-        const float4 r = __ldg(reinterpret_cast<const float4*>(src));
-        v[0] = r.x; v[1] = r.y; v[2] = r.z; v[3] = r.w;
-    }
-    __device__ static void store(float* dst, const float* v) { *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]); }
-};
-
 template <typename T, int K>
 __global__ void __launch_bounds__(128)
 ssm_conv_vec_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, const float* __restrict__ taps,
                     const float* __restrict__ bias, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                     const float* __restrict__ kept, size_t slot_stride, const int* __restrict__ row_seg,
                     const int* __restrict__ cu_rows, const int* __restrict__ seg_pos, const int* __restrict__ seg_slot,
-                    T* __restrict__ out, float* __restrict__ dt_out, float* __restrict__ da_out, int n, int C, int H, int conv_blocks) {
+                    T* __restrict__ out, float* __restrict__ dt_out, float* __restrict__ da_out, int n, int C, int H, int conv_blocks, int act) {
     kp_pdl_begin();
     constexpr int W = SsVec<T>::W;
     const int r0 = blockIdx.y * SV_ROWS;
@@ -145,10 +114,9 @@ ssm_conv_vec_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, c
             const float4 t = __ldg(t4 + i);
             flat[4 * i] = t.x; flat[4 * i + 1] = t.y; flat[4 * i + 2] = t.z; flat[4 * i + 3] = t.w;
         }
-        const float4* b4 = reinterpret_cast<const float4*>(bias + c);
 #pragma unroll
         for (int i = 0; i < W / 4; i++) {
-            const float4 t = __ldg(b4 + i);
+            const float4 t = bias ? __ldg(reinterpret_cast<const float4*>(bias + c) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
             bs[4 * i] = t.x; bs[4 * i + 1] = t.y; bs[4 * i + 2] = t.z; bs[4 * i + 3] = t.w;
         }
 #pragma unroll
@@ -182,29 +150,8 @@ ssm_conv_vec_kernel(const T* __restrict__ p, int ld, int conv_col, int dt_col, c
             }
         }
 #pragma unroll
-        for (int e = 0; e < W; e++) acc[e] = ss_silu(acc[e]);
+        for (int e = 0; e < W; e++) acc[e] = act ? ss_silu(acc[e]) : acc[e];
         SsVec<T>::store(out + (size_t)r * C + c, acc);
-    }
-}
-
-// The inputs a request keeps behind a segment of len rows: its last taps - 1, from the rows of this step and, where the
-// segment is shorter than that, from what was kept before (zero for a fresh sequence).
-template <typename T>
-__global__ void __launch_bounds__(128)
-ssm_conv_keep_kernel(const T* __restrict__ p, int ld, int conv_col, float* __restrict__ kept, size_t slot_stride,
-                     const int* __restrict__ cu_rows, const int* __restrict__ seg_pos, const int* __restrict__ seg_slot, int C, int K) {
-    kp_pdl_begin();
-    const int seg = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
-    if (c >= C) return;
-    const int row0 = cu_rows[seg], row1 = cu_rows[seg + 1], len = row1 - row0;
-    const bool fresh = seg_pos[seg] == 0;
-    float* kp = kept + (size_t)seg_slot[seg] * slot_stride;
-    for (int j = 0; j < K - 1; j++) {                       // ascending: index len + j is read before it is written
-        const int rr = row1 - (K - 1) + j;
-        float v;
-        if (rr >= row0) v = to_f32(p[(size_t)rr * ld + conv_col + c]);
-        else v = fresh ? 0.f : kp[(size_t)(len + j) * C + c];
-        kp[(size_t)j * C + c] = v;
     }
 }
 
@@ -569,16 +516,16 @@ ssm_chunk_out_kernel(const T* __restrict__ xbc, int ldx, int c_col, const float*
 
 extern "C" {
 
-// The convolution with bias and silu over the C channels at conv_col of p, dt and the decay's logarithm of the H heads
-// at dt_col.  taps [C][K], bias [C], dt_bias, a_log [H].  kept: a slot's last K - 1 inputs at `kept + slot *
+// The convolution over the C channels at conv_col of p, with a bias unless it is null and silu where act is 1, and dt and
+// the decay's logarithm of the H heads at dt_col (H = 0: none, the channels alone).  taps [C][K], bias [C], dt_bias, a_log [H].  kept: a slot's last K - 1 inputs at `kept + slot *
 // slot_stride`.  single_rows != 0: every segment has one row and the kept inputs are renewed here; else they are
 // renewed by a second launch behind the first unless keep == 0.
 int kp_ssm_conv(const void* p, int ld, int conv_col, int dt_col, const float* taps, const float* bias, const float* dt_bias,
                 const float* a_log, float* kept, long long slot_stride, const int* row_seg, const int* cu_rows, const int* seg_pos,
                 const int* seg_slot, void* out, float* dt_out, float* da_out, int n, int n_seg, int C, int H, int K, int single_rows,
-                int keep, int dtype, void* stream) {
+                int keep, int act, int dtype, void* stream) {
     if (n <= 0) return 0;
-    if (C < 1 || H < 1 || K < 1 || K > SS_MAX_TAPS || n > 65535 || n_seg > 65535) return KP_ERR_UNSUPPORTED;
+    if (C < 1 || H < 0 || act < 0 || act > 1 || K < 1 || K > SS_MAX_TAPS || n > 65535 || n_seg > 65535) return KP_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const int fused = single_rows && keep;
     const int vw = dtype == KP_DTYPE_F32 ? 4 : 8;
@@ -590,13 +537,13 @@ int kp_ssm_conv(const void* p, int ld, int conv_col, int dt_col, const float* ta
 #define SV_LAUNCH(KK)                                                                                                        \
         KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(ssm_conv_vec_kernel<T, KK>, grid, dim3(128), 0, s, (const T*)p, ld, conv_col, dt_col, taps,  \
                                                    bias, dt_bias, a_log, (const float*)kept, (size_t)slot_stride, row_seg, cu_rows, seg_pos, \
-                                                   seg_slot, (T*)out, dt_out, da_out, n, C, H, conv_blocks)))
+                                                   seg_slot, (T*)out, dt_out, da_out, n, C, H, conv_blocks, act)))
         if (K == 1) SV_LAUNCH(1); else if (K == 2) SV_LAUNCH(2); else if (K == 3) SV_LAUNCH(3); else SV_LAUNCH(4);
 #undef SV_LAUNCH
     } else {
         KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(ssm_conv_kernel<T>, dim3((C + H + 127) / 128, n), dim3(128), 0, s, (const T*)p, ld, conv_col,
                                                    dt_col, taps, bias, dt_bias, a_log, kept, (size_t)slot_stride, row_seg, cu_rows, seg_pos,
-                                                   seg_slot, (T*)out, dt_out, da_out, C, H, K, fused)));
+                                                   seg_slot, (T*)out, dt_out, da_out, C, H, K, fused, act)));
     }
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;

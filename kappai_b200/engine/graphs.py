@@ -316,8 +316,7 @@ class DecodeGraphs:
         r = self.runner
         # the eager warm-up run changes fixed-size state (and rewrites this step's keys, harmlessly);
         # keep a copy of the state tensors and put them back before the captured run replays the step
-        from ..cache.storage import StateView
-        states = [v.tensor for v in r.storage.views if isinstance(v, StateView) and v.writes]
+        states = r.storage.state_tensors()
         saved = [t.clone() for t in states]
         torch.cuda.current_stream().synchronize()
         r.model.forward(g.ctx, r.storage.views)

@@ -34,7 +34,7 @@ class Model:
             side = self._make("side", ls.side) if ls.side is not None else None
             p1 = self._make("norm", ls.mixer_post_norm) if ls.mixer_post_norm is not None else None
             p2 = self._make("norm", ls.ffn_post_norm) if ls.ffn_post_norm is not None else None
-            block = make_part("block", PartSpec(ls.block, dict(ls.block_params)), env)
+            block = self._make("block", PartSpec(ls.block, dict(ls.block_params), ls.block_prefix, dict(ls.block_rename)))
             # (an arrangement registered from outside may not know of side parts or of norms behind the sublayers: it is
             # asked only where there is one)
             if p1 is not None or p2 is not None:
@@ -46,10 +46,13 @@ class Model:
         self.schedule = list(spec.schedule)
         self.entry = self._make("entry", spec.entry) if spec.entry is not None else None
         self.token_table = self._make("embedding", spec.token_table) if spec.token_table is not None else None
-        parts = [self.embedding, self.final_norm, self.head, self.entry, self.token_table]
+        self.residual = self._make("residual", spec.residual) if spec.residual is not None else None
+        parts = [self.embedding, self.final_norm, self.head, self.entry, self.token_table, self.residual]
         for b in self.blocks:
             parts += [b, b.mixer, b.ffn, b.mixer_norm, b.ffn_norm, getattr(b, "side", None),
                       getattr(b, "mixer_post_norm", None), getattr(b, "ffn_post_norm", None)]
+        for p in parts:                        # (grows as it is walked: parts of parts too)
+            parts += list(getattr(p, "inner_parts", ()))
         # a decode step may be captured in a CUDA graph only if every part reads its tables from the device
         self.graph_safe = all(getattr(p, "graph_safe", False) for p in parts if p is not None)
         # parts that build tables of their own for every step, one builder per key
@@ -127,6 +130,8 @@ class Model:
                 K.scale_cast(x, None, h0, 1.0)
             else:
                 K.cast(x, h0)
+        if self.residual is not None:
+            x = self.residual.enter(x)
         for i, e in enumerate(self.schedule):
             if e.enter:
                 x = self.entry.forward(x, h0)
@@ -135,10 +140,12 @@ class Model:
             ctx.next_block = self.blocks[nxt.layer] if nxt is not None and not nxt.enter else None
             self.blocks[e.layer].forward(x, ctx, cache_views[i])
             if observer is not None:
-                observer(i, x)
+                observer(i, x if self.residual is None else self.residual.rows(x))
         if ctx.n_out == 0:
             return None
-        if self.final_norm is not None:
+        if self.residual is not None:
+            h = self.residual.normed(x, self.final_norm, rows=ctx.logit_rows)
+        elif self.final_norm is not None:
             h = self.final_norm.forward(x, rows=ctx.logit_rows)
         else:
             h = x.index_select(0, ctx.logit_rows.long()).to(self.env.dtype)

@@ -20,7 +20,7 @@ from typing import Dict, Hashable, List, Optional, Sequence, Tuple
 import torch
 
 from ..cache.manager import CacheManager, OutOfPages
-from ..cache.spec import PagedKVSpec, StateSpec
+from ..cache.spec import PagedKVSpec, StateSpec, leaf_specs
 from ..cache.storage import CacheStorage
 from ..config.registry import load_config
 from ..parts.base import BuildEnv
@@ -93,7 +93,7 @@ class ModelRunner:
         elt = torch.empty((), dtype=self.dtype).element_size()
         needs: Dict[Hashable, GroupNeed] = {}
         state_bytes = 0
-        for s in specs:
+        for s in (leaf for spec in specs for leaf in leaf_specs(spec)):
             if isinstance(s, PagedKVSpec):
                 g = needs.setdefault(s.group_key, GroupNeed(s.group_key, 0, s.window, s.keep_first if s.window is not None else 0))
                 g.bytes_per_token += 2 * s.num_kv_heads * s.head_dim * elt

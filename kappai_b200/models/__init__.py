@@ -4,3 +4,4 @@ from . import tizusun  # noqa: F401
 from . import vekuzen  # noqa: F401
 from . import tupalorn  # noqa: F401
 from . import vumotar  # noqa: F401
+from . import gosulorn  # noqa: F401

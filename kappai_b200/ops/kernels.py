@@ -752,10 +752,41 @@ def ssm_conv(p: torch.Tensor, conv_col: int, dt_col: int, taps: torch.Tensor, bi
         raise KernelError(f"ssm_conv: {K} taps exceed {SSM_MAX_TAPS}")
     _run("ssm_conv", load_library("ssm").kp_ssm_conv, _ptr(p), _rows_2d(p, "p"), int(conv_col), int(dt_col), _ptr(taps), _ptr(bias),
          _ptr(dt_bias), _ptr(a_log), _ptr(kept), ctypes.c_longlong(kept.stride(0)), _ptr(row_seg), _ptr(cu_rows), _ptr(seg_pos),
-         _ptr(seg_slot), _ptr(out), _ptr(dt_out), _ptr(da_out), n, int(n_seg), C, H, K, int(bool(single_rows)), int(bool(keep)),
+         _ptr(seg_slot), _ptr(out), _ptr(dt_out), _ptr(da_out), n, int(n_seg), C, H, K, int(bool(single_rows)), int(bool(keep)), 1,
          dtype_code(p.dtype), STREAM)
     if keep and not single_rows and K > 1:
         LAUNCHES[0] += 1
+
+
+def channel_conv(p: torch.Tensor, conv_col: int, taps: torch.Tensor, kept: torch.Tensor, row_seg: torch.Tensor,
+                 cu_rows: torch.Tensor, seg_pos: torch.Tensor, seg_slot: torch.Tensor, out: torch.Tensor, n_seg: int,
+                 single_rows: bool, keep: bool = True, activation: Optional[str] = None,
+                 bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The convolution of :func:`ssm_conv` alone: ``out = act(conv(p[:, conv_col : conv_col + C]) (+ bias))``, act = silu
+    or none.  ``kept`` as there."""
+    _need(p, "p", contiguous=False); _need(out, "out", p.dtype); _need(kept, "kept", torch.float32, contiguous=False)
+    _need(taps, "taps", torch.float32)
+    for t, nm in ((row_seg, "row_seg"), (cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (seg_slot, "seg_slot")):
+        _need(t, nm, torch.int32)
+    n, C = out.shape
+    K = taps.shape[1]
+    if (p.shape[0] != n or tuple(taps.shape) != (C, K) or conv_col + C > p.shape[1] or kept.dim() != 2 or kept.stride(1) != 1
+            or kept.shape[1] < (K - 1) * C):
+        raise KernelError("channel_conv: shape mismatch")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != C:
+            raise KernelError("channel_conv: bias size")
+    if K > SSM_MAX_TAPS or activation not in ("silu", None):
+        raise KernelError(f"channel_conv: {K} taps (at most {SSM_MAX_TAPS}), activation '{activation}' (silu or none)")
+    none = _ptr(None)
+    _run("channel_conv", load_library("ssm").kp_ssm_conv, _ptr(p), _rows_2d(p, "p"), int(conv_col), 0, _ptr(taps), _ptr(bias),
+         none, none, _ptr(kept), ctypes.c_longlong(kept.stride(0)), _ptr(row_seg), _ptr(cu_rows), _ptr(seg_pos), _ptr(seg_slot),
+         _ptr(out), none, none, n, int(n_seg), C, 0, K, int(bool(single_rows)), int(bool(keep)), int(activation == "silu"),
+         dtype_code(p.dtype), STREAM)
+    if keep and not single_rows and K > 1:
+        LAUNCHES[0] += 1
+    return out
 
 
 def _ssm_check(what, xbc, dt, da, D, state, y, H, G, N, P):
@@ -816,6 +847,176 @@ def ssm_chunks(xbc: torch.Tensor, dt: torch.Tensor, da: torch.Tensor, D: torch.T
          int(bool(write_state)), dtype_code(xbc.dtype), STREAM, work=(4 * n * H * N * P, 0))
     LAUNCHES[0] += 3
     return y
+
+
+# ------------------------------------------------------------------ recurrences with data-dependent decays
+
+RECUR_MAX_DIM = 256        # key rows of a head's state
+RECUR_MAX_TAPS = SSM_MAX_TAPS
+
+
+def delta_prep(p: torch.Tensor, conv_col: int, b_col: int, a_col: int, taps: torch.Tensor, neg_a: torch.Tensor, dt_bias: torch.Tensor,
+               kept: torch.Tensor, row_seg: torch.Tensor, cu_rows: torch.Tensor, seg_pos: torch.Tensor, seg_slot: torch.Tensor,
+               out: torch.Tensor, beta: torch.Tensor, lg: torch.Tensor, n_seg: int, H: int, G: int, D: int, P: int, q_scale: float,
+               per_channel: bool, single_rows: bool, keep: bool = True) -> None:
+    """What stands between the projections ``p`` and a delta recurrence.  ``out`` float32 [n, C]: the C = 2 G D + H P
+    channels [q | k | v] from ``conv_col``, each behind its causal convolution (taps [C, K], the last on the current
+    row) and silu, q and k as unit vectors a head, q times ``q_scale``.  ``beta`` [n, H] = sigmoid of the H columns from
+    ``b_col``.  ``lg``: the logarithms of the decays, ``neg_a_h * softplus(z + dt_bias)`` with ``neg_a`` = -exp(A_log): a head
+    (z the H columns from ``a_col``; lg [n, H]) or, ``per_channel``, a key channel (lg [n, H D] holds z and is changed in place).
+    ``kept`` and ``single_rows`` as in :func:`ssm_conv`."""
+    _need(p, "p", contiguous=False); _need(kept, "kept", torch.float32, contiguous=False)
+    for t, nm in ((taps, "taps"), (neg_a, "neg_a"), (dt_bias, "dt_bias"), (out, "out"), (beta, "beta"), (lg, "lg")):
+        _need(t, nm, torch.float32)
+    for t, nm in ((row_seg, "row_seg"), (cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (seg_slot, "seg_slot")):
+        _need(t, nm, torch.int32)
+    n, C, K = p.shape[0], 2 * G * D + H * P, taps.shape[1]
+    n_dec = H * D if per_channel else H
+    if (tuple(out.shape) != (n, C) or tuple(taps.shape) != (C, K) or neg_a.numel() != H or dt_bias.numel() != n_dec
+            or tuple(beta.shape) != (n, H) or tuple(lg.shape) != (n, n_dec) or conv_col + C > p.shape[1] or b_col + H > p.shape[1]
+            or (not per_channel and a_col + H > p.shape[1]) or kept.dim() != 2 or kept.stride(1) != 1 or kept.shape[1] < (K - 1) * C):
+        raise KernelError("delta_prep: shape mismatch")
+    if K > RECUR_MAX_TAPS or D > RECUR_MAX_DIM:
+        raise KernelError(f"delta_prep: {K} taps or heads of {D} exceed {RECUR_MAX_TAPS} or {RECUR_MAX_DIM}")
+    _run("delta_prep", load_library("recurrence").kp_delta_prep, _ptr(p), _rows_2d(p, "p"), int(conv_col), int(b_col), int(a_col), _ptr(taps),
+         _ptr(neg_a), _ptr(dt_bias), _ptr(kept), ctypes.c_longlong(kept.stride(0)), _ptr(row_seg), _ptr(cu_rows), _ptr(seg_pos),
+         _ptr(seg_slot), _ptr(out), _ptr(beta), _ptr(lg), n, int(n_seg), H, G, D, P, K, ctypes.c_float(q_scale), int(bool(per_channel)),
+         int(bool(single_rows)), int(bool(keep)), dtype_code(p.dtype), STREAM, work=(0, n * C * (p.element_size() + 4)))
+    if keep and not single_rows and K > 1:
+        LAUNCHES[0] += 1
+
+
+def log_decay_sigmoid(z: torch.Tensor, tau: float) -> torch.Tensor:
+    """z <- log(sigmoid(z)^(1 / tau)), in place, float32."""
+    _need(z, "z", torch.float32)
+    _run("log_decay_sigmoid", load_library("recurrence").kp_log_decay_sigmoid, _ptr(z), ctypes.c_longlong(z.numel()),
+         ctypes.c_float(1.0 / float(tau)), STREAM, work=(0, 8 * z.numel()))
+    return z
+
+
+def _recur_check(what, q, k, v, lg, beta, state, out, H, G, D, P, per_channel):
+    for t, nm in ((q, "q"), (k, "k"), (v, "v")):
+        _need(t, nm, q.dtype, contiguous=False)
+    _need(lg, "lg", torch.float32); _need(out, "out", torch.float32); _need(state, "state", torch.float32, contiguous=False)
+    n = q.shape[0]
+    if (q.stride(0) != k.stride(0) or q.stride(0) != v.stride(0) or tuple(q.shape) != (n, G * D) or tuple(k.shape) != (n, G * D)
+            or tuple(v.shape) != (n, H * P) or H % G or tuple(lg.shape) != (n, H * D if per_channel else H)
+            or tuple(out.shape) != (n, H * P) or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < H * D * P):
+        raise KernelError(f"{what}: shape mismatch")
+    if beta is not None:
+        _need(beta, "beta", torch.float32)
+        if tuple(beta.shape) != (n, H):
+            raise KernelError(f"{what}: beta's shape")
+        if q.dtype != torch.float32:
+            raise KernelError(f"{what}: the delta recurrence reads float32 vectors (what delta_prep leaves)")
+    elif not per_channel:
+        raise KernelError(f"{what}: the gated recurrence has one decay a key channel")
+    if D > RECUR_MAX_DIM:
+        raise KernelError(f"{what}: heads of {D} exceed {RECUR_MAX_DIM}")
+    return n
+
+
+def recur_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, lg: torch.Tensor, beta: Optional[torch.Tensor], q_scale: float,
+               state: torch.Tensor, cu_rows: torch.Tensor, seg_pos: torch.Tensor, seg_slot: torch.Tensor, out: torch.Tensor,
+               n_seg: int, H: int, G: int, D: int, P: int, per_channel: bool, write_state: bool = True) -> torch.Tensor:
+    """``S <- exp(lg) S; u = beta (v - S^T k), or v without ``beta``; S <- S + k u^T; o = S^T (q_scale q)`` row after row of
+    every segment, from the state in the segment's slot (zero at position 0) and back into it.  ``q``, ``k`` [n, G D] and ``v``
+    [n, H P] are columns of rows of one pitch; ``lg`` float32 [n, H], or with ``per_channel`` [n, H D]; ``state``
+    float32 [slots, stride] whose rows begin with [H, D, P]; ``out`` float32 [n, H P]."""
+    n = _recur_check("recur_scan", q, k, v, lg, beta, state, out, H, G, D, P, per_channel)
+    for t, nm in ((cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (seg_slot, "seg_slot")):
+        _need(t, nm, torch.int32)
+    _run("recur_scan", load_library("recurrence").kp_recur_scan, _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(lg), _ptr(beta),
+         ctypes.c_float(q_scale), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(cu_rows), _ptr(seg_pos), _ptr(seg_slot), _ptr(out),
+         _rows_2d(out, "out"), int(n_seg), H, G, D, P, int(bool(per_channel)), int(bool(write_state)), dtype_code(q.dtype), STREAM,
+         tag=f" {'delta' if beta is not None else 'gated'}", work=((6 if beta is not None else 4) * n * H * D * P, 8 * n_seg * H * D * P))
+    return out
+
+
+def recur_chunk_rows() -> int:
+    return int(load_library("recurrence").kp_recur_chunk_rows())
+
+
+def recur_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, lg: torch.Tensor, beta: Optional[torch.Tensor], q_scale: float,
+                 state: torch.Tensor, cu_rows: torch.Tensor, seg_pos: torch.Tensor, seg_slot: torch.Tensor, chunk_seg: torch.Tensor,
+                 chunk_row0: torch.Tensor, seg_chunk0: torch.Tensor, n_chunks: int, out: torch.Tensor, n_seg: int, H: int, G: int,
+                 D: int, P: int, per_channel: bool, write_state: bool = True) -> torch.Tensor:
+    """The recurrence of :func:`recur_scan` for segments of many rows: chunks of rows as small matrix products (tensor
+    cores, tf32 with both operands in two parts), in three passes (see csrc/recurrence.cu).  The chunk lists as in
+    :func:`lightning_chunks`.  Sums have another order than the scan's."""
+    n = _recur_check("recur_chunks", q, k, v, lg, beta, state, out, H, G, D, P, per_channel)
+    for t, nm in ((cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (seg_slot, "seg_slot"), (chunk_seg, "chunk_seg"),
+                  (chunk_row0, "chunk_row0"), (seg_chunk0, "seg_chunk0")):
+        _need(t, nm, torch.int32)
+    if chunk_seg.numel() < n_chunks or chunk_row0.numel() < n_chunks or seg_chunk0.numel() < n_seg + 1:
+        raise KernelError("recur_chunks: chunk lists too short")
+    lib = load_library("recurrence")
+    lib.kp_recur_chunks_scratch.restype = ctypes.c_longlong
+    scratch = torch.empty(int(lib.kp_recur_chunks_scratch(int(n_chunks), H, D, P, int(beta is not None))), dtype=torch.float32,
+                          device=q.device)
+    _run("recur_chunks", lib.kp_recur_chunks, _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(lg), _ptr(beta), ctypes.c_float(q_scale),
+         _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(cu_rows), _ptr(seg_pos), _ptr(seg_slot), _ptr(chunk_seg), _ptr(chunk_row0),
+         _ptr(seg_chunk0), int(n_chunks), _ptr(scratch), _ptr(out), _rows_2d(out, "out"), int(n_seg), H, G, D, P, int(bool(per_channel)),
+         int(bool(write_state)), dtype_code(q.dtype), STREAM, tag=f" {'delta' if beta is not None else 'gated'}",
+         work=((6 if beta is not None else 4) * n * H * D * P, 0))
+    LAUNCHES[0] += 2
+    return out
+
+
+# ------------------------------------------------------------------ a residual of several streams
+
+STREAMS_MAX = 8
+
+
+def streams_enter(e: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
+    """x[r, s] = e[r] for every stream s: ``e`` float32 [n, d], ``x`` float32 [n, S, d]."""
+    _need(e, "e", torch.float32); _need(x, "x", torch.float32)
+    n, S, d = x.shape
+    if tuple(e.shape) != (n, d):
+        raise KernelError("streams_enter: shape mismatch")
+    _run("streams_enter", load_library("streams").kp_streams_enter, _ptr(e), _ptr(x), n, d, S, STREAM)
+    return x
+
+
+def streams_rows(x: torch.Tensor, y: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                 out_w: Optional[torch.Tensor] = None, in_w: Optional[torch.Tensor] = None, norm_w: Optional[torch.Tensor] = None,
+                 eps: float = 0.0, centred: bool = True, h: Optional[torch.Tensor] = None,
+                 rows: Optional[torch.Tensor] = None) -> None:
+    """One pass over rows of several streams, ``x`` float32 [n, S, d].  With ``y`` (float32 [n, d], left cleared):
+    ``x_t <- sum_s mix[s, t] x_s + out_w[t] y``.  With ``h`` ([rows, d] in the storage type): ``h = norm(sum_t in_w[t] x_t) *
+    norm_w`` of the new streams (``in_w`` None: their sum), the norm centred (a layer norm without a shift) or the RMS
+    norm.  ``rows`` (without ``y``): the rows to read."""
+    _need(x, "x", torch.float32)
+    n, S, d = x.shape
+    if S > STREAMS_MAX:
+        raise KernelError(f"streams_rows: {S} streams exceed {STREAMS_MAX}")
+    if y is not None:
+        for t, nm, size in ((y, "y", n * d), (mix, "mix", S * S), (out_w, "out_w", S)):
+            _need(t, nm, torch.float32)
+            if t.numel() != size:
+                raise KernelError(f"streams_rows: size of {nm}")
+        if rows is not None:
+            raise KernelError("streams_rows: picked rows are read, not changed")
+    if h is not None:
+        _need(h, "h"); _need(norm_w, "norm_w", torch.float32)
+        if rows is not None:
+            _need(rows, "rows", torch.int32)
+        n_out = n if rows is None else rows.numel()
+        if tuple(h.shape) != (n_out, d) or norm_w.numel() != d:
+            raise KernelError("streams_rows: shape mismatch")
+        if in_w is not None:
+            _need(in_w, "in_w", torch.float32)
+            if in_w.numel() != S:
+                raise KernelError("streams_rows: size of in_w")
+    elif y is None or rows is not None:
+        raise KernelError("streams_rows: nothing to do")
+    n_rows = n if rows is None else rows.numel()
+    if n_rows > MAX_STEP_ROWS:
+        raise KernelError("streams_rows: too many rows")
+    _run("streams_rows", load_library("streams").kp_streams_rows, _ptr(x), _ptr(y), _ptr(mix), _ptr(out_w), _ptr(in_w), _ptr(norm_w),
+         ctypes.c_float(eps), int(bool(centred)), _ptr(rows), _ptr(h), n_rows, d, S, dtype_code(h.dtype if h is not None else torch.float32),
+         STREAM, work=(0, n_rows * d * (4 * S * (2 if y is not None else 1) + (8 if y is not None else 0)
+                                        + (h.element_size() if h is not None else 0))))
 
 
 # ------------------------------------------------------------------ attention

@@ -43,12 +43,18 @@ sequence stay visible to every later row, at their true places, and their pages 
 ``value_dim`` of its own: the norm's mean is then taken over ``head_dim`` columns of the wider cache head.  An odd
 ``head_dim`` without a position encoding is stored wider in the same way.
 
+``conv_kernel`` (taps; default 0, none): q, k and v each pass a causal convolution a channel over time, right behind the
+projection and its bias and before the norm and the rotation (tensors ``q_conv.weight`` and so on, [channels, taps], the
+last tap on the current token, no bias); their last ``conv_kernel - 1`` projected values are state in the request's slot
+beside the paged keys and values.  ``out_scale`` (default 1) multiplies the mixer's output; the values' taps and the
+output bias carry it, so it goes with ``conv_kernel``.
+
 Sizes and constants (params): hidden_size, num_heads, num_kv_heads, head_dim,
 value_dim, scale, qk_norm_eps (None: no q/k norm), qk_norm ("per_head" |
 "projection"), window (None: all keys), cache_window, block (None), values
 ("projection" | "keys"), kv ("own" | "borrowed"), gate (None | "sigmoid" |
 "head_sigmoid"), softmax_weights ("operand" | "float32"), position (a
-``position`` PartSpec), bias, keep_first, sink (None | "zero" | "learned"), q_temp.
+``position`` PartSpec), bias, keep_first, sink (None | "zero" | "learned"), q_temp, conv_kernel, out_scale.
 """
 from __future__ import annotations
 
@@ -57,7 +63,7 @@ from typing import Dict, Optional
 import numpy as np
 import torch
 
-from ..cache.spec import PagedKVSpec
+from ..cache.spec import CompositeSpec, PagedKVSpec, StateSpec
 from ..config.schema import ConfigError, PartSpec
 from ..ops import kernels as K
 from ..ops.linear import linear
@@ -260,8 +266,8 @@ class Attention(PagedAttentionKernels, Part):
         pos_given = self._p("position", None) is not None
         if self.qk_norm == "projection" or self.vdim != self.dim or (self.dim % 2 and not pos_given):
             # (an odd head size without a rotation is stored wider too: the kernels take even sizes)
-            if self.values_are_keys or self.bias:
-                raise ConfigError("attention: values='keys' and biases want value_dim = head_dim and the per-head norm")
+            if self.values_are_keys or (self.bias and self.qk_norm == "projection"):
+                raise ConfigError("attention: values='keys' wants value_dim = head_dim; it and biases want the per-head norm")
             if min(self.dim, self.vdim) < 1:
                 raise ConfigError("attention: head sizes must be positive")
             self.hd = -(-max(self.dim, self.vdim) // 16) * 16
@@ -296,6 +302,14 @@ class Attention(PagedAttentionKernels, Part):
             raise ConfigError("attention: values='keys' needs a position encoding that runs in the fused q/k kernel")
         if self.qk_norm == "projection" and (not hasattr(self.position, "fused_rotary") or self.position.fused_rotary()[2]):
             raise ConfigError("attention: qk_norm='projection' runs without a rotation")
+        self.taps = int(self._p("conv_kernel", 0) or 0)
+        self.out_scale = float(self._p("out_scale", 1.0))
+        if not (0 <= self.taps <= K.SSM_MAX_TAPS):
+            raise ConfigError(f"attention: conv_kernel={self.taps} outside 0..{K.SSM_MAX_TAPS}")
+        if self.taps and (self.values_are_keys or self.borrows):
+            raise ConfigError("attention: conv_kernel wants key and value matrices of the mixer's own")
+        if self.out_scale != 1.0 and not self.taps:
+            raise ConfigError("attention: out_scale is carried by the values' convolution (conv_kernel)")
         self._tile_setup()
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -317,9 +331,11 @@ class Attention(PagedAttentionKernels, Part):
         if self.sink == "learned":
             s["sink"] = WeightSpec((H,), "bias")
         if self.bias:
-            hd = self.hd                      # (biases go with value_dim = head_dim)
-            for n, sz in (("q_proj", H * hd), ("k_proj", G * hd), ("v_proj", G * hd), ("out_proj", d)):
+            for n, sz in (("q_proj", H * self.dim), ("k_proj", G * self.dim), ("v_proj", G * self.vdim), ("out_proj", d)):
                 s[n + ".bias"] = WeightSpec((sz,), "bias")
+        if self.taps:
+            for n, sz in (("q", H * self.dim), ("k", G * self.dim), ("v", G * self.vdim)):
+                s[n + "_conv.weight"] = WeightSpec((sz, self.taps), "conv")
         return s
 
     def _pad_heads(self, w, heads, width):
@@ -351,8 +367,16 @@ class Attention(PagedAttentionKernels, Part):
         self.w_o = self._pad_heads(w["out_proj.weight"].t().contiguous(), H, self.vdim).t().contiguous()
         self.b_qkv = self.b_o = None
         if self.bias:
-            self.b_qkv = torch.cat([w[n + ".bias"].float() for n in ("q_proj", "k_proj", "v_proj")]).contiguous()
-            self.b_o = w["out_proj.bias"].float().contiguous()
+            b = [self._pad_heads(w[n + ".bias"].float(), heads, width)
+                 for n, heads, width in (("q_proj", H, self.dim), ("k_proj", G, self.dim), ("v_proj", G, self.vdim))]
+            b.append(torch.zeros(self.w_qkv.shape[0] - sum(x.shape[0] for x in b), dtype=torch.float32, device=self.w_qkv.device))
+            self.b_qkv = torch.cat(b).contiguous()
+            self.b_o = (w["out_proj.bias"].float() * self.out_scale).contiguous()
+        self.conv_w = None
+        if self.taps:
+            self.conv_w = torch.cat([self._pad_heads(w["q_conv.weight"].float(), H, self.dim),
+                                     self._pad_heads(w["k_conv.weight"].float(), G, self.dim),
+                                     self._pad_heads(w["v_conv.weight"].float() * self.out_scale, G, self.vdim)], 0).contiguous()
         self.q_w = self.k_w = None
         if self.qk_norm == "projection":
             self.q_w = self._pad_heads(w["q_norm.weight"].float(), H, self.dim)
@@ -366,14 +390,39 @@ class Attention(PagedAttentionKernels, Part):
 
     def cache_spec(self):
         # (a borrower names what it reads, so that the engine can see that lender and borrower agree)
-        return PagedKVSpec(self.G, self.hd, self.cache_window, None if self.block is None else int(self.block),
-                           self.keep_first if self.cache_window is not None else 0)
+        kv = PagedKVSpec(self.G, self.hd, self.cache_window, None if self.block is None else int(self.block),
+                         self.keep_first if self.cache_window is not None else 0)
+        if self.taps < 2:
+            return kv
+        return CompositeSpec((kv, StateSpec(((self.taps - 1) * (self.H + 2 * self.G) * self.hd,), "float32")))
+
+    def input_product(self):
+        return self.w_qkv, self.b_qkv
+
+    def drop_input_product(self):
+        self.w_qkv = self.b_qkv = None
 
     def forward(self, h, residual, ctx, cache):
-        """``cache``: a :class:`~kappai_b200.cache.storage.KVLayerView`."""
+        """``cache``: a :class:`~kappai_b200.cache.storage.KVLayerView` (with a convolution of two taps or more, that and the
+        :class:`~kappai_b200.cache.storage.StateView` of its kept inputs)."""
+        self.forward_projected(linear(h, self.w_qkv, self.b_qkv), residual, ctx, cache)
+
+    def _convolve(self, qkv, ctx, kept, keep):
+        """q, k and v behind their convolutions; the columns behind them (a gate) stay where they are."""
+        out = torch.empty((ctx.n_rows, (self.H + 2 * self.G) * self.hd), dtype=qkv.dtype, device=qkv.device)
+        return K.channel_conv(qkv, 0, self.conv_w, kept, ctx.row_seg, ctx.cu_rows, ctx.seg_pos, ctx.seg_slot, out, ctx.n_seg,
+                              ctx.decode_only, keep)
+
+    def forward_projected(self, qkv, residual, ctx, cache):
+        """``qkv``: the rows of the input product (``input_product``), possibly columns of a wider one."""
         H, G, hd = self.H, self.G, self.hd
+        proj = qkv
+        if self.taps > 1:
+            cache, conv = cache.parts
+            qkv = self._convolve(qkv, ctx, conv.tensor, conv.writes)
+        elif self.taps == 1:
+            qkv = self._convolve(qkv, ctx, torch.empty((1, 1), dtype=torch.float32, device=qkv.device), False)
         view = ctx.paged[cache.group]
-        qkv = linear(h, self.w_qkv, self.b_qkv)
         q = torch.empty((ctx.n_rows, H * hd), dtype=qkv.dtype, device=qkv.device)
         kv_out = cache.tensor if cache.writes else None
         if self.borrows and cache.writes:
@@ -396,9 +445,9 @@ class Attention(PagedAttentionKernels, Part):
                               view.page_size, H, G, hd)
         o = self._attend(q, ctx, view, cache)
         if self.head_gate:
-            K.head_gate(o, qkv[:, self.gate_col:self.gate_col + H], H, hd)
+            K.head_gate(o, proj[:, self.gate_col:self.gate_col + H], H, hd)
         elif self.gated:
-            K.sigmoid_gate(o, qkv[:, self.gate_col:self.gate_col + H * hd])
+            K.sigmoid_gate(o, proj[:, self.gate_col:self.gate_col + H * hd])
         linear(o, self.w_o, self.b_o, out=residual, accumulate=True)
 
 

@@ -30,6 +30,13 @@ any             optionally ``step_tables_key`` and ``step_tables(segs)``: int32
 ``entry``         ``forward(x, h0)`` -> the new residual at the head of a
                   schedule entry marked ``enter`` (``h0``: the embedding output
                   in the compute type).
+``residual``      how the residual is kept between the layers where it is not one
+                  float32 row: ``enter(x)`` makes it of the embedding output,
+                  ``rows(x)`` gives the float32 rows it stands for (for an
+                  observer), ``normed(x, norm, rows=None)`` norms picked rows of
+                  those.
+
+A mixer made of other parts lists them in ``inner_parts``.
 """
 from __future__ import annotations
 
@@ -46,11 +53,16 @@ class WeightSpec:
     """One tensor a part binds.  ``role`` picks the random-weights
     distribution and the storage dtype of a written model folder:
     ``matrix`` / ``embedding`` (bfloat16), ``norm`` / ``conv`` / ``bias``
-    (float32)."""
+    (float32), ``stream`` (float32).  A size of -1 is taken from the weight file
+    (``free``: the size that random weights give it)."""
 
     shape: Tuple[int, ...]
     role: str = "matrix"
     optional: bool = False
+    free: int = 16
+
+    def fits(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(w in (-1, n) for w, n in zip(self.shape, shape))
 
 
 @dataclass
@@ -67,6 +79,7 @@ class Part:
     # its host_* lists or other host values that change from step to step): such a part can be captured
     # in a CUDA graph.  Parts registered from outside are not assumed to be.
     graph_safe = False
+    inner_parts = ()           # the parts that a part is made of, if any
 
     def __init__(self, params: Dict[str, Any], env: BuildEnv):
         self.params = dict(params)
@@ -101,7 +114,7 @@ class Part:
 
 
 _REGISTRY: Dict[Tuple[str, str], Callable[..., Part]] = {}
-CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "side", "entry")
+CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "side", "entry", "residual")
 
 
 def register_part(category: str, kind: str, factory: Callable[..., Part], *, replace: bool = False) -> None:
@@ -138,4 +151,4 @@ def _ensure_builtin() -> None:
     global _builtin
     if not _builtin:
         _builtin = True
-        from . import norm, position, attention, shortconv, lightning, ssm, ffn, block, embedding, side  # noqa: F401
+        from . import norm, position, attention, shortconv, lightning, ssm, gated, parallel, ffn, block, embedding, side, streams  # noqa: F401

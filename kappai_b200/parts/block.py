@@ -25,13 +25,23 @@ one kernel norms the branch, adds it to the residual, clears the branch for
 its next use and, where another norm follows at once (the feed-forward's, or
 the first norm of the layer that runs next), norms the new residual for it in
 the same pass.
+
+``streams_residual``: the residual is several float32 streams a row (streams.py).
+A sublayer reads ``norm(sum_t in[t] x_t)`` and its output y joins every stream
+while the streams are mixed, ``x_t <- sum_s mix[s, t] x_s + out[t] y``; mixer
+and feed-forward each with coefficients of their own (``hc1``, ``hc2``:
+``in`` [streams], ``out`` [streams], ``mix`` [streams, streams], indexed from,
+to).  As above a sublayer adds into a zeroed float32 branch, and one kernel
+reads the branch, changes the streams, clears the branch and norms the weighted
+sum that the next sublayer reads (of this layer or the one that runs next).
 """
 from __future__ import annotations
 
 import torch
 
 from ..ops import kernels as K
-from .base import Part, register_part
+from .base import Part, WeightSpec, register_part
+from .streams import stream_norm
 
 
 class PreNormResidualBlock(Part):
@@ -124,6 +134,16 @@ class ParallelResidualBlock(Part):
             self.side.forward(x, ctx)
 
 
+def branch_rows(n, d, ctx, device):
+    """The float32 rows a sublayer adds its output into: one zeroed buffer a step, shared by the layers (the
+    kernel that reads a branch clears it)."""
+    y = getattr(ctx, "branch_buffer", None)
+    if y is None or tuple(y.shape) != (n, d):
+        y = torch.zeros((n, d), dtype=torch.float32, device=device)
+        ctx.branch_buffer = y
+    return y
+
+
 class SandwichResidualBlock(Part):
     category = "block"
     graph_safe = True
@@ -138,18 +158,8 @@ class SandwichResidualBlock(Part):
         self.mixer_post_norm, self.ffn_post_norm = p1, p2
         return self
 
-    @staticmethod
-    def _branch(x, ctx):
-        """The float32 rows a sublayer adds its output into: one zeroed buffer a step, shared by the layers (the
-        kernel that reads a branch clears it)."""
-        y = getattr(ctx, "sandwich_branch", None)
-        if y is None or y.shape != x.shape:
-            y = torch.zeros_like(x)
-            ctx.sandwich_branch = y
-        return y
-
     def forward(self, x, ctx, cache):
-        y = self._branch(x, ctx)
+        y = branch_rows(x.shape[0], x.shape[1], ctx, x.device)
         # the input of this layer's mixer: left by the layer before for this very residual, or made here
         carry = getattr(ctx, "sandwich_carry", None)
         ctx.sandwich_carry = None
@@ -179,6 +189,68 @@ class SandwichResidualBlock(Part):
             self.side.forward(x, ctx)
 
 
+class StreamsResidualBlock(Part):
+    category = "block"
+    graph_safe = True
+
+    def __init__(self, params, env):
+        super().__init__(params, env)
+        self.S = int(self._p("streams"))
+        self.sublayers = int(self._p("sublayers", 2))           # 1: a layer without a feed-forward
+
+    def weight_specs(self):
+        S = self.S
+        return {f"hc{q}.{n}": WeightSpec(shape, "stream") for q in range(1, self.sublayers + 1)
+                for n, shape in (("in", (S,)), ("out", (S,)), ("mix", (S, S)))}
+
+    def bind(self, w):
+        self.hc = [{n: w[f"hc{q}.{n}"].float().contiguous() for n in ("in", "out", "mix")} for q in range(1, self.sublayers + 1)]
+
+    def assemble(self, mixer, ffn, mixer_norm, ffn_norm, side=None):
+        if side is not None:
+            raise ValueError("streams_residual: no side part in this arrangement")
+        if self.sublayers != (1 if ffn is None else 2):
+            raise ValueError("streams_residual: coefficients for every sublayer the layer has, and no more")
+        self.mixer, self.ffn, self.mixer_norm, self.ffn_norm, self.side = mixer, ffn, mixer_norm, ffn_norm, None
+        self.centred = [stream_norm(n) for n in (mixer_norm, ffn_norm)[:self.sublayers]]
+        return self
+
+    def _step(self, x, y, q, nxt, j, last):
+        """Sublayer q's output y joins the streams; the normed input of block ``nxt``'s sublayer j leaves (unless ``last``)."""
+        hc = self.hc[q]
+        if last:
+            K.streams_rows(x, y, hc["mix"], hc["out"])
+            return None
+        norm = (nxt.mixer_norm, nxt.ffn_norm)[j]
+        h = torch.empty((x.shape[0], x.shape[2]), dtype=self.env.dtype, device=x.device)
+        K.streams_rows(x, y, hc["mix"], hc["out"], nxt.hc[j]["in"], norm.weight, norm.eps, nxt.centred[j], h)
+        return h
+
+    def forward(self, x, ctx, cache):
+        """``x``: float32 [rows, streams, hidden]."""
+        y = branch_rows(x.shape[0], x.shape[2], ctx, x.device)
+        carry = getattr(ctx, "streams_carry", None)
+        ctx.streams_carry = None
+        if carry is not None and carry[0] is x and carry[1] is self:
+            h = carry[2]
+        else:
+            h = torch.empty((x.shape[0], x.shape[2]), dtype=self.env.dtype, device=x.device)
+            n1 = self.mixer_norm
+            K.streams_rows(x, in_w=self.hc[0]["in"], norm_w=n1.weight, eps=n1.eps, centred=self.centred[0], h=h)
+        self.mixer.forward(h, y, ctx, cache)
+        q = 0
+        if self.ffn is not None:
+            h = self._step(x, y, 0, self, 1, False)
+            self.ffn.forward(h, y, ctx)
+            q = 1
+        nxt = getattr(ctx, "next_block", None)
+        follows = isinstance(nxt, StreamsResidualBlock) and nxt.S == self.S
+        h = self._step(x, y, q, nxt, 0, not follows)
+        if follows:
+            ctx.streams_carry = (x, nxt, h)
+
+
+register_part("block", "streams_residual", StreamsResidualBlock)
 register_part("block", "sandwich_residual", SandwichResidualBlock)
 register_part("block", "prenorm_residual", PreNormResidualBlock)
 register_part("block", "parallel_residual", ParallelResidualBlock)

@@ -11,7 +11,8 @@ may be smaller than the head size (the rest of the head is left as it is).
 frequencies by their wavelength ``l = 2 pi / f``: a frequency with
 ``l < original / high`` is kept, one with ``l > original / low`` is divided by
 ``factor``, and between the two, with ``s = (original / l - low) / (high - low)``,
-it becomes ``(1 - s) f / factor + s f``.
+it becomes ``(1 - s) f / factor + s f``.  With the key ``factor`` alone every
+frequency is divided by it.
 
 ``none``: no rotation.
 """
@@ -26,9 +27,11 @@ from .base import Part, register_part
 
 def scaled_frequencies(f: np.ndarray, scaling) -> np.ndarray:
     """Rotary frequencies rescaled by wavelength (see the module's text); ``scaling`` is
-    (factor, low, high, original) or None."""
+    (factor, low, high, original), (factor,) or None."""
     if scaling is None:
         return f
+    if len(scaling) == 1:
+        return f / scaling[0]
     factor, low, high, original = scaling
     lam = 2.0 * np.pi / f
     s = (original / lam - low) / (high - low)
@@ -52,7 +55,11 @@ class RotaryEncoding(Part):
         self.interleaved = pairing == "interleaved"
         scaling = self._p("scaling", None)
         self.scaling = None
-        if scaling:
+        if scaling and set(scaling) == {"factor"}:
+            self.scaling = (float(scaling["factor"]),)
+            if not self.scaling[0] > 0:
+                raise ConfigError("rope: scaling wants factor > 0")
+        elif scaling:
             try:
                 self.scaling = tuple(float(scaling[k]) for k in ("factor", "low", "high", "original"))
             except (KeyError, TypeError, ValueError):

@@ -67,7 +67,7 @@ def load_weights(model, model_dir: str) -> None:
         for n, ws in table.items():
             if n in where:
                 _, shape = where[n].info(n)
-                if tuple(shape) != tuple(ws.shape):
+                if not ws.fits(tuple(shape)):
                     wrong.append(f"{n}: file has {list(shape)}, model wants {list(ws.shape)}")
         if missing or unexpected or wrong:
             lines = [f"{model_dir}: the weight files do not fit the model"]

@@ -6,7 +6,8 @@ and the tensor's name, so a tensor's values do not depend on which other
 tensors exist or in what order they are made.  Distributions by role:
 matrices and embeddings N(0, 0.02), stored in bfloat16; norm weights
 1 + N(0, 0.1); convolution weights U(-1/sqrt(3), 1/sqrt(3)); biases N(0, 0.02);
-these three stored in float32.  (The reference has random weights only in its
+stream coefficients about the mean of the streams (a vector) or the identity (a
+matrix); these four stored in float32.  (The reference has random weights only in its
 tests: src/test/test_synth_gguf.c:50-68,349-460.)
 """
 from __future__ import annotations
@@ -41,6 +42,9 @@ def random_tensor(seed: int, name: str, shape, role: str) -> torch.Tensor:
         return torch.from_numpy(g.uniform(-b, b, shape).astype(np.float32))
     if role == "bias":
         return torch.from_numpy(g.standard_normal(shape, dtype=np.float32) * np.float32(0.02))
+    if role == "stream":
+        base = np.eye(shape[0]) if len(shape) == 2 else np.full(shape, 1.0 / shape[0])
+        return torch.from_numpy((base + 0.05 * g.standard_normal(shape)).astype(np.float32))
     raise ValueError(f"no random distribution for tensor role '{role}'")
 
 
@@ -50,7 +54,8 @@ def random_weights(config_dict: Dict[str, Any], seed: int) -> Dict[str, torch.Te
     arch, cfg = config_from_dict(config_dict)
     spec = arch.build_spec(cfg)
     model = Model(spec, BuildEnv(torch.device("cpu"), torch.float32, max_positions=1))
-    return {name: random_tensor(seed, name, ws.shape, ws.role) for name, ws in model.weight_table().items()}
+    return {name: random_tensor(seed, name, tuple(ws.free if n < 0 else n for n in ws.shape), ws.role)
+            for name, ws in model.weight_table().items()}
 
 
 def write_random_model(config_dict: Dict[str, Any], out_dir: str, seed: int) -> str:
