@@ -71,13 +71,17 @@ delta_prep_kernel(const T* __restrict__ p, int ld, int conv_col, int b_col, int 
     const int seg = row_seg[r], row0 = cu_rows[seg];
     const bool fresh = seg_pos[seg] == 0;
     float* kp = kept + (size_t)seg_slot[seg] * slot_stride;
+    // (lane l keeps channels 4 l .. 4 l + 3 where heads are a multiple of 4 wide, so that a head's sum of squares is added in the
+    // order of the other form below)
+    const bool quads = D % 4 == 0;
+    auto place = [&](int j) { return quads ? (j >> 2) * 128 + lane * 4 + (j & 3) : lane + 32 * j; };
     float y[8];
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < 8; j++) {
         y[j] = 0.f;
-        const int c = base + lane + 32 * j;
-        if (lane + 32 * j >= count) continue;
+        const int c = base + place(j);
+        if (place(j) >= count) continue;
         float acc = 0.f;
         for (int m = 0; m < K; m++) {
             const int rr = r - (K - 1) + m;
@@ -100,7 +104,7 @@ delta_prep_kernel(const T* __restrict__ p, int ld, int conv_col, int b_col, int 
     float* dst = out + (size_t)r * C + base;
 #pragma unroll
     for (int j = 0; j < 8; j++)
-        if (lane + 32 * j < count) dst[lane + 32 * j] = y[j] * scale;
+        if (place(j) < count) dst[place(j)] = y[j] * scale;
 }
 
 // The same for steps of several rows where heads are multiples of 4 wide and rows start on 8 (16) bytes: a lane takes four

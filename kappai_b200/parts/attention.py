@@ -41,7 +41,7 @@ sequence stay visible to every later row, at their true places, and their pages 
 ``q_temp`` = {coef, every}: the query of position p is multiplied by
 ``1 + coef ln(floor((p + 1) / every) + 1)`` (float32, in the fused q/k kernel).  The per-head q/k norm goes with a
 ``value_dim`` of its own: the norm's mean is then taken over ``head_dim`` columns of the wider cache head.  An odd
-``head_dim`` without a position encoding is stored wider in the same way.
+``head_dim`` is stored wider in the same way (with a rotation only where there is no q/k norm).
 
 ``conv_kernel`` (taps; default 0, none): q, k and v each pass a causal convolution a channel over time, right behind the
 projection and its bias and before the norm and the rotation (tensors ``q_conv.weight`` and so on, [channels, taps], the
@@ -263,9 +263,11 @@ class Attention(PagedAttentionKernels, Part):
         # dim, vdim: the heads as the model has them; hd: as the cache and the kernels see them
         self.dim = self.hd
         self.vdim = int(self._p("value_dim", self.dim))
-        pos_given = self._p("position", None) is not None
-        if self.qk_norm == "projection" or self.vdim != self.dim or (self.dim % 2 and not pos_given):
-            # (an odd head size without a rotation is stored wider too: the kernels take even sizes)
+        pos = self._p("position", None)
+        kind = None if pos is None else (pos["kind"] if isinstance(pos, dict) else pos.kind)
+        odd_ok = kind in (None, "none") or (kind == "rope" and self.qk_norm_eps is None)
+        if self.qk_norm == "projection" or self.vdim != self.dim or (self.dim % 2 and odd_ok):
+            # (an odd head size is stored wider too: the kernels take even sizes, and rotate a head's first dimensions only)
             if self.values_are_keys or (self.bias and self.qk_norm == "projection"):
                 raise ConfigError("attention: values='keys' wants value_dim = head_dim; it and biases want the per-head norm")
             if min(self.dim, self.vdim) < 1:
@@ -278,7 +280,6 @@ class Attention(PagedAttentionKernels, Part):
         if self.hd % 2 or not (2 <= self.hd <= 256):
             raise ConfigError(f"attention: head_dim={self.dim} is not supported by the kernels "
                               "(an even number from 2 to 256)")
-        pos = self._p("position", None)
         if pos is None:
             pos = PartSpec("none")
         elif isinstance(pos, dict):

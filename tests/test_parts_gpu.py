@@ -47,10 +47,10 @@ class Batch:
     """Several requests, each cut in two steps; builds StepContexts through the real cache manager."""
 
     def __init__(self, specs, lens, cuts, page, dtype):
-        from kappai_b200.cache import CacheManager, PagedKVSpec
+        from kappai_b200.cache import CacheManager, PagedKVSpec, leaf_specs
         from kappai_b200.cache.storage import CacheStorage
         self.lens, self.cuts, self.page = lens, cuts, page
-        gks = {s.group_key: s for s in specs if isinstance(s, PagedKVSpec)}
+        gks = {s.group_key: s for spec in specs for s in leaf_specs(spec) if isinstance(s, PagedKVSpec)}
         n_pages = sum(-(-L // page) for L in lens) + 2
         self.storage = CacheStorage(specs, [None] * len(specs), {g: n_pages for g in gks}, page, len(lens) + 1,
                                     dtype, torch.device("cuda:0"))
