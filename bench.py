@@ -479,6 +479,26 @@ def vumotar_config(width, H, G, hd, E, top, ff_e):
                        for t, m in (("attention", att), ("attention_2", att2), ("latent_attention", latent))]}
 
 
+GOSULORN_WINDOW = 1024
+GOSULORN_STREAMS = 4
+
+
+def gosulorn_config(width, H, G, hd, ff):
+    """Four layers of the sizes of the other designs': the gated delta rule (half as many query/key heads), gated linear
+    attention, the two mixers side by side, and the delta layer's tensors run again; four streams."""
+    delta = {"heads": H, "kv_heads": max(1, H // 2), "dim": hd, "vdim": hd, "conv": 4}
+    gla = {"heads": H, "dim": hd, "vdim": hd, "tau": 16.0}
+    left = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "conv": 3, "scale": hd ** -0.5, "mask": {"size": GOSULORN_WINDOW},
+            "rot": {"dims": hd // 2, "base": 500000.0, "scaling": {"factor": 8.0}}}
+    right = {"heads": H, "kv_heads": H, "dim": hd, "vdim": hd, "conv": 4}
+    mlp = {"kind": "dense", "ff": ff}
+    layers = [{"type": "delta", "mixer": delta, "mlp": dict(mlp)}, {"type": "gla", "mixer": gla, "mlp": dict(mlp)},
+              {"type": "parallel", "mixer": {"left": left, "left_scale": 1.0, "right": right, "right_scale": 0.5}, "mlp": dict(mlp)},
+              {"type": "delta", "mixer": delta, "mlp": dict(mlp), "weights_of": 0}]
+    return {"architecture": "Gosulorn", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-5}, "streams": GOSULORN_STREAMS,
+            "layers": layers}
+
+
 def lfm2_like_config(width, H, G, hd, ff, n_layers):
     return dict(architectures=["Lfm2ForCausalLM"], vocab_size=DESIGN_VOCAB, hidden_size=width, num_hidden_layers=n_layers,
                 num_attention_heads=H, num_key_value_heads=G, head_dim=hd, layer_types=["full_attention"] * n_layers,
@@ -525,7 +545,8 @@ def run_design(a) -> int:
     import kappai_b200.models.tizusun as tz
     import kappai_b200.models.vekuzen as vk
     import kappai_b200.models.vumotar as vm
-    tz.SOFTMAX_WEIGHTS = vk.SOFTMAX_WEIGHTS = vm.SOFTMAX_WEIGHTS = a.softmax_weights
+    import kappai_b200.models.gosulorn as gs
+    tz.SOFTMAX_WEIGHTS = vk.SOFTMAX_WEIGHTS = vm.SOFTMAX_WEIGHTS = gs.SOFTMAX_WEIGHTS = a.softmax_weights
     pk = peaks()
     T, B, ctx_len = PROMPT_LEN, a.batch, PROMPT_LEN + 256
     warmup = max(a.warmup, 3)
@@ -533,8 +554,10 @@ def run_design(a) -> int:
     vekuzen = a.design == "vekuzen"
     tupalorn = a.design == "tupalorn"
     vumotar = a.design == "vumotar"
+    gosulorn = a.design == "gosulorn"
     out = {"design": a.design.capitalize(),
-           "beside": ("Tizusun mixture layers of the same sizes" if vumotar else
+           "beside": ("Tupalorn layers of the same sizes" if gosulorn else
+                      "Tizusun mixture layers of the same sizes" if vumotar else
                       "dense Vekuzen layers of the same sizes" if tupalorn else "Tizusun layers of the same sizes" if vekuzen
                       else "LFM2 attention layers of the same sizes"), "dtype": "bf16",
            "softmax_weights": a.softmax_weights,
@@ -546,11 +569,12 @@ def run_design(a) -> int:
         if a.size and a.size != name:
             continue
         rec = {}
-        if tupalorn:
+        if tupalorn or gosulorn:
             layers = "dddd"
         if vumotar:
             layers = "mmm"
-        pair = ((("vumotar", vumotar_config(width, H, G, hd, E, top, ff_e)),
+        pair = ((("gosulorn", gosulorn_config(width, H, G, hd, ff)), ("tupalorn", tupalorn_config(width, H, G, hd, ff))) if gosulorn else
+                (("vumotar", vumotar_config(width, H, G, hd, E, top, ff_e)),
                  ("tizusun", tizusun_config(width, H, G, hd, ff, E, top, ff_e, layers))) if vumotar else
                 (("tupalorn", tupalorn_config(width, H, G, hd, ff)),
                  ("vekuzen", vekuzen_config(width, H, G, hd, ff, E, top, ff_e, layers))) if tupalorn else
@@ -701,7 +725,7 @@ def main() -> int:
                     help="with --workload: launch every kernel on its own between CUDA events and print the device "
                          "time by kernel class (the run's throughput is then not the engine's)")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="prompt length of --probe")
-    ap.add_argument("--design", choices=["tizusun", "vekuzen", "tupalorn", "vumotar"], default=None,
+    ap.add_argument("--design", choices=["tizusun", "vekuzen", "tupalorn", "vumotar", "gosulorn"], default=None,
                     help="time another design at a few layer sizes beside the closest existing model of the same sizes "
                          "(tizusun beside LFM2 attention layers, vekuzen beside tizusun, tupalorn beside dense vekuzen layers) "
                          "(prefill, decode, device time by kernel class) instead of the default line")

@@ -355,26 +355,36 @@ recur_scan_kernel(const T* __restrict__ qp, const T* __restrict__ kp, const T* _
 // (in the gated recurrence u = v), and
 //   o_i = (exp(G_i) q_i)^T S + sum_{j <= i} B_ij u_j ,                        B_ij = sum_d q_i k_j exp(G_i - G_j) ,
 //   S'  = exp(G_last) S + sum_j (exp(G_last - G_j) k_j) u_j^T .
-// Three passes: (0) for all chunks side by side what does not need S: A and B, the system solved for the right hand
-// sides beta v and beta exp(G) k, so that u = Wv - Wk S; (1) a serial pass a (segment, head, 32 value columns): u and S',
-// leaving every chunk's S; (2) for all chunks side by side the outputs.  Every exponent is <= 0: where a product of two
-// exponentials stands for exp(G_i - G_j) with factors a channel, its reference is the sum in front of i's 16 rows, which
-// lies between the two; inside 16 rows every pair takes its own exponential.
+// The system is solved for the right hand sides beta v and beta exp(G) k, so that u = Wv - Wk S; with K' the rows
+// exp(G_last - G_j) k_j and Q the rows exp(G_i) q_i everything that depends on S is then one product:
+//   S' = M S + N ,   M = diag(exp(G_last)) - K'^T Wk ,   N = K'^T Wv ;        o = (Q - B Wk) S + B Wv .
+// Three passes: (0) for all chunks side by side M, N, Q - B Wk, and B Wv into the output rows; (1) a serial pass that walks
+// a segment's chunks and leaves every chunk's S in N's place (the gated recurrence: S' = diag(exp(G_last)) S + N, element
+// by element); (2) for all chunks side by side the products with S, added to the output rows.
 //
-// The matrix products run on the tensor cores in tf32 with both operands cut into a rounded part and what it leaves
-// (three products a pair: what is dropped is 2^-22 of a term), float32 sums.
+// Every exponent is <= 0: where a product of two exponentials stands for exp(G_i - G_j) with factors a channel, its
+// reference is a sum that lies between the two; inside eight rows every pair takes its own exponential.
+//
+// The matrix products run on the tensor cores in tf32 with both operands cut into their upper eleven bits and what those
+// leave (three products a pair: what is dropped is about 2^-21 of a term), float32 sums.  What one pass leaves for the
+// next lies in the order of the product's register fragments: a tile [16, 8] as 32 lanes of four floats.  As the left
+// operand of a product, a result tile's columns 2t and 2t + 1 stand in the places t and t + 4 of the inner index (the
+// right operand is read in the same order), so a result is a left operand as it is.
 #define RC_C 64
-#define RC_THREADS 256
-#define RC_PT 32                 // value columns of a block of pass 1
-#define RC_LDU 40                // row pitch of [.., 32] operands read by columns (40 % 32 == 8: no bank conflicts)
 #define RC_LDB 68                // row pitch of the 64 x 64 matrices
-#define RC_MAX_D 256
+#define RC_MAX_D 128
+#define RC_MAX_P 256
 #define RC_LOG2E 1.4426950408889634f
 
+// 2^x for x <= 0 (the special function unit alone: two units in the last place, below 2^-126 zero)
+__device__ __forceinline__ float rc_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ void rc_split(float x, uint32_t& hi, uint32_t& lo) {
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
-    const float rest = x - __uint_as_float(hi);
-    asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(lo) : "f"(rest));
+    hi = __float_as_uint(x) & 0xffffe000u;                       // (by a mask: conversions run at a fraction of its rate)
+    lo = __float_as_uint(x - __uint_as_float(hi));               // exact; the product reads its upper bits
 }
 __device__ __forceinline__ void rc_mma(float* c, const uint32_t* a, const uint32_t* b) {
     asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -403,11 +413,24 @@ __device__ __forceinline__ void rc_load_at(RcA& f, const float* s, int ld, int m
     rc_split(p[4 * ld], f.hi[2], f.lo[2]);
     rc_split(p[4 * ld + 8], f.hi[3], f.lo[3]);
 }
+// The same from fragment order (see above)
+__device__ __forceinline__ void rc_frag_a(RcA& f, const float4 v) {
+    rc_split(v.x, f.hi[0], f.lo[0]);
+    rc_split(v.y, f.hi[1], f.lo[1]);
+    rc_split(v.z, f.hi[2], f.lo[2]);
+    rc_split(v.w, f.hi[3], f.lo[3]);
+}
 // A tile [8, 8] of a right operand stored [k][col]
 __device__ __forceinline__ void rc_load_b(RcB& f, const float* s, int ld, int k0, int n0, int g, int t) {
     const float* p = s + (k0 + t) * ld + n0 + g;
     rc_split(p[0], f.hi[0], f.lo[0]);
     rc_split(p[4 * ld], f.hi[1], f.lo[1]);
+}
+// The same in the inner order that goes with a left operand in fragment order
+__device__ __forceinline__ void rc_load_b2(RcB& f, const float* s, int ld, int k0, int n0, int g, int t) {
+    const float* p = s + (k0 + 2 * t) * ld + n0 + g;
+    rc_split(p[0], f.hi[0], f.lo[0]);
+    rc_split(p[ld], f.hi[1], f.lo[1]);
 }
 // The same of one stored [col][k]
 __device__ __forceinline__ void rc_load_bt(RcB& f, const float* s, int ld, int k0, int n0, int g, int t) {
@@ -416,153 +439,193 @@ __device__ __forceinline__ void rc_load_bt(RcB& f, const float* s, int ld, int k
     rc_split(p[4], f.hi[1], f.lo[1]);
 }
 
-// What pass 0 leaves of a (chunk, head): exp(G_last - G_j) k_j [64][D], exp(G_i) q_i [64][D], with DELTA Wk [64][D], Wv (v in
-// the gated recurrence; pass 1 puts u in its place) [64][P], B [64][64], exp(G_last) [D].  All pieces start on 16 bytes.
-struct RcRec { size_t kh, qt, wk, wv, bm, el, size; };
-__host__ __device__ inline RcRec rc_record(int D, int P, bool delta) {
-    RcRec r;
-    r.kh = 0;
-    r.qt = r.kh + (size_t)RC_C * D;
-    r.wk = r.qt + (size_t)RC_C * D;
-    r.wv = r.wk + (delta ? (size_t)RC_C * D : 0);
-    r.bm = r.wv + (size_t)RC_C * P;
-    r.el = r.bm + (size_t)RC_C * RC_C;
-    r.size = (r.el + D + 3) / 4 * 4;
+// Sizes: key channels in tiles of 16, value columns in tiles of 8.  What pass 0 leaves of a (chunk, head), in floats: N (then
+// S), [D16 / 16][P8 / 8] tiles; Q - B Wk, [4][D16 / 8] tiles; M, [D16 / 16][D16 / 8] tiles, or with the gated recurrence
+// exp(G_last) [D16].
+struct RcDims { int D16, P8, ld, ldw; };
+__host__ __device__ inline RcDims rc_dims(int D, int P, bool delta) {
+    RcDims r;
+    r.D16 = (D + 15) / 16 * 16;
+    r.P8 = (P + 7) / 8 * 8;
+    r.ld = (D + 31) / 32 * 32 + 4;                                // (4 beyond a multiple of 32: no bank conflicts by rows)
+    r.ldw = (r.P8 + (delta ? r.D16 : 0) + 31) / 32 * 32 + 8;      // (8 beyond: none by columns)
     return r;
 }
+struct RcRec { size_t n, q, m, size; };
+__host__ __device__ inline RcRec rc_record(int D, int P, bool delta) {
+    const RcDims s = rc_dims(D, P, delta);
+    RcRec r;
+    r.n = 0;
+    r.q = (size_t)s.D16 * s.P8;
+    r.m = r.q + (size_t)RC_C * s.D16;
+    r.size = r.m + (delta ? (size_t)s.D16 * s.D16 : s.D16);
+    return r;
+}
+// floats of shared memory of pass 0: K and Q rows, B, exp(G_last), beta, and the sums G and A, whose place W takes later
+__host__ inline size_t rc_prepare_floats(int D, int P, bool delta, bool chan) {
+    const RcDims s = rc_dims(D, P, delta);
+    const size_t ga = (chan ? (size_t)RC_C * s.ld : RC_C) + (delta ? (size_t)RC_C * RC_LDB : 0), w = (size_t)RC_C * s.ldw;
+    return 2 * (size_t)RC_C * s.ld + (size_t)RC_C * RC_LDB + s.D16 + RC_C + (ga > w ? ga : w);
+}
 
-// Pass 0, one block a (chunk, head).
-template <typename T, bool DELTA, bool CHAN>
-__global__ void __launch_bounds__(RC_THREADS)
+// Pass 0, one block a (chunk, head).  NTH threads: at least P8 + D16 with the delta rule.
+template <typename T, bool DELTA, bool CHAN, int NTH>
+__global__ void __launch_bounds__(NTH, 512 / NTH)
 recur_chunk_prepare_kernel(const T* __restrict__ qp, const T* __restrict__ kp, const T* __restrict__ vp, int ldi,
                            const float* __restrict__ lg, const float* __restrict__ beta, float q_scale,
                            const int* __restrict__ cu_rows, const int* __restrict__ chunk_seg, const int* __restrict__ chunk_row0,
-                           float* __restrict__ rec, int H, int G, int D, int P) {
+                           float* __restrict__ rec, float* __restrict__ out, int ldo, int H, int G, int D, int P) {
     kp_pdl_begin();
+    constexpr int WARPS = NTH / 32;
     extern __shared__ __align__(16) float rc_sm[];
-    const int Dp = (D + 31) & ~31, ld = Dp + 4;
+    const RcDims Z = rc_dims(D, P, DELTA);
+    const int ld = Z.ld, Dp = ld - 4;
     float* Ks = rc_sm;                                           // [64][ld]
     float* Qs = Ks + RC_C * ld;                                  // [64][ld]
-    float* As = Qs + RC_C * ld;                                  // [64][RC_LDB] (with DELTA)
-    float* bt = As + (DELTA ? RC_C * RC_LDB : 0);                // [64]
-    float* Gs = bt + RC_C;                                       // [64][ld], or [64]: sums of base-2 logarithms
+    float* Bs = Qs + RC_C * ld;                                  // [64][RC_LDB]
+    float* el = Bs + RC_C * RC_LDB;                              // [D16]
+    float* bt = el + Z.D16;                                      // [64]
+    float* Ws = bt + RC_C;                                       // [64][ldw], once the next two are done with
+    float* As = Ws;                                              // [64][RC_LDB] (with DELTA)
+    float* Gs = As + (DELTA ? RC_C * RC_LDB : 0);                // [64][ld], or [64]: sums of base-2 logarithms
     const int chunk = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = lane >> 2, t = lane & 3;
     const int grp = head / (H / G);
     const int t0 = chunk_row0[chunk], n = min(RC_C, cu_rows[chunk_seg[chunk] + 1] - t0);
     const RcRec R = rc_record(D, P, DELTA);
-    float* out = rec + ((size_t)chunk * H + head) * R.size;
-    for (int i = warp; i < RC_C; i += RC_THREADS / 32) {
-        const bool live = i < n;
-        const size_t row = (size_t)(t0 + i) * ldi + (size_t)grp * D;
-        for (int d = lane; d < Dp; d += 32) {
-            const bool ok = live && d < D;
-            Ks[i * ld + d] = ok ? to_f32(kp[row + d]) : 0.f;
-            Qs[i * ld + d] = ok ? to_f32(qp[row + d]) * q_scale : 0.f;
-            if (CHAN) Gs[i * ld + d] = ok ? lg[((size_t)(t0 + i) * H + head) * D + d] * RC_LOG2E : 0.f;
+    float* dst = rec + ((size_t)chunk * H + head) * R.size;
+    // (a warp's rows are fetched together: their loads are all under way before the first is waited for)
+    constexpr int ROWS = RC_C / WARPS;
+    for (int d = lane; d < Dp; d += 32) {
+        float kv[ROWS], qv[ROWS], gv[ROWS];
+#pragma unroll
+        for (int x = 0; x < ROWS; x++) {
+            const int i = warp + x * WARPS;
+            const bool ok = i < n && d < D;
+            const size_t at = (size_t)(t0 + i) * ldi + (size_t)grp * D + d;
+            kv[x] = ok ? to_f32(kp[at]) : 0.f;
+            qv[x] = ok ? to_f32(qp[at]) : 0.f;
+            gv[x] = CHAN && ok ? lg[((size_t)(t0 + i) * H + head) * D + d] : 0.f;
+        }
+#pragma unroll
+        for (int x = 0; x < ROWS; x++) {
+            const int i = warp + x * WARPS;
+            Ks[i * ld + d] = kv[x];
+            Qs[i * ld + d] = qv[x] * q_scale;
+            if (CHAN) Gs[i * ld + d] = gv[x] * RC_LOG2E;
         }
     }
     if (tid < RC_C) {
         bt[tid] = DELTA && tid < n ? beta[(size_t)(t0 + tid) * H + head] : 0.f;
         if (!CHAN) Gs[tid] = tid < n ? lg[(size_t)(t0 + tid) * H + head] * RC_LOG2E : 0.f;
     }
+    for (int x = tid; x < RC_C * RC_LDB; x += NTH) Bs[x] = 0.f;  // (what lies above the diagonal is read as part of tiles)
     __syncthreads();
     if (CHAN) {
-        for (int d = tid; d < Dp; d += RC_THREADS) {
+        for (int d = tid; d < Dp; d += NTH) {
             float acc = 0.f;
-#pragma unroll 8
+#pragma unroll 16
             for (int i = 0; i < RC_C; i++) {
                 acc += Gs[i * ld + d];
                 Gs[i * ld + d] = acc;
             }
         }
-    } else if (tid == 0) {
-        float acc = 0.f;
-#pragma unroll 8
-        for (int i = 0; i < RC_C; i++) {
-            acc += Gs[i];
-            Gs[i] = acc;
+    } else if (warp == 0) {
+        const float a = Gs[2 * lane], b = a + Gs[2 * lane + 1];
+        float sum = b;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += up;
         }
+        float before = __shfl_up_sync(0xffffffffu, sum, 1);
+        if (lane == 0) before = 0.f;
+        Gs[2 * lane] = before + a;
+        Gs[2 * lane + 1] = before + b;
     }
     __syncthreads();
-    const int g = lane >> 2, t = lane & 3;
-    float* Bm = out + R.bm;
     if (!CHAN) {
-        // rows 16 (warp & 3) .., four tiles of eight columns
-        const int m0 = (warp & 3) * 16, nt0 = (warp >> 2) * 4;
-        float ca[4][4], cb[4][4];
+        // the ten pieces [16, 16] on and below the diagonal, the warps in turn
+        for (int x = warp; x < 10; x += WARPS) {
+            const int a = x < 1 ? 0 : (x < 3 ? 1 : (x < 6 ? 2 : 3)), b = x - a * (a + 1) / 2;
+            const int m0 = 16 * a, n0 = 16 * b;
+            float ca[2][4], cb[2][4];
 #pragma unroll
-        for (int x = 0; x < 4; x++)
+            for (int y = 0; y < 2; y++)
 #pragma unroll
-            for (int y = 0; y < 4; y++) { ca[x][y] = 0.f; cb[x][y] = 0.f; }
-        if (nt0 * 8 <= m0 + 15) {
+                for (int z = 0; z < 4; z++) { ca[y][z] = 0.f; cb[y][z] = 0.f; }
             for (int k0 = 0; k0 < D; k0 += 8) {
                 RcA fk, fq;
                 if (DELTA) rc_load_a(fk, Ks, ld, m0, k0, g, t);
                 rc_load_a(fq, Qs, ld, m0, k0, g, t);
 #pragma unroll
-                for (int x = 0; x < 4; x++) {
-                    if ((nt0 + x) * 8 > m0 + 15) continue;
+                for (int y = 0; y < 2; y++) {
                     RcB fb;
-                    rc_load_bt(fb, Ks, ld, k0, (nt0 + x) * 8, g, t);
-                    if (DELTA) rc_mma3(ca[x], fk, fb);
-                    rc_mma3(cb[x], fq, fb);
+                    rc_load_bt(fb, Ks, ld, k0, n0 + 8 * y, g, t);
+                    if (DELTA) rc_mma3(ca[y], fk, fb);
+                    rc_mma3(cb[y], fq, fb);
                 }
             }
+#pragma unroll
+            for (int y = 0; y < 2; y++)
+#pragma unroll
+                for (int z = 0; z < 4; z++) {
+                    const int i = m0 + g + (z >> 1) * 8, j = n0 + 8 * y + 2 * t + (z & 1);
+                    const float w = j <= i ? rc_exp2(Gs[i] - Gs[j]) : 0.f;
+                    if (DELTA) As[i * RC_LDB + j] = j < i ? bt[i] * (w * ca[y][z]) : 0.f;
+                    Bs[i * RC_LDB + j] = w * cb[y][z];
+                }
         }
-#pragma unroll
-        for (int x = 0; x < 4; x++)
-#pragma unroll
-            for (int y = 0; y < 4; y++) {
-                const int i = m0 + g + (y >> 1) * 8, j = (nt0 + x) * 8 + 2 * t + (y & 1);
-                const float w = j <= i ? exp2f(Gs[i] - Gs[j]) : 0.f;
-                if (DELTA) As[i * RC_LDB + j] = j < i ? bt[i] * (w * ca[x][y]) : 0.f;
-                Bm[i * RC_C + j] = w * cb[x][y];
-            }
     } else {
-        // pairs of 16 rows and 16 earlier rows of another sixteen: both factors by the sum in front of the later sixteen
-        if (warp < 6) {
-            const int a = warp == 0 ? 1 : (warp < 3 ? 2 : 3), b = warp == 0 ? 0 : (warp < 3 ? warp - 1 : warp - 3);
-            const int m0 = 16 * a, n0 = 16 * b;
-            const float* Gr = Gs + (m0 - 1) * ld;
+        // pieces whose rows lie behind their columns: sixteen rows against sixteen earlier ones (six of them), and the upper
+        // eight rows of a sixteen against its lower eight (four; their other rows count for nothing).  Both factors by the sum
+        // in front of the later rows.
+        for (int x = warp; x < 10; x += WARPS) {
+            const bool inner = x >= 6;
+            const int a = inner ? x - 6 : (x < 1 ? 1 : (x < 3 ? 2 : 3)), b = inner ? a : (x < 1 ? 0 : (x < 3 ? x - 1 : x - 3));
+            const int m0 = 16 * a, n0 = 16 * b, ref = inner ? m0 + 7 : m0 - 1;
+            const float* Gr = Gs + ref * ld;
             float ca[2][4], cb[2][4];
 #pragma unroll
-            for (int x = 0; x < 2; x++)
+            for (int y = 0; y < 2; y++)
 #pragma unroll
-                for (int y = 0; y < 4; y++) { ca[x][y] = 0.f; cb[x][y] = 0.f; }
+                for (int z = 0; z < 4; z++) { ca[y][z] = 0.f; cb[y][z] = 0.f; }
             for (int k0 = 0; k0 < D; k0 += 8) {
                 RcA fk, fq;
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int i = m0 + g + (e & 1) * 8, d = k0 + t + (e >> 1) * 4;
-                    const float w = exp2f(Gs[i * ld + d] - Gr[d]);
+                    const float w = i > ref ? rc_exp2(Gs[i * ld + d] - Gr[d]) : 0.f;
                     if (DELTA) rc_split(Ks[i * ld + d] * w, fk.hi[e], fk.lo[e]);
                     rc_split(Qs[i * ld + d] * w, fq.hi[e], fq.lo[e]);
                 }
 #pragma unroll
-                for (int x = 0; x < 2; x++) {
+                for (int y = 0; y < 2; y++) {
+                    if (inner && y) continue;
                     RcB fb;
 #pragma unroll
                     for (int e = 0; e < 2; e++) {
-                        const int jj = n0 + x * 8 + g, d = k0 + t + e * 4;
-                        rc_split(Ks[jj * ld + d] * exp2f(Gr[d] - Gs[jj * ld + d]), fb.hi[e], fb.lo[e]);
+                        const int jj = n0 + y * 8 + g, d = k0 + t + e * 4;
+                        rc_split(Ks[jj * ld + d] * rc_exp2(Gr[d] - Gs[jj * ld + d]), fb.hi[e], fb.lo[e]);
                     }
-                    if (DELTA) rc_mma3(ca[x], fk, fb);
-                    rc_mma3(cb[x], fq, fb);
+                    if (DELTA) rc_mma3(ca[y], fk, fb);
+                    rc_mma3(cb[y], fq, fb);
                 }
             }
 #pragma unroll
-            for (int x = 0; x < 2; x++)
+            for (int y = 0; y < 2; y++)
 #pragma unroll
-                for (int y = 0; y < 4; y++) {
-                    const int i = m0 + g + (y >> 1) * 8, jj = n0 + x * 8 + 2 * t + (y & 1);
-                    if (DELTA) As[i * RC_LDB + jj] = bt[i] * ca[x][y];
-                    Bm[i * RC_C + jj] = cb[x][y];
+                for (int z = 0; z < 4; z++) {
+                    const int i = m0 + g + (z >> 1) * 8, jj = n0 + y * 8 + 2 * t + (z & 1);
+                    if (i <= ref || (inner && y)) continue;
+                    if (DELTA) As[i * RC_LDB + jj] = bt[i] * ca[y][z];
+                    Bs[i * RC_LDB + jj] = cb[y][z];
                 }
         }
-        // pairs inside sixteen rows: a warp a row, the lanes over the channels (two rows of every sixteen a warp, 17 pairs)
-        for (int blk = 0; blk < RC_C / 16; blk++)
-            for (int half = 0; half < 2; half++) {
-                const int i = 16 * blk + (half ? 15 - warp : warp);
+        // pairs inside eight rows: the lanes over the channels
+        for (int blk = warp % 8; blk < 8; blk += 8)
+            for (int r = warp / 8; r < 8; r += WARPS / 8) {
+                const int i = 8 * blk + (WARPS == 8 ? r : (r & 2 ? r ^ 1 : r));
                 float ki[RC_MAX_D / 32], qi[RC_MAX_D / 32], gi[RC_MAX_D / 32];
 #pragma unroll
                 for (int m = 0; m < RC_MAX_D / 32; m++) {
@@ -572,269 +635,350 @@ recur_chunk_prepare_kernel(const T* __restrict__ qp, const T* __restrict__ kp, c
                     qi[m] = ok ? Qs[i * ld + d] : 0.f;
                     gi[m] = ok ? Gs[i * ld + d] : 0.f;
                 }
-                for (int jj = 16 * blk; jj < 16 * blk + 16; jj++) {
+                for (int jj = 8 * blk; jj <= i; jj++) {
                     float sa = 0.f, sb = 0.f;
-                    if (jj <= i) {
 #pragma unroll
-                        for (int m = 0; m < RC_MAX_D / 32; m++) {
-                            const int d = lane + 32 * m;
-                            if (d < Dp) {
-                                const float x = Ks[jj * ld + d] * exp2f(gi[m] - Gs[jj * ld + d]);
-                                if (DELTA) sa = fmaf(ki[m], x, sa);
-                                sb = fmaf(qi[m], x, sb);
-                            }
+                    for (int m = 0; m < RC_MAX_D / 32; m++) {
+                        const int d = lane + 32 * m;
+                        if (d < Dp) {
+                            const float x = Ks[jj * ld + d] * rc_exp2(gi[m] - Gs[jj * ld + d]);
+                            if (DELTA) sa = fmaf(ki[m], x, sa);
+                            sb = fmaf(qi[m], x, sb);
                         }
-                        if (DELTA) sa = warp_sum(sa);
-                        sb = warp_sum(sb);
                     }
+                    if (DELTA) sa = warp_sum(sa);
+                    sb = warp_sum(sb);
                     if (lane == 0) {
                         if (DELTA) As[i * RC_LDB + jj] = jj < i ? bt[i] * sa : 0.f;
-                        Bm[i * RC_C + jj] = sb;
+                        Bs[i * RC_LDB + jj] = sb;
                     }
                 }
             }
     }
     __syncthreads();
-    // the system, one right hand side a thread; the gated recurrence takes v as it is
-    for (int c = tid; c < (DELTA ? P + D : P); c += RC_THREADS) {
-        const bool is_v = c < P;
-        if (!DELTA) {
-            for (int i = 0; i < RC_C; i++)
-                out[R.wv + (size_t)i * P + c] = i < n ? to_f32(vp[(size_t)(t0 + i) * ldi + (size_t)head * P + c]) : 0.f;
-            continue;
-        }
-        const int d = c - P;
-        float w[RC_C];
-        if (is_v) {
+    // the right hand sides, one column a thread: beta v, then beta exp(G) k; without DELTA u = v
+    const int n_col = Z.P8 + (DELTA ? Z.D16 : 0);
+    float w[RC_C];
+    if (tid < n_col) {
+        const int d = tid - Z.P8;
+        if (d < 0) {
+            const bool ok = tid < P;
+            const T* src = vp + (size_t)t0 * ldi + (size_t)head * P + tid;
 #pragma unroll
-            for (int i = 0; i < RC_C; i++) w[i] = i < n ? to_f32(vp[(size_t)(t0 + i) * ldi + (size_t)head * P + c]) : 0.f;
+            for (int i = 0; i < RC_C; i++) w[i] = ok && i < n ? to_f32(src[(size_t)i * ldi]) : 0.f;
+            if (DELTA) {
 #pragma unroll
-            for (int i = 0; i < RC_C; i++) w[i] *= bt[i];
-        } else {
-#pragma unroll
-            for (int i = 0; i < RC_C; i++) w[i] = bt[i] * (Ks[i * ld + d] * exp2f(CHAN ? Gs[i * ld + d] : Gs[i]));
-        }
-#pragma unroll
-        for (int i = 1; i < RC_C; i++) {
-            float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-            const float4* row = reinterpret_cast<const float4*>(As + i * RC_LDB);
-#pragma unroll
-            for (int q = 0; q < (i + 3) / 4; q++) {
-                const float4 r4 = row[q];
-                a0 = fmaf(r4.x, w[4 * q], a0);
-                if (4 * q + 1 < i) a1 = fmaf(r4.y, w[4 * q + 1], a1);
-                if (4 * q + 2 < i) a2 = fmaf(r4.z, w[4 * q + 2], a2);
-                if (4 * q + 3 < i) a3 = fmaf(r4.w, w[4 * q + 3], a3);
+                for (int i = 0; i < RC_C; i++) w[i] *= bt[i];
             }
-            w[i] -= (a0 + a1) + (a2 + a3);
-        }
-        float* dst = is_v ? out + R.wv + c : out + R.wk + d;
-        const int step = is_v ? P : D;
+        } else if (d < Dp) {
 #pragma unroll
-        for (int i = 0; i < RC_C; i++) dst[(size_t)i * step] = w[i];
-    }
-    for (int i = warp; i < RC_C; i += RC_THREADS / 32)
-        for (int d = lane; d < D; d += 32) {
-            const float gi = CHAN ? Gs[i * ld + d] : Gs[i], gl = CHAN ? Gs[(RC_C - 1) * ld + d] : Gs[RC_C - 1];
-            out[R.kh + (size_t)i * D + d] = Ks[i * ld + d] * exp2f(gl - gi);
-            out[R.qt + (size_t)i * D + d] = Qs[i * ld + d] * exp2f(gi);
+            for (int i = 0; i < RC_C; i++) w[i] = bt[i] * (Ks[i * ld + d] * rc_exp2(CHAN ? Gs[i * ld + d] : Gs[i]));
         }
-    for (int d = tid; d < D; d += RC_THREADS) out[R.el + d] = exp2f(CHAN ? Gs[(RC_C - 1) * ld + d] : Gs[RC_C - 1]);
-}
-
-__device__ __forceinline__ void rc_cp16(float* dst, const float* src) {
-    const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src) : "memory");
-}
-// rows x cols floats from global (row pitch src_ld) to shared memory (row pitch ld); vec: everything starts on 16 bytes
-__device__ __forceinline__ void rc_fetch(float* dst, int ld, const float* src, int src_ld, int rows, int cols, bool vec, int warp, int lane) {
-    for (int i = warp; i < rows; i += RC_THREADS / 32) {
-        if (vec) for (int x = lane * 4; x < cols; x += 128) rc_cp16(dst + i * ld + x, src + (size_t)i * src_ld + x);
-        else for (int x = lane; x < cols; x += 32) dst[i * ld + x] = src[(size_t)i * src_ld + x];
-    }
-}
-
-// Pass 1, one block a (32 value columns, head, segment): S[chunk] <- the state at the chunk's head; u in the place of Wv;
-// the segment's slot <- the state behind its last chunk.  stages: 2 fetches a chunk's operands while the one before runs.
-template <bool DELTA>
-__global__ void __launch_bounds__(RC_THREADS)
-recur_chunk_states_kernel(float* __restrict__ rec, float* __restrict__ heads_s, float* __restrict__ state, size_t slot_stride,
-                          const int* __restrict__ seg_pos, const int* __restrict__ seg_slot, const int* __restrict__ seg_chunk0,
-                          int H, int D, int P, int write_state, int stages, int vec) {
-    kp_pdl_begin();
-    extern __shared__ __align__(16) float rc_sm[];
-    const int Dp = (D + 31) & ~31, lda = Dp + 4, ldb = Dp + 8;
-    const int stage_floats = (DELTA ? RC_C * lda : 0) + RC_C * ldb + RC_C * RC_LDU;
-    float* Ss = rc_sm;                                           // [Dp][RC_LDU]
-    float* st0 = Ss + Dp * RC_LDU;
-    const int tile = blockIdx.x, head = blockIdx.y, seg = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int g = lane >> 2, t = lane & 3;
-    const int j0 = tile * RC_PT, cols = min(RC_PT, P - j0);
-    const RcRec R = rc_record(D, P, DELTA);
-    // (columns and rows behind the sizes stay zero: nothing is fetched into them)
-    for (int x = tid; x < Dp * RC_LDU + stages * stage_floats; x += RC_THREADS) rc_sm[x] = 0.f;
-    __syncthreads();
-    float* st = state + (size_t)seg_slot[seg] * slot_stride + (size_t)head * D * P;
-    if (seg_pos[seg] != 0)
-        for (int i = warp; i < D; i += RC_THREADS / 32)
-            if (lane < cols) Ss[i * RC_LDU + lane] = st[(size_t)i * P + j0 + lane];
-    const int c_begin = seg_chunk0[seg], c_end = seg_chunk0[seg + 1];
-    auto fetch = [&](int c, int s) {
-        const float* src = rec + ((size_t)c * H + head) * R.size;
-        float* wk = st0 + s * stage_floats;
-        float* kh = wk + (DELTA ? RC_C * lda : 0);
-        float* wv = kh + RC_C * ldb;
-        if (DELTA) rc_fetch(wk, lda, src + R.wk, D, RC_C, D, vec, warp, lane);
-        rc_fetch(kh, ldb, src + R.kh, D, RC_C, D, vec, warp, lane);
-        rc_fetch(wv, RC_LDU, src + R.wv + j0, P, RC_C, cols, vec, warp, lane);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    if (c_begin < c_end) fetch(c_begin, 0);
-    for (int c = c_begin; c < c_end; c++) {
-        const int s = stages == 2 ? (c - c_begin) & 1 : 0;
-        if (stages == 2 && c + 1 < c_end) {
-            fetch(c + 1, s ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        float* wk = st0 + s * stage_floats;
-        float* kh = wk + (DELTA ? RC_C * lda : 0);
-        float* us = kh + RC_C * ldb;
-        float* dst = heads_s + ((size_t)c * H + head) * D * P + j0;
-        for (int i = warp; i < D; i += RC_THREADS / 32)
-            if (lane < cols) dst[(size_t)i * P + lane] = Ss[i * RC_LDU + lane];
-        float* rc = rec + ((size_t)c * H + head) * R.size;
         if (DELTA) {
-            const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 16;
-            float acc[2][4];
 #pragma unroll
-            for (int x = 0; x < 2; x++)
+            for (int i = 1; i < RC_C; i++) {
+                float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+                const float4* row = reinterpret_cast<const float4*>(As + i * RC_LDB);
 #pragma unroll
-                for (int y = 0; y < 4; y++) acc[x][y] = 0.f;
-#pragma unroll 2
-            for (int k0 = 0; k0 < D; k0 += 8) {
-                RcA fa;
-                rc_load_a(fa, wk, lda, m0, k0, g, t);
-#pragma unroll
-                for (int x = 0; x < 2; x++) {
-                    RcB fb;
-                    rc_load_b(fb, Ss, RC_LDU, k0, n0 + 8 * x, g, t);
-                    rc_mma3(acc[x], fa, fb);
+                for (int q = 0; q < (i + 3) / 4; q++) {
+                    const float4 r4 = row[q];
+                    a0 = fmaf(r4.x, w[4 * q], a0);
+                    if (4 * q + 1 < i) a1 = fmaf(r4.y, w[4 * q + 1], a1);
+                    if (4 * q + 2 < i) a2 = fmaf(r4.z, w[4 * q + 2], a2);
+                    if (4 * q + 3 < i) a3 = fmaf(r4.w, w[4 * q + 3], a3);
                 }
+                w[i] -= (a0 + a1) + (a2 + a3);
             }
-#pragma unroll
-            for (int x = 0; x < 2; x++)
-#pragma unroll
-                for (int y = 0; y < 4; y++) {
-                    const int i = m0 + g + (y >> 1) * 8, j = n0 + 8 * x + 2 * t + (y & 1);
-                    const float u = us[i * RC_LDU + j] - acc[x][y];
-                    us[i * RC_LDU + j] = u;
-                    if (j < cols) rc[R.wv + (size_t)i * P + j0 + j] = u;
-                }
         }
-        __syncthreads();
-        for (int m0 = warp * 16; m0 < D; m0 += 16 * (RC_THREADS / 32)) {
-            float acc[4][4];
-            const float e0 = m0 + g < D ? rc[R.el + m0 + g] : 0.f, e1 = m0 + g + 8 < D ? rc[R.el + m0 + g + 8] : 0.f;
-#pragma unroll
-            for (int x = 0; x < 4; x++)
-#pragma unroll
-                for (int y = 0; y < 4; y++)
-                    acc[x][y] = (y < 2 ? e0 : e1) * Ss[(m0 + g + (y >> 1) * 8) * RC_LDU + 8 * x + 2 * t + (y & 1)];
-#pragma unroll 2
-            for (int k0 = 0; k0 < RC_C; k0 += 8) {
-                RcA fa;
-                rc_load_at(fa, kh, ldb, m0, k0, g, t);
-#pragma unroll
-                for (int x = 0; x < 4; x++) {
-                    RcB fb;
-                    rc_load_b(fb, us, RC_LDU, k0, 8 * x, g, t);
-                    rc_mma3(acc[x], fa, fb);
-                }
-            }
-#pragma unroll
-            for (int x = 0; x < 4; x++)
-#pragma unroll
-                for (int y = 0; y < 4; y++)
-                    Ss[(m0 + g + (y >> 1) * 8) * RC_LDU + 8 * x + 2 * t + (y & 1)] = acc[x][y];
-        }
-        __syncthreads();
-        if (stages == 1 && c + 1 < c_end) fetch(c + 1, 0);
     }
-    if (write_state)
-        for (int i = warp; i < D; i += RC_THREADS / 32)
-            if (lane < cols) st[(size_t)i * P + j0 + lane] = Ss[i * RC_LDU + lane];
-}
-
-// Pass 2, one block a (PT value columns, chunk, head): o = exp(G) q S + B u.
-template <int PT>
-__global__ void __launch_bounds__(RC_THREADS)
-recur_chunk_out_kernel(const float* __restrict__ rec, const float* __restrict__ heads_s, const int* __restrict__ cu_rows,
-                       const int* __restrict__ chunk_seg, const int* __restrict__ chunk_row0, float* __restrict__ out, int ldo,
-                       int H, int D, int P, int delta, int vec) {
-    kp_pdl_begin();
-    constexpr int LDP = PT + 8;                                  // (PT 32 or 64: 8 beyond a multiple of 32)
-    constexpr int NT = PT / 16;                                  // tiles of eight columns a warp
-    extern __shared__ __align__(16) float rc_sm[];
-    const int Dp = (D + 31) & ~31, lda = Dp + 4;
-    float* Qt = rc_sm;                                           // [64][lda]
-    float* Ss = Qt + RC_C * lda;                                 // [Dp][LDP]
-    float* Bs = Ss + Dp * LDP;                                   // [64][RC_LDB]
-    float* us = Bs + RC_C * RC_LDB;                              // [64][LDP]
-    const int chunk = blockIdx.y, head = blockIdx.z, tile = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int g = lane >> 2, t = lane & 3;
-    const int t0 = chunk_row0[chunk], n = min(RC_C, cu_rows[chunk_seg[chunk] + 1] - t0);
-    const int j0 = tile * PT, cols = min(PT, P - j0);
-    const RcRec R = rc_record(D, P, delta != 0);
-    const float* rc = rec + ((size_t)chunk * H + head) * R.size;
-    if (D < Dp || cols < PT) {                                   // zeros where nothing is fetched
-        for (int x = tid; x < RC_C * lda + Dp * LDP; x += RC_THREADS) rc_sm[x] = 0.f;
-        for (int x = tid; x < RC_C * LDP; x += RC_THREADS) us[x] = 0.f;
-        __syncthreads();
-    }
-    rc_fetch(Qt, lda, rc + R.qt, D, RC_C, D, vec, warp, lane);
-    rc_fetch(Ss, LDP, heads_s + ((size_t)chunk * H + head) * D * P + j0, P, D, cols, vec, warp, lane);
-    rc_fetch(Bs, RC_LDB, rc + R.bm, RC_C, RC_C, RC_C, true, warp, lane);
-    rc_fetch(us, LDP, rc + R.wv + j0, P, RC_C, cols, vec, warp, lane);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * (PT / 2);
-    if (m0 >= n) return;
-    float acc[NT][4];
-#pragma unroll
-    for (int x = 0; x < NT; x++)
-#pragma unroll
-        for (int y = 0; y < 4; y++) acc[x][y] = 0.f;
-#pragma unroll 2
-    for (int k0 = 0; k0 < D; k0 += 8) {
-        RcA fa;
-        rc_load_a(fa, Qt, lda, m0, k0, g, t);
-#pragma unroll
-        for (int x = 0; x < NT; x++) {
-            RcB fb;
-            rc_load_b(fb, Ss, LDP, k0, n0 + 8 * x, g, t);
-            rc_mma3(acc[x], fa, fb);
+    // K and Q rows become exp(G_last - G) k and exp(G) q
+    for (int i = warp; i < RC_C; i += WARPS)
+        for (int d = lane; d < Dp; d += 32) {
+            const float gi = CHAN ? Gs[i * ld + d] : Gs[i], gl = CHAN ? Gs[(RC_C - 1) * ld + d] : Gs[RC_C - 1];
+            Ks[i * ld + d] *= rc_exp2(gl - gi);
+            Qs[i * ld + d] *= rc_exp2(gi);
         }
+    for (int d = tid; d < Z.D16; d += NTH) {
+        const float e = d < D ? rc_exp2(CHAN ? Gs[(RC_C - 1) * ld + d] : Gs[RC_C - 1]) : 0.f;
+        el[d] = e;
+        if (!DELTA) dst[R.m + d] = e;
     }
-    for (int k0 = 0; k0 < m0 + 16; k0 += 8) {
-        RcA fa;
-        rc_load_a(fa, Bs, RC_LDB, m0, k0, g, t);
+    __syncthreads();
+    if (tid < n_col) {
 #pragma unroll
-        for (int x = 0; x < NT; x++) {
-            RcB fb;
-            rc_load_b(fb, us, LDP, k0, n0 + 8 * x, g, t);
-            rc_mma3(acc[x], fa, fb);
+        for (int i = 0; i < RC_C; i++) Ws[i * Z.ldw + tid] = w[i];
+    }
+    __syncthreads();
+    // the products with W: K'^T W (rows: key channels), then B W (rows: the chunk's), four tiles of eight columns an item
+    const int mt1 = Z.D16 / 16, tiles = n_col / 8, groups = (tiles + 3) / 4, ks = Z.D16 / 8, nts = Z.P8 / 8;
+    for (int x = warp; x < (mt1 + 4) * groups; x += WARPS) {
+        const int m = x / groups, n1 = (x - m * groups) * 4;
+        const bool first = m < mt1;
+        const int m0 = (first ? m : m - mt1) * 16, k_end = first ? RC_C : m0 + 16;
+        float acc[4][4];
+#pragma unroll
+        for (int y = 0; y < 4; y++)
+#pragma unroll
+            for (int z = 0; z < 4; z++) acc[y][z] = 0.f;
+        for (int k0 = 0; k0 < k_end; k0 += 8) {
+            RcA fa;
+            if (first) rc_load_at(fa, Ks, ld, m0, k0, g, t);
+            else rc_load_a(fa, Bs, RC_LDB, m0, k0, g, t);
+#pragma unroll
+            for (int y = 0; y < 4; y++) {
+                RcB fb;
+                rc_load_b(fb, Ws, Z.ldw, k0, (n1 + y) * 8, g, t);
+                rc_mma3(acc[y], fa, fb);
+            }
         }
-    }
-#pragma unroll
-    for (int x = 0; x < NT; x++)
 #pragma unroll
         for (int y = 0; y < 4; y++) {
-            const int i = m0 + g + (y >> 1) * 8, j = n0 + 8 * x + 2 * t + (y & 1);
-            if (i < n && j < cols) out[(size_t)(t0 + i) * ldo + (size_t)head * P + j0 + j] = acc[x][y];
+            const int nt = n1 + y;
+            if (nt >= tiles) continue;
+            float* c = acc[y];
+            if (nt < nts) {
+                if (first) {
+                    *reinterpret_cast<float4*>(dst + R.n + ((size_t)(m * nts + nt) * 32 + lane) * 4) = make_float4(c[0], c[1], c[2], c[3]);
+                } else {
+#pragma unroll
+                    for (int z = 0; z < 4; z++) {
+                        const int i = m0 + g + (z >> 1) * 8, j = nt * 8 + 2 * t + (z & 1);
+                        if (i < n && j < P) out[(size_t)(t0 + i) * ldo + (size_t)head * P + j] = c[z];
+                    }
+                }
+            } else if (DELTA) {
+                const int k = nt - nts, d = k * 8 + 2 * t;
+                if (first) {
+                    const int r0 = m0 + g, r1 = r0 + 8;
+                    *reinterpret_cast<float4*>(dst + R.m + ((size_t)(m * ks + k) * 32 + lane) * 4) =
+                        make_float4((r0 == d ? el[d] : 0.f) - c[0], (r1 == d ? el[d] : 0.f) - c[2],
+                                    (r0 == d + 1 ? el[d + 1] : 0.f) - c[1], (r1 == d + 1 ? el[d + 1] : 0.f) - c[3]);
+                } else {
+                    const float* q0 = Qs + (m0 + g) * ld + d;
+                    const float* q1 = q0 + 8 * ld;
+                    *reinterpret_cast<float4*>(dst + R.q + ((size_t)((m - mt1) * ks + k) * 32 + lane) * 4) =
+                        make_float4(q0[0] - c[0], q1[0] - c[2], q0[1] - c[1], q1[1] - c[3]);
+                }
+            }
+        }
+    }
+    if (!DELTA) {
+        for (int x = warp; x < 4 * ks; x += WARPS) {
+            const float* q0 = Qs + (x / ks * 16 + g) * ld + (x % ks) * 8 + 2 * t;
+            const float* q1 = q0 + 8 * ld;
+            *reinterpret_cast<float4*>(dst + R.q + ((size_t)x * 32 + lane) * 4) = make_float4(q0[0], q1[0], q0[1], q1[1]);
+        }
+    }
+}
+
+// Pass 1 with the delta rule, one block a (16 value columns, head, segment), a warp 16 rows of the state.  In place: N[chunk] <-
+// the state at the chunk's head; the segment's slot <- the state behind its last chunk.  The tiles of M come through a ring in
+// shared memory, four a stage, RT_STAGES - 1 stages ahead; a lane reads what it has copied itself, so nothing but its own
+// copies is waited for.
+#define RT_COLS 16
+#define RT_STAGES 6
+#define RT_LD 20                 // (20 % 16 == 4: the right operand's reads, rows 2t and 2t + 1, hit every bank once)
+template <int KS>
+__global__ void __launch_bounds__(KS * 16, KS == 16 ? 2 : 1)
+recur_chunk_states_kernel(float* __restrict__ rec, float* __restrict__ state, size_t slot_stride, const int* __restrict__ seg_pos,
+                          const int* __restrict__ seg_slot, const int* __restrict__ seg_chunk0, int H, int D, int P, int write_state) {
+    kp_pdl_begin();
+    __shared__ __align__(16) float Ss[2][KS * 8 * RT_LD];
+    extern __shared__ __align__(16) float rc_sm[];               // [RT_STAGES][4][threads] tiles' float4s
+    constexpr int NTH = KS * 16, SPC = KS / 4;                   // stages a chunk
+    const int head = blockIdx.y, seg = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = lane >> 2, t = lane & 3;
+    const RcDims Z = rc_dims(D, P, true);
+    const RcRec R = rc_record(D, P, true);
+    const int ks = Z.D16 / 8, nts = Z.P8 / 8, nt0 = blockIdx.x * 2;
+    const bool two = nt0 + 1 < nts;
+    const size_t step = (size_t)H * R.size;
+    const int c0 = seg_chunk0[seg], c1 = seg_chunk0[seg + 1];
+    float* base = rec + ((size_t)c0 * H + head) * R.size;
+    float* st = state + (size_t)seg_slot[seg] * slot_stride + (size_t)head * D * P;
+    const bool fresh = seg_pos[seg] == 0;
+    float s[2][4];
+#pragma unroll
+    for (int y = 0; y < 2; y++)
+#pragma unroll
+        for (int z = 0; z < 4; z++) {
+            const int d = warp * 16 + g + (z >> 1) * 8, j = (nt0 + y) * 8 + 2 * t + (z & 1);
+            s[y][z] = !fresh && d < D && j < P ? st[(size_t)d * P + j] : 0.f;
+        }
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 nf[2];
+    const int total = (c1 - c0) * SPC;
+    int put = 0, put_slot = 0, get_slot = 0;                     // the stage to fetch next, its slot, the slot to read next
+    auto fetch = [&]() {
+        if (put < total) {
+            const int c = put / SPC, k0 = put % SPC * 4;
+            const float4* src = reinterpret_cast<const float4*>(base + (size_t)c * step + R.m) + (size_t)(warp * ks + k0) * 32 + lane;
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+                if (k0 + i < ks) {
+                    const uint32_t a = (uint32_t)__cvta_generic_to_shared(rc_sm + ((put_slot * 4 + i) * NTH + tid) * 4);
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src + i * 32) : "memory");
+                }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        put++;
+        put_slot = put_slot + 1 == RT_STAGES ? 0 : put_slot + 1;
+    };
+    auto n_tile = [&](int c, int y) {
+        return c < c1 && (y == 0 || two) ? reinterpret_cast<const float4*>(base + (size_t)(c - c0) * step + R.n)[(size_t)(warp * nts + nt0 + y) * 32 + lane]
+                                         : zero;
+    };
+#pragma unroll
+    for (int i = 0; i < RT_STAGES - 1; i++) fetch();
+    nf[0] = n_tile(c0, 0);
+    nf[1] = n_tile(c0, 1);
+    for (int c = c0; c < c1; c++) {
+        float* buf = Ss[(c - c0) & 1];
+        float4* ns = reinterpret_cast<float4*>(base + (size_t)(c - c0) * step + R.n) + (size_t)(warp * nts + nt0) * 32 + lane;
+#pragma unroll
+        for (int y = 0; y < 2; y++) {
+            float* p = buf + (warp * 16 + g) * RT_LD + y * 8 + 2 * t;
+            *reinterpret_cast<float2*>(p) = make_float2(s[y][0], s[y][1]);
+            *reinterpret_cast<float2*>(p + 8 * RT_LD) = make_float2(s[y][2], s[y][3]);
+            if (y == 0 || two) ns[y * 32] = make_float4(s[y][0], s[y][1], s[y][2], s[y][3]);
+        }
+        float hi[2][4], lo[2][4];
+#pragma unroll
+        for (int y = 0; y < 2; y++) {
+            hi[y][0] = nf[y].x; hi[y][1] = nf[y].y; hi[y][2] = nf[y].z; hi[y][3] = nf[y].w;
+            nf[y] = n_tile(c + 1, y);
+#pragma unroll
+            for (int z = 0; z < 4; z++) lo[y][z] = 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int part = 0; part < SPC; part++) {
+            asm volatile("cp.async.wait_group %0;" ::"n"(RT_STAGES - 2) : "memory");
+            const float* tiles = rc_sm + ((size_t)get_slot * 4 * NTH + tid) * 4;
+            get_slot = get_slot + 1 == RT_STAGES ? 0 : get_slot + 1;
+            float4 m4[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) m4[i] = *reinterpret_cast<const float4*>(tiles + i * NTH * 4);
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const int k = part * 4 + i;
+                if (k >= ks) continue;
+                RcA fa;
+                rc_frag_a(fa, m4[i]);
+#pragma unroll
+                for (int y = 0; y < 2; y++) {
+                    RcB fb;
+                    rc_load_b2(fb, buf, RT_LD, k * 8, y * 8, g, t);
+                    rc_mma(lo[y], fa.lo, fb.hi);
+                    rc_mma(lo[y], fa.hi, fb.lo);
+                    rc_mma(hi[y], fa.hi, fb.hi);
+                }
+            }
+            fetch();                                             // (into the slot read one stage ago)
+        }
+#pragma unroll
+        for (int y = 0; y < 2; y++)
+#pragma unroll
+            for (int z = 0; z < 4; z++) s[y][z] = hi[y][z] + lo[y][z];
+    }
+    if (write_state) {
+#pragma unroll
+        for (int y = 0; y < 2; y++)
+#pragma unroll
+            for (int z = 0; z < 4; z++) {
+                const int d = warp * 16 + g + (z >> 1) * 8, j = (nt0 + y) * 8 + 2 * t + (z & 1);
+                if (d < D && j < P) st[(size_t)d * P + j] = s[y][z];
+            }
+    }
+}
+
+// Pass 1 of the gated recurrence, element by element: N[chunk] <- the state at the chunk's head, S' = exp(G_last) S + N.
+__global__ void __launch_bounds__(256)
+recur_chunk_decay_kernel(float* __restrict__ rec, float* __restrict__ state, size_t slot_stride, const int* __restrict__ seg_pos,
+                         const int* __restrict__ seg_slot, const int* __restrict__ seg_chunk0, int H, int D, int P, int write_state) {
+    kp_pdl_begin();
+    const int head = blockIdx.y, seg = blockIdx.z;
+    const int e = blockIdx.x * blockDim.x + threadIdx.x;         // a place in fragment order
+    const RcDims Z = rc_dims(D, P, false);
+    const RcRec R = rc_record(D, P, false);
+    if (e >= Z.D16 * Z.P8) return;
+    const int tile = e >> 7, lane = (e >> 2) & 31, z = e & 3, nts = Z.P8 / 8;
+    const int d = tile / nts * 16 + (lane >> 2) + (z >> 1) * 8, j = tile % nts * 8 + 2 * (lane & 3) + (z & 1);
+    float* st = state + (size_t)seg_slot[seg] * slot_stride + ((size_t)head * D + d) * P + j;
+    const bool real = d < D && j < P;
+    float S = real && seg_pos[seg] != 0 ? *st : 0.f;
+    const size_t step = (size_t)H * R.size;
+    const int c_end = seg_chunk0[seg + 1];
+    for (int c0 = seg_chunk0[seg]; c0 < c_end; c0 += 8) {
+        float* p = rec + ((size_t)c0 * H + head) * R.size;
+        float u[8], w[8];
+#pragma unroll
+        for (int k = 0; k < 8; k++)
+            if (c0 + k < c_end) {
+                u[k] = p[k * step + R.n + e];
+                w[k] = p[k * step + R.m + d];
+            }
+#pragma unroll
+        for (int k = 0; k < 8; k++)
+            if (c0 + k < c_end) {
+                p[k * step + R.n + e] = S;
+                S = fmaf(w[k], S, u[k]);
+            }
+    }
+    if (write_state && real) *st = S;
+}
+
+// Pass 2, one block a (64 value columns, chunk, head): out += (Q - B Wk) S.
+#define RO_COLS 64
+#define RO_LD 68                 // (68 % 16 == 4)
+#define RO_THREADS 256
+__global__ void __launch_bounds__(RO_THREADS)
+recur_chunk_out_kernel(const float* __restrict__ rec, const int* __restrict__ cu_rows, const int* __restrict__ chunk_seg,
+                       const int* __restrict__ chunk_row0, float* __restrict__ out, int ldo, int H, int D, int P, int delta) {
+    kp_pdl_begin();
+    __shared__ __align__(16) float Ss[RC_MAX_D * RO_LD];
+    const int chunk = blockIdx.y, head = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = lane >> 2, t = lane & 3;
+    const int t0 = chunk_row0[chunk], n = min(RC_C, cu_rows[chunk_seg[chunk] + 1] - t0);
+    const RcDims Z = rc_dims(D, P, delta != 0);
+    const RcRec R = rc_record(D, P, delta != 0);
+    const float* src = rec + ((size_t)chunk * H + head) * R.size;
+    const int ks = Z.D16 / 8, nts = Z.P8 / 8, nt0 = blockIdx.x * (RO_COLS / 8), tiles = min(RO_COLS / 8, nts - nt0);
+    for (int x = warp; x < (Z.D16 / 16) * (RO_COLS / 8); x += RO_THREADS / 32) {
+        const int m = x / (RO_COLS / 8), y = x % (RO_COLS / 8);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (y < tiles) v = __ldg(reinterpret_cast<const float4*>(src + R.n) + (size_t)(m * nts + nt0 + y) * 32 + lane);
+        float* p = Ss + (m * 16 + g) * RO_LD + y * 8 + 2 * t;
+        *reinterpret_cast<float2*>(p) = make_float2(v.x, v.y);
+        *reinterpret_cast<float2*>(p + 8 * RO_LD) = make_float2(v.z, v.w);
+    }
+    __syncthreads();
+    const int m = warp & 3, n0 = (warp >> 2) * 4;                // 16 rows, four tiles of eight columns
+    if (m * 16 >= n || n0 >= tiles) return;
+    float acc[4][4];
+#pragma unroll
+    for (int y = 0; y < 4; y++)
+#pragma unroll
+        for (int z = 0; z < 4; z++) acc[y][z] = 0.f;
+    const float4* qf = reinterpret_cast<const float4*>(src + R.q) + (size_t)m * ks * 32 + lane;
+#pragma unroll 4
+    for (int k = 0; k < ks; k++) {
+        RcA fa;
+        rc_frag_a(fa, __ldg(qf + (size_t)k * 32));
+#pragma unroll
+        for (int y = 0; y < 4; y++) {
+            RcB fb;
+            rc_load_b2(fb, Ss, RO_LD, k * 8, (n0 + y) * 8, g, t);
+            rc_mma3(acc[y], fa, fb);
+        }
+    }
+#pragma unroll
+    for (int y = 0; y < 4; y++)
+#pragma unroll
+        for (int z = 0; z < 4; z++) {
+            const int i = m * 16 + g + (z >> 1) * 8, j = (nt0 + n0 + y) * 8 + 2 * t + (z & 1);
+            if (i < n && j < P) out[(size_t)(t0 + i) * ldo + (size_t)head * P + j] += acc[y][z];
         }
 }
 
@@ -933,43 +1077,40 @@ int kp_recur_scan(const void* q, const void* k, const void* v, int ldi, const fl
 }
 
 int kp_recur_chunk_rows() { return RC_C; }
-// floats of scratch that kp_recur_chunks wants: the records of pass 0, then every chunk's state a head
+int kp_recur_chunks_ok(int D, int P) { return D >= 1 && P >= 1 && D <= RC_MAX_D && P <= RC_MAX_P; }
+// floats of scratch that kp_recur_chunks wants: the records of pass 0
 long long kp_recur_chunks_scratch(int n_chunks, int H, int D, int P, int delta) {
-    return (long long)n_chunks * H * ((long long)rc_record(D, P, delta != 0).size + (long long)D * P);
+    return (long long)n_chunks * H * (long long)rc_record(D, P, delta != 0).size;
 }
 
 // The chunked form: the arguments of kp_recur_scan and the list of chunks (chunk_seg, chunk_row0 [n_chunks]: every chunk's
 // segment, numbered among the n_seg segments given here, and first row; seg_chunk0 [n_seg + 1]: the first chunk of every
-// segment).  scratch: kp_recur_chunks_scratch floats, 16-byte aligned.
+// segment).  scratch: kp_recur_chunks_scratch floats, 16-byte aligned.  KP_ERR_UNSUPPORTED for sizes that
+// kp_recur_chunks_ok does not take.
 int kp_recur_chunks(const void* q, const void* k, const void* v, int ldi, const float* lg, const float* beta, float q_scale, float* state,
                     long long slot_stride, const int* cu_rows, const int* seg_pos, const int* seg_slot, const int* chunk_seg,
                     const int* chunk_row0, const int* seg_chunk0, int n_chunks, float* scratch, float* out, int ldo, int n_seg, int H,
                     int G, int D, int P, int per_channel, int write_state, int dtype, void* stream) {
     if (n_seg <= 0 || n_chunks <= 0) return 0;
     if (H < 1 || G < 1 || H % G || D < 1 || P < 1 || (uintptr_t)scratch % 16) return KP_ERR_BAD_ARG;
-    if (D > RC_MAX_D || H > 65535 || n_seg > 65535 || n_chunks > 65535) return KP_ERR_UNSUPPORTED;
+    if (!kp_recur_chunks_ok(D, P) || H > 65535 || n_seg > 65535 || n_chunks > 65535) return KP_ERR_UNSUPPORTED;
     const bool delta = beta != nullptr;
-    const int Dp = (D + 31) & ~31, ld = Dp + 4;
-    const size_t sm0 = ((size_t)(per_channel ? 3 : 2) * RC_C * ld + (delta ? RC_C * RC_LDB : 0) + 2 * RC_C) * sizeof(float);
-    const size_t stage = ((delta ? (size_t)RC_C * ld : 0) + (size_t)RC_C * (Dp + 8) + (size_t)RC_C * RC_LDU) * sizeof(float);
-    const size_t keep1 = (size_t)Dp * RC_LDU * sizeof(float);
-    const int stages = keep1 + 2 * stage <= 227 * 1024 ? 2 : 1;
-    const size_t sm1 = keep1 + stages * stage;
-    const int pt = P > 32 ? 64 : 32;
-    const size_t sm2 = ((size_t)RC_C * ld + (size_t)Dp * (pt + 8) + (size_t)RC_C * RC_LDB + (size_t)RC_C * (pt + 8)) * sizeof(float);
-    const int vec = D % 4 == 0 && P % 4 == 0;
-    float* rec = scratch;
-    float* hs = scratch + (size_t)n_chunks * H * rc_record(D, P, delta).size;
+    const RcDims Z = rc_dims(D, P, delta);
+    const size_t sm0 = rc_prepare_floats(D, P, delta, per_channel != 0) * sizeof(float);
+    // (256 threads, two blocks an SM, where a column a thread and the shared memory allow it)
+    const bool small = Z.P8 + (delta ? Z.D16 : 0) <= 256 && sm0 <= 112 * 1024;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
-#define RC_PREPARE(T, DL, CH)                                                                                                \
+#define RC_PREPARE_N(T, DL, CH, NTH)                                                                                         \
     do {                                                                                                                     \
-        if ((e = cudaFuncSetAttribute(recur_chunk_prepare_kernel<T, DL, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm0)) != cudaSuccess) return (int)e; \
-        kp_launch_pdl(recur_chunk_prepare_kernel<T, DL, CH>, dim3(n_chunks, H), dim3(RC_THREADS), sm0, s, (const T*)q, (const T*)k, (const T*)v, \
-                      ldi, lg, beta, q_scale, cu_rows, chunk_seg, chunk_row0, rec, H, G, D, P);                              \
+        if ((e = cudaFuncSetAttribute(recur_chunk_prepare_kernel<T, DL, CH, NTH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm0)) != cudaSuccess) \
+            return (int)e;                                                                                                   \
+        kp_launch_pdl(recur_chunk_prepare_kernel<T, DL, CH, NTH>, dim3(n_chunks, H), dim3(NTH), sm0, s, (const T*)q, (const T*)k, (const T*)v, \
+                      ldi, lg, beta, q_scale, cu_rows, chunk_seg, chunk_row0, scratch, out, ldo, H, G, D, P);                \
     } while (0)
+#define RC_PREPARE(T, DL, CH) do { if (small) RC_PREPARE_N(T, DL, CH, 256); else RC_PREPARE_N(T, DL, CH, 512); } while (0)
     if (delta) {
-        if (dtype != KP_DTYPE_F32) return KP_ERR_UNSUPPORTED;
+        if (dtype != KP_DTYPE_F32) return KP_ERR_UNSUPPORTED;          // (what delta_prep leaves)
         if (per_channel) RC_PREPARE(float, true, true);
         else RC_PREPARE(float, true, false);
     } else {
@@ -977,28 +1118,30 @@ int kp_recur_chunks(const void* q, const void* k, const void* v, int ldi, const 
         KP_DISPATCH_DTYPE(dtype, T, RC_PREPARE(T, false, true));
     }
 #undef RC_PREPARE
+#undef RC_PREPARE_N
     if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
-    const dim3 grid1((P + RC_PT - 1) / RC_PT, H, n_seg);
     if (delta) {
-        if ((e = cudaFuncSetAttribute(recur_chunk_states_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return (int)e;
-        kp_launch_pdl(recur_chunk_states_kernel<true>, grid1, dim3(RC_THREADS), sm1, s, rec, hs, state, (size_t)slot_stride, seg_pos, seg_slot,
-                      seg_chunk0, H, D, P, write_state, stages, vec);
+        const dim3 grid((Z.P8 + RT_COLS - 1) / RT_COLS, H, n_seg), block(Z.D16 * 2);
+        // (a ring as wide as the kernel's largest block: its pitch does not depend on the block that is launched)
+#define RC_STATES(KS)                                                                                                        \
+        do {                                                                                                                 \
+            const size_t ring = (size_t)RT_STAGES * 4 * (KS * 16) * 16;                                                      \
+            if ((e = cudaFuncSetAttribute(recur_chunk_states_kernel<KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ring)) != cudaSuccess) \
+                return (int)e;                                                                                               \
+            kp_launch_pdl(recur_chunk_states_kernel<KS>, grid, block, ring, s, scratch, state, (size_t)slot_stride, seg_pos, seg_slot, \
+                          seg_chunk0, H, D, P, write_state);                                                                 \
+        } while (0)
+        if (D <= 32) RC_STATES(4);
+        else if (D <= 64) RC_STATES(8);
+        else RC_STATES(16);
+#undef RC_STATES
     } else {
-        if ((e = cudaFuncSetAttribute(recur_chunk_states_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1)) != cudaSuccess) return (int)e;
-        kp_launch_pdl(recur_chunk_states_kernel<false>, grid1, dim3(RC_THREADS), sm1, s, rec, hs, state, (size_t)slot_stride, seg_pos, seg_slot,
-                      seg_chunk0, H, D, P, write_state, stages, vec);
+        kp_launch_pdl(recur_chunk_decay_kernel, dim3((Z.D16 * Z.P8 + 255) / 256, H, n_seg), dim3(256), 0, s, scratch, state, (size_t)slot_stride,
+                      seg_pos, seg_slot, seg_chunk0, H, D, P, write_state);
     }
     if ((e = cudaGetLastError()) != cudaSuccess) return (int)e;
-    const dim3 grid2((P + pt - 1) / pt, n_chunks, H);
-    if (pt == 64) {
-        if ((e = cudaFuncSetAttribute(recur_chunk_out_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm2)) != cudaSuccess) return (int)e;
-        kp_launch_pdl(recur_chunk_out_kernel<64>, grid2, dim3(RC_THREADS), sm2, s, (const float*)rec, (const float*)hs, cu_rows, chunk_seg, chunk_row0,
-                      out, ldo, H, D, P, (int)delta, vec);
-    } else {
-        if ((e = cudaFuncSetAttribute(recur_chunk_out_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm2)) != cudaSuccess) return (int)e;
-        kp_launch_pdl(recur_chunk_out_kernel<32>, grid2, dim3(RC_THREADS), sm2, s, (const float*)rec, (const float*)hs, cu_rows, chunk_seg, chunk_row0,
-                      out, ldo, H, D, P, (int)delta, vec);
-    }
+    kp_launch_pdl(recur_chunk_out_kernel, dim3((Z.P8 + RO_COLS - 1) / RO_COLS, n_chunks, H), dim3(RO_THREADS), 0, s, (const float*)scratch, cu_rows,
+                  chunk_seg, chunk_row0, out, ldo, H, D, P, (int)delta);
     return kp_launch_status();
 }
 

@@ -93,52 +93,52 @@ streams_rows_kernel(float* x, float* y, const float* __restrict__ mix, const flo
     for (int i = threadIdx.x; i < d; i += ST_THREADS) h[(size_t)blockIdx.x * d + i] = from_f32<T>((read(i) - mean) * scale * w[i]);
 }
 
-// The same for 16-byte aligned rows of at most 1024 PER floats (d % 4 == 0): u stays in registers, so streams and y are read
-// once and leave in 16-byte stores.  Which form runs depends on the row's length and the buffers' alignment alone.
-template <typename T, int S, int PER>
-__global__ void __launch_bounds__(ST_THREADS)
+// The same for 16-byte aligned rows of at most 4 NTH PER floats (d % 4 == 0): a thread fetches what it needs of the row at once
+// and keeps u in registers, so streams and y are read once and leave in 16-byte stores.  Which form runs depends on the
+// row's length and the buffers' alignment alone.
+template <typename T, int S, int NTH, int PER, bool MIX>
+__global__ void __launch_bounds__(NTH)
 streams_rows_vec_kernel(float* x, float* y, const float* __restrict__ mix, const float* __restrict__ outw, const float* __restrict__ inw,
                         const float* __restrict__ w, float eps, int centred, const int* __restrict__ rows, T* __restrict__ h, int d) {
     kp_pdl_begin();
     __shared__ float red[32];
-    const int r = rows ? rows[blockIdx.x] : (int)blockIdx.x;
+    const int r = !MIX && rows ? rows[blockIdx.x] : (int)blockIdx.x;
     const int n4 = d >> 2;
     float4* xr = reinterpret_cast<float4*>(x + (size_t)r * S * d);
-    float4* yr = y ? reinterpret_cast<float4*>(y + (size_t)r * d) : nullptr;
+    float4* yr = reinterpret_cast<float4*>(y + (size_t)r * d);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 v[PER][S], yv[PER], u[PER];
+#pragma unroll
+    for (int j = 0; j < PER; j++) {
+        const int i = threadIdx.x + j * NTH;
+        const bool ok = i < n4;
+#pragma unroll
+        for (int s = 0; s < S; s++) v[j][s] = ok ? xr[(size_t)s * n4 + i] : zero;
+        yv[j] = MIX && ok ? yr[i] : zero;
+    }
     StCoef<S> k;
-    k.load(mix, outw, inw, y != nullptr);
-    float4 u[PER];
+    k.load(mix, outw, inw, MIX);
     float sum = 0.f;
 #pragma unroll
     for (int j = 0; j < PER; j++) {
-        const int i = threadIdx.x + j * ST_THREADS;
-        u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (i >= n4) continue;
-        float4 v[S];
+        const int i = threadIdx.x + j * NTH;
+        u[j] = zero;
 #pragma unroll
-        for (int s = 0; s < S; s++) v[s] = xr[(size_t)s * n4 + i];
-        if (yr) {
-            const float4 yv = yr[i];
-            yr[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-            for (int t = 0; t < S; t++) {
-                float4 z = make_float4(k.out[t] * yv.x, k.out[t] * yv.y, k.out[t] * yv.z, k.out[t] * yv.w);
+        for (int t = 0; t < S; t++) {
+            float4 z = v[j][t];
+            if (MIX) {
+                z = make_float4(k.out[t] * yv[j].x, k.out[t] * yv[j].y, k.out[t] * yv[j].z, k.out[t] * yv[j].w);
 #pragma unroll
                 for (int s = 0; s < S; s++) {
                     const float m = k.mix[s][t];
-                    z.x = fmaf(m, v[s].x, z.x); z.y = fmaf(m, v[s].y, z.y); z.z = fmaf(m, v[s].z, z.z); z.w = fmaf(m, v[s].w, z.w);
+                    z.x = fmaf(m, v[j][s].x, z.x); z.y = fmaf(m, v[j][s].y, z.y); z.z = fmaf(m, v[j][s].z, z.z); z.w = fmaf(m, v[j][s].w, z.w);
                 }
-                xr[(size_t)t * n4 + i] = z;
-                u[j].x = fmaf(k.in[t], z.x, u[j].x); u[j].y = fmaf(k.in[t], z.y, u[j].y);
-                u[j].z = fmaf(k.in[t], z.z, u[j].z); u[j].w = fmaf(k.in[t], z.w, u[j].w);
+                if (i < n4) xr[(size_t)t * n4 + i] = z;
             }
-        } else {
-#pragma unroll
-            for (int t = 0; t < S; t++) {
-                u[j].x = fmaf(k.in[t], v[t].x, u[j].x); u[j].y = fmaf(k.in[t], v[t].y, u[j].y);
-                u[j].z = fmaf(k.in[t], v[t].z, u[j].z); u[j].w = fmaf(k.in[t], v[t].w, u[j].w);
-            }
+            u[j].x = fmaf(k.in[t], z.x, u[j].x); u[j].y = fmaf(k.in[t], z.y, u[j].y);
+            u[j].z = fmaf(k.in[t], z.z, u[j].z); u[j].w = fmaf(k.in[t], z.w, u[j].w);
         }
+        if (MIX && i < n4) yr[i] = zero;
         sum += (u[j].x + u[j].y) + (u[j].z + u[j].w);
     }
     if (!h) return;
@@ -146,7 +146,7 @@ streams_rows_vec_kernel(float* x, float* y, const float* __restrict__ mix, const
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < PER; j++) {
-        if (threadIdx.x + j * ST_THREADS >= n4) continue;
+        if (threadIdx.x + j * NTH >= n4) continue;
         u[j].x -= mean; u[j].y -= mean; u[j].z -= mean; u[j].w -= mean;
         ss = fmaf(u[j].x, u[j].x, ss); ss = fmaf(u[j].y, u[j].y, ss); ss = fmaf(u[j].z, u[j].z, ss); ss = fmaf(u[j].w, u[j].w, ss);
     }
@@ -154,7 +154,7 @@ streams_rows_vec_kernel(float* x, float* y, const float* __restrict__ mix, const
     const float scale = 1.0f / sqrtf(ss / (float)d + eps);
 #pragma unroll
     for (int j = 0; j < PER; j++) {
-        const int i = threadIdx.x + j * ST_THREADS;
+        const int i = threadIdx.x + j * NTH;
         if (i >= n4) continue;
         const float4 ww = __ldg(reinterpret_cast<const float4*>(w) + i);
         st_store4<T>(h + (size_t)blockIdx.x * d + 4 * i, u[j].x * scale * ww.x, u[j].y * scale * ww.y, u[j].z * scale * ww.z,
@@ -165,19 +165,29 @@ streams_rows_vec_kernel(float* x, float* y, const float* __restrict__ mix, const
 template <int S>
 static int st_rows(float* x, float* y, const float* mix, const float* outw, const float* inw, const float* w, float eps, int centred,
                    const int* rows, void* h, int n, int d, int dtype, cudaStream_t s) {
-    const bool vec = (d & 3) == 0 && d <= 8192 && !(((uintptr_t)x | (uintptr_t)y | (uintptr_t)w | (uintptr_t)h) & 15);
-#define ST_VEC(PER)                                                                                                          \
-    KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(streams_rows_vec_kernel<T, S, PER>, dim3(n), dim3(ST_THREADS), 0, s, x, y, mix, outw, inw, w, eps, \
-                                               centred, rows, (T*)h, d)))
+    // (more than four streams: a thread holds one float4 of each, for rows of at most 2,048)
+    constexpr bool few = S <= 4;
+    const bool vec = (d & 3) == 0 && d <= (few ? 8192 : 2048) && !(((uintptr_t)x | (uintptr_t)y | (uintptr_t)w | (uintptr_t)h) & 15);
+#define ST_VEC_M(NTH, PER, MIX)                                                                                              \
+    KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(streams_rows_vec_kernel<T, S, NTH, PER, MIX>, dim3(n), dim3(NTH), 0, s, x, y, mix, outw, inw, w, \
+                                               eps, centred, rows, (T*)h, d)))
+#define ST_VEC(NTH, PER) do { if (y) ST_VEC_M(NTH, PER, true); else ST_VEC_M(NTH, PER, false); } while (0)
     if (vec) {
-        if (d <= 2048) ST_VEC(2);
-        else if (d <= 4096) ST_VEC(4);
-        else ST_VEC(8);
+        if constexpr (few) {
+            if (d <= 1024) ST_VEC(128, 2);
+            else if (d <= 2048) ST_VEC(256, 2);
+            else if (d <= 4096) ST_VEC(512, 2);
+            else ST_VEC(1024, 2);
+        } else {
+            if (d <= 1024) ST_VEC(256, 1);
+            else ST_VEC(512, 1);
+        }
     } else {
         KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(streams_rows_kernel<T, S>, dim3(n), dim3(ST_THREADS), 0, s, x, y, mix, outw, inw, w, eps,
                                                    centred, rows, (T*)h, d)));
     }
 #undef ST_VEC
+#undef ST_VEC_M
     return kp_launch_status();
 }
 

@@ -937,6 +937,14 @@ def recur_chunk_rows() -> int:
     return int(load_library("recurrence").kp_recur_chunk_rows())
 
 
+RECUR_CHUNK_MAX_DIM = 128        # key rows and value columns of a head that the chunked form takes
+RECUR_CHUNK_MAX_VALUE = 256
+
+
+def recur_chunks_ok(D: int, P: int) -> bool:
+    return D <= RECUR_CHUNK_MAX_DIM and P <= RECUR_CHUNK_MAX_VALUE
+
+
 def recur_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, lg: torch.Tensor, beta: Optional[torch.Tensor], q_scale: float,
                  state: torch.Tensor, cu_rows: torch.Tensor, seg_pos: torch.Tensor, seg_slot: torch.Tensor, chunk_seg: torch.Tensor,
                  chunk_row0: torch.Tensor, seg_chunk0: torch.Tensor, n_chunks: int, out: torch.Tensor, n_seg: int, H: int, G: int,
@@ -950,6 +958,8 @@ def recur_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, lg: torch.Te
         _need(t, nm, torch.int32)
     if chunk_seg.numel() < n_chunks or chunk_row0.numel() < n_chunks or seg_chunk0.numel() < n_seg + 1:
         raise KernelError("recur_chunks: chunk lists too short")
+    if not recur_chunks_ok(D, P):
+        raise KernelError(f"recur_chunks: heads of {D} x {P} exceed {RECUR_CHUNK_MAX_DIM} x {RECUR_CHUNK_MAX_VALUE}")
     lib = load_library("recurrence")
     lib.kp_recur_chunks_scratch.restype = ctypes.c_longlong
     scratch = torch.empty(int(lib.kp_recur_chunks_scratch(int(n_chunks), H, D, P, int(beta is not None))), dtype=torch.float32,

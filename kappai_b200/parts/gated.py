@@ -95,7 +95,7 @@ class _Recurrence(Part):
         if self.D > K.RECUR_MAX_DIM:
             raise ConfigError(f"{what}: head_dim={self.D} is not supported by the kernels (at most {K.RECUR_MAX_DIM})")
         self.state_len = self.H * self.D * self.P
-        self.chunked = self.env.dtype != torch.float32 and self.env.device.type == "cuda"
+        self.chunked = self.env.dtype != torch.float32 and K.recur_chunks_ok(self.D, self.P) and self.env.device.type == "cuda"
         if self.chunked:
             self.chunk_rows = K.recur_chunk_rows()
             self.step_tables_key = ("lightning_chunks", self.chunk_rows)

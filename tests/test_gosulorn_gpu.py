@@ -73,9 +73,10 @@ SIZES = [  # kernel, heads, q/k heads, key channels, value columns, a decay a ke
     ("scan", 2, 2, 128, 64, False, True), ("scan", 2, 1, 256, 36, True, True), ("scan", 3, 3, 64, 33, True, False),
     ("scan", 1, 1, 1, 1, True, False), ("scan", 2, 2, 130, 20, True, False),
     ("chunks", 4, 2, 16, 16, False, True), ("chunks", 3, 1, 24, 40, True, True), ("chunks", 5, 5, 5, 3, True, True),
-    ("chunks", 2, 2, 128, 64, False, True), ("chunks", 4, 2, 128, 128, True, True), ("chunks", 2, 1, 256, 36, True, True),
-    ("chunks", 3, 1, 250, 70, False, True), ("chunks", 3, 3, 64, 33, True, False), ("chunks", 1, 1, 1, 1, True, False),
-    ("chunks", 2, 2, 160, 96, True, False), ("chunks", 2, 2, 64, 128, True, False)]
+    ("chunks", 2, 2, 128, 64, False, True), ("chunks", 4, 2, 128, 128, True, True), ("chunks", 2, 1, 100, 36, True, True),
+    ("chunks", 3, 1, 30, 256, False, True), ("chunks", 2, 1, 128, 256, True, True), ("chunks", 2, 2, 64, 9, False, True),
+    ("chunks", 3, 3, 64, 33, True, False), ("chunks", 1, 1, 1, 1, True, False), ("chunks", 1, 1, 1, 1, False, True),
+    ("chunks", 2, 2, 120, 96, True, False), ("chunks", 2, 2, 64, 256, True, False), ("chunks", 2, 2, 128, 128, True, False)]
 
 
 def _recurrence_case(kernel, H, G, D, Pv, chan, delta, dtype, lens, cut, extra, draw_lg, rng, tol):
