@@ -774,10 +774,10 @@ recur_chunk_prepare_kernel(const T* __restrict__ qp, const T* __restrict__ kp, c
 
 // Pass 1 with the delta rule, one block a (16 value columns, head, segment), a warp 16 rows of the state.  In place: N[chunk] <-
 // the state at the chunk's head; the segment's slot <- the state behind its last chunk.  The tiles of M come through a ring in
-// shared memory, four a stage, RT_STAGES - 1 stages ahead; a lane reads what it has copied itself, so nothing but its own
+// shared memory, four a stage, STAGES - 1 stages ahead; a lane reads what it has copied itself, so nothing but its own
 // copies is waited for.
 #define RT_COLS 16
-#define RT_STAGES 6
+#define RT_STAGES(KS) ((KS) == 16 ? 5 : 6)     // (two blocks an SM at 128 key channels)
 #define RT_LD 20                 // (20 % 16 == 4: the right operand's reads, rows 2t and 2t + 1, hit every bank once)
 template <int KS>
 __global__ void __launch_bounds__(KS * 16, KS == 16 ? 2 : 1)
@@ -785,8 +785,8 @@ recur_chunk_states_kernel(float* __restrict__ rec, float* __restrict__ state, si
                           const int* __restrict__ seg_slot, const int* __restrict__ seg_chunk0, int H, int D, int P, int write_state) {
     kp_pdl_begin();
     __shared__ __align__(16) float Ss[2][KS * 8 * RT_LD];
-    extern __shared__ __align__(16) float rc_sm[];               // [RT_STAGES][4][threads] tiles' float4s
-    constexpr int NTH = KS * 16, SPC = KS / 4;                   // stages a chunk
+    extern __shared__ __align__(16) float rc_sm[];               // [STAGES][4][threads] tiles' float4s
+    constexpr int NTH = KS * 16, SPC = KS / 4, STAGES = RT_STAGES(KS);      // (SPC stages a chunk)
     const int head = blockIdx.y, seg = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int g = lane >> 2, t = lane & 3;
     const RcDims Z = rc_dims(D, P, true);
@@ -823,14 +823,14 @@ recur_chunk_states_kernel(float* __restrict__ rec, float* __restrict__ state, si
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
         put++;
-        put_slot = put_slot + 1 == RT_STAGES ? 0 : put_slot + 1;
+        put_slot = put_slot + 1 == STAGES ? 0 : put_slot + 1;
     };
     auto n_tile = [&](int c, int y) {
         return c < c1 && (y == 0 || two) ? reinterpret_cast<const float4*>(base + (size_t)(c - c0) * step + R.n)[(size_t)(warp * nts + nt0 + y) * 32 + lane]
                                          : zero;
     };
 #pragma unroll
-    for (int i = 0; i < RT_STAGES - 1; i++) fetch();
+    for (int i = 0; i < STAGES - 1; i++) fetch();
     nf[0] = n_tile(c0, 0);
     nf[1] = n_tile(c0, 1);
     for (int c = c0; c < c1; c++) {
@@ -854,9 +854,9 @@ recur_chunk_states_kernel(float* __restrict__ rec, float* __restrict__ state, si
         __syncthreads();
 #pragma unroll
         for (int part = 0; part < SPC; part++) {
-            asm volatile("cp.async.wait_group %0;" ::"n"(RT_STAGES - 2) : "memory");
+            asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
             const float* tiles = rc_sm + ((size_t)get_slot * 4 * NTH + tid) * 4;
-            get_slot = get_slot + 1 == RT_STAGES ? 0 : get_slot + 1;
+            get_slot = get_slot + 1 == STAGES ? 0 : get_slot + 1;
             float4 m4[4];
 #pragma unroll
             for (int i = 0; i < 4; i++) m4[i] = *reinterpret_cast<const float4*>(tiles + i * NTH * 4);
@@ -1125,7 +1125,7 @@ int kp_recur_chunks(const void* q, const void* k, const void* v, int ldi, const 
         // (a ring as wide as the kernel's largest block: its pitch does not depend on the block that is launched)
 #define RC_STATES(KS)                                                                                                        \
         do {                                                                                                                 \
-            const size_t ring = (size_t)RT_STAGES * 4 * (KS * 16) * 16;                                                      \
+            const size_t ring = (size_t)RT_STAGES(KS) * 4 * (KS * 16) * 16;                                                      \
             if ((e = cudaFuncSetAttribute(recur_chunk_states_kernel<KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ring)) != cudaSuccess) \
                 return (int)e;                                                                                               \
             kp_launch_pdl(recur_chunk_states_kernel<KS>, grid, block, ring, s, scratch, state, (size_t)slot_stride, seg_pos, seg_slot, \
