@@ -53,6 +53,11 @@ latent attention with a window, learned sinks and head gates; mixtures whose sig
 inputs, with a shared unit) beside a Tizusun model of mixture layers of the same sizes, the closest design the engine
 has (grouped-query attention with a mask, mixture feed-forwards, whole softmax weights).
 
+``--design gosulorn`` does the same for the Gosulorn design (a residual of four streams; the gated delta rule, gated
+linear attention, windowed attention with short convolutions side by side with a delta rule mixer; one layer's weights
+run twice) beside Tupalorn layers of the same sizes, the closest design the engine has (recurrent mixers with float32
+states and convolutions, windowed attention, gated units).
+
 Only one GPU is used; ``--gpus N`` with N > 1 prints a line that says so and
 exits with 2.
 """

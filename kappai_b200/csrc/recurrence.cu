@@ -1,9 +1,10 @@
 // Linear recurrences with data-dependent decays.  A head keeps a float32 state S [D, P] a request and follows, row after
 // row,
 //
-//   S <- diag(g) S ;   u = v                       ("gated": gated linear attention)
-//                  or  u = beta (v - S^T k)        ("delta": the gated delta rule: what S holds for k is taken off v first)
-//   S <- S + k u^T ;   o = S^T q ,
+//   F = g S          what is left of the state of the row before
+//   e = v            ("gated": gated linear attention), or
+//   e = beta (v - F^T k)     ("delta": the gated delta rule: what F holds for k is taken off v first)
+//   S' = F + k e^T ,     o = S'^T q ,
 //
 // g one factor in (0, 1] a head, or one a key channel (a row of S), given by its logarithm.  Several heads may share a
 // query and key (head h reads q/k head h / (H / G)).
@@ -45,7 +46,7 @@ __device__ __forceinline__ void rc_gate_entry(const T* __restrict__ prow, int b_
 
 // p: rows [n, ld] in the storage type with the channels [q: G heads of D | k: G heads of D | v: H heads of P] side by side
 // from conv_col.  out: [n, C] float32, the same channels behind convolution and silu, q and k as unit vectors a head
-// (x / sqrt(sum x^2 + 1e-6)), q times q_scale.  A warp takes one q or k head, or 128 channels of v, or 128 gate entries, of
+// (divided by the root of their sum of squares + 1e-6), q times q_scale.  A warp takes one q or k head, or 128 channels of v, or 128 gate entries, of
 // one row.  single_rows: every segment has one row, and the lane that read a channel's kept inputs writes the new ones.
 #define RP_UNIT_EPS 1e-6f
 template <typename T>

@@ -1,6 +1,6 @@
 // A residual of several streams: x [rows][S][d], float32.  A sublayer reads one weighted sum of a row's streams, normed;
 // behind it every stream becomes a weighted sum of all the old streams plus its share of the sublayer's output:
-//   x_t <- sum_s mix[s][t] x_s + out[t] y ;   u = sum_t in[t] x_t ;   h = norm(u) * w
+//   x'_b = out_b y + sum_a mix_ab x_a ,     h = w * norm(sum_b in_b x'_b)
 // in one pass over the row (the y it read is cleared for whoever adds into it next; h in the storage type is what the next
 // sublayer reads).  norm: a layer norm without a shift (centred: mean taken off, variance about the mean), or the RMS norm.
 // All float32 with a fixed tree a row.

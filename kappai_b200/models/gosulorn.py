@@ -1,9 +1,9 @@
 """Gosulorn: a decoder whose residual is several streams, with three kinds of linear-time mixer.
 
     x_1 .. x_s = embed[token]                                                    (``streams`` copies)
-    a sublayer:  u = sum_t in[t] x_t ;  y = sublayer(LN(u)) ;  x_t <- sum_s mix[s, t] x_s + out[t] y
+    a sublayer:  y = f(LN(sum_b in_b x_b)) ;  x'_b = out_b y + sum_a mix_ab x_a
     a layer:     its mixer, then its feed-forward, as such sublayers             (coefficients hc1, hc2; norms norm1, norm2)
-    output:      logits = embed . LN(sum_t x_t)                                  (the table is the head; LN has no shift)
+    output:      logits = embed . LN(sum_b x_b)                                  (the table is the head; LN has no shift)
 
 The mixers: ``gla`` (gated linear attention, one data-dependent factor a key channel; parts/gated.py), ``delta`` (the gated
 delta rule, one factor a head, a silu gate; there too) and ``parallel`` (parts/parallel.py), the sum of two mixers on the
@@ -12,12 +12,12 @@ biases, short convolutions on q, k and v and a rotation of a head's first dimens
 (parts/attention.py), on the right the gated delta rule with one factor a key channel, low-rank projections for factors and
 gate, and a sigmoid gate.  The feed-forward is a gated unit with the tanh form of gelu.
 
-A layer with ``weights_of: j`` runs layer j's tensors again with a cache or state of its own: it is one more entry of the
-schedule that names layer j.
+Where an entry says ``weights_of: j`` the schedule simply names layer j once more; what is remembered of a sequence belongs
+to schedule entries, so the second run keeps its own.
 
-This file is the only place that knows the design's ``config.json`` keys and tensor names.  ``layers`` lists the layers, each
-with its ``type`` (the mixer), the mixer's sizes (``mixer``) and its feed-forward (``mlp``, or null for none); layer i's
-tensors start with ``l<i>.``.  Every size and constant is read from there or, for the low ranks, from the tensors' shapes;
+This file is the only place that knows the design's ``config.json`` keys and tensor names: an
+entry of ``layers`` holds ``type``, ``mixer`` and ``mlp`` (null where there is none), and tensors are named by the entry's
+number, ``l0.`` on.  All sizes and constants come from the file or, for the low ranks, from the tensors' shapes;
 what the design fixes (activations, the kinds of gate, norm and decay, the tied head) is written below.  ``mask``, ``rot`` and
 ``rot.scaling`` may be left out (every earlier key is read; nothing is rotated; frequencies as they are).
 """

@@ -919,7 +919,7 @@ def _recur_check(what, q, k, v, lg, beta, state, out, H, G, D, P, per_channel):
 def recur_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, lg: torch.Tensor, beta: Optional[torch.Tensor], q_scale: float,
                state: torch.Tensor, cu_rows: torch.Tensor, seg_pos: torch.Tensor, seg_slot: torch.Tensor, out: torch.Tensor,
                n_seg: int, H: int, G: int, D: int, P: int, per_channel: bool, write_state: bool = True) -> torch.Tensor:
-    """``S <- exp(lg) S; u = beta (v - S^T k), or v without ``beta``; S <- S + k u^T; o = S^T (q_scale q)`` row after row of
+    """``F = exp(lg) S; e = beta (v - F^T k)``, or v without ``beta``; ``S = F + k e^T; o = S^T (q_scale q)`` row after row of
     every segment, from the state in the segment's slot (zero at position 0) and back into it.  ``q``, ``k`` [n, G D] and ``v``
     [n, H P] are columns of rows of one pitch; ``lg`` float32 [n, H], or with ``per_channel`` [n, H D]; ``state``
     float32 [slots, stride] whose rows begin with [H, D, P]; ``out`` float32 [n, H P]."""
@@ -993,7 +993,7 @@ def streams_rows(x: torch.Tensor, y: Optional[torch.Tensor] = None, mix: Optiona
                  eps: float = 0.0, centred: bool = True, h: Optional[torch.Tensor] = None,
                  rows: Optional[torch.Tensor] = None) -> None:
     """One pass over rows of several streams, ``x`` float32 [n, S, d].  With ``y`` (float32 [n, d], left cleared):
-    ``x_t <- sum_s mix[s, t] x_s + out_w[t] y``.  With ``h`` ([rows, d] in the storage type): ``h = norm(sum_t in_w[t] x_t) *
+    ``x'_b = out_w_b y + sum_a mix_ab x_a``.  With ``h`` ([rows, d] in the storage type): ``h = norm(sum_t in_w[t] x_t) *
     norm_w`` of the new streams (``in_w`` None: their sum), the norm centred (a layer norm without a shift) or the RMS
     norm.  ``rows`` (without ``y``): the rows to read."""
     _need(x, "x", torch.float32)

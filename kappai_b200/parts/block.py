@@ -27,8 +27,8 @@ the first norm of the layer that runs next), norms the new residual for it in
 the same pass.
 
 ``streams_residual``: the residual is several float32 streams a row (streams.py).
-A sublayer reads ``norm(sum_t in[t] x_t)`` and its output y joins every stream
-while the streams are mixed, ``x_t <- sum_s mix[s, t] x_s + out[t] y``; mixer
+A sublayer reads ``norm(sum_b in_b x_b)`` and its output y joins every stream
+while the streams are mixed, ``x'_b = out_b y + sum_a mix_ab x_a``; mixer
 and feed-forward each with coefficients of their own (``hc1``, ``hc2``:
 ``in`` [streams], ``out`` [streams], ``mix`` [streams, streams], indexed from,
 to).  As above a sublayer adds into a zeroed float32 branch, and one kernel

@@ -4,10 +4,10 @@ Every head keeps a float32 state ``S`` [head_dim, value_dim] a request, zero at 
 
 ``gated_delta``: ``q, k, v`` (q and k with ``num_qk_heads`` heads, head h reads q/k head ``h // (num_heads / num_qk_heads)``)
 each pass a causal convolution a channel (``conv_kernel`` taps, the last on the current token, no bias) and silu; q
-and k become unit vectors a head, ``x / sqrt(sum x^2 + 1e-6)``, q times ``head_dim^-1/2``; ``beta = sigmoid(h Wb^T)``, one
-a head; then, in this order,
+and k become unit vectors a head (1e-6 joins the sum of squares under the root), q times ``head_dim^-1/2``; ``beta = sigmoid(h Wb^T)``, one
+a head; then every row decays the state, corrects what it holds for the row's key, and reads the corrected state:
 
-    S <- g S ;  u = beta (v - S^T k) ;  S <- S + k u^T ;  o = S^T q .
+    F = g S_before ;  e = beta (v - F^T k) ;  S = F + k e^T ;  o = S^T q .
 
 ``decay`` = ``"head"``: one factor a head, ``g = exp(-exp(A_log) softplus(h Wa^T + dt_bias))``; ``"channel"``: one a key
 channel (a row of S), with the low-rank projection ``(h Wa1^T) Wa2^T`` in the place of ``h Wa^T`` and ``dt_bias``
@@ -16,7 +16,7 @@ times ``gate``: ``"silu"`` (``silu(h Wg^T)``) or ``"sigmoid"``, the projection w
 (``"low"``: ``(h Wg1^T) Wg2^T``); then the output matrix.  Ranks are taken from the tensors' shapes.
 
 ``gated_linear``: ``q = h Wq^T head_dim^-1/2``, ``k``, ``v`` with as many heads each and no convolution; a factor a key
-channel ``g = sigmoid(z)^(1/tau)``, ``z = (h Wa1^T) Wa2^T + b``; ``S_t = diag(g_t) S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t``;
+channel ``g = sigmoid(z)^(1/tau)``, ``z = (h Wa1^T) Wa2^T + b``; each row multiplies the state's rows by their factors, adds ``k v^T`` and reads with q;
 the same norm a head, times ``silu(h Wg^T)``, then the output matrix.
 
 Everything that reads the layer's input is one product; what enters the recurrence behind the projections (unit norms,

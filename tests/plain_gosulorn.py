@@ -123,7 +123,7 @@ def windowed_attention(q, k, v, scale, window):
 
 
 def gated_scan(q, k, v, g, state=None):
-    """S_t = diag(g_t) S_(t-1) + k_t v_t^T ; o_t = S_t^T q_t.  q, k, g [T, H, dim], v [T, H, vdim]; o and the last state."""
+    """Each row: the state's rows times their factors, plus the outer product of k and v; q reads.  q, k, g [T, H, dim], v [T, H, vdim]; o and the last state."""
     T, H, D = q.shape
     S = np.zeros((H, D, v.shape[2])) if state is None else np.array(state, dtype=np.float64)
     o = np.zeros((T, H, v.shape[2]))
@@ -134,7 +134,7 @@ def gated_scan(q, k, v, g, state=None):
 
 
 def delta_scan(q, k, v, g, beta, state=None):
-    """S <- g S ; u = beta (v - S^T k) ; S <- S + k u^T ; o = S^T q.  q, k [T, H, dim], v [T, H, vdim], beta [T, H],
+    """Each row: F = g S, S' = F + k (beta (v - F^T k))^T; q reads S'.  q, k [T, H, dim], v [T, H, vdim], beta [T, H],
     g [T, H, dim] or [T, H, 1]; o and the last state."""
     T, H, D = q.shape
     S = np.zeros((H, D, v.shape[2])) if state is None else np.array(state, dtype=np.float64)
@@ -221,7 +221,7 @@ def streams_read(xs, w_in):
 
 
 def streams_write(xs, y, mix, out):
-    """Every stream from the old ones: x_t <- sum_s mix[s, t] x_s + out[t] y."""
+    """Every stream b from the old ones: out_b y + sum_a mix_ab x_a."""
     return np.einsum("nsd,st->ntd", xs, mix) + out[None, :, None] * y[:, None, :]
 
 

@@ -157,7 +157,7 @@ def test_caches_of_several_memories():
 # ----------------------------------------------------------------------------------- the plain mechanisms by hand
 
 def test_delta_rule_by_hand_and_carried_state():
-    # one head, a state of one row and one column, k = 1: S <- g S ; S <- S + beta (v - S) ; o = S q
+    # one head, a state of one row and one column, k = 1: F = g S, then S = F + beta (v - F), read by q
     one = lambda *a: np.array(a, dtype=float).reshape(-1, 1, 1)
     g, beta, v, q = one(0.5, 0.5, 1.0), np.array([[1.0], [0.5], [0.25]]), one(2.0, 4.0, -1.0), one(1.0, 3.0, 1.0)
     o, S = P.delta_scan(q, one(1, 1, 1), v, g, beta)
@@ -226,3 +226,20 @@ def test_linear_frequency_scaling():
     assert np.allclose(plain.cos[3].numpy(), np.cos(3 * np.array([1.0, 0.1])))
     with pytest.raises(ConfigError):
         make_part("position", PartSpec("rope", {"rotary_dim": 4, "theta": 100.0, "scaling": {"factor": -1.0}}), env)
+
+
+def test_the_bench_configurations_are_valid_models():
+    """``bench.py --design gosulorn`` times these layer sizes: every one of them reads as a model with all three mixers whose
+    last layer runs the first one's weights."""
+    import importlib.util
+    import os
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    spec = importlib.util.spec_from_file_location("bench_for_test", os.path.join(root, "bench.py"))
+    bench = importlib.util.module_from_spec(spec)
+    spec.loader.exec_module(bench)
+    for name, width, H, G, hd, ff, *_ in bench.DESIGN_SIZES:
+        m = _spec(bench.gosulorn_config(width, H, G, hd, ff))
+        assert [l.mixer.kind for l in m.layers] == ["gated_delta", "gated_linear", "parallel"], name
+        assert [e.layer for e in m.schedule] == [0, 1, 2, 0] and m.residual.params["streams"] == bench.GOSULORN_STREAMS
+        left = m.layers[2].mixer.params["mixers"]["left"].params
+        assert left["window"] == bench.GOSULORN_WINDOW and left["head_dim"] == left["value_dim"] == hd
