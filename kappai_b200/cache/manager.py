@@ -41,7 +41,7 @@ class PagePool:
     """Pages of one layer group."""
 
     def __init__(self, n_pages: int, page_size: int, window: Optional[int] = None, block: Optional[int] = None,
-                 keep_first: int = 0):
+                 keep_first: int = 0, every: int = 1):
         if n_pages < 1 or page_size < 1:
             raise CacheError("a page pool needs at least one page and a positive page size")
         if window is not None and window < 1:
@@ -50,6 +50,9 @@ class PagePool:
             raise CacheError("block must be positive")
         if keep_first < 0:
             raise CacheError("keep_first must not be negative")
+        if every < 1 or (every > 1 and (window is not None or block is not None)):
+            raise CacheError("every must be positive, and a pool with an entry for several positions keeps all of them")
+        self.every = int(every)                                       # positions an entry stands for
         self.n_pages, self.page_size, self.window, self.block = n_pages, page_size, window, block
         self.keep_first = int(keep_first)                             # the first keys of a sequence are read for good
         self._free: List[int] = list(range(n_pages - 1, -1, -1))      # stack: lowest page first
@@ -75,9 +78,26 @@ class PagePool:
         the same name: a copy of the table elsewhere knows by it when it is stale."""
         return self._version[req]
 
+    def pages_for(self, n_tokens: int) -> int:
+        """Pages that the entries of ``n_tokens`` positions fill."""
+        return _ceil_div(n_tokens // self.every, self.page_size)
+
     def pages_needed(self, req: Hashable, new_len: int) -> int:
         have = len(self._tables.get(req, ()))
-        return max(0, _ceil_div(new_len, self.page_size) - have)
+        return max(0, self.pages_for(new_len) - have)
+
+    def slot(self, req: Hashable, pos: int) -> int:
+        """Physical slot (page * page_size + offset) of the entry that position ``pos`` writes: its own, or in a pool
+        with an entry for several positions the one it completes (-1 if it completes none)."""
+        e = pos
+        if self.every > 1:
+            if (pos + 1) % self.every:
+                return -1
+            e = pos // self.every
+        page = self._tables[req][e // self.page_size]
+        if page == RELEASED:
+            raise CacheError(f"position {pos} of {req!r} lies in a released page")
+        return page * self.page_size + e % self.page_size
 
     # -- changes
     def _stamp(self) -> int:
@@ -213,8 +233,9 @@ class CacheManager:
     """All page groups and the slot pool of one engine.
 
     ``groups`` maps a group key to ``(n_pages, page_size, window)``,
-    ``(n_pages, page_size, window, block)`` or
-    ``(n_pages, page_size, window, block, keep_first)``.  Each
+    ``(n_pages, page_size, window, block)``,
+    ``(n_pages, page_size, window, block, keep_first)`` or
+    ``(n_pages, page_size, window, block, keep_first, every)``.  Each
     request gets one slot (used by every state-holding layer) and one block
     table per group.
     """
@@ -283,8 +304,15 @@ class CacheManager:
         return self.pools[group].table(req)
 
     def token_slots(self, req: Hashable, group: Hashable, start: int, n: int) -> List[int]:
-        """Physical token slot (page * page_size + offset) of positions start..start+n-1."""
+        """Physical slot (page * page_size + offset) of the entries that positions start..start+n-1 write (-1 where a
+        position writes none: see :meth:`PagePool.slot`)."""
         pool = self.pools[group]
+        if pool.every > 1:
+            first = -(start + 1) % pool.every                        # the first of these positions that completes an entry
+            out = [-1] * n
+            for i in range(first, n, pool.every):
+                out[i] = pool.slot(req, start + i)
+            return out
         t, ps = pool.table(req), pool.page_size
         if n > 32:
             # a prompt portion: by arrays (a Python loop over 2048 positions costs 0.3 ms a step and page group)
@@ -294,13 +322,7 @@ class CacheManager:
                 bad = int(pos[pages == RELEASED][0])
                 raise CacheError(f"position {bad} of {req!r} lies in a released page")
             return (pages * ps + pos % ps).tolist()
-        out = []
-        for pos in range(start, start + n):
-            page = t[pos // ps]
-            if page == RELEASED:
-                raise CacheError(f"position {pos} of {req!r} lies in a released page")
-            out.append(page * ps + pos % ps)
-        return out
+        return [pool.slot(req, pos) for pos in range(start, start + n)]
 
     def check(self) -> None:
         for p in self.pools.values():

@@ -8,7 +8,11 @@ recurrent/conv state of fixed size per layer):
   pages.  Mixers with the same (kv heads, head dim, window) form a *group*
   that shares block tables; groups with different needs have pages of their
   own.  A windowed group may keep the first ``keep_first`` keys of every
-  sequence readable: the pages that hold them are never given back early.
+  sequence readable: the pages that hold them are never given back early.  A
+  group may keep one entry for every ``every`` positions instead of one a
+  position (entry e stands for the positions e every .. e every + every - 1 and
+  exists once the last of them does), and one row a position instead of a key
+  and a value row (``planes`` = 1: a latent that both are made of).
 * :class:`StateSpec` — a fixed-size tensor per request; kept in a slot.
 
 A mixer that needs several of these at once (keys and values beside the last
@@ -27,6 +31,8 @@ class PagedKVSpec:
     window: Optional[int] = None      # keys older than this many positions are never read again
     block: Optional[int] = None       # a position reads no key from before its own block of this many positions
     keep_first: int = 0               # with a window: the first keys of a sequence stay readable for good
+    every: int = 1                    # positions an entry stands for
+    planes: int = 2                   # rows an entry: a key and a value, or one row for both
 
     @property
     def group_key(self) -> Tuple:
@@ -35,6 +41,10 @@ class PagedKVSpec:
             key += (("block", self.block),)
         if self.keep_first and self.window is not None:
             key += (("keep_first", self.keep_first),)
+        if self.every != 1:
+            key += (("every", self.every),)
+        if self.planes != 2:
+            key += (("planes", self.planes),)
         return key
 
 

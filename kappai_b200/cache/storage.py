@@ -1,8 +1,8 @@
 """Device memory of the cache: page pools and state slots.
 
 For a page group with ``L`` caches (one per schedule entry that keeps keys and
-values in it) the pool is one tensor ``[L, n_pages, 2, G, page_size, hd]`` in
-the compute dtype: page ``p`` exists in all ``L`` layers at once, so one block
+values in it) the pool is one tensor ``[L, n_pages, 2, G, page_size, hd]`` (1 in
+the place of 2 where an entry is one row) in the compute dtype: page ``p`` exists in all ``L`` layers at once, so one block
 table serves the whole group (the reference keeps ``[layer][kv head][pos][hd]``
 per session, src/backend/cpu/common.c:1494-1601).  State of fixed size is one
 tensor ``[n_slots, *shape]`` per schedule entry that keeps one.  An entry whose
@@ -21,7 +21,7 @@ from .spec import CompositeSpec, PagedKVSpec, StateSpec, leaf_specs
 @dataclass
 class KVLayerView:
     """One schedule entry's keys and values: ``tensor`` is
-    [n_pages, 2, G, page_size, hd]; ``writes`` is False for an entry that only
+    [n_pages, planes, G, page_size, hd]; ``writes`` is False for an entry that only
     reads another entry's cache."""
 
     group: Hashable
@@ -57,7 +57,7 @@ class CacheStorage:
         self.pools: Dict[Hashable, torch.Tensor] = {}
         for gk, n_caches in members.items():
             s = self.groups[gk]
-            self.pools[gk] = torch.zeros((n_caches, n_pages[gk], 2, s.num_kv_heads, page_size, s.head_dim),
+            self.pools[gk] = torch.zeros((n_caches, n_pages[gk], s.planes, s.num_kv_heads, page_size, s.head_dim),
                                          dtype=dtype, device=device)
         taken = {gk: 0 for gk in members}
 
@@ -82,6 +82,7 @@ class CacheStorage:
                 self.views[i] = _read_only(v)
 
     def bytes_per_token(self, group: Hashable) -> int:
+        """Bytes an entry takes in all caches of the group (a token, where the group keeps one entry a position)."""
         t = self.pools[group]
         return t[:, 0, :, :, 0, :].numel() * t.element_size()
 

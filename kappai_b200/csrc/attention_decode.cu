@@ -17,6 +17,11 @@
 // nothing of kept keys), a second small launch of the kernel below (`front`) computes the kept keys alone, into slots
 // of their own behind the window's chunks (`slot0` on), and the merge is told where they are.  `sink` (one float32 number a query head, or null): exp(sink_h) is added to the softmax's
 // denominator, once a row, by the merge (the chunk kernels know nothing of it).
+//
+// Three more: `cap` > 0 bounds the scores (cap tanh(s / cap)); `out_scale` multiplies a row's output (in the merge);
+// `pool` > 0 (with a window): a row also reads the means of the blocks of `pool` positions that lie wholly before its
+// window.  They are keys 0 .. n - 1 of a cache and a block table of their own: the chunk kernel runs once more over
+// those (`front` = 2), into slots behind the window's chunks, and the merge takes them in front, as kept keys.
 #include "common.cuh"
 
 #define AD_CHUNK 256
@@ -62,7 +67,8 @@ __device__ __forceinline__ int chunk_at(int i, int n_front, int c_lo, int front_
 }
 // (front_slot0 >= 0: the kept keys' chunks, of AD_CHUNK keys each, lie in slots of their own and hold kept keys only)
 #define AD_CHUNK_KEYS 256
-__device__ __forceinline__ int merge_front(int first_hi, int chunk_keys, int c_lo, int front_slot0) {
+__device__ __forceinline__ int merge_front(int first_hi, int chunk_keys, int c_lo, int front_slot0, int pos, int window, int pool) {
+    if (pool > 0) return (kp_pooled_count(pos, window, pool) + AD_CHUNK_KEYS - 1) / AD_CHUNK_KEYS;
     return front_slot0 >= 0 ? (first_hi + AD_CHUNK_KEYS - 1) / AD_CHUNK_KEYS : front_chunks(first_hi, chunk_keys, c_lo);
 }
 
@@ -73,7 +79,7 @@ __global__ void __launch_bounds__(AD_THREADS)
 attn_split_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ cache, const int* __restrict__ block_table,
                   int max_blocks, const int* __restrict__ row_seg, const int* __restrict__ positions,
                   float* __restrict__ part_acc, float* __restrict__ part_ml, int n_chunks, float scale, int window,
-                  int page_size, int H, int G, int hd_rt, int block, int keep_first, int slot0, int front) {
+                  int page_size, int H, int G, int hd_rt, int block, int keep_first, int slot0, int front, float cap, int pool) {
     kp_pdl_begin();
     extern __shared__ float smem[];
     const int hd = HD ? HD : hd_rt;
@@ -90,7 +96,8 @@ attn_split_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ cache,
     key_range(positions[row], window, block, k_lo, k_hi);
     const int c0 = chunk * AD_CHUNK;
     int first_hi = min(keep_first, k_lo);                       // keys below it are read although they lie before the window
-    if (front) { k_hi = first_hi - 1; k_lo = 0; first_hi = 0; } // the kept keys alone (none: no chunk passes the test below)
+    if (front == 1) { k_hi = first_hi - 1; k_lo = 0; first_hi = 0; } // the kept keys alone (none: no chunk passes the test below)
+    if (front == 2) { k_hi = kp_pooled_count(k_hi, window, pool) - 1; k_lo = 0; }   // the pooled entries alone
     if (c0 > k_hi || (c0 + AD_CHUNK - 1 < k_lo && c0 >= first_hi)) return;          // the chunk holds none of this row's keys
     const int* bt = block_table + (size_t)row_seg[row] * max_blocks;
     const size_t page_stride = (size_t)2 * G * page_size * hd;
@@ -144,7 +151,7 @@ attn_split_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ cache,
 #pragma unroll
     for (int r = 0; r < AD_RMAX; r++) {
         if (r < R) {
-            s[r] = valid ? s[r] * scale : -INFINITY;
+            s[r] = valid ? kp_capped(s[r] * scale, cap) : -INFINITY;
             const float m = warp_max(s[r]);
             if (lane == 0) wred[warp][r] = m;
         }
@@ -253,7 +260,7 @@ template <typename T>
 __global__ void attn_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                   const int* __restrict__ positions, T* __restrict__ out, int ldo, int n_chunks,
                                   int chunk_keys, int window, int H, int hd, int block, int keep_first,
-                                  const float* __restrict__ sink, int front_slot0) {
+                                  const float* __restrict__ sink, int front_slot0, float out_scale, int pool) {
     kp_pdl_begin_early_if(gridDim.y > 1);
     extern __shared__ __align__(16) float merge_sm[];       // [MERGE_BATCH], [n_chunks] l_c, [n_chunks] exp(m_c - m), [32]
     const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
@@ -262,7 +269,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_acc, const floa
     // (a position beyond the chunks the caller gave is the caller's fault; the clamp keeps the reads inside
     // the scratch and the shared arrays all the same)
     const int c_hi = min(k_hi / chunk_keys, n_chunks - 1), c_lo = min(k_lo / chunk_keys, c_hi);
-    const int n_front = merge_front(min(keep_first, k_lo), chunk_keys, c_lo, front_slot0), n = n_front + c_hi - c_lo + 1;
+    const int n_front = merge_front(min(keep_first, k_lo), chunk_keys, c_lo, front_slot0, k_hi, window, pool), n = n_front + c_hi - c_lo + 1;
     float* s_acc = merge_sm;
     float* s_l = merge_sm + MERGE_BATCH;
     float* s_w = s_l + n_chunks;
@@ -303,7 +310,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_acc, const floa
     __syncthreads();
     float l = sink ? expf(sink[h] - m) : 0.f;               // the sink: in the denominator once, with no value
     for (int c = 0; c < n; c++) l = __fmaf_rn(s_l[c], s_w[c], l);
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    const float inv = l > 0.f ? out_scale / l : 0.f;
     float v = 0.f;
     for (int c0 = 0; c0 < n; c0 += mb) {
         const int nb = min(mb, n - c0);
@@ -331,7 +338,7 @@ template <typename T>
 __global__ void attn_merge_warp_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                                        const int* __restrict__ positions, T* __restrict__ out, int ldo, int n_chunks,
                                        int chunk_keys, int window, int H, int hd, int n_rows, int block, int keep_first,
-                                       const float* __restrict__ sink, int front_slot0) {
+                                       const float* __restrict__ sink, int front_slot0, float out_scale, int pool) {
     kp_pdl_begin_early_if(n_rows > 1);
     const int lane = threadIdx.x & 31;
     const int item = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);          // (row, head)
@@ -340,7 +347,7 @@ __global__ void attn_merge_warp_kernel(const float* __restrict__ part_acc, const
     int k_lo, k_hi;
     key_range(positions[row], window, block, k_lo, k_hi);
     const int c_hi = min(k_hi / chunk_keys, n_chunks - 1), c_lo = min(k_lo / chunk_keys, c_hi);
-    const int n_front = merge_front(min(keep_first, k_lo), chunk_keys, c_lo, front_slot0), n = n_front + c_hi - c_lo + 1;
+    const int n_front = merge_front(min(keep_first, k_lo), chunk_keys, c_lo, front_slot0, k_hi, window, pool), n = n_front + c_hi - c_lo + 1;
     const float* pa = part_acc + ((size_t)row * H + h) * n_chunks * hd;
     const float* ml = part_ml + ((size_t)row * H + h) * n_chunks * 2;
     // the sums of the first MERGE_WARP_BLOCK chunks are on their way while the statistics are worked out
@@ -377,7 +384,7 @@ __global__ void attn_merge_warp_kernel(const float* __restrict__ part_acc, const
             }
         }
     }
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    const float inv = l > 0.f ? out_scale / l : 0.f;
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int d = lane + 32 * i;
@@ -390,13 +397,13 @@ static size_t merge_smem_bytes(int n_chunks) { return sizeof(float) * ((size_t)2
 template <typename T>
 static int launch_merge(const float* part_acc, const float* part_ml, const int* positions, void* out, int ldo,
                         int n_chunks, int chunk_keys, int window, int block, int keep_first, const float* sink, int n, int H,
-                        int hd, cudaStream_t s, int front_slot0 = -1) {
+                        int hd, cudaStream_t s, int front_slot0 = -1, float out_scale = 1.f, int pool = 0) {
     if (window <= 0) keep_first = 0;
-    if (keep_first == 0) front_slot0 = -1;
+    if (keep_first == 0 && pool == 0) front_slot0 = -1;
     if (n_chunks <= MERGE_WARP_CHUNKS && hd <= 128) {
         const int warps = 8;
         kp_launch_pdl(attn_merge_warp_kernel<T>, dim3((n * H + warps - 1) / warps), dim3(warps * 32), 0, s, part_acc, part_ml,
-                      positions, (T*)out, ldo, n_chunks, chunk_keys, window, H, hd, n, block, keep_first, sink, front_slot0);
+                      positions, (T*)out, ldo, n_chunks, chunk_keys, window, H, hd, n, block, keep_first, sink, front_slot0, out_scale, pool);
         return kp_launch_status();
     }
     const size_t smem = merge_smem_bytes(n_chunks);
@@ -407,7 +414,7 @@ static int launch_merge(const float* part_acc, const float* part_ml, const int* 
     }
     if (hd > MERGE_THREADS || (hd & 3)) return KP_ERR_UNSUPPORTED;
     kp_launch_pdl(attn_merge_kernel<T>, dim3(H, n), dim3(MERGE_THREADS), smem, s, part_acc, part_ml, positions, (T*)out, ldo,
-                  n_chunks, chunk_keys, window, H, hd, block, keep_first, sink, front_slot0);
+                  n_chunks, chunk_keys, window, H, hd, block, keep_first, sink, front_slot0, out_scale, pool);
     return kp_launch_status();
 }
 
@@ -427,11 +434,18 @@ long long kp_attention_split_scratch(int n_rows, int H, int hd, int n_chunks) {
 // n_chunks: chunks of 256 keys the grid covers; must reach the largest position in the batch.
 // block: 0, or the size of the blocks of positions that a row's keys do not reach beyond (see key_range).
 // keep_first: the first keys of the sequence that stay readable behind a window; sink: [H] float32 or null.
-int kp_attention_split_sink(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
-                            const int* row_seg, const int* positions, void* out, int ldo, float* scratch, int n_chunks,
-                            float scale, int window, int block, int keep_first, const float* sink, int page_size, int n,
-                            int H, int G, int hd, int dtype, void* stream) {
+// cap: 0, or the bound of the scores; out_scale: factor of the output; pool: 0, or the positions of a pooled block, whose
+// means lie in pool_cache / pool_table, n_pool_chunks chunks of 256 of them at most (the scratch then has n_chunks +
+// n_pool_chunks slots a row and head).
+int kp_attention_split_pooled(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
+                              const int* row_seg, const int* positions, void* out, int ldo, float* scratch, int n_chunks,
+                              float scale, int window, int block, int keep_first, const float* sink, float cap, float out_scale,
+                              int pool, const void* pool_cache, const int* pool_table, int max_pool_blocks, int n_pool_chunks,
+                              int page_size, int n, int H, int G, int hd, int dtype, void* stream) {
     if (n <= 0) return 0;
+    if (cap < 0.f || pool < 0 || (pool > 0 && (window <= 0 || block > 0 || keep_first > 0 || !pool_cache || !pool_table || n_pool_chunks < 1)))
+        return KP_ERR_BAD_ARG;
+    if (pool == 0) n_pool_chunks = 0;
     if (keep_first < 0 || (keep_first > 0 && block > 0)) return KP_ERR_BAD_ARG;
     if (window <= 0) keep_first = 0;
     if (hd < 16 || hd > KP_MAX_HEAD_DIM || (hd & 15)) return KP_ERR_UNSUPPORTED;
@@ -440,14 +454,14 @@ int kp_attention_split_sink(const void* q, int ldq, const void* cache, const int
     const int R = H / G;
     const size_t smem = split_smem_bytes(R, hd);
     float* part_acc = scratch;
-    float* part_ml = scratch + (size_t)n * H * n_chunks * hd;
+    const int n_slots = n_chunks + n_pool_chunks;
+    float* part_ml = scratch + (size_t)n * H * n_slots * hd;
     cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(n_chunks, G, n);
     constexpr int SLOT0 = 0, FRONT = 0;
 #define AD_LAUNCH(T, HD, RR)                                                                                      \
-    kp_launch_pdl(attn_split_kernel<T, HD, RR>, dim3(grid), dim3(AD_THREADS), smem, s, (const T*)q, ldq, (const T*)cache, block_table,       \
+    kp_launch_pdl(attn_split_kernel<T, HD, RR>, dim3(n_chunks, G, n), dim3(AD_THREADS), smem, s, (const T*)q, ldq, (const T*)cache, block_table,       \
                                                                 max_blocks, row_seg, positions, part_acc, part_ml,    \
-                                                                n_chunks, scale, window, page_size, H, G, hd, block, keep_first, SLOT0, FRONT)
+                                                                n_slots, scale, window, page_size, H, G, hd, block, keep_first, SLOT0, FRONT, cap, 0)
     KP_DISPATCH_DTYPE(dtype, T, {
         cudaError_t e0;
         if (hd == 64 && R == 4) e0 = AD_LAUNCH(T, 64, 4);
@@ -455,10 +469,25 @@ int kp_attention_split_sink(const void* q, int ldq, const void* cache, const int
         else if (hd == 128) e0 = AD_LAUNCH(T, 128, 0);
         else e0 = AD_LAUNCH(T, 0, 0);
         if (e0 != cudaSuccess) { cudaGetLastError(); return (int)e0; }      // the first launch that failed
-        return launch_merge<T>(part_acc, part_ml, positions, out, ldo, n_chunks, AD_CHUNK, window, block, keep_first, sink, n, H, hd, s);
+        if (pool > 0) {
+            kp_launch_pdl(attn_split_kernel<T, 0, 0>, dim3(n_pool_chunks, G, n), dim3(AD_THREADS), smem, s, (const T*)q, ldq, (const T*)pool_cache,
+                          pool_table, max_pool_blocks, row_seg, positions, part_acc, part_ml, n_slots, scale, window, page_size, H, G,
+                          hd, 0, 0, n_chunks, 2, cap, pool);
+        }
+        return launch_merge<T>(part_acc, part_ml, positions, out, ldo, n_slots, AD_CHUNK, window, block, keep_first, sink, n, H, hd, s,
+                               pool > 0 ? n_chunks : -1, out_scale, pool);
     });
 #undef AD_LAUNCH
     return kp_launch_status();
+}
+
+int kp_attention_split_sink(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
+                            const int* row_seg, const int* positions, void* out, int ldo, float* scratch, int n_chunks,
+                            float scale, int window, int block, int keep_first, const float* sink, int page_size, int n,
+                            int H, int G, int hd, int dtype, void* stream) {
+    return kp_attention_split_pooled(q, ldq, cache, block_table, max_blocks, row_seg, positions, out, ldo, scratch, n_chunks, scale,
+                                     window, block, keep_first, sink, 0.f, 1.f, 0, nullptr, nullptr, 0, 0, page_size, n, H, G, hd,
+                                     dtype, stream);
 }
 
 int kp_attention_split_masked(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
@@ -493,21 +522,31 @@ int kp_attention_front_chunks(const void* q, int ldq, const void* cache, const i
     float* part_ml = scratch + (size_t)n * H * n_chunks * hd;
     KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(attn_split_kernel<T, 0, 0>, dim3(n_front, G, n), dim3(AD_THREADS), smem, (cudaStream_t)stream,
                                                (const T*)q, ldq, (const T*)cache, block_table, max_blocks, row_seg, positions, part_acc,
-                                               part_ml, n_chunks, scale, window, page_size, H, G, hd, 0, keep_first, front_slot0, 1)));
+                                               part_ml, n_chunks, scale, window, page_size, H, G, hd, 0, keep_first, front_slot0, 1, 0.f, 0)));
     return kp_launch_status();
 }
 
 // front_slot0: -1, or the slot from which the kept first keys' chunks lie (see kp_attention_front_chunks).
-int kp_attention_merge_sink(const int* positions, void* out, int ldo, const float* scratch, int n_chunks,
-                            int chunk_keys, int window, int block, int keep_first, const float* sink, int front_slot0, int n,
-                            int H, int hd, int dtype, void* stream) {
+// out_scale: factor of the output; pool > 0: the slots from front_slot0 on hold chunks of 256 pooled entries instead.
+int kp_attention_merge_pooled(const int* positions, void* out, int ldo, const float* scratch, int n_chunks,
+                              int chunk_keys, int window, int block, int keep_first, const float* sink, int front_slot0,
+                              float out_scale, int pool, int n, int H, int hd, int dtype, void* stream) {
+    if (pool < 0 || (pool > 0 && (window <= 0 || keep_first > 0 || front_slot0 < 0))) return KP_ERR_BAD_ARG;
     if (n <= 0) return 0;
     if (hd < 16 || hd > KP_MAX_HEAD_DIM || n > 65535 || chunk_keys < 1) return KP_ERR_UNSUPPORTED;
     const float* part_acc = scratch;
     const float* part_ml = scratch + (size_t)n * H * n_chunks * hd;
     KP_DISPATCH_DTYPE(dtype, T, return launch_merge<T>(part_acc, part_ml, positions, out, ldo, n_chunks, chunk_keys, window,
-                                                       block, keep_first, sink, n, H, hd, (cudaStream_t)stream, front_slot0));
+                                                       block, keep_first, sink, n, H, hd, (cudaStream_t)stream, front_slot0,
+                                                       out_scale, pool));
     return kp_launch_status();
+}
+
+int kp_attention_merge_sink(const int* positions, void* out, int ldo, const float* scratch, int n_chunks,
+                            int chunk_keys, int window, int block, int keep_first, const float* sink, int front_slot0, int n,
+                            int H, int hd, int dtype, void* stream) {
+    return kp_attention_merge_pooled(positions, out, ldo, scratch, n_chunks, chunk_keys, window, block, keep_first, sink, front_slot0,
+                                     1.f, 0, n, H, hd, dtype, stream);
 }
 
 int kp_attention_merge_masked(const int* positions, void* out, int ldo, const float* scratch, int n_chunks,

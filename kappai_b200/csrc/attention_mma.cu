@@ -16,59 +16,19 @@
 //    causal limit, double-buffered.
 //
 // Formulas as in attention.cu (src/backend/cpu/scalar/core.c:383-433).  Tiles
+// Variants, each an argument: `cap` > 0 bounds the scores (cap tanh(s / cap); these instantiations always keep the
+// softmax weights whole); `pool` > 0 (with a window): the rows also read the means of the blocks of `pool` positions
+// that lie wholly before their windows, from a cache and a block table of their own.  The prefill kernel takes their
+// tiles first; the split kernels run once more over them, into slots of their own (slot0 on), which the merge takes
+// in front of the window's chunks.  Tiles
 // start at multiples of 64 of the absolute key index, chunks at multiples of
 // 256, so the order of summation does not depend on how a prompt was cut or
 // what else is in the batch.
-#include "tma.cuh"
+#include "mma.cuh"
 
 #define AM_TILE 64
 #define AM_CHUNK 256
 #define AM_RMAX 8
-
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
-    const int sz = valid ? 16 : 0;                  // size 0: the 16 bytes are filled with zeros
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(sz) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
-                                         uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
-                 "{%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-// `bytes` (a multiple of 16, both addresses 16-byte aligned) from global to shared memory; completes on `bar`
-__device__ __forceinline__ void kp_bulk_g2s(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                 ::"r"(kp_smem_u32(dst)), "l"(src), "r"(bytes), "r"(kp_smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<uint32_t*>(&v);
-}
-
-// Softmax weights in full: a float32 value is the exact sum of three bfloat16 parts (8 significant bits each), so
-// the product with V can be taken part by part on the tensor cores and added up in float32 without rounding the
-// weights.  Packs the next part of (a, b) and leaves in them what it did not take.
-__device__ __forceinline__ uint32_t pack_bf16_part(float& a, float& b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    a -= __low2float(h);
-    b -= __high2float(h);
-    return *reinterpret_cast<const uint32_t*>(&h);
-}
 
 // A tile in shared memory: 64 rows (keys) of HD bf16, as HD / 64 halves of 64 rows x 128 bytes; in a half the
 // 16-byte chunk c of row r lies at chunk c ^ (r & 7).  This is what a TMA box of 64 columns with the 128-byte
@@ -142,13 +102,13 @@ __device__ __forceinline__ void pv_tile(float (&o)[HD / 8][4], const uint32_t (&
 // it, and a multiple of 8.  Boxes wholly outside the row's keys are not loaded; V rows outside them are zeroed.
 KP_STATUS_WORD(g_attn_status, attention_mma)          // 0 ok; 1: a bounded wait gave up
 
-template <int HD, int NW, bool TMA, bool EXACT>
+template <int HD, int NW, bool TMA, int MODE>
 __global__ void __launch_bounds__(NW * 32)
 attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __restrict__ q, int ldq, const bf16* __restrict__ cache,
                       const int* __restrict__ block_table, int max_blocks, const int* __restrict__ row_seg,
                       const int* __restrict__ positions, float* __restrict__ part_acc, float* __restrict__ part_ml,
-                      int n_chunks, float scale, int window, int page_size, int H, int G, int block) {
-    constexpr bool exact_p = EXACT;                               // the softmax weights enter the product with V whole
+                      int n_slots, int slot0, float scale, int window, int page_size, int H, int G, int block, float cap, int pool) {
+    constexpr bool exact_p = MODE >= 1;                           // the softmax weights enter the product with V whole
     kp_pdl_begin_early_if(gridDim.z > 1);
     extern __shared__ unsigned char smem_dyn[];
     unsigned char* smem_raw = reinterpret_cast<unsigned char*>(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023);
@@ -164,7 +124,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __res
     const int chunk = blockIdx.x, kvh = blockIdx.y, row = blockIdx.z;
     const int R = H / G;
     const int pos = positions[row];
-    const int k_lo = kp_key_lo(pos, window, block), k_hi = pos;
+    const int k_lo = pool > 0 ? 0 : kp_key_lo(pos, window, block), k_hi = pool > 0 ? kp_pooled_count(pos, window, pool) - 1 : pos;
     const int c0 = chunk * CHUNK;
     if (c0 > k_hi || c0 + CHUNK - 1 < k_lo) return;
     const int* bt = block_table + (size_t)row_seg[row] * max_blocks;
@@ -246,7 +206,8 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __res
 #pragma unroll
         for (int i = 0; i < 2; i++) {
             const int key = t0 + nt * 8 + 2 * t + i;
-            const float v = (key >= k_lo && key <= k_hi) ? s[nt][i] * scale : -INFINITY;
+            const float sv = MODE == 2 ? kp_capped(s[nt][i] * scale, cap) : s[nt][i] * scale;
+            const float v = (key >= k_lo && key <= k_hi) ? sv : -INFINITY;
             s[nt][i] = v;
             m = fmaxf(m, v);
         }
@@ -304,7 +265,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __res
             const float mw = wm[w * AM_RMAX + r];
             if (mw != -INFINITY) acc = fmaf(wO[((size_t)w * AM_RMAX + r) * HD + d], expf(mw - M), acc);
         }
-        part_acc[(((size_t)row * H + kvh * R + r) * n_chunks + chunk) * HD + d] = acc;
+        part_acc[(((size_t)row * H + kvh * R + r) * n_slots + slot0 + chunk) * HD + d] = acc;
     }
     if (tid < R) {
         float M = -INFINITY, L = 0.f;
@@ -313,7 +274,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __res
             const float mw = wm[w * AM_RMAX + tid];
             if (mw != -INFINITY) L = fmaf(wl[w * AM_RMAX + tid], expf(mw - M), L);
         }
-        float* ml = part_ml + (((size_t)row * H + kvh * R + tid) * n_chunks + chunk) * 2;
+        float* ml = part_ml + (((size_t)row * H + kvh * R + tid) * n_slots + slot0 + chunk) * 2;
         ml[0] = M;
         ml[1] = L;
     }
@@ -343,13 +304,14 @@ static size_t ar_smem_bytes() {
            AR_GROUPS * sizeof(float) * (AR_NW * AM_RMAX * HD + 2 * AR_NW * AM_RMAX) + 32;
 }
 
-template <int HD, bool EXACT>
+template <int HD, int MODE>
 __global__ void __launch_bounds__(AR_THREADS)
 attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __restrict__ q, int ldq,
                        const int* __restrict__ block_table, int max_blocks, const int* __restrict__ row_seg,
                        const int* __restrict__ positions, float* __restrict__ part_acc, float* __restrict__ part_ml,
-                       int n_chunks, float scale, int window, int page_size, int H, int G, int n_rows, int block) {
-    constexpr bool exact_p = EXACT;
+                       int n_chunks, int n_slots, int slot0, float scale, int window, int page_size, int H, int G, int n_rows,
+                       int block, float cap, int pool) {
+    constexpr bool exact_p = MODE >= 1;
     kp_pdl_begin_early_if(n_rows > 1);
     extern __shared__ unsigned char smem_dyn[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023);
@@ -389,8 +351,8 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
                 c_kvh = rest % G;
                 c_row = rest / G;
                 const int pos = positions[c_row];
-                c_lo = kp_key_lo(pos, window, block);
-                c_hi = pos;
+                c_lo = pool > 0 ? 0 : kp_key_lo(pos, window, block);
+                c_hi = pool > 0 ? kp_pooled_count(pos, window, pool) - 1 : pos;
                 const int c0 = c_chunk * AR_CHUNK;
                 valid = !(c0 > c_hi || c0 + AR_CHUNK - 1 < c_lo);
                 if (valid) c_seg = row_seg[c_row];
@@ -505,7 +467,8 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
 #pragma unroll
             for (int i = 0; i < 2; i++) {
                 const int key = t0 + nt * 8 + 2 * t + i;
-                const float v = (key >= k_lo && key <= k_hi) ? sc[nt][i] * scale : -INFINITY;
+                const float sv = MODE == 2 ? kp_capped(sc[nt][i] * scale, cap) : sc[nt][i] * scale;
+                const float v = (key >= k_lo && key <= k_hi) ? sv : -INFINITY;
                 sc[nt][i] = v;
                 m = fmaxf(m, v);
             }
@@ -565,7 +528,7 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
                 const float mw = wm[w * AM_RMAX + r];
                 if (mw != -INFINITY) acc = fmaf(wO[((size_t)w * AM_RMAX + r) * HD + d], expf(mw - M), acc);
             }
-            part_acc[(((size_t)me.row * H + me.kvh * R + r) * n_chunks + me.chunk) * HD + d] = acc;
+            part_acc[(((size_t)me.row * H + me.kvh * R + r) * n_slots + slot0 + me.chunk) * HD + d] = acc;
         }
         if (gtid < R) {
             float M = -INFINITY, L = 0.f;
@@ -574,7 +537,7 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
                 const float mw = wm[w * AM_RMAX + gtid];
                 if (mw != -INFINITY) L = fmaf(wl[w * AM_RMAX + gtid], expf(mw - M), L);
             }
-            float* ml = part_ml + (((size_t)me.row * H + me.kvh * R + gtid) * n_chunks + me.chunk) * 2;
+            float* ml = part_ml + (((size_t)me.row * H + me.kvh * R + gtid) * n_slots + slot0 + me.chunk) * 2;
             ml[0] = M;
             ml[1] = L;
         }
@@ -588,14 +551,17 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
 // that hold them come first, then the tiles of the window, the tiles in between are left out.  sink (one float32 a
 // query head, or null): a row's running maximum and sum start at (sink_h, 1) instead of (-inf, 0), which is a key
 // with that score and no value.
-template <int HD, bool EXACT>
+// MODE 0: softmax weights rounded to bfloat16; 1: whole; 2: whole, with soft-capped scores and pooled blocks.
+template <int HD, int MODE>
 __global__ void __launch_bounds__(128)
 attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restrict__ cache,
                         const int* __restrict__ block_table, int max_blocks, const int* __restrict__ cu_rows,
                         const int* __restrict__ seg_pos, const int* __restrict__ tile_seg,
                         const int* __restrict__ tile_row0, bf16* __restrict__ out, int ldo, float scale, int window,
-                        int page_size, int H, int G, int block, int keep_first, const float* __restrict__ sink) {
-    constexpr bool exact_p = EXACT;
+                        int page_size, int H, int G, int block, int keep_first, const float* __restrict__ sink, float cap,
+                        float out_scale, int pool, const bf16* __restrict__ pool_cache, const int* __restrict__ pool_table,
+                        int max_pool_blocks) {
+    constexpr bool exact_p = MODE >= 1;
     kp_pdl_begin();
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* Ks = reinterpret_cast<bf16*>(smem_raw);                 // [2][64][HD]
@@ -616,7 +582,11 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
     const int k_hi_all = pos0 + n_rows - 1;
     const int k_lo_all = kp_key_lo(pos0, window, block);
     const int tile_lo = k_lo_all / AM_TILE, tile_hi = k_hi_all / AM_TILE;
-    const int n_front = keep_first > 0 ? min(tile_lo, (keep_first + AM_TILE - 1) / AM_TILE) : 0;   // tiles of kept first keys
+    const bool pooled = MODE == 2 && pool > 0;
+    const int n_pool = pooled ? kp_pooled_count(k_hi_all, window, pool) : 0;          // pooled entries the tile's last row sees
+    const int n_front = pooled ? (n_pool + AM_TILE - 1) / AM_TILE                     // tiles of pooled entries, or of kept first keys
+                               : (keep_first > 0 ? min(tile_lo, (keep_first + AM_TILE - 1) / AM_TILE) : 0);
+    const int* ptab = pooled ? pool_table + (size_t)seg * max_pool_blocks : nullptr;
     const int n_kt = n_front + tile_hi - tile_lo + 1;
 
     // this warp's 16 rows: rows r0 = warp*16 + g and r0 + 8
@@ -645,16 +615,22 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
     const float m_start = sink ? sink[h] : -INFINITY, l_start = sink ? 1.f : 0.f;
     float m_a = m_start, m_b = m_start, l_a = l_start, l_b = l_start;
 
-    load_kv_tile<HD>(Ks, Vs, cache, bt, page_stride, k_off, v_off, page_size, (n_front ? 0 : tile_lo) * AM_TILE, k_lo_all, k_hi_all,
-                     tid, 128, keep_first);
+    auto load = [&](int it, int buf) {                             // the it-th tile of the walk into buffer buf
+        bf16* kd = Ks + buf * AM_TILE * HD;
+        bf16* vd = Vs + buf * AM_TILE * HD;
+        if (MODE == 2 && pooled && it < n_front)
+            load_kv_tile<HD>(kd, vd, pool_cache, ptab, page_stride, k_off, v_off, page_size, it * AM_TILE, 0, n_pool - 1, tid, 128);
+        else
+            load_kv_tile<HD>(kd, vd, cache, bt, page_stride, k_off, v_off, page_size, (it < n_front ? it : tile_lo + (it - n_front)) * AM_TILE,
+                             k_lo_all, k_hi_all, tid, 128, keep_first);
+    };
+    load(0, 0);
     cp_async_commit();
     for (int it = 0; it < n_kt; it++) {
         const int kt = it < n_front ? it : tile_lo + (it - n_front);
         const int buf = it & 1;
         if (it + 1 < n_kt) {
-            const int kt_next = it + 1 < n_front ? it + 1 : tile_lo + (it + 1 - n_front);
-            load_kv_tile<HD>(Ks + (buf ^ 1) * AM_TILE * HD, Vs + (buf ^ 1) * AM_TILE * HD, cache, bt, page_stride, k_off,
-                             v_off, page_size, kt_next * AM_TILE, k_lo_all, k_hi_all, tid, 128, keep_first);
+            load(it + 1, buf ^ 1);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -665,7 +641,11 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
         // a warp whose rows all lie before this tile (causal) or after its window has nothing to do in it
         const int w_pos_hi = pos0 + min(warp * 16 + 15, n_rows - 1);
         const int w_lo = kp_key_lo(pos0 + warp * 16, window, block);
-        if (warp * 16 < n_rows && t0 <= w_pos_hi && (t0 + AM_TILE - 1 >= w_lo || t0 < keep_first)) {
+        // (a tile of pooled entries: a row reads the entries below its own count)
+        const bool front = MODE == 2 && pooled && it < n_front;
+        const int cnt_a = front ? kp_pooled_count(pos_a, window, pool) : 0, cnt_b = front ? kp_pooled_count(pos_b, window, pool) : 0;
+        if (warp * 16 < n_rows && (front ? t0 < kp_pooled_count(w_pos_hi, window, pool)
+                                         : t0 <= w_pos_hi && (t0 + AM_TILE - 1 >= w_lo || t0 < keep_first))) {
             float s[8][4];
             qk_tile<HD>(s, qf, Ks + buf * AM_TILE * HD, lane);
             float mx_a = -INFINITY, mx_b = -INFINITY;
@@ -674,8 +654,12 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
 #pragma unroll
                 for (int i = 0; i < 2; i++) {
                     const int key = t0 + nt * 8 + 2 * t + i;
-                    const float va = (has_a && key <= pos_a && (key >= lo_a || key < keep_first)) ? s[nt][i] * scale : -INFINITY;
-                    const float vb = (has_b && key <= pos_b && (key >= lo_b || key < keep_first)) ? s[nt][2 + i] * scale : -INFINITY;
+                    const bool in_a = front ? key < cnt_a : key <= pos_a && (key >= lo_a || key < keep_first);
+                    const bool in_b = front ? key < cnt_b : key <= pos_b && (key >= lo_b || key < keep_first);
+                    const float ca_ = MODE == 2 ? kp_capped(s[nt][i] * scale, cap) : s[nt][i] * scale;
+                    const float cb_ = MODE == 2 ? kp_capped(s[nt][2 + i] * scale, cap) : s[nt][2 + i] * scale;
+                    const float va = has_a && in_a ? ca_ : -INFINITY;
+                    const float vb = has_b && in_b ? cb_ : -INFINITY;
                     s[nt][i] = va; s[nt][2 + i] = vb;
                     mx_a = fmaxf(mx_a, va); mx_b = fmaxf(mx_b, vb);
                 }
@@ -724,7 +708,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
         }
         __syncthreads();                                          // the buffer is free for the load after next
     }
-    const float ia = l_a > 0.f ? 1.0f / l_a : 0.f, ib = l_b > 0.f ? 1.0f / l_b : 0.f;
+    const float ia = l_a > 0.f ? out_scale / l_a : 0.f, ib = l_b > 0.f ? out_scale / l_b : 0.f;
     if (has_a) {
         bf16* oa = out + (size_t)(row0 + ra) * ldo + (size_t)h * HD;
 #pragma unroll
@@ -755,7 +739,8 @@ static int am_n_sm() {
 template <int HD, int NW>
 static int launch_split(const void* q, int ldq, const void* cache, long long n_pages, const int* block_table,
                         int max_blocks, const int* row_seg, const int* positions, float* part_acc, float* part_ml,
-                        int n_chunks, float scale, int window, int block, int exact_p, int page_size, int n, int H, int G, cudaStream_t s) {
+                        int n_chunks, int n_slots, int slot0, float scale, int window, int block, int mode, float cap, int pool,
+                        int page_size, int n, int H, int G, cudaStream_t s) {
     const size_t smem = 1024 + (size_t)2 * NW * AM_TILE * HD * 2 + sizeof(float) * (NW * AM_RMAX * HD + 2 * NW * AM_RMAX) + 16;
     alignas(64) CUtensorMap tm = {};
     // tiles by TMA where the pages allow it (and the cache is known by its size), else by cp.async
@@ -769,44 +754,47 @@ static int launch_split(const void* q, int ldq, const void* cache, long long n_p
             const size_t rs = ar_smem_bytes<HD>();
             static bool ready = false;
             if (!ready) {
-                cudaError_t e = cudaFuncSetAttribute(attn_split_ring_kernel<HD, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rs);
-                if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_ring_kernel<HD, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rs);
+                cudaError_t e = cudaFuncSetAttribute(attn_split_ring_kernel<HD, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rs);
+                if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_ring_kernel<HD, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rs);
+                if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_ring_kernel<HD, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rs);
                 if (e != cudaSuccess) return (int)e;
                 ready = true;
             }
             const long long items = (long long)n * G * n_chunks;
             const int sms = am_n_sm();
-            kp_launch_pdl(exact_p ? attn_split_ring_kernel<HD, true> : attn_split_ring_kernel<HD, false>,
+            kp_launch_pdl(mode == 2 ? attn_split_ring_kernel<HD, 2> : (mode ? attn_split_ring_kernel<HD, 1> : attn_split_ring_kernel<HD, 0>),
                           dim3((unsigned)(items < sms ? items : sms)), dim3(AR_THREADS), rs, s, tm,
-                          (const bf16*)q, ldq, block_table, max_blocks, row_seg, positions, part_acc, part_ml, n_chunks, scale,
-                          window, page_size, H, G, n, block);
+                          (const bf16*)q, ldq, block_table, max_blocks, row_seg, positions, part_acc, part_ml, n_chunks, n_slots, slot0,
+                          scale, window, page_size, H, G, n, block, cap, pool);
             return kp_launch_status();
         }
     }
-    auto kern = tma ? (exact_p ? attn_split_mma_kernel<HD, NW, true, true> : attn_split_mma_kernel<HD, NW, true, false>)
-                    : (exact_p ? attn_split_mma_kernel<HD, NW, false, true> : attn_split_mma_kernel<HD, NW, false, false>);
+    auto kern = tma ? (mode == 2 ? attn_split_mma_kernel<HD, NW, true, 2> : (mode ? attn_split_mma_kernel<HD, NW, true, 1> : attn_split_mma_kernel<HD, NW, true, 0>))
+                    : (mode == 2 ? attn_split_mma_kernel<HD, NW, false, 2> : (mode ? attn_split_mma_kernel<HD, NW, false, 1> : attn_split_mma_kernel<HD, NW, false, 0>));
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
     kp_launch_pdl(kern, dim3(dim3(n_chunks, G, n)), dim3(NW * 32), smem, s, tm,
         (const bf16*)q, ldq, (const bf16*)cache, block_table, max_blocks, row_seg, positions, part_acc, part_ml,
-        n_chunks, scale, window, page_size, H, G, block);
+        n_slots, slot0, scale, window, page_size, H, G, block, cap, pool);
     return kp_launch_status();
 }
 
 template <int HD>
 static int launch_prefill(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
                           const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0, int n_tiles,
-                          void* out, int ldo, float scale, int window, int block, int keep_first, const float* sink, int exact_p,
+                          void* out, int ldo, float scale, int window, int block, int keep_first, const float* sink, int mode,
+                          float cap, float out_scale, int pool, const void* pool_cache, const int* pool_table, int max_pool_blocks,
                           int page_size, int H, int G, cudaStream_t s) {
     const size_t smem = (size_t)4 * AM_TILE * HD * 2;
-    auto kern = exact_p ? attn_prefill_mma_kernel<HD, true> : attn_prefill_mma_kernel<HD, false>;
+    auto kern = mode == 2 ? attn_prefill_mma_kernel<HD, 2> : (mode ? attn_prefill_mma_kernel<HD, 1> : attn_prefill_mma_kernel<HD, 0>);
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     kp_launch_pdl(kern, dim3(dim3(n_tiles, H)), dim3(128), smem, s, 
         (const bf16*)q, ldq, (const bf16*)cache, block_table, max_blocks, cu_rows, seg_pos, tile_seg, tile_row0,
-        (bf16*)out, ldo, scale, window, page_size, H, G, block, window > 0 ? keep_first : 0, sink);
+        (bf16*)out, ldo, scale, window, page_size, H, G, block, window > 0 ? keep_first : 0, sink, cap, out_scale, pool,
+        (const bf16*)pool_cache, pool_table, max_pool_blocks);
     return kp_launch_status();
 }
 
@@ -815,21 +803,27 @@ extern "C" {
 // The chunk partials of the split pass (bfloat16, head size 64 or 128, H/G <= 8); chunks of `chunk_keys` keys
 // (64, 128 or 256), n_chunks of them, into `scratch` (n * H * n_chunks * (hd + 2) floats).  The caller runs the
 // merge of attention_decode.cu afterwards (kp_attention_merge, same chunk size) on the same scratch.
-int kp_attention_split_mma_masked(const void* q, int ldq, const void* cache, long long n_pages, const int* block_table,
+// n_slots: slots a (row, head) has in the scratch; the chunks go to slots slot0 on.  cap: 0, or the bound of the scores
+// (the weights are then kept whole); pool > 0: `cache` and `block_table` hold the means of blocks of `pool` positions, and
+// a row reads those that lie wholly before its window.
+int kp_attention_split_mma_pooled(const void* q, int ldq, const void* cache, long long n_pages, const int* block_table,
                                   int max_blocks, const int* row_seg, const int* positions, float* scratch, int n_chunks,
-                                  int chunk_keys, float scale, int window, int block, int exact_p, int page_size, int n, int H,
-                                  int G, int hd, void* stream) {
+                                  int n_slots, int slot0, int chunk_keys, float scale, int window, int block, int exact_p,
+                                  float cap, int pool, int page_size, int n, int H, int G, int hd, void* stream) {
     if (n <= 0) return 0;
-    if (block < 0) return KP_ERR_BAD_ARG;
+    if (block < 0 || cap < 0.f || pool < 0 || slot0 < 0 || (pool > 0 && window <= 0)) return KP_ERR_BAD_ARG;
+    // (the chunks that no row reaches need no slots: only those below n_slots - slot0 are run)
+    if (n_chunks > n_slots - slot0) return KP_ERR_BAD_ARG;
+    const int mode = cap > 0.f ? 2 : (exact_p ? 1 : 0);
     if ((hd != 64 && hd != 128) || G < 1 || H % G || H / G > AM_RMAX || page_size < 1 || n_chunks < 1 || n > 65535 ||
         G > 65535 || (ldq & 1) || (chunk_keys != 64 && chunk_keys != 128 && chunk_keys != 256))
         return KP_ERR_UNSUPPORTED;
     float* part_acc = scratch;
-    float* part_ml = scratch + (size_t)n * H * n_chunks * hd;
+    float* part_ml = scratch + (size_t)n * H * n_slots * hd;
     cudaStream_t s = (cudaStream_t)stream;
 #define AM_SPLIT(HD, NW)                                                                                          \
     return launch_split<HD, NW>(q, ldq, cache, n_pages, block_table, max_blocks, row_seg, positions, part_acc, part_ml, \
-                                n_chunks, scale, window, block, exact_p, page_size, n, H, G, s)
+                                n_chunks, n_slots, slot0, scale, window, block, mode, cap, pool, page_size, n, H, G, s)
     if (hd == 64) {
         if (chunk_keys == 64) AM_SPLIT(64, 1);
         if (chunk_keys == 128) AM_SPLIT(64, 2);
@@ -839,6 +833,14 @@ int kp_attention_split_mma_masked(const void* q, int ldq, const void* cache, lon
     if (chunk_keys == 128) AM_SPLIT(128, 2);
     AM_SPLIT(128, 4);
 #undef AM_SPLIT
+}
+
+int kp_attention_split_mma_masked(const void* q, int ldq, const void* cache, long long n_pages, const int* block_table,
+                                  int max_blocks, const int* row_seg, const int* positions, float* scratch, int n_chunks,
+                                  int chunk_keys, float scale, int window, int block, int exact_p, int page_size, int n, int H,
+                                  int G, int hd, void* stream) {
+    return kp_attention_split_mma_pooled(q, ldq, cache, n_pages, block_table, max_blocks, row_seg, positions, scratch, n_chunks,
+                                         n_chunks, 0, chunk_keys, scale, window, block, exact_p, 0.f, 0, page_size, n, H, G, hd, stream);
 }
 
 int kp_attention_split_mma(const void* q, int ldq, const void* cache, long long n_pages, const int* block_table, int max_blocks,
@@ -852,19 +854,36 @@ int kp_attention_split_mma(const void* q, int ldq, const void* cache, long long 
 // block: 0, or the size of the blocks of positions beyond whose start a row reads no key.  exact_p: 1 takes the
 // softmax weights into the product with V whole (three bfloat16 parts), 0 rounded to bfloat16.
 // keep_first: the first keys of the sequence that stay readable behind a window; sink: [H] float32 or null.
-int kp_attention_prefill_mma_sink(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
-                                  const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0,
-                                  int n_tiles, void* out, int ldo, float scale, int window, int block, int keep_first,
-                                  const float* sink, int exact_p, int page_size, int H, int G, int hd, void* stream) {
+// cap: 0, or the bound of the scores; out_scale: factor of the output; pool: 0, or the positions of a pooled block, whose
+// means lie in pool_cache / pool_table.
+int kp_attention_prefill_mma_pooled(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
+                                    const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0,
+                                    int n_tiles, void* out, int ldo, float scale, int window, int block, int keep_first,
+                                    const float* sink, int exact_p, float cap, float out_scale, int pool, const void* pool_cache,
+                                    const int* pool_table, int max_pool_blocks, int page_size, int H, int G, int hd, void* stream) {
     if (n_tiles <= 0) return 0;
+    if (cap < 0.f || pool < 0 || (pool > 0 && (window <= 0 || block > 0 || keep_first > 0 || !pool_cache || !pool_table)))
+        return KP_ERR_BAD_ARG;
+    const int mode = (cap > 0.f || pool > 0) ? 2 : (exact_p ? 1 : 0);
     if (block < 0 || keep_first < 0 || (keep_first > 0 && block > 0)) return KP_ERR_BAD_ARG;
     if ((hd != 64 && hd != 128) || G < 1 || H % G || page_size < 1 || H > 65535 || (ldq & 1) || (ldo & 1))
         return KP_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     if (hd == 64) return launch_prefill<64>(q, ldq, cache, block_table, max_blocks, cu_rows, seg_pos, tile_seg, tile_row0,
-                                            n_tiles, out, ldo, scale, window, block, keep_first, sink, exact_p, page_size, H, G, s);
+                                            n_tiles, out, ldo, scale, window, block, keep_first, sink, mode, cap, out_scale, pool,
+                                            pool_cache, pool_table, max_pool_blocks, page_size, H, G, s);
     return launch_prefill<128>(q, ldq, cache, block_table, max_blocks, cu_rows, seg_pos, tile_seg, tile_row0, n_tiles,
-                               out, ldo, scale, window, block, keep_first, sink, exact_p, page_size, H, G, s);
+                               out, ldo, scale, window, block, keep_first, sink, mode, cap, out_scale, pool, pool_cache, pool_table,
+                               max_pool_blocks, page_size, H, G, s);
+}
+
+int kp_attention_prefill_mma_sink(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,
+                                  const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0,
+                                  int n_tiles, void* out, int ldo, float scale, int window, int block, int keep_first,
+                                  const float* sink, int exact_p, int page_size, int H, int G, int hd, void* stream) {
+    return kp_attention_prefill_mma_pooled(q, ldq, cache, block_table, max_blocks, cu_rows, seg_pos, tile_seg, tile_row0, n_tiles, out,
+                                           ldo, scale, window, block, keep_first, sink, exact_p, 0.f, 1.f, 0, nullptr, nullptr, 0,
+                                           page_size, H, G, hd, stream);
 }
 
 int kp_attention_prefill_mma_masked(const void* q, int ldq, const void* cache, const int* block_table, int max_blocks,

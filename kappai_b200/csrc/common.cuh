@@ -45,6 +45,13 @@ __device__ __forceinline__ float kp_act_rt(int act, float g) {
     return act == KP_ACT_RELU ? kp_act<KP_ACT_RELU>(g) : (act == KP_ACT_GELU_TANH ? kp_act<KP_ACT_GELU_TANH>(g) : kp_act<KP_ACT_SILU>(g));
 }
 
+// The ungated units' activations (the same codes, and the square of relu).
+#define KP_ACT_RELU_SQ 4
+__device__ __forceinline__ float kp_act_plain(int act, float v) {
+    if (act == KP_ACT_RELU_SQ) { const float r = fmaxf(v, 0.f); return r * r; }
+    return kp_act_rt(act, v);
+}
+
 // For the epilogues of the products (a choice at run time: silu unless another is asked for).  A launcher's
 // `epi` argument carries the activation of its gated epilogue in bits 8 and up.
 __device__ __forceinline__ float kp_act_epilogue(int act, float g) {
@@ -75,6 +82,12 @@ __device__ __forceinline__ int kp_key_lo(int pos, int window, int block) {
     if (block > 0) lo = max(lo, (pos / block) * block);
     return lo;
 }
+
+// The blocks of `pool` positions that a row at position `pos` sees the means of: those that lie wholly before its window
+// of `window` keys, blocks 0 .. count - 1.  Non-decreasing in pos.
+__device__ __forceinline__ int kp_pooled_count(int pos, int window, int pool) { return max(0, pos - window + 1) / pool; }
+// A score bounded smoothly by `cap` (0: as it is).
+__device__ __forceinline__ float kp_capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

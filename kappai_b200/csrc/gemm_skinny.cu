@@ -23,6 +23,7 @@
 #define EPI_STORE_F32 1
 #define EPI_ACCUM_F32 2
 #define EPI_SWIGLU 3
+#define EPI_ACT 6        // store bf16 behind an ungated activation (common.cuh, kp_act_plain)
 
 #define SK_WARPS 8
 #define SK_U 4                 // k-blocks of 32 a warp has in flight per stage
@@ -166,6 +167,8 @@ gemm_skinny_kernel(const SkinnyArgs p) {
             ((bf16*)p.C)[o] = from_f32<bf16>(kp_gated_epilogue(p.act, gq, uq, p.glu_limit, p.glu_alpha, p.glu_shift));
         } else if (EPI == EPI_STORE) {
             ((bf16*)p.C)[o] = from_f32<bf16>(v);
+        } else if (EPI == EPI_ACT) {
+            ((bf16*)p.C)[o] = from_f32<bf16>(kp_act_plain(p.act, v));
         } else if (EPI == EPI_STORE_F32) {
             ((float*)p.C)[o] = v;
         } else {
@@ -199,6 +202,7 @@ static int launch_epi(const SkinnyArgs& a, int epi, cudaStream_t s) {
         case EPI_STORE_F32: return launch_pdl(gemm_skinny_kernel<MT, HALF, EPI_STORE_F32>, grid, s, a);
         case EPI_ACCUM_F32: return launch_pdl(gemm_skinny_kernel<MT, HALF, EPI_ACCUM_F32>, grid, s, a);
         case EPI_SWIGLU: return launch_pdl(gemm_skinny_kernel<MT, HALF, EPI_SWIGLU>, grid, s, a);
+        case EPI_ACT: return launch_pdl(gemm_skinny_kernel<MT, HALF, EPI_ACT>, grid, s, a);
         default: return KP_ERR_BAD_ARG;
     }
 }
@@ -245,7 +249,8 @@ static int skinny_run(const void* A, int lda, const void* W, int ldw, const floa
     SkinnyArgs a = {};
     a.act = KP_EPI_ACT(epi);
     epi = KP_EPI_KIND(epi);
-    if (a.act != KP_ACT_SILU && a.act != KP_ACT_RELU && a.act != KP_ACT_GELU_TANH && !(a.act == KP_ACT_GLU_CLAMPED && glu)) return KP_ERR_UNSUPPORTED;
+    if (a.act != KP_ACT_SILU && a.act != KP_ACT_RELU && a.act != KP_ACT_GELU_TANH && !(a.act == KP_ACT_GLU_CLAMPED && glu) &&
+        !(a.act == KP_ACT_RELU_SQ && epi == EPI_ACT)) return KP_ERR_UNSUPPORTED;
     if (glu) { a.glu_limit = glu[0]; a.glu_alpha = glu[1]; a.glu_shift = glu[2]; }
     int st = check_common(M, N, K, ldw, W, epi, &a.ff);
     if (st) return st;

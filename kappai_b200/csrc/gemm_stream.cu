@@ -33,6 +33,7 @@
 #define EPI_STORE_F32 1
 #define EPI_ACCUM_F32 2
 #define EPI_SWIGLU 3
+#define EPI_ACT 6                            // store bf16 behind an ungated activation (common.cuh, kp_act_plain)
 #define EPI_CONV_STEP 4                      // W = [B; C; X] rows (in_proj of the gated short convolution): the conv step of
                                              // one-row segments runs in the epilogue, with the state update
 
@@ -322,6 +323,8 @@ gemm_stream_kernel(const StreamArgs p) {
                 ((bf16*)p.C)[o] = from_f32<bf16>(kp_gated_epilogue(p.act, gq, uq, p.glu_limit, p.glu_alpha, p.glu_shift));
             } else if (EPI == EPI_STORE) {
                 ((bf16*)p.C)[o] = from_f32<bf16>(v);
+            } else if (EPI == EPI_ACT) {
+                ((bf16*)p.C)[o] = from_f32<bf16>(kp_act_plain(p.act, v));
             } else if (EPI == EPI_STORE_F32) {
                 ((float*)p.C)[o] = v;
             } else {
@@ -388,6 +391,7 @@ static int launch_epi(StreamArgs a, int epi, cudaStream_t s) {
         case EPI_STORE_F32: return launch_pdl(gemm_stream_kernel<MT, HALF, EPI_STORE_F32, WIDE>, grid, sm, s, a);
         case EPI_ACCUM_F32: return launch_pdl(gemm_stream_kernel<MT, HALF, EPI_ACCUM_F32, WIDE>, grid, sm, s, a);
         case EPI_SWIGLU: return launch_pdl(gemm_stream_kernel<MT, HALF, EPI_SWIGLU, false>, grid, sm, s, a);
+        case EPI_ACT: return launch_pdl(gemm_stream_kernel<MT, HALF, EPI_ACT, WIDE>, grid, sm, s, a);
         case EPI_CONV_STEP:
             // at most 16 rows: from 32 rows on the tensor-core kernel and the separate conv kernel are faster (measured)
             if constexpr (MT == 1) return launch_pdl(gemm_stream_kernel<MT, HALF, EPI_CONV_STEP, false>, grid, sm, s, a);
@@ -441,7 +445,8 @@ static int stream_run(const void* A, int lda, const void* W, int ldw, const floa
     StreamArgs a = {};
     a.act = KP_EPI_ACT(epi);
     epi = KP_EPI_KIND(epi);
-    if (a.act != KP_ACT_SILU && a.act != KP_ACT_RELU && a.act != KP_ACT_GELU_TANH && !(a.act == KP_ACT_GLU_CLAMPED && glu)) return KP_ERR_UNSUPPORTED;
+    if (a.act != KP_ACT_SILU && a.act != KP_ACT_RELU && a.act != KP_ACT_GELU_TANH && !(a.act == KP_ACT_GLU_CLAMPED && glu) &&
+        !(a.act == KP_ACT_RELU_SQ && epi == EPI_ACT)) return KP_ERR_UNSUPPORTED;
     if (glu) { a.glu_limit = glu[0]; a.glu_alpha = glu[1]; a.glu_shift = glu[2]; }
     int st = check_common(a, M, N, K, ldw, W, epi);
     if (st) return st;

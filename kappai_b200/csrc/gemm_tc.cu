@@ -42,6 +42,7 @@
 #define EPI_STORE_F32 1
 #define EPI_ACCUM_F32 2
 #define EPI_SWIGLU 3
+#define EPI_ACT 6                            // store bf16 behind an ungated activation (common.cuh, kp_act_plain)
 #define EPI_GLU 4                            // inside this file only: EPI_SWIGLU whose unit is the one with limits (act code 3)
 #define TC_GATED(E) ((E) == EPI_SWIGLU || (E) == EPI_GLU)
 
@@ -104,10 +105,11 @@ __device__ __forceinline__ void tc_finish(const TcArgs& p, int n_lim, const floa
             const float gq = to_f32(from_f32<bf16>(x)), uq = to_f32(from_f32<bf16>(up));
             x = EPI == EPI_GLU ? kp_glu_clamped(gq, uq, p.glu_limit, p.glu_alpha, p.glu_shift) : kp_act_epilogue(p.act, gq) * uq;
         }
+        if (EPI == EPI_ACT) x = kp_act_plain(p.act, x);
         v[j] = x;
     }
     const bool whole = p.vec_ok && n_base + W <= n_lim;                  // vector stores of the whole piece
-    if (EPI == EPI_STORE || TC_GATED(EPI)) {
+    if (EPI == EPI_STORE || EPI == EPI_ACT || TC_GATED(EPI)) {
         bf16* dst = (bf16*)p.C + (size_t)m * p.ldc + n_base;
         if (whole && W >= 8) {
 #pragma unroll
@@ -513,6 +515,7 @@ static int tc_max_clusters(int bn, int epi, int cluster, int a_rows) {
         case EPI_STORE: TC_MC_BN(EPI_STORE)
         case EPI_STORE_F32: TC_MC_BN(EPI_STORE_F32)
         case EPI_ACCUM_F32: TC_MC_BN(EPI_ACCUM_F32)
+        case EPI_ACT: TC_MC_BN(EPI_ACT)
         case EPI_SWIGLU: TC_MC_BN(EPI_SWIGLU)
         default: return 0;
     }
@@ -522,7 +525,8 @@ static int tc_max_clusters(int bn, int epi, int cluster, int a_rows) {
 
 extern "C" {
 
-// epi: 0 store bf16, 1 store f32, 2 accumulate into f32, 3 SwiGLU (W = [gate; up], N = 2*ff, output [M, ff] bf16).
+// epi: 0 store bf16, 1 store f32, 2 accumulate into f32, 3 SwiGLU (W = [gate; up], N = 2*ff, output [M, ff] bf16),
+// 6 store bf16 behind the activation of bits 8 and up.
 // split: products of 17 to 1024 rows may be cut along K (0: never).
 // glu: limit, alpha and shift of the gated unit with limits (activation code 3 in epi), else null.
 static int tc_run(const void* A, int lda, const void* W, int ldw, const float* bias, void* C, int ldc, int M, int N,
@@ -544,14 +548,15 @@ static int tc_run(const void* A, int lda, const void* W, int ldw, const float* b
     if (M <= 0 || N <= 0) return 0;
     const int act = KP_EPI_ACT(epi);
     epi = KP_EPI_KIND(epi);
-    if (act != KP_ACT_SILU && act != KP_ACT_RELU && act != KP_ACT_GELU_TANH && !(act == KP_ACT_GLU_CLAMPED && glu)) return KP_ERR_UNSUPPORTED;
+    if (act != KP_ACT_SILU && act != KP_ACT_RELU && act != KP_ACT_GELU_TANH && !(act == KP_ACT_GLU_CLAMPED && glu) &&
+        !(act == KP_ACT_RELU_SQ && epi == EPI_ACT)) return KP_ERR_UNSUPPORTED;
     if (K < 8 || (K & 7) || (lda & 7) || (ldw & 7) || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return KP_ERR_UNSUPPORTED;
     if ((long long)((M + TC_BM - 1) / TC_BM) > 65535) return KP_ERR_UNSUPPORTED;
     TcArgs a = {};
     a.bias = bias; a.C = C; a.ldc = ldc; a.M = M; a.N = N; a.K = K; a.ff = 0; a.act = act;
     if (glu) { a.glu_limit = glu[0]; a.glu_alpha = glu[1]; a.glu_shift = glu[2]; }
     {
-        const int esz = (epi == EPI_STORE || epi == EPI_SWIGLU) ? 2 : 4;
+        const int esz = (epi == EPI_STORE || epi == EPI_SWIGLU || epi == EPI_ACT) ? 2 : 4;
         a.vec_ok = (((uintptr_t)C & 15) == 0 && ((size_t)ldc * esz) % 16 == 0) ? 1 : 0;
     }
     if (epi == EPI_SWIGLU) {
@@ -637,6 +642,7 @@ static int tc_run(const void* A, int lda, const void* W, int ldw, const float* b
         case EPI_STORE: TC_PICK(EPI_STORE)
         case EPI_STORE_F32: TC_PICK(EPI_STORE_F32)
         case EPI_ACCUM_F32: TC_PICK(EPI_ACCUM_F32)
+        case EPI_ACT: TC_PICK(EPI_ACT)
         case EPI_SWIGLU:
             if (a.act == KP_ACT_GLU_CLAMPED) {           // an instantiation of its own: the others' epilogues stay as they were
                 switch (bn) {

@@ -1,0 +1,806 @@
+// Attention over a cache of latents: keys and values are expanded from one low-rank latent a token, k_h = Wuk_h c and
+// v_h = Wuv_h c, beside a rotated key part that all heads share, and only the latent c and that part are kept.
+//
+//   cache row of a token: [ c (rank, normed; zeros up to rankp) | rotated key part (rot_dim; zeros up to rotp) ]
+//   s_h(t) = (q_h . Wuk_h c_t + qr_h . kr_t) scale ,  o_h = sum_t softmax(s_h)_t Wuv_h c_t        (causal)
+//
+// rankp and rotp are rank and rot_dim rounded up to 16; a row has W = rankp + rotp elements and lies in pages
+// [page][1][1][page_size][W].  Two ways of computing the same:
+//
+//  * absorbed (decoded tokens, short portions, the 32-bit mode): the expanding matrices move to the other side of the
+//    sums, q'_h = Wuk_h^T q_h once a row, s_h(t) = ([q'_h | qr_h] . row_t) scale, u_h = sum_t softmax(s_h)_t c_t and
+//    o_h = Wuv_h u_h.  All heads read the same rows, so a cache row is fetched once for up to 16 heads.  Per-head
+//    products (head_gemm), a pass over chunks of 256 keys (latent_split: bfloat16 on the tensor cores, or scalar) that
+//    leaves each chunk's maximum, sum and unnormalised latent, and a merge in chunk order.
+//  * expanded (prompt portions): the latents of the request's whole context are gathered from its pages, one product
+//    expands them, and latent_prefill runs tiles of 64 query rows over the expanded rows.
+//
+// The softmax statistics are float32; its weights enter the products whole, as three bfloat16 parts.  Chunks lie at
+// multiples of 256 of the absolute key index and tiles at multiples of 32 or 64, so the order of a row's sums does not
+// depend on how its prompt was cut or on what else is in the batch.
+#include "mma.cuh"
+
+#define LA_CHUNK 256               // keys a chunk of the absorbed pass
+#define LA_TILE 32                 // keys a tile of its tensor-core form
+#define LA_MAX_STAGES 4
+#define LA_SCALAR_HEADS 4          // heads a CTA of its scalar form
+#define LP_TILE 64                 // query rows and keys a tile of the expanded form
+
+KP_STATUS_WORD(g_latent_status, latent)          // 0 ok; 1: a bounded wait gave up
+
+// ------------------------------------------------------------------------------------------------ preparation
+// One block a row of the input product p = [.. q: H heads of (dimp unrotated | rotp rotated) .. | latent (rankp) and key
+// part (rotp) ..]: the latent normed over `rank` columns with weight w, and the key part rotated, go to the row's cache
+// page; every head's rotated query part is rotated where it is, and for rows below n_absorbed also stored behind
+// the place of the head's absorbed query in qa [n_absorbed][H][W].  rot: dimensions rotated (tables cos/sin
+// [positions][rot / 2], which may carry a factor; null: no rotation).
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(T* __restrict__ p, int ld, int q_col, int c_col, int H, int dimp, int rotp, int rank, int rankp,
+                   const float* __restrict__ w, float eps, const float* __restrict__ cos_tab, const float* __restrict__ sin_tab,
+                   int rot, int interleaved, const int* __restrict__ positions, const int* __restrict__ slot_map,
+                   T* __restrict__ cache, int page_size, T* __restrict__ qa, int n_absorbed) {
+    kp_pdl_begin_early_if(gridDim.x > 1);
+    __shared__ float red[32];
+    const int row = blockIdx.x, tid = threadIdx.x, W = rankp + rotp;
+    T* pr = p + (size_t)row * ld;
+    const T* c = pr + c_col;
+    const int pos = positions[row];
+    const int half = cos_tab ? rot >> 1 : 0;
+    const float* ct = cos_tab ? cos_tab + (size_t)pos * half : nullptr;
+    const float* st = cos_tab ? sin_tab + (size_t)pos * half : nullptr;
+    float ss = 0.f;
+    for (int i = tid; i < rank; i += 256) { const float v = to_f32(c[i]); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, red);
+    const float scale = 1.0f / sqrtf(ss / (float)rank + eps);
+    const int slot = cache ? slot_map[row] : -1;
+    if (slot >= 0) {
+        T* dst = cache + ((size_t)(slot / page_size) * page_size + slot % page_size) * W;
+        for (int i = tid; i < rankp; i += 256) dst[i] = from_f32<T>(i < rank ? (to_f32(c[i]) * scale) * w[i] : 0.f);
+        // (the key part's columns behind its own are zero in the product already)
+        for (int i = tid; i < rotp; i += 256) {
+            float v = to_f32(c[rankp + i]);
+            if (i < 2 * half) {
+                const int j = interleaved ? i >> 1 : (i < half ? i : i - half);
+                const bool second = interleaved ? (i & 1) : i >= half;
+                const float o = to_f32(c[rankp + (interleaved ? i ^ 1 : (second ? i - half : i + half))]);
+                v = second ? o * st[j] + v * ct[j] : v * ct[j] - o * st[j];
+            }
+            dst[rankp + i] = from_f32<T>(v);
+        }
+    }
+    const int Dq = dimp + rotp;
+    for (int i = tid; i < H * half; i += 256) {
+        const int h = i / half, j = i - h * half;
+        T* q = pr + q_col + (size_t)h * Dq + dimp;
+        const int ia = interleaved ? 2 * j : j, ib = interleaved ? 2 * j + 1 : j + half;
+        const float a = to_f32(q[ia]), b = to_f32(q[ib]);
+        const T ra = from_f32<T>(a * ct[j] - b * st[j]), rb = from_f32<T>(a * st[j] + b * ct[j]);
+        q[ia] = ra;
+        q[ib] = rb;
+        if (row < n_absorbed) {
+            T* d = qa + ((size_t)row * H + h) * W + rankp;
+            d[ia] = ra;
+            d[ib] = rb;
+        }
+    }
+    if (row < n_absorbed && rotp > 2 * half) {                     // what is not rotated passes on as it is
+        const int rest = rotp - 2 * half;
+        for (int i = tid; i < H * rest; i += 256) {
+            const int h = i / rest, j = 2 * half + i % rest;
+            qa[((size_t)row * H + h) * W + rankp + j] = pr[q_col + (size_t)h * Dq + dimp + j];
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------------------- per-head products
+// out[m, h, n] = sum_k a[m, h, k] b[h][n][k]   (times sigmoid(gate[m, h, n]) if gate).  Row and head strides are given.
+// One CTA: 16 MT rows x 32 columns of one head, four warps of 8 columns; k in stretches of 64, double-buffered.
+struct HeadGemmArgs {
+    const void* a; const void* b; const void* gate; void* out;
+    long long a_row, o_row, g_row;
+    int a_head, o_head, g_head;
+    int M, N, K, H;
+};
+
+template <int MT>
+__global__ void __launch_bounds__(128)
+head_gemm_mma_kernel(const HeadGemmArgs p) {
+    constexpr int BK = 64, PITCH = BK + 8;
+    kp_pdl_begin_early_if(p.M > 1);
+    __shared__ __align__(16) bf16 As[2][MT * 16][PITCH], Bs[2][32][PITCH];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int n0 = blockIdx.x * 32, h = blockIdx.y, m0 = blockIdx.z * MT * 16;
+    const bf16* A = (const bf16*)p.a + (size_t)h * p.a_head;
+    const bf16* B = (const bf16*)p.b + (size_t)h * p.N * p.K;
+    auto load = [&](int k0, int buf) {
+        for (int i = tid; i < MT * 16 * 8; i += 128) {
+            const int r = i >> 3, c = (i & 7) * 8;
+            const bool ok = m0 + r < p.M && k0 + c < p.K;
+            cp_async16(&As[buf][r][c], ok ? A + (size_t)(m0 + r) * p.a_row + k0 + c : A, ok);
+        }
+        for (int i = tid; i < 32 * 8; i += 128) {
+            const int r = i >> 3, c = (i & 7) * 8;
+            const bool ok = n0 + r < p.N && k0 + c < p.K;
+            cp_async16(&Bs[buf][r][c], ok ? B + (size_t)(n0 + r) * p.K + k0 + c : B, ok);
+        }
+        cp_async_commit();
+    };
+    float acc[MT][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) acc[m][i] = 0.f;
+    const int n_k = (p.K + BK - 1) / BK;
+    load(0, 0);
+    for (int it = 0; it < n_k; it++) {
+        const int buf = it & 1;
+        if (it + 1 < n_k) { load((it + 1) * BK, buf ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+#pragma unroll
+        for (int ks = 0; ks < BK / 16; ks += 2) {
+            uint32_t b[4];                                         // 8 columns x 32 of k
+            ldmatrix_x4(b, &Bs[buf][warp * 8 + (lane & 7)][ks * 16 + (lane >> 3) * 8]);
+#pragma unroll
+            for (int m = 0; m < MT; m++) {
+                uint32_t a0[4], a1[4];
+                ldmatrix_x4(a0, &As[buf][m * 16 + (lane & 15)][ks * 16 + (lane >> 4) * 8]);
+                ldmatrix_x4(a1, &As[buf][m * 16 + (lane & 15)][ks * 16 + 16 + (lane >> 4) * 8]);
+                mma_bf16(acc[m], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
+                mma_bf16(acc[m], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
+            }
+        }
+        __syncthreads();
+    }
+    const int n = n0 + warp * 8 + 2 * t;
+    if (n >= p.N) return;                                          // (N is a multiple of 16: a pair is inside or outside)
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int half = 0; half < 2; half++) {
+            const int r = m0 + m * 16 + g + half * 8;
+            if (r >= p.M) continue;
+            float v0 = acc[m][half * 2], v1 = acc[m][half * 2 + 1];
+            if (p.gate) {
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>((const bf16*)p.gate + (size_t)r * p.g_row + (size_t)h * p.g_head + n));
+                v0 /= 1.0f + expf(-z.x);
+                v1 /= 1.0f + expf(-z.y);
+            }
+            *reinterpret_cast<uint32_t*>((bf16*)p.out + (size_t)r * p.o_row + (size_t)h * p.o_head + n) = pack_bf16(v0, v1);
+        }
+}
+
+// The same on the CUDA cores (float32 mode): 16 rows x 64 columns a CTA.
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_gemm_simt_kernel(const HeadGemmArgs p) {
+    kp_pdl_begin();
+    constexpr int BM = 16, BN = 64, BK = 16;
+    __shared__ float As[BK][BM + 1], Bs[BK][BN + 1];
+    const int tid = threadIdx.x, tx = tid & 63, ty = tid >> 6;     // column, row group of 4
+    const int n0 = blockIdx.x * BN, h = blockIdx.y, m0 = blockIdx.z * BM;
+    const T* A = (const T*)p.a + (size_t)h * p.a_head;
+    const T* B = (const T*)p.b + (size_t)h * p.N * p.K;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k0 = 0; k0 < p.K; k0 += BK) {
+        {
+            const int r = tid >> 4, c = tid & 15;
+            As[c][r] = (m0 + r < p.M && k0 + c < p.K) ? to_f32(A[(size_t)(m0 + r) * p.a_row + k0 + c]) : 0.f;
+        }
+        for (int i = tid; i < BN * BK; i += 256) {
+            const int r = i >> 4, c = i & 15;
+            Bs[c][r] = (n0 + r < p.N && k0 + c < p.K) ? to_f32(B[(size_t)(n0 + r) * p.K + k0 + c]) : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < BK; k++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) acc[i] = fmaf(As[k][ty * 4 + i], Bs[k][tx], acc[i]);
+        __syncthreads();
+    }
+    const int n = n0 + tx;
+    if (n >= p.N) return;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int r = m0 + ty * 4 + i;
+        if (r >= p.M) continue;
+        float v = acc[i];
+        if (p.gate) v /= 1.0f + expf(-to_f32(((const T*)p.gate)[(size_t)r * p.g_row + (size_t)h * p.g_head + n]));
+        ((T*)p.out)[(size_t)r * p.o_row + (size_t)h * p.o_head + n] = from_f32<T>(v);
+    }
+}
+
+// --------------------------------------------------------------------------------- absorbed pass, tensor cores
+// One CTA: one chunk of 256 keys, up to 16 heads, one row.  Tiles of 32 cache rows come by bulk copies (one a key,
+// issued by the lanes of warp 0) into a ring; S = Q K^T by all 8 warps (8 keys x half of W each), the softmax of the
+// 16 x 32 scores by half-warps (a head each), then every warp sums its own columns of the latent, P V with V = the
+// latent columns of the same tile.  PT: pairs of 8-column tiles a warp (rank <= 128 PT).
+template <int PT>
+__global__ void __launch_bounds__(256, 2)
+latent_split_mma_kernel(const bf16* __restrict__ qa, const bf16* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
+                        const int* __restrict__ row_seg, const int* __restrict__ positions, float* __restrict__ part_acc,
+                        float* __restrict__ part_ml, int n_chunks, float scale, int page_size, int H, int rankp, int W, int n_stages) {
+    kp_pdl_begin_early_if(gridDim.z > 1);
+    extern __shared__ __align__(128) unsigned char la_smem[];
+    const int pitch = W + 8;                                       // (an odd number of 16-byte pieces: ldmatrix rows do not collide)
+    bf16* Ks = reinterpret_cast<bf16*>(la_smem);                   // [n_stages][LA_TILE][pitch]
+    bf16* Qs = Ks + (size_t)n_stages * LA_TILE * pitch;            // [16][pitch]
+    bf16* Ps = Qs + (size_t)16 * pitch;                            // [3][16][40]
+    float* Sp = reinterpret_cast<float*>(Ps + 3 * 16 * 40);        // [2][16][36]
+    float* corr_s = Sp + 2 * 16 * 36;                              // [16]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(corr_s + 16);     // [n_stages]
+
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int chunk = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
+    const int k_hi = positions[row], c0 = chunk * LA_CHUNK;
+    if (c0 > k_hi) return;
+    const int n_keys = min(k_hi + 1 - c0, LA_CHUNK), n_tiles = (n_keys + LA_TILE - 1) / LA_TILE;
+    const int* bt = block_table + (size_t)row_seg[row] * max_blocks;
+    const int nh = min(16, H - h0);
+
+    if (tid == 0) {
+        for (int s = 0; s < n_stages; s++) kp_mbar_init(&bars[s], 1);
+        kp_mbar_init_fence();
+    }
+    __syncthreads();
+    auto load = [&](int it) {                                      // warp 0: tile it into its stage
+        const int s = it % n_stages, r = it * LA_TILE + lane;
+        if (lane == 0) kp_mbar_expect_tx(&bars[s], (uint32_t)min(LA_TILE, n_keys - it * LA_TILE) * W * 2);
+        __syncwarp();
+        if (r < n_keys) {
+            const int key = c0 + r;
+            kp_bulk_g2s(Ks + ((size_t)s * LA_TILE + lane) * pitch,
+                        cache + ((size_t)bt[key / page_size] * page_size + key % page_size) * W, (uint32_t)W * 2, &bars[s]);
+        }
+    };
+    if (warp == 0)
+        for (int it = 0; it < min(n_stages, n_tiles); it++) load(it);
+    {
+        const int per = W >> 3;                                    // 16-byte pieces a row
+        const bf16* src = qa + ((size_t)row * H + h0) * W;
+        for (int i = tid; i < 16 * per; i += 256) {
+            const int r = i / per, c = (i - r * per) * 8;
+            *reinterpret_cast<uint4*>(Qs + (size_t)r * pitch + c) =
+                r < nh ? *reinterpret_cast<const uint4*>(src + (size_t)r * W + c) : make_uint4(0, 0, 0, 0);
+        }
+    }
+    float o[PT][2][4];
+#pragma unroll
+    for (int j = 0; j < PT; j++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) o[j][0][i] = o[j][1][i] = 0.f;
+    float m_run = -INFINITY, l_run = 0.f;                          // of head tid / 16, the same in its 16 lanes
+    const int KS = W >> 4, nt = warp & 3, kh = warp >> 2;
+    const int ks_lo = kh ? KS / 2 : 0, ks_hi = kh ? KS : KS / 2;
+    __syncthreads();                                               // Q is there
+
+    bool ok = true;
+    for (int it = 0; it < n_tiles; it++) {
+        const int s = it % n_stages;
+        const bf16* Kt = Ks + (size_t)s * LA_TILE * pitch;
+        const int valid = min(LA_TILE, n_keys - it * LA_TILE);
+        ok = kp_mbar_wait_bounded(&bars[s], (it / n_stages) & 1);
+        if (valid < LA_TILE) {                                     // the chunk's last tile: rows that no copy filled
+            const int per = W >> 3;
+            for (int i = tid; i < (LA_TILE - valid) * per; i += 256) {
+                const int r = i / per;
+                *reinterpret_cast<uint4*>(const_cast<bf16*>(Kt) + (size_t)(valid + r) * pitch + (i - r * per) * 8) = make_uint4(0, 0, 0, 0);
+            }
+            __syncthreads();
+        }
+        float sa[4] = {0.f, 0.f, 0.f, 0.f}, sb[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int ks = ks_lo; ks < ks_hi; ks++) {
+            uint32_t a[4], b[2];
+            ldmatrix_x4(a, Qs + (size_t)(lane & 15) * pitch + ks * 16 + (lane >> 4) * 8);
+            ldmatrix_x2(b, Kt + (size_t)(nt * 8 + (lane & 7)) * pitch + ks * 16 + ((lane >> 3) & 1) * 8);
+            if ((ks - ks_lo) & 1) mma_bf16(sb, a[0], a[1], a[2], a[3], b[0], b[1]);
+            else mma_bf16(sa, a[0], a[1], a[2], a[3], b[0], b[1]);
+        }
+        {
+            float* d = Sp + (size_t)kh * 16 * 36 + nt * 8 + 2 * t;
+            *reinterpret_cast<float2*>(d + g * 36) = make_float2(sa[0] + sb[0], sa[1] + sb[1]);
+            *reinterpret_cast<float2*>(d + (g + 8) * 36) = make_float2(sa[2] + sb[2], sa[3] + sb[3]);
+        }
+        if (!__syncthreads_and(ok)) { ok = false; break; }         // (all threads leave together)
+        {
+            const int hr = tid >> 4, kk = (tid & 15) * 2;
+            const float2 x = *reinterpret_cast<const float2*>(Sp + hr * 36 + kk), y = *reinterpret_cast<const float2*>(Sp + 16 * 36 + hr * 36 + kk);
+            float p0 = kk < valid ? (x.x + y.x) * scale : -INFINITY, p1 = kk + 1 < valid ? (x.y + y.y) * scale : -INFINITY;
+            float mx = fmaxf(p0, p1);
+#pragma unroll
+            for (int d = 8; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+            const float m_new = fmaxf(m_run, mx);                  // (finite: the first key of every tile is the row's)
+            const float corr = m_run == -INFINITY ? 0.f : expf(m_run - m_new);
+            p0 = kk < valid ? expf(p0 - m_new) : 0.f;
+            p1 = kk + 1 < valid ? expf(p1 - m_new) : 0.f;
+            float sum = p0 + p1;
+#pragma unroll
+            for (int d = 8; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+            l_run = l_run * corr + sum;
+            m_run = m_new;
+#pragma unroll
+            for (int part = 0; part < 3; part++)
+                *reinterpret_cast<uint32_t*>(Ps + (size_t)(part * 16 + hr) * 40 + kk) = pack_bf16_part(p0, p1);
+            if ((tid & 15) == 0) corr_s[hr] = corr;
+        }
+        __syncthreads();
+        const float ca = corr_s[g], cb = corr_s[g + 8];
+        uint32_t pf[3][2][4];
+#pragma unroll
+        for (int part = 0; part < 3; part++)
+#pragma unroll
+            for (int ks = 0; ks < 2; ks++) ldmatrix_x4(pf[part][ks], Ps + (size_t)(part * 16 + (lane & 15)) * 40 + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int j = 0; j < PT; j++) {
+            const int c = (warp + 8 * j) * 16;                     // this warp's j-th stretch of 16 columns
+            if (c < rankp) {
+#pragma unroll
+                for (int i = 0; i < 2; i++) { o[j][i][0] *= ca; o[j][i][1] *= ca; o[j][i][2] *= cb; o[j][i][3] *= cb; }
+#pragma unroll
+                for (int ks = 0; ks < 2; ks++) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, Kt + (size_t)(ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * pitch + c + (lane >> 4) * 8);
+#pragma unroll
+                    for (int part = 0; part < 3; part++) {
+                        mma_bf16(o[j][0], pf[part][ks][0], pf[part][ks][1], pf[part][ks][2], pf[part][ks][3], b[0], b[1]);
+                        mma_bf16(o[j][1], pf[part][ks][0], pf[part][ks][1], pf[part][ks][2], pf[part][ks][3], b[2], b[3]);
+                    }
+                }
+            }
+        }
+        __syncthreads();                                           // the stage, the scores and the weights are free
+        if (warp == 0 && it + n_stages < n_tiles) load(it + n_stages);
+    }
+    if (!ok) {
+        if (tid == 0) atomicExch(&g_latent_status, 1);
+        kp_linger_after_failure();
+        return;
+    }
+#pragma unroll
+    for (int j = 0; j < PT; j++) {
+        const int c = (warp + 8 * j) * 16;
+        if (c >= rankp) continue;
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int col = c + i * 8 + 2 * t;
+            if (g < nh)
+                *reinterpret_cast<float2*>(part_acc + (((size_t)row * H + h0 + g) * n_chunks + chunk) * rankp + col) = make_float2(o[j][i][0], o[j][i][1]);
+            if (g + 8 < nh)
+                *reinterpret_cast<float2*>(part_acc + (((size_t)row * H + h0 + g + 8) * n_chunks + chunk) * rankp + col) = make_float2(o[j][i][2], o[j][i][3]);
+        }
+    }
+    if ((tid & 15) == 0 && (tid >> 4) < nh)
+        *reinterpret_cast<float2*>(part_ml + (((size_t)row * H + h0 + (tid >> 4)) * n_chunks + chunk) * 2) = make_float2(m_run, l_run);
+}
+
+// ------------------------------------------------------------------------------------- absorbed pass, CUDA cores
+// The same for any sizes and both storage types: one CTA a (chunk, up to 4 heads, row); a key a thread for the scores,
+// a column a thread for the sums.
+template <typename T>
+__global__ void __launch_bounds__(LA_CHUNK)
+latent_split_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
+                    const int* __restrict__ row_seg, const int* __restrict__ positions, float* __restrict__ part_acc,
+                    float* __restrict__ part_ml, int n_chunks, float scale, int page_size, int H, int rankp, int W) {
+    kp_pdl_begin();
+    constexpr int R = LA_SCALAR_HEADS;
+    extern __shared__ __align__(16) float ls_smem[];               // [R][W] queries, [R][256] weights, [32], [256] row offsets
+    float* qs = ls_smem;
+    float* ps = qs + R * W;
+    float* red = ps + R * LA_CHUNK;
+    int* where = reinterpret_cast<int*>(red + 32);
+    const int tid = threadIdx.x, chunk = blockIdx.x, h0 = blockIdx.y * R, row = blockIdx.z;
+    const int k_hi = positions[row], c0 = chunk * LA_CHUNK;
+    if (c0 > k_hi) return;
+    const int n_keys = min(k_hi + 1 - c0, LA_CHUNK), nh = min(R, H - h0);
+    const int* bt = block_table + (size_t)row_seg[row] * max_blocks;
+    for (int i = tid; i < R * W; i += LA_CHUNK) qs[i] = i < nh * W ? to_f32(qa[((size_t)row * H + h0) * W + i]) : 0.f;
+    const int key = c0 + tid;
+    where[tid] = tid < n_keys ? bt[key / page_size] * page_size + key % page_size : 0;
+    __syncthreads();
+    float s[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) s[r] = 0.f;
+    if (tid < n_keys) {
+        const T* kp = cache + (size_t)where[tid] * W;
+        constexpr int VN = 16 / sizeof(T);
+        for (int i = 0; i < W; i += VN) {                          // (W is a multiple of 16)
+            const uint4 raw = *reinterpret_cast<const uint4*>(kp + i);
+            const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+            for (int j = 0; j < VN; j++) {
+                const float kv = to_f32(e[j]);
+#pragma unroll
+                for (int r = 0; r < R; r++) s[r] = fmaf(qs[r * W + i + j], kv, s[r]);
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+        const float v = tid < n_keys ? s[r] * scale : -INFINITY;
+        const float m = block_max(v, red);
+        const float p = tid < n_keys ? expf(v - m) : 0.f;
+        const float l = block_sum(p, red);
+        ps[r * LA_CHUNK + tid] = p;
+        if (tid == 0 && r < nh) {
+            float* ml = part_ml + (((size_t)row * H + h0 + r) * n_chunks + chunk) * 2;
+            ml[0] = m;
+            ml[1] = l;
+        }
+    }
+    __syncthreads();
+    for (int c = tid; c < rankp; c += LA_CHUNK) {
+        float acc[R];
+#pragma unroll
+        for (int r = 0; r < R; r++) acc[r] = 0.f;
+#pragma unroll 4
+        for (int k = 0; k < n_keys; k++) {
+            const float v = to_f32(cache[(size_t)where[k] * W + c]);
+#pragma unroll
+            for (int r = 0; r < R; r++) acc[r] = fmaf(ps[r * LA_CHUNK + k], v, acc[r]);
+        }
+#pragma unroll
+        for (int r = 0; r < R; r++)
+            if (r < nh) part_acc[(((size_t)row * H + h0 + r) * n_chunks + chunk) * rankp + c] = acc[r];
+    }
+}
+
+// The chunks of a (head, row) put together in chunk order: u = sum_c acc_c exp(m_c - m) / sum_c l_c exp(m_c - m).
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, const int* __restrict__ positions,
+                    T* __restrict__ out, int n_chunks, int H, int rankp) {
+    kp_pdl_begin_early_if(gridDim.y > 1);
+    extern __shared__ float lm_w[];                                // [n_chunks] weights, [32]
+    float* red = lm_w + n_chunks;
+    const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x;
+    const int n = min(positions[row] / LA_CHUNK + 1, n_chunks);
+    const float* ml = part_ml + ((size_t)row * H + h) * n_chunks * 2;
+    float m = -INFINITY;
+    for (int c = tid; c < n; c += 128) { const float v = ml[2 * c]; lm_w[c] = v; m = fmaxf(m, v); }
+    m = block_max(m, red);
+    for (int c = tid; c < n; c += 128) lm_w[c] = expf(lm_w[c] - m);
+    __syncthreads();
+    float l = 0.f;
+    for (int c = 0; c < n; c++) l = fmaf(ml[2 * c + 1], lm_w[c], l);
+    const float inv = 1.0f / l;
+    const float* pa = part_acc + ((size_t)row * H + h) * n_chunks * rankp;
+    for (int i = tid * 4; i < rankp; i += 512) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int c = 0; c < n; c++) {
+            const float4 a = *reinterpret_cast<const float4*>(pa + (size_t)c * rankp + i);
+            const float w = lm_w[c];
+            v.x = fmaf(a.x, w, v.x); v.y = fmaf(a.y, w, v.y); v.z = fmaf(a.z, w, v.z); v.w = fmaf(a.w, w, v.w);
+        }
+        T* o = out + ((size_t)row * H + h) * rankp + i;
+        o[0] = from_f32<T>(v.x * inv); o[1] = from_f32<T>(v.y * inv); o[2] = from_f32<T>(v.z * inv); o[3] = from_f32<T>(v.w * inv);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------- expanded pass
+// The cache rows of the contexts of some segments, side by side: row ctx_base[i] + t of `out` [T][W] is key t of segment i
+// (segments without rows there have ctx_base[i] == ctx_base[i + 1]).  A warp a row.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const bf16* __restrict__ cache, const int* __restrict__ block_table, int max_blocks, const int* __restrict__ ctx_base,
+                     int n_seg, bf16* __restrict__ out, int n_rows, int page_size, int W) {
+    kp_pdl_begin();
+    const int lane = threadIdx.x & 31, r = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (r >= n_rows) return;
+    int lo = 0, hi = n_seg;                                        // the last segment with ctx_base <= r
+    while (hi - lo > 1) {
+        const int mid = (lo + hi) >> 1;
+        if (ctx_base[mid] <= r) lo = mid; else hi = mid;
+    }
+    const int key = r - ctx_base[lo];
+    const uint4* src = reinterpret_cast<const uint4*>(cache + ((size_t)block_table[(size_t)lo * max_blocks + key / page_size] * page_size + key % page_size) * W);
+    uint4* dst = reinterpret_cast<uint4*>(out + (size_t)r * W);
+    for (int i = lane; i < W >> 3; i += 32) dst[i] = src[i];
+}
+
+// One CTA: 64 query rows of a segment, one head: 4 warps x 16 rows over tiles of 64 keys, double-buffered (cp.async).  A
+// tile's key rows are [expanded unrotated part | shared rotated part], its value rows the expanded values.  KS, VT: the most
+// 16-column steps of a key and 8-column tiles of a value.
+struct LatentPrefillArgs {
+    const bf16* q; const bf16* ex; const bf16* rows; bf16* out;
+    const int* cu_rows; const int* seg_pos; const int* tile_seg; const int* tile_row0; const int* ctx_base;
+    int ldq, ldo, ld_ex, W, rankp, dimp, rotp, vdimp, v_col, n_tiles;
+    float scale;
+};
+
+template <int KS, int VT>
+__global__ void __launch_bounds__(128)
+latent_prefill_kernel(const LatentPrefillArgs p) {
+    kp_pdl_begin();
+    extern __shared__ __align__(128) unsigned char lp_smem[];
+    const int Dq = p.dimp + p.rotp, kp = Dq + 8, vp = p.vdimp + 8;
+    bf16* Ks = reinterpret_cast<bf16*>(lp_smem);                   // [2][64][kp]
+    bf16* Vs = Ks + (size_t)2 * LP_TILE * kp;                      // [2][64][vp]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.y, tile = p.n_tiles - 1 - blockIdx.x;   // (later rows of a prompt read more keys: they go first)
+    const int seg = p.tile_seg[tile], row0 = p.tile_row0[tile];
+    const int n_rows = min(LP_TILE, p.cu_rows[seg + 1] - row0);
+    const int pos0 = p.seg_pos[seg] + (row0 - p.cu_rows[seg]);
+    const int k_hi = pos0 + n_rows - 1, n_kt = k_hi / LP_TILE + 1;
+    const size_t base = p.ctx_base[seg];
+    const int nks = Dq >> 4, nvt = p.vdimp >> 3;
+    const int kc = p.dimp >> 3, rc = p.rotp >> 3, vc = p.vdimp >> 3;       // 16-byte pieces
+
+    auto load = [&](int kt, int buf) {
+        bf16* kd = Ks + (size_t)buf * LP_TILE * kp;
+        bf16* vd = Vs + (size_t)buf * LP_TILE * vp;
+        const int per = kc + rc + vc;
+        for (int i = tid; i < LP_TILE * per; i += 128) {
+            const int r = i / per, c = i - r * per, key = kt * LP_TILE + r;
+            const bool ok = key <= k_hi;
+            const size_t er = base + (ok ? key : 0);
+            const bf16* src;
+            bf16* dst;
+            if (c < kc) { src = p.ex + er * p.ld_ex + (size_t)h * p.dimp + c * 8; dst = kd + (size_t)r * kp + c * 8; }
+            else if (c < kc + rc) { src = p.rows + er * p.W + p.rankp + (c - kc) * 8; dst = kd + (size_t)r * kp + c * 8; }
+            else { src = p.ex + er * p.ld_ex + p.v_col + (size_t)h * p.vdimp + (c - kc - rc) * 8; dst = vd + (size_t)r * vp + (c - kc - rc) * 8; }
+            cp_async16(dst, src, ok);
+        }
+        cp_async_commit();
+    };
+    load(0, 0);
+
+    const int ra = warp * 16 + g, rb = ra + 8;
+    const int pos_a = pos0 + ra, pos_b = pos0 + rb;
+    const bool has_a = ra < n_rows, has_b = rb < n_rows;
+    uint32_t qf[KS][4];
+    {
+        const bf16* qa = p.q + (size_t)(row0 + min(ra, n_rows - 1)) * p.ldq + (size_t)h * Dq;
+        const bf16* qb = p.q + (size_t)(row0 + min(rb, n_rows - 1)) * p.ldq + (size_t)h * Dq;
+#pragma unroll
+        for (int ks = 0; ks < KS; ks++) {
+            if (ks < nks) {
+                qf[ks][0] = *reinterpret_cast<const uint32_t*>(qa + ks * 16 + 2 * t);
+                qf[ks][1] = *reinterpret_cast<const uint32_t*>(qb + ks * 16 + 2 * t);
+                qf[ks][2] = *reinterpret_cast<const uint32_t*>(qa + ks * 16 + 8 + 2 * t);
+                qf[ks][3] = *reinterpret_cast<const uint32_t*>(qb + ks * 16 + 8 + 2 * t);
+            }
+        }
+    }
+    float o[VT][4];
+#pragma unroll
+    for (int d = 0; d < VT; d++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) o[d][i] = 0.f;
+    float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
+
+    for (int kt = 0; kt < n_kt; kt++) {
+        const int buf = kt & 1;
+        if (kt + 1 < n_kt) { load(kt + 1, buf ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        const int t0 = kt * LP_TILE;
+        const int w_hi = pos0 + min(warp * 16 + 15, n_rows - 1);
+        if (warp * 16 < n_rows && t0 <= w_hi) {
+            const bf16* Kt = Ks + (size_t)buf * LP_TILE * kp;
+            const bf16* Vt = Vs + (size_t)buf * LP_TILE * vp;
+            float s[8][4];
+#pragma unroll
+            for (int nt = 0; nt < 8; nt++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) s[nt][i] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks < KS; ks++) {
+                if (ks < nks) {
+#pragma unroll
+                    for (int nt = 0; nt < 8; nt += 2) {
+                        uint32_t b[4];
+                        ldmatrix_x4(b, Kt + (size_t)((nt + (lane >> 4)) * 8 + (lane & 7)) * kp + ks * 16 + ((lane >> 3) & 1) * 8);
+                        mma_bf16(s[nt], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b[0], b[1]);
+                        mma_bf16(s[nt + 1], qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3], b[2], b[3]);
+                    }
+                }
+            }
+            float mx_a = -INFINITY, mx_b = -INFINITY;
+#pragma unroll
+            for (int nt = 0; nt < 8; nt++) {
+#pragma unroll
+                for (int i = 0; i < 2; i++) {
+                    const int key = t0 + nt * 8 + 2 * t + i;
+                    s[nt][i] = has_a && key <= pos_a ? s[nt][i] * p.scale : -INFINITY;
+                    s[nt][2 + i] = has_b && key <= pos_b ? s[nt][2 + i] * p.scale : -INFINITY;
+                    mx_a = fmaxf(mx_a, s[nt][i]);
+                    mx_b = fmaxf(mx_b, s[nt][2 + i]);
+                }
+            }
+            mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
+            mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
+            mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
+            mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
+            const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
+            const float ca = m_a == -INFINITY ? 0.f : expf(m_a - mn_a), cb = m_b == -INFINITY ? 0.f : expf(m_b - mn_b);
+            float sa = 0.f, sb = 0.f;
+#pragma unroll
+            for (int nt = 0; nt < 8; nt++) {
+#pragma unroll
+                for (int i = 0; i < 2; i++) {
+                    s[nt][i] = mn_a == -INFINITY ? 0.f : expf(s[nt][i] - mn_a);
+                    s[nt][2 + i] = mn_b == -INFINITY ? 0.f : expf(s[nt][2 + i] - mn_b);
+                    sa += s[nt][i];
+                    sb += s[nt][2 + i];
+                }
+            }
+            sa += __shfl_xor_sync(0xffffffffu, sa, 1); sa += __shfl_xor_sync(0xffffffffu, sa, 2);
+            sb += __shfl_xor_sync(0xffffffffu, sb, 1); sb += __shfl_xor_sync(0xffffffffu, sb, 2);
+            l_a = l_a * ca + sa; l_b = l_b * cb + sb;
+            m_a = mn_a; m_b = mn_b;
+#pragma unroll
+            for (int d = 0; d < VT; d++) { o[d][0] *= ca; o[d][1] *= ca; o[d][2] *= cb; o[d][3] *= cb; }
+#pragma unroll
+            for (int kk = 0; kk < 4; kk++) {                       // 16 keys at a time: their weights' three parts, then V once
+                uint32_t pf[3][4];
+#pragma unroll
+                for (int part = 0; part < 3; part++) {
+                    pf[part][0] = pack_bf16_part(s[2 * kk][0], s[2 * kk][1]);
+                    pf[part][1] = pack_bf16_part(s[2 * kk][2], s[2 * kk][3]);
+                    pf[part][2] = pack_bf16_part(s[2 * kk + 1][0], s[2 * kk + 1][1]);
+                    pf[part][3] = pack_bf16_part(s[2 * kk + 1][2], s[2 * kk + 1][3]);
+                }
+#pragma unroll
+                for (int d = 0; d < VT; d += 2) {
+                    if (d < nvt) {
+                        uint32_t b[4];
+                        ldmatrix_x4_trans(b, Vt + (size_t)(kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * vp + (d + (lane >> 4)) * 8);
+#pragma unroll
+                        for (int part = 0; part < 3; part++) {
+                            mma_bf16(o[d], pf[part][0], pf[part][1], pf[part][2], pf[part][3], b[0], b[1]);
+                            mma_bf16(o[d + 1], pf[part][0], pf[part][1], pf[part][2], pf[part][3], b[2], b[3]);
+                        }
+                    }
+                }
+            }
+        }
+        __syncthreads();                                           // the buffer is free for the load after next
+    }
+    const float ia = l_a > 0.f ? 1.0f / l_a : 0.f, ib = l_b > 0.f ? 1.0f / l_b : 0.f;
+#pragma unroll
+    for (int d = 0; d < VT; d++) {
+        if (d >= nvt) continue;
+        const size_t col = (size_t)h * p.vdimp + d * 8 + 2 * t;
+        if (has_a) *reinterpret_cast<uint32_t*>(p.out + (size_t)(row0 + ra) * p.ldo + col) = pack_bf16(o[d][0] * ia, o[d][1] * ia);
+        if (has_b) *reinterpret_cast<uint32_t*>(p.out + (size_t)(row0 + rb) * p.ldo + col) = pack_bf16(o[d][2] * ib, o[d][3] * ib);
+    }
+}
+
+static size_t la_fixed_bytes(int W) { return (size_t)16 * (W + 8) * 2 + 3 * 16 * 40 * 2 + 2 * 16 * 36 * 4 + 16 * 4 + LA_MAX_STAGES * 8; }
+static size_t la_tile_bytes(int W) { return (size_t)LA_TILE * (W + 8) * 2; }
+#define LA_SMEM_BUDGET (112 * 1024)                                // two CTAs an SM
+
+template <typename F>
+static int la_set_smem(F kern, size_t sm) {
+    if (sm <= 48 * 1024) return 0;
+    return (int)cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+}
+
+extern "C" {
+
+int kp_latent_prep(void* p, int ld, int q_col, int c_col, int H, int dimp, int rotp, int rank, int rankp, const float* w, float eps,
+                   const float* cos_tab, const float* sin_tab, int rot, int interleaved, const int* positions, const int* slot_map,
+                   void* cache, int page_size, void* qa, int n_absorbed, int n, int dtype, void* stream) {
+    if (n <= 0) return 0;
+    if (H < 1 || rank < 1 || rank > rankp || (rankp & 15) || (rotp & 15) || rotp < 0 || page_size < 1 || (cos_tab && (rot < 2 || (rot & 1) || rot > rotp)) ||
+        n_absorbed < 0 || n_absorbed > n || (n_absorbed > 0 && !qa))
+        return KP_ERR_BAD_ARG;
+    KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(latent_prep_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, (T*)p, ld, q_col, c_col, H,
+                                               dimp, rotp, rank, rankp, w, eps, cos_tab, sin_tab, rot, interleaved, positions,
+                                               slot_map, (T*)cache, page_size, (T*)qa, n_absorbed)));
+    return kp_launch_status();
+}
+
+// out[m, h, :N] = a[m, h, :K] b[h]^T, b [H][N][K]; strides in elements.  N and K multiples of 16.
+int kp_head_gemm(const void* a, long long a_row, int a_head, const void* b, void* out, long long o_row, int o_head, const void* gate,
+                 long long g_row, int g_head, int M, int N, int K, int H, int dtype, void* stream) {
+    if (M <= 0) return 0;
+    if (N < 1 || K < 1 || H < 1 || (N & 15) || (K & 15) || H > 65535) return KP_ERR_BAD_ARG;
+    HeadGemmArgs p = {a, b, gate, out, a_row, o_row, g_row, a_head, o_head, g_head, M, N, K, H};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == KP_DTYPE_BF16 && !(((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & 15) && !(a_row & 7) && !(a_head & 7) && !(o_row & 1) &&
+        !(o_head & 1) && (!gate || (!((uintptr_t)gate & 3) && !(g_row & 1) && !(g_head & 1)))) {
+        const int gx = (N + 31) / 32;
+        if (M <= 16) kp_launch_pdl(head_gemm_mma_kernel<1>, dim3(gx, H, 1), dim3(128), 0, s, p);
+        else if (M <= 32) kp_launch_pdl(head_gemm_mma_kernel<2>, dim3(gx, H, 1), dim3(128), 0, s, p);
+        else kp_launch_pdl(head_gemm_mma_kernel<4>, dim3(gx, H, (M + 63) / 64), dim3(128), 0, s, p);
+        return kp_launch_status();
+    }
+    KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(head_gemm_simt_kernel<T>, dim3((N + 63) / 64, H, (M + 15) / 16), dim3(256), 0, s, p)));
+    return kp_launch_status();
+}
+
+long long kp_latent_split_scratch(int n, int H, int rankp, int n_chunks) { return (long long)n * H * n_chunks * (rankp + 2); }
+
+// qa [n][H][W] -> u [n][H][rankp]; scratch: kp_latent_split_scratch floats; n_chunks chunks of 256 keys must reach the
+// largest position.
+int kp_latent_split(const void* qa, const void* cache, const int* block_table, int max_blocks, const int* row_seg, const int* positions,
+                    float* scratch, int n_chunks, void* u, float scale, int page_size, int n, int H, int rankp, int rotp, int dtype,
+                    int tensor_cores, void* stream) {
+    if (n <= 0) return 0;
+    if (n > 65535 || H < 1 || n_chunks < 1 || page_size < 1 || (rankp & 15) || (rotp & 15) || rankp < 16) return KP_ERR_BAD_ARG;
+    const int W = rankp + rotp;
+    float* part_acc = scratch;
+    float* part_ml = scratch + (size_t)n * H * n_chunks * rankp;
+    cudaStream_t s = (cudaStream_t)stream;
+    int st = 0;
+    const size_t fixed = la_fixed_bytes(W), tile = la_tile_bytes(W);
+    if (tensor_cores && dtype == KP_DTYPE_BF16 && rankp <= 512 && fixed + 2 * tile <= 2 * LA_SMEM_BUDGET && !(((uintptr_t)qa | (uintptr_t)cache) & 15)) {
+        const size_t budget = fixed + 2 * tile <= LA_SMEM_BUDGET ? LA_SMEM_BUDGET : 2 * LA_SMEM_BUDGET;
+        int stages = (int)((budget - fixed) / tile);
+        if (stages > LA_MAX_STAGES) stages = LA_MAX_STAGES;
+        const size_t sm = fixed + stages * tile;
+        dim3 grid(n_chunks, (H + 15) / 16, n);
+#define LA_MMA(PT)                                                                                                        \
+    do {                                                                                                                  \
+        st = la_set_smem(latent_split_mma_kernel<PT>, sm);                                                                \
+        if (st) return st;                                                                                                \
+        kp_launch_pdl(latent_split_mma_kernel<PT>, grid, dim3(256), sm, s, (const bf16*)qa, (const bf16*)cache, block_table, max_blocks, \
+                      row_seg, positions, part_acc, part_ml, n_chunks, scale, page_size, H, rankp, W, stages);            \
+    } while (0)
+        if (rankp <= 128) LA_MMA(1); else if (rankp <= 256) LA_MMA(2); else LA_MMA(4);
+#undef LA_MMA
+    } else {
+        const size_t sm = ((size_t)LA_SCALAR_HEADS * (W + LA_CHUNK) + 32 + LA_CHUNK) * sizeof(float);
+        if (sm > 200 * 1024) return KP_ERR_UNSUPPORTED;
+        dim3 grid(n_chunks, (H + LA_SCALAR_HEADS - 1) / LA_SCALAR_HEADS, n);
+        KP_DISPATCH_DTYPE(dtype, T, {
+            st = la_set_smem(latent_split_kernel<T>, sm);
+            if (st) return st;
+            kp_launch_pdl(latent_split_kernel<T>, grid, dim3(LA_CHUNK), sm, s, (const T*)qa, (const T*)cache, block_table, max_blocks, row_seg,
+                          positions, part_acc, part_ml, n_chunks, scale, page_size, H, rankp, W);
+        });
+    }
+    st = kp_launch_status();
+    if (st) return st;
+    const size_t msm = ((size_t)n_chunks + 32) * sizeof(float);
+    if (msm > 200 * 1024) return KP_ERR_UNSUPPORTED;
+    KP_DISPATCH_DTYPE(dtype, T, {
+        st = la_set_smem(latent_merge_kernel<T>, msm);
+        if (st) return st;
+        kp_launch_pdl(latent_merge_kernel<T>, dim3(H, n), dim3(128), msm, s, part_acc, part_ml, positions, (T*)u, n_chunks, H, rankp);
+    });
+    return kp_launch_status();
+}
+
+int kp_latent_gather(const void* cache, const int* block_table, int max_blocks, const int* ctx_base, int n_seg, void* out, int n_rows,
+                     int page_size, int W, void* stream) {
+    if (n_rows <= 0) return 0;
+    if (n_seg < 1 || page_size < 1 || (W & 7)) return KP_ERR_BAD_ARG;
+    kp_launch_pdl(latent_gather_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, (cudaStream_t)stream, (const bf16*)cache, block_table, max_blocks,
+                  ctx_base, n_seg, (bf16*)out, n_rows, page_size, W);
+    return kp_launch_status();
+}
+
+// q: rows of H heads of dimp + rotp; ex [T][ld_ex]: the expanded keys (H heads of dimp) and, from v_col on, values (H
+// heads of vdimp); rows [T][W]: the gathered cache rows; tile_seg / tile_row0: n_tiles tiles of 64 rows.
+int kp_latent_prefill(const void* q, int ldq, const void* ex, int ld_ex, int v_col, const void* rows, int rankp, int dimp, int rotp,
+                      int vdimp, const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0, const int* ctx_base,
+                      int n_tiles, void* out, int ldo, float scale, int H, void* stream) {
+    if (n_tiles <= 0) return 0;
+    if ((dimp & 15) || (rotp & 15) || (vdimp & 15) || (rankp & 15) || H < 1 || H > 65535) return KP_ERR_BAD_ARG;
+    if ((ldq & 1) || (ldo & 1) || (ld_ex & 7) || (v_col & 7) || (((uintptr_t)ex | (uintptr_t)rows) & 15)) return KP_ERR_UNSUPPORTED;
+    const int Dq = dimp + rotp;
+    LatentPrefillArgs a = {(const bf16*)q, (const bf16*)ex, (const bf16*)rows, (bf16*)out, cu_rows, seg_pos, tile_seg, tile_row0, ctx_base,
+                           ldq, ldo, ld_ex, rankp + rotp, rankp, dimp, rotp, vdimp, v_col, n_tiles, scale};
+    const size_t sm = (size_t)2 * LP_TILE * (Dq + 8 + vdimp + 8) * 2;
+    if (sm > 200 * 1024) return KP_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    int st;
+#define LP_LAUNCH(KS, VT)                                                                                                 \
+    do {                                                                                                                  \
+        st = la_set_smem(latent_prefill_kernel<KS, VT>, sm);                                                              \
+        if (st) return st;                                                                                                \
+        kp_launch_pdl(latent_prefill_kernel<KS, VT>, dim3(n_tiles, H), dim3(128), sm, s, a);                              \
+        return kp_launch_status();                                                                                        \
+    } while (0)
+    if (Dq <= 128 && vdimp <= 64) LP_LAUNCH(8, 8);
+    if (Dq <= 128 && vdimp <= 128) LP_LAUNCH(8, 16);
+    if (Dq <= 192 && vdimp <= 128) LP_LAUNCH(12, 16);
+    if (Dq <= 256 && vdimp <= 256) LP_LAUNCH(16, 32);
+#undef LP_LAUNCH
+    return KP_ERR_UNSUPPORTED;
+}
+
+}  // extern "C"

@@ -10,6 +10,10 @@
 // constant, not renormalised.  The last `n_identity` router outputs may stand for experts without weights that
 // return their input: their pairs get places in the layout but no tiles, and the combine adds weight * h for them.
 //
+// In that way the choice may be made from groups of experts (`n_groups` equal stretches of neighbours, 0 or 1: no groups):
+// a group is as good as its best expert, and only experts of the `keep` best groups can be chosen; and with `renorm` the
+// weights are divided by their sum (+ 1e-20) before the constant.
+//
 // A third (`mode` 2): the `top` largest logits are chosen, as in the first, and the weight of a chosen expert is
 // sigmoid(z) times the constant, each on its own, not renormalised.
 //
@@ -39,7 +43,8 @@
 // One warp chooses for one row.  z [E]: the row's router logits in shared memory (mode 0: bias already added); they
 // are overwritten.  s [E]: room for the scores of mode 1.
 __device__ __forceinline__ void moe_choose(float* z, float* s, int E, int top, int mode, const float* __restrict__ bias,
-                                           float wscale, int* __restrict__ idx_out, float* __restrict__ w_out) {
+                                           float wscale, int n_groups, int keep, int renorm, int* __restrict__ idx_out,
+                                           float* __restrict__ w_out) {
     const int lane = threadIdx.x & 31;
     if (mode == 1) {
         // scores over all outputs; the choice runs over score + correction, the weight is the score
@@ -55,6 +60,29 @@ __device__ __forceinline__ void moe_choose(float* z, float* s, int E, int top, i
             z[e] = sc + (bias ? bias[e] : 0.f);
         }
         __syncwarp();
+        if (n_groups > 1 && keep < n_groups) {
+            const int per = E / n_groups;
+            unsigned long long kept = 0ull;                     // bit c: group c is kept (at most 64 groups)
+            for (int k = 0; k < keep; k++) {
+                float best = -INFINITY;                         // the best expert outside the groups kept so far
+                int bi = 0x7fffffff;
+                for (int e = lane; e < E; e += 32) {
+                    const float v = z[e];
+                    if (v > best && !((kept >> (e / per)) & 1ull)) { best = v; bi = e; }
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+                    if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+                }
+                if (bi == 0x7fffffff) break;                    // (a row of NaN: the choice below keeps the indices legal)
+                kept |= 1ull << (bi / per);
+            }
+            for (int e = lane; e < E; e += 32)
+                if (!((kept >> (e / per)) & 1ull)) z[e] = -INFINITY;
+            __syncwarp();
+        }
     }
     float my_z = -INFINITY;
     int my_e = 0;
@@ -77,9 +105,11 @@ __device__ __forceinline__ void moe_choose(float* z, float* s, int E, int top, i
         __syncwarp();
     }
     if (mode == 1) {
+        float wt = lane < top ? s[my_e] : 0.f;
+        if (renorm) wt /= warp_sum(wt) + 1e-20f;
         if (lane < top) {
             idx_out[lane] = my_e;
-            w_out[lane] = s[my_e] * wscale;
+            w_out[lane] = wt * wscale;
         }
         return;
     }
@@ -101,7 +131,7 @@ __device__ __forceinline__ void moe_choose(float* z, float* s, int E, int top, i
 
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int n, int E, int top, int mode,
-                 float wscale, int* __restrict__ idx_out, float* __restrict__ w_out) {
+                 float wscale, int n_groups, int keep, int renorm, int* __restrict__ idx_out, float* __restrict__ w_out) {
     kp_pdl_begin();
     extern __shared__ float route_sm[];                         // [warps][2 E]: logits, scores
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -110,7 +140,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
     float* z = route_sm + (size_t)warp * 2 * E;
     for (int e = lane; e < E; e += 32) z[e] = logits[(size_t)r * E + e] + (mode == 0 && bias ? bias[e] : 0.f);
     __syncwarp();
-    moe_choose(z, z + E, E, top, mode, bias, wscale, idx_out + (size_t)r * top, w_out + (size_t)r * top);
+    moe_choose(z, z + E, E, top, mode, bias, wscale, n_groups, keep, renorm, idx_out + (size_t)r * top, w_out + (size_t)r * top);
 }
 
 // The router as one kernel: logits z = h Wr^T + b in float32 (h is widened from its storage type; a row's
@@ -122,7 +152,8 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
 template <typename T, int RB>
 __global__ void __launch_bounds__(256)
 moe_router_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ wr, const float* __restrict__ bias, int n,
-                  int E, int d, int top, int mode, float wscale, int* __restrict__ idx_out, float* __restrict__ w_out) {
+                  int E, int d, int top, int mode, float wscale, int n_groups, int keep, int renorm, int* __restrict__ idx_out,
+                  float* __restrict__ w_out) {
     kp_pdl_begin();
     extern __shared__ __align__(16) float router_sm[];          // [RB][d] rows, [RB][2 E] logits and scores
     float* hs = router_sm;
@@ -172,7 +203,8 @@ moe_router_kernel(const T* __restrict__ h, int ldh, const float* __restrict__ wr
     __syncthreads();
     if (warp >= nr) return;
     float* z = zs + (size_t)warp * 2 * E;                        // warp r chooses for row r
-    moe_choose(z, z + E, E, top, mode, bias, wscale, idx_out + (size_t)(row0 + warp) * top, w_out + (size_t)(row0 + warp) * top);
+    moe_choose(z, z + E, E, top, mode, bias, wscale, n_groups, keep, renorm, idx_out + (size_t)(row0 + warp) * top,
+               w_out + (size_t)(row0 + warp) * top);
 }
 
 // ------------------------------------------------------------------------------------------------- sort
@@ -768,9 +800,15 @@ int kp_moe_max_tiles(int n, int E, int top) {
 // logits [n, E] float32 -> idx [n, top], weights [n, top], and the layout (see kp_moe_layout_ints).
 // mode 0: the largest logits (+ bias), weights = softmax over the chosen; mode 1: scores = softmax over all, the largest
 // score + bias chosen, weights = score * wscale; mode 2: the largest logits, weights = sigmoid(logit) * wscale.  The last n_identity of the E outputs are experts without weights.
+// n_groups, keep, renorm: the choice from groups and the renormalised weights of mode 1 (0, 0, 0: neither).
+static bool moe_groups_ok(int E, int top, int mode, int n_groups, int keep, int renorm) {
+    if (n_groups <= 1) return n_groups >= 0 && (!renorm || mode == 1);
+    return mode == 1 && n_groups <= 64 && E % n_groups == 0 && keep >= 1 && keep <= n_groups && top <= keep * (E / n_groups);
+}
 int kp_moe_route(const float* logits, const float* bias, int n, int E, int top, int mode, float wscale, int n_identity,
-                 int* idx, float* weights, int* layout, void* stream) {
+                 int n_groups, int keep, int renorm, int* idx, float* weights, int* layout, void* stream) {
     if (n <= 0) return 0;
+    if (!moe_groups_ok(E, top, mode, n_groups, keep, renorm)) return KP_ERR_UNSUPPORTED;
     if (E < 1 || top < 1 || top > E || top > MOE_MAX_TOP || mode < 0 || mode > 2 || n_identity < 0 || n_identity >= E)
         return KP_ERR_UNSUPPORTED;
     const size_t route_sm = (size_t)8 * 2 * E * sizeof(float), sort_sm = ((size_t)3 * E + 1) * sizeof(int);
@@ -780,7 +818,8 @@ int kp_moe_route(const float* logits, const float* bias, int n, int E, int top, 
         cudaError_t e = cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)route_sm);
         if (e != cudaSuccess) return (int)e;
     }
-    kp_launch_pdl(moe_route_kernel, dim3((n + 7) / 8), dim3(256), route_sm, s, logits, bias, n, E, top, mode, wscale, idx, weights);
+    kp_launch_pdl(moe_route_kernel, dim3((n + 7) / 8), dim3(256), route_sm, s, logits, bias, n, E, top, mode, wscale, n_groups, keep, renorm,
+                  idx, weights);
     cudaError_t e0 = cudaGetLastError();
     if (e0 != cudaSuccess) return (int)e0;
     int* offsets = layout;
@@ -797,8 +836,10 @@ int kp_moe_route(const float* logits, const float* bias, int n, int E, int top, 
 // and the layout.  KP_ERR_UNSUPPORTED where the rows do not fit the kernel's shared memory or alignment (the caller
 // then computes the logits with a matrix product and calls kp_moe_route).
 int kp_moe_router(const void* h, int ldh, const float* wr, const float* bias, int n, int E, int d, int top, int mode,
-                  float wscale, int n_identity, int* idx, float* weights, int* layout, int dtype, void* stream) {
+                  float wscale, int n_identity, int n_groups, int keep, int renorm, int* idx, float* weights, int* layout, int dtype,
+                  void* stream) {
     if (n <= 0) return 0;
+    if (!moe_groups_ok(E, top, mode, n_groups, keep, renorm)) return KP_ERR_UNSUPPORTED;
     if (E < 1 || top < 1 || top > E || top > MOE_MAX_TOP || mode < 0 || mode > 2 || n_identity < 0 || n_identity >= E)
         return KP_ERR_UNSUPPORTED;
     const size_t sort_sm = ((size_t)3 * E + 1) * sizeof(int);
@@ -814,7 +855,7 @@ int kp_moe_router(const void* h, int ldh, const float* wr, const float* bias, in
             if (e != cudaSuccess) return (int)e;                                                                          \
         }                                                                                                                 \
         kp_launch_pdl(moe_router_kernel<T, RB>, dim3((n + RB - 1) / RB), dim3(256), sm, s, (const T*)h, ldh, wr, bias, n, E, d, \
-                      top, mode, wscale, idx, weights);                                                                   \
+                      top, mode, wscale, n_groups, keep, renorm, idx, weights);                                                                   \
     } while (0)
     KP_DISPATCH_DTYPE(dtype, T, { if (rb == 8) MOE_ROUTER_LAUNCH(T, 8); else MOE_ROUTER_LAUNCH(T, 1); });
 #undef MOE_ROUTER_LAUNCH

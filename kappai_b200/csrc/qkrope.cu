@@ -16,6 +16,8 @@
 // `norm_dim` (<= hd): the number the norm's mean is taken over, for heads stored wider than they are with
 // zeros behind their own columns.  A query temperature (temp_every > 0): the query heads of the row at position
 // p leave multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1), computed in float32.
+// `norm_after`: instead of the norm in front of the rotation q and k are divided by their root mean square behind it
+// (no weight).
 #include "common.cuh"
 
 #define KP_MAX_HEAD_DIM 256
@@ -31,7 +33,8 @@ qk_norm_rope_kv_kernel(const T* qkv, int ld, const float* __restrict__ q_w,
                        const float* __restrict__ sin_tab, int rot, int interleaved,
                        const int* __restrict__ positions, const int* __restrict__ slot_map,
                        T* q_out, int ldq, T* __restrict__ cache, int page_size,
-                       int H, int G, int hd, int write_kv, int v_col, int norm_dim, float temp_coef, float temp_every) {
+                       int H, int G, int hd, int write_kv, int v_col, int norm_dim, float temp_coef, float temp_every,
+                       int norm_after) {
     kp_pdl_begin();
     __shared__ float buf[4][KP_MAX_HEAD_DIM];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -72,6 +75,13 @@ qk_norm_rope_kv_kernel(const T* qkv, int ld, const float* __restrict__ q_w,
         }
         __syncwarp();
     }
+    if (norm_after && kind != 2) {
+        float sq = 0.f;
+        for (int i = lane; i < hd; i += 32) sq = fmaf(x[i], x[i], sq);
+        sq = warp_sum(sq);
+        const float scale = 1.0f / sqrtf(sq / (float)norm_dim + eps);
+        for (int i = lane; i < hd; i += 32) x[i] *= scale;
+    }
     if (kind == 0 && temp_every > 0.f) {
         const float tq = kp_query_temperature(positions[row], temp_coef, temp_every);
         for (int i = lane; i < hd; i += 32) x[i] *= tq;
@@ -103,7 +113,7 @@ qk_norm_rope_kv_vec_kernel(const bf16* __restrict__ qkv, int ld, const float* __
                            const float* __restrict__ sin_tab, const int* __restrict__ positions,
                            const int* __restrict__ slot_map, bf16* __restrict__ q_out, int ldq,
                            bf16* __restrict__ cache, int page_size, int H, int G, int write_kv, int v_col, int rot,
-                           int norm_dim, float temp_coef, float temp_every) {
+                           int norm_dim, float temp_coef, float temp_every, int norm_after) {
     kp_pdl_begin_early();
     constexpr int L = HD / 8;                          // lanes a head
     constexpr int HPB = 128 / L;                       // heads a block
@@ -150,6 +160,18 @@ qk_norm_rope_kv_vec_kernel(const bf16* __restrict__ qkv, int ld, const float* __
             if (kind != 2 && rotated) x[i] = lower ? x[i] * cc[i] - other * sn[i] : other * sn[i] + x[i] * cc[i];
         }
     }
+    if (norm_after) {                                  // (every lane takes part in the shuffles)
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) ss = fmaf(x[i], x[i], ss);
+#pragma unroll
+        for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float scale = 1.0f / sqrtf(ss / (float)norm_dim + eps);
+        if (kind != 2) {
+#pragma unroll
+            for (int i = 0; i < 8; i++) x[i] *= scale;
+        }
+    }
     if (!live || (kind != 0 && !write_kv)) return;
     if (kind == 0 && temp_every > 0.f) {
         const float tq = kp_query_temperature(positions[row], temp_coef, temp_every);
@@ -175,12 +197,13 @@ qk_norm_rope_kv_vec_kernel(const bf16* __restrict__ qkv, int ld, const float* __
     *reinterpret_cast<uint4*>(dst + lane_in * 8) = o;
 }
 
-extern "C" int kp_qk_norm_rope_kv_temp(const void* qkv, int ld, const float* q_w, const float* k_w, float eps,
-                                       const float* cos_tab, const float* sin_tab, int rot, int interleaved,
-                                       const int* positions, const int* slot_map, void* q_out, int ldq, void* cache,
-                                       int page_size, int n, int H, int G, int hd, int write_kv, int v_col, int norm_dim,
-                                       float temp_coef, float temp_every, int dtype, void* stream) {
+extern "C" int kp_qk_norm_rope_kv_after(const void* qkv, int ld, const float* q_w, const float* k_w, float eps,
+                                        const float* cos_tab, const float* sin_tab, int rot, int interleaved,
+                                        const int* positions, const int* slot_map, void* q_out, int ldq, void* cache,
+                                        int page_size, int n, int H, int G, int hd, int write_kv, int v_col, int norm_dim,
+                                        float temp_coef, float temp_every, int norm_after, int dtype, void* stream) {
     if (n <= 0) return 0;
+    if (norm_after && (q_w || k_w || q_out == nullptr)) return KP_ERR_BAD_ARG;
     if (norm_dim <= 0) norm_dim = hd;
     if (norm_dim > hd || temp_every < 0.f) return KP_ERR_BAD_ARG;
     if (v_col < 0) v_col = (H + G) * hd;
@@ -199,18 +222,27 @@ extern "C" int kp_qk_norm_rope_kv_temp(const void* qkv, int ld, const float* q_w
         if (hd == 64)
             kp_launch_pdl(qk_norm_rope_kv_vec_kernel<64>, dim3(vgrid), dim3(128), 0, (cudaStream_t)stream, (const bf16*)qkv, ld, q_w,
                           k_w, eps, cos_tab, sin_tab, positions, slot_map, (bf16*)q_out, ldq, (bf16*)cache, page_size, H, G, write_kv, v_col, rot,
-                          norm_dim, temp_coef, temp_every);
+                          norm_dim, temp_coef, temp_every, norm_after);
         else
             kp_launch_pdl(qk_norm_rope_kv_vec_kernel<128>, dim3(vgrid), dim3(128), 0, (cudaStream_t)stream, (const bf16*)qkv, ld, q_w,
                           k_w, eps, cos_tab, sin_tab, positions, slot_map, (bf16*)q_out, ldq, (bf16*)cache, page_size, H, G, write_kv, v_col, rot,
-                          norm_dim, temp_coef, temp_every);
+                          norm_dim, temp_coef, temp_every, norm_after);
         return kp_launch_status();
     }
     dim3 grid((H + 2 * G + 3) / 4, n);
     KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(qk_norm_rope_kv_kernel<T>, dim3(grid), dim3(128), 0, (cudaStream_t)stream, 
         (const T*)qkv, ld, q_w, k_w, eps, cos_tab, sin_tab, rot, interleaved, positions, slot_map, (T*)q_out, ldq,
-        (T*)cache, page_size, H, G, hd, write_kv, v_col, norm_dim, temp_coef, temp_every)));
+        (T*)cache, page_size, H, G, hd, write_kv, v_col, norm_dim, temp_coef, temp_every, norm_after)));
     return kp_launch_status();
+}
+
+extern "C" int kp_qk_norm_rope_kv_temp(const void* qkv, int ld, const float* q_w, const float* k_w, float eps,
+                                       const float* cos_tab, const float* sin_tab, int rot, int interleaved,
+                                       const int* positions, const int* slot_map, void* q_out, int ldq, void* cache,
+                                       int page_size, int n, int H, int G, int hd, int write_kv, int v_col, int norm_dim,
+                                       float temp_coef, float temp_every, int dtype, void* stream) {
+    return kp_qk_norm_rope_kv_after(qkv, ld, q_w, k_w, eps, cos_tab, sin_tab, rot, interleaved, positions, slot_map, q_out, ldq,
+                                    cache, page_size, n, H, G, hd, write_kv, v_col, norm_dim, temp_coef, temp_every, 0, dtype, stream);
 }
 
 extern "C" int kp_qk_norm_rope_kv(const void* qkv, int ld, const float* q_w, const float* k_w, float eps,
@@ -277,5 +309,72 @@ extern "C" int kp_qk_rownorm_kv(const void* qkv, int ld, int k_col, int v_col, c
     KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(qk_rownorm_kv_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, (const T*)qkv, ld,
                                                k_col, v_col, q_w, k_w, eps, count_q, count_k, slot_map, (T*)q_out, ldq, (T*)cache,
                                                page_size, H, G, hd, write_kv)));
+    return kp_launch_status();
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// Means of blocks of `pool` positions: where a row of this step completes a block (its position p has (p + 1) % pool ==
+// 0), the block's keys and values as the cache holds them are averaged (float32, summed in the order of the positions,
+// whatever steps brought them there) and the means stored as entry p / pool of the request's pooled pages.
+// pool_slot_map: the entry's slot a row, -1 for a row that completes no block.  VEC: elements a thread takes.
+template <typename T, int VEC> struct PoolVec;
+template <> struct PoolVec<bf16, 8> { typedef uint4 V; };
+template <> struct PoolVec<float, 4> { typedef float4 V; };
+template <> struct PoolVec<bf16, 1> { typedef bf16 V; };
+template <> struct PoolVec<float, 1> { typedef float V; };
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128)
+pool_blocks_kernel(const T* __restrict__ cache, const int* __restrict__ block_table, int max_blocks, const int* __restrict__ row_seg,
+                   const int* __restrict__ positions, const int* __restrict__ pool_slot_map, T* __restrict__ pool_cache, int pool,
+                   int page_size, int planes_heads, int hd) {
+    kp_pdl_begin();
+    typedef typename PoolVec<T, VEC>::V V;
+    const int row = blockIdx.y;
+    const int slot = pool_slot_map[row];
+    if (slot < 0) return;
+    const int per = hd / VEC;
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;            // (K or V, head, stretch of the head)
+    if (i >= planes_heads * per) return;
+    const int head = i / per, c = (i - head * per) * VEC;
+    const int p0 = positions[row] - pool + 1;
+    const int* bt = block_table + (size_t)row_seg[row] * max_blocks;
+    float acc[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; j++) acc[j] = 0.f;
+#pragma unroll 4
+    for (int k = 0; k < pool; k++) {
+        const int pos = p0 + k;
+        const V v = *reinterpret_cast<const V*>(cache + (((size_t)bt[pos / page_size] * planes_heads + head) * page_size + pos % page_size) * hd + c);
+        const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+        for (int j = 0; j < VEC; j++) acc[j] += to_f32(e[j]);
+    }
+    V o;
+    T* e = reinterpret_cast<T*>(&o);
+#pragma unroll
+    for (int j = 0; j < VEC; j++) e[j] = from_f32<T>(acc[j] / (float)pool);
+    *reinterpret_cast<V*>(pool_cache + (((size_t)(slot / page_size) * planes_heads + head) * page_size + slot % page_size) * hd + c) = o;
+}
+
+extern "C" int kp_pool_blocks(const void* cache, const int* block_table, int max_blocks, const int* row_seg, const int* positions,
+                              const int* pool_slot_map, void* pool_cache, int pool, int page_size, int n, int G, int hd, int dtype,
+                              void* stream) {
+    if (n <= 0) return 0;
+    if (pool < 1 || page_size < 1 || G < 1 || hd < 1 || n > 65535) return KP_ERR_BAD_ARG;
+    const int ph = 2 * G;
+    cudaStream_t s = (cudaStream_t)stream;
+#define POOL_LAUNCH(T, VEC)                                                                                               \
+    kp_launch_pdl(pool_blocks_kernel<T, VEC>, dim3((ph * (hd / VEC) + 127) / 128, n), dim3(128), 0, s, (const T*)cache, block_table, \
+                  max_blocks, row_seg, positions, pool_slot_map, (T*)pool_cache, pool, page_size, ph, hd)
+    const bool aligned = !(((uintptr_t)cache | (uintptr_t)pool_cache) & 15);
+    if (dtype == KP_DTYPE_BF16) {
+        if (aligned && hd % 8 == 0) POOL_LAUNCH(bf16, 8); else POOL_LAUNCH(bf16, 1);
+    } else if (dtype == KP_DTYPE_F32) {
+        if (aligned && hd % 4 == 0) POOL_LAUNCH(float, 4); else POOL_LAUNCH(float, 1);
+    } else {
+        return KP_ERR_BAD_ARG;
+    }
+#undef POOL_LAUNCH
     return kp_launch_status();
 }

@@ -42,6 +42,15 @@ __global__ void rmsnorm_rows_kernel(const float* __restrict__ x, const float* __
 }
 
 // four consecutive outputs in one store (the destination is 8- or 16-byte aligned: d % 4 == 0)
+__device__ __forceinline__ void load4(const float* src, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(src);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void load4(const bf16* src, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(src);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+    v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+}
 __device__ __forceinline__ void store4(float* dst, float a, float b, float c, float d) {
     *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
 }
@@ -496,6 +505,86 @@ rmsnorm_add_norm_rows_vec_kernel(float* __restrict__ y, const float* __restrict_
     }
 }
 
+// A sublayer's output joins the residual scaled a channel and gated element by element:
+//   x += (ls * sigmoid(g)) * y ;  y <- 0        (ls [d] or null: 1; g [n, d] in the storage type, rows ldg apart, or null: 1)
+// and, with h_out, the norm in front of the next sublayer: h_out = x / sqrt(mean(x^2) + eps) * wn.  One block a row; the
+// row stays in registers (PER float4s a thread), or where it is too long or unaligned in memory (PER = 0).
+template <typename T, int PER>
+__global__ void __launch_bounds__(256)
+gated_add_norm_rows_kernel(float* __restrict__ y, const T* __restrict__ g, int ldg, const float* __restrict__ ls, float* __restrict__ x,
+                           const float* __restrict__ wn, float eps, T* __restrict__ h_out, int d) {
+    kp_pdl_begin_early_if(gridDim.x > 1);
+    __shared__ float red[32];
+    const int r = blockIdx.x;
+    float* yr = y + (size_t)r * d;
+    float* xr = x + (size_t)r * d;
+    const T* gr = g ? g + (size_t)r * ldg : nullptr;
+    auto gate = [](float z) { return 1.0f / (1.0f + expf(-z)); };
+    float ss = 0.f;
+    if constexpr (PER > 0) {
+        const int d4 = d >> 2;
+        float4 v[PER];
+#pragma unroll
+        for (int j = 0; j < PER; j++) {
+            const int i = threadIdx.x + j * 256;
+            if (i < d4) {
+                const float4 b = reinterpret_cast<const float4*>(yr)[i];
+                float4 a = reinterpret_cast<const float4*>(xr)[i];
+                float f[4] = {1.f, 1.f, 1.f, 1.f};
+                if (gr) {
+                    float z[4];
+                    load4(gr + 4 * i, z);
+#pragma unroll
+                    for (int k = 0; k < 4; k++) f[k] = gate(z[k]);
+                }
+                if (ls) {
+                    const float4 w = __ldg(reinterpret_cast<const float4*>(ls) + i);
+                    f[0] *= w.x; f[1] *= w.y; f[2] *= w.z; f[3] *= w.w;
+                }
+                a.x = fmaf(f[0], b.x, a.x); a.y = fmaf(f[1], b.y, a.y); a.z = fmaf(f[2], b.z, a.z); a.w = fmaf(f[3], b.w, a.w);
+                reinterpret_cast<float4*>(xr)[i] = a;
+                reinterpret_cast<float4*>(yr)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                v[j] = a;
+                ss = fmaf(a.x, a.x, ss); ss = fmaf(a.y, a.y, ss); ss = fmaf(a.z, a.z, ss); ss = fmaf(a.w, a.w, ss);
+            }
+        }
+        if (h_out == nullptr) return;
+        ss = block_sum(ss, red);
+        const float sn = 1.0f / sqrtf(ss / (float)d + eps);
+        T* hr = h_out + (size_t)r * d;
+#pragma unroll
+        for (int j = 0; j < PER; j++) {
+            const int i = threadIdx.x + j * 256;
+            if (i < d4) {
+                const float4 w = __ldg(reinterpret_cast<const float4*>(wn) + i);
+                store4(hr + 4 * i, (v[j].x * sn) * w.x, (v[j].y * sn) * w.y, (v[j].z * sn) * w.z, (v[j].w * sn) * w.w);
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < d; i += 256) {
+            const float f = (gr ? gate(to_f32(gr[i])) : 1.f) * (ls ? ls[i] : 1.f);
+            const float a = fmaf(f, yr[i], xr[i]);
+            xr[i] = a;
+            yr[i] = 0.f;
+            ss = fmaf(a, a, ss);
+        }
+        if (h_out == nullptr) return;
+        ss = block_sum(ss, red);
+        const float sn = 1.0f / sqrtf(ss / (float)d + eps);
+        T* hr = h_out + (size_t)r * d;
+        for (int i = threadIdx.x; i < d; i += 256) hr[i] = from_f32<T>((xr[i] * sn) * wn[i]);
+    }
+}
+
+// An activation by itself, element by element (an ungated unit), from the float32 product to the storage type.
+template <typename T>
+__global__ void __launch_bounds__(256)
+activate_kernel(const float* __restrict__ in, T* __restrict__ out, size_t n, int act) {
+    kp_pdl_begin();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
+        out[i] = from_f32<T>(kp_act_plain(act, in[i]));
+}
+
 // out[r, :] += sigmoid(h[r, :] . wg) * y[r, :]: a branch weighed by one gate a row, the gate's logit computed here
 // (float32 sum in a fixed order, h widened from its storage type).
 template <typename T>
@@ -914,6 +1003,31 @@ int kp_rmsnorm_add_norm_rows(float* y, const float* wb, float eps_b, float* x, c
     }
     KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(rmsnorm_add_norm_rows_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, y, wb,
                                                eps_b, x, wn, eps_n, (T*)h_out, d)));
+    return kp_launch_status();
+}
+
+int kp_gated_add_norm_rows(float* y, const void* g, int ldg, const float* ls, float* x, const float* wn, float eps, void* h_out,
+                           int n, int d, int dtype, void* stream) {
+    if (n <= 0) return 0;
+    if (d < 1 || ((wn == nullptr) != (h_out == nullptr))) return KP_ERR_BAD_ARG;
+    const bool vec = (d & 3) == 0 && d <= 8192 && (ldg & 3) == 0 &&
+                     !(((uintptr_t)y | (uintptr_t)x | (uintptr_t)wn | (uintptr_t)h_out | (uintptr_t)ls | (uintptr_t)g) & 15);
+#define GATED_ADD(PER)                                                                                                     \
+    KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(gated_add_norm_rows_kernel<T, PER>, dim3(n), dim3(256), 0, (cudaStream_t)stream, y, \
+                                               (const T*)g, ldg, ls, x, wn, eps, (T*)h_out, d)))
+    if (!vec) GATED_ADD(0);
+    else if (d <= 2048) GATED_ADD(2);
+    else if (d <= 4096) GATED_ADD(4);
+    else GATED_ADD(8);
+#undef GATED_ADD
+    return kp_launch_status();
+}
+
+int kp_activate(const float* in, void* out, long long n, int act, int dtype, void* stream) {
+    if (n <= 0) return 0;
+    const long long blocks = (n + 255) / 256;
+    KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(activate_kernel<T>, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0,
+                                               (cudaStream_t)stream, in, (T*)out, (size_t)n, act)));
     return kp_launch_status();
 }
 

@@ -134,14 +134,15 @@ def build_step_context(segments: Sequence[Segment], groups: Dict[Hashable, int],
 
 
 def lay_out_step(segments: Sequence[Segment], groups: Dict[Hashable, int], vocab_size: int, max_positions: int,
-                 table_builders: Optional[Dict[Hashable, object]] = None, round_blocks=None, round_context=None
-                 ) -> HostStep:
+                 table_builders: Optional[Dict[Hashable, object]] = None, round_blocks=None, round_context=None,
+                 every: Optional[Dict[Hashable, int]] = None) -> HostStep:
     """Validate the segments and lay their tables out on the host.
 
     ``round_blocks`` / ``round_context`` (for steps that may be captured): the width of the block tables and the
     step's largest context are rounded up by them, so that steps that differ a little share a signature.
 
-    ``groups`` maps each page group to its page size.  Everything that could
+    ``groups`` maps each page group to its page size, ``every`` those with an entry for several positions to that
+    number.  Everything that could
     make a kernel read or write out of bounds is refused here, before any
     launch (token ids: src/context.c:866-867; positions: src/context.c:998-999).
     ``table_builders`` maps a key to a part whose ``step_tables(StepSegments)``
@@ -219,7 +220,7 @@ def lay_out_step(segments: Sequence[Segment], groups: Dict[Hashable, int], vocab
             n = len(s.tokens)
             if t is None or ts is None or len(ts) != n:
                 raise BatchError(f"request {s.req!r}: no block table / token slots for page group {gk!r}")
-            need = -(-(s.pos_start + n) // page_size)
+            need = -(-((s.pos_start + n) // (every or {}).get(gk, 1)) // page_size)
             if len(t) < need:
                 raise BatchError(f"request {s.req!r}: block table covers {len(t)} blocks, {need} needed")
             bt[i, :len(t)] = t

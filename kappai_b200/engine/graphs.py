@@ -140,7 +140,7 @@ class _DecodeGraph:
                     bt[j, :len(t)] = t
                     bt[j, len(t):] = 0
                     keys[j] = key
-                sm[j] = t[lens[j] // ps] * ps + lens[j] % ps
+                sm[j] = t[lens[j] // ps] * ps + lens[j] % ps if pool.every == 1 else pool.slot(r, lens[j])
         if self.part_layout:
             self._fill_part_tables(lens)
         np.copyto(self.pinned_np[i], a)

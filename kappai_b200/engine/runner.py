@@ -95,8 +95,9 @@ class ModelRunner:
         state_bytes = 0
         for s in (leaf for spec in specs for leaf in leaf_specs(spec)):
             if isinstance(s, PagedKVSpec):
-                g = needs.setdefault(s.group_key, GroupNeed(s.group_key, 0, s.window, s.keep_first if s.window is not None else 0))
-                g.bytes_per_token += 2 * s.num_kv_heads * s.head_dim * elt
+                g = needs.setdefault(s.group_key, GroupNeed(s.group_key, 0, s.window, s.keep_first if s.window is not None else 0,
+                                                            s.every))
+                g.bytes_per_token += s.planes * s.num_kv_heads * s.head_dim * elt
             elif isinstance(s, StateSpec):
                 n = 1
                 for d in s.shape:
@@ -113,9 +114,11 @@ class ModelRunner:
         self.storage = CacheStorage(specs, borrowing, plan.pages, page_size, max_requests, self.dtype, self.device)
         self.cache = CacheManager({gk: (plan.pages[gk], page_size, self.storage.groups[gk].window,
                                         self.storage.groups[gk].block,
-                                        self.storage.groups[gk].keep_first if self.storage.groups[gk].window is not None else 0)
+                                        self.storage.groups[gk].keep_first if self.storage.groups[gk].window is not None else 0,
+                                        self.storage.groups[gk].every)
                                    for gk in group_keys}, max_requests)
         self.group_page_size = {gk: page_size for gk in group_keys}
+        self.group_every = {gk: self.storage.groups[gk].every for gk in group_keys}
         self.vocab_size = self.spec.vocab_size
         self.last_h2d_bytes = 0
         self.observer = None               # called with the residual behind every layer of a step (debugging): see Model.forward
@@ -138,7 +141,7 @@ class ModelRunner:
             return self.cache.can_extend(req, self.cache.requests[req].length + n_new)
         if not self.cache.can_admit():
             return False
-        return all(-(-n_new // p.page_size) <= p.n_free for p in self.cache.pools.values())
+        return all(p.pages_for(n_new) <= p.n_free for p in self.cache.pools.values())
 
     def check_status(self) -> None:
         """Wait for the device and raise if a kernel gave up a bounded wait since the last check (its output
@@ -196,7 +199,8 @@ class ModelRunner:
         g = self.graphs if capturable else None
         host = lay_out_step(segs, self.group_page_size, self.vocab_size, self.max_model_len, self.model.table_builders,
                             round_blocks=g.round_blocks if g else None,
-                            round_context=(lambda t: min(self.max_model_len, g.round_context(t))) if g else None)
+                            round_context=(lambda t: min(self.max_model_len, g.round_context(t))) if g else None,
+                            every=self.group_every)
         return host, [(req, new_len) for req, _, new_len in plan]
 
     def prepare(self, entries: Sequence[StepEntry]) -> Tuple[StepContext, List[Tuple[Hashable, int]]]:

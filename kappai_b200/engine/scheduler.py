@@ -159,7 +159,7 @@ class Scheduler:
                and self.cache.can_admit()):
             r = self.waiting[0]
             n = min(r.n_tokens, budget)
-            if not all(-(-n // p.page_size) <= p.n_free for p in self.cache.pools.values()):
+            if not all(p.pages_for(n) <= p.n_free for p in self.cache.pools.values()):
                 if not self.running and not entries:
                     # nothing runs, every page is free, and the first portion still does not fit
                     self.waiting.popleft()

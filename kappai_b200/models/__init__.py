@@ -5,3 +5,4 @@ from . import vekuzen  # noqa: F401
 from . import tupalorn  # noqa: F401
 from . import vumotar  # noqa: F401
 from . import gosulorn  # noqa: F401
+from . import ladedra  # noqa: F401

@@ -173,7 +173,7 @@ def _rows_2d(t: torch.Tensor, name: str) -> int:
 # issuing work and returns.  The engine reads the words of a step with the step's own device-to-host copy.
 
 _STATUS_LIBS = (("gemm_tc", "tc"), ("gemm_stream", "stream"), ("attention_mma", "attention_mma"),
-                ("attention_tc", "attention_tc"), ("moe", "moe_tc"))
+                ("attention_tc", "attention_tc"), ("moe", "moe_tc"), ("latent", "latent"))
 
 
 def read_status() -> dict:
@@ -379,6 +379,15 @@ def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: f
 ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2}     # codes of the gated units' activations (csrc/common.cuh)
 
 
+PLAIN_ACTIVATIONS = dict(ACTIVATIONS, relu_squared=4)    # the ungated units have one more
+
+
+def plain_activation_code(name: str) -> int:
+    if name not in PLAIN_ACTIVATIONS:
+        raise KernelError(f"activation '{name}' (expected one of {', '.join(PLAIN_ACTIVATIONS)})")
+    return PLAIN_ACTIVATIONS[name]
+
+
 def activation_code(name: str) -> int:
     try:
         return ACTIVATIONS[name]
@@ -518,6 +527,47 @@ def rmsnorm_add_norm_rows(y: torch.Tensor, w_branch: torch.Tensor, eps_branch: f
          ctypes.c_float(eps_branch), _ptr(x), _ptr(w_next), ctypes.c_float(eps_next), _ptr(h_out), n, d,
          dtype_code(h_out.dtype if h_out is not None else torch.float32), STREAM)
     return x
+
+
+def gated_add_norm_rows(y: torch.Tensor, gate: Optional[torch.Tensor], scale: Optional[torch.Tensor], x: torch.Tensor,
+                        w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0,
+                        h_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += scale * sigmoid(gate) * y (float32; ``scale`` [d] or None: 1, ``gate`` [n, d] in the compute type, its rows may be
+    strided, or None: 1), y cleared; with ``w_next`` and ``h_out`` also ``h_out = rmsnorm(x) * w_next`` of the new x."""
+    _need(y, "y", torch.float32); _need(x, "x", torch.float32)
+    n, d = x.shape
+    if tuple(y.shape) != (n, d) or (w_next is None) != (h_out is None):
+        raise KernelError("gated_add_norm_rows: shape mismatch")
+    dt = gate.dtype if gate is not None else (h_out.dtype if h_out is not None else torch.float32)
+    if gate is not None:
+        _need(gate, "gate", contiguous=False)
+        if tuple(gate.shape) != (n, d):
+            raise KernelError("gated_add_norm_rows: gate shape")
+    if scale is not None:
+        _need(scale, "scale", torch.float32)
+        if scale.numel() != d:
+            raise KernelError("gated_add_norm_rows: scale size")
+    if h_out is not None:
+        _need(w_next, "w_next", torch.float32); _need(h_out, "h_out", dt)
+        if tuple(h_out.shape) != (n, d) or w_next.numel() != d:
+            raise KernelError("gated_add_norm_rows: shape mismatch")
+    if n > MAX_STEP_ROWS:
+        raise KernelError("gated_add_norm_rows: too many rows")
+    _run("gated_add_norm_rows", load_library("rowwise").kp_gated_add_norm_rows, _ptr(y), _ptr(gate),
+         _rows_2d(gate, "gate") if gate is not None else 0, _ptr(scale), _ptr(x), _ptr(w_next), ctypes.c_float(eps_next), _ptr(h_out),
+         n, d, dtype_code(dt), STREAM,
+         work=(0, n * d * (16 + (gate.element_size() if gate is not None else 0) + (h_out.element_size() if h_out is not None else 0))))
+    return x
+
+
+def activate(x: torch.Tensor, out: torch.Tensor, activation: str) -> torch.Tensor:
+    """out = act(x), element by element (float32 in, ``out`` in the compute type)."""
+    _need(x, "x", torch.float32); _need(out, "out")
+    if x.shape != out.shape:
+        raise KernelError("activate: shape mismatch")
+    _run("activate", load_library("rowwise").kp_activate, _ptr(x), _ptr(out), ctypes.c_longlong(x.numel()), plain_activation_code(activation),
+         dtype_code(out.dtype), STREAM)
+    return out
 
 
 def row_gate_add(h: torch.Tensor, w_gate: torch.Tensor, y: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -1036,7 +1086,7 @@ def qk_norm_rope_kv(qkv: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optiona
                     interleaved: bool, positions: torch.Tensor, slot_map: Optional[torch.Tensor],
                     q_out: Optional[torch.Tensor], cache: Optional[torch.Tensor], page_size: int, H: int, G: int,
                     hd: int, v_col: Optional[int] = None, norm_dim: Optional[int] = None,
-                    q_temp: Optional[Tuple[float, float]] = None) -> Optional[torch.Tensor]:
+                    q_temp: Optional[Tuple[float, float]] = None, norm_after: bool = False) -> Optional[torch.Tensor]:
     """Norm + rotate q and k; write q to ``q_out`` and, if ``cache`` is given,
     k and v to their pages.  ``cache`` is one layer's [pages, 2, G, page_size, hd].
     With ``q_out`` None, q and k are changed in place and no cache is written.
@@ -1044,7 +1094,8 @@ def qk_norm_rope_kv(qkv: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optiona
     ``H * hd`` makes the values the key projections themselves, before norm and rotation).  Columns behind
     q, k and v are left alone.  ``norm_dim``: the number the norm's mean is taken over where a head is stored
     wider than it is (zeros behind its own columns; default ``hd``).  ``q_temp`` = (coef, every): the queries of
-    the row at position p leave multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)`` (float32)."""
+    the row at position p leave multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)`` (float32).  ``norm_after``: q
+    and k are divided by their root mean square (``eps``, no weight) behind the rotation, not in front of it."""
     _need(qkv, "qkv", contiguous=False)
     _need(positions, "positions", torch.int32)
     n = qkv.shape[0]
@@ -1077,16 +1128,18 @@ def qk_norm_rope_kv(qkv: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optiona
     nd = hd if norm_dim is None else int(norm_dim)
     if not (1 <= nd <= hd):
         raise KernelError("qk_norm_rope_kv: norm_dim")
+    if norm_after and (q_w is not None or k_w is not None or q_out is None):
+        raise KernelError("qk_norm_rope_kv: the norm behind the rotation has no weights and no in-place form")
     coef, every = (0.0, 0.0) if q_temp is None else (float(q_temp[0]), float(q_temp[1]))
     if q_temp is not None and not every > 0:
         raise KernelError("qk_norm_rope_kv: the query temperature's period must be positive")
     lib = load_library("qkrope")
-    _run("qk_norm_rope_kv", lib.kp_qk_norm_rope_kv_temp, _ptr(qkv), _rows_2d(qkv, "qkv"), _ptr(q_w), _ptr(k_w), ctypes.c_float(eps),
+    _run("qk_norm_rope_kv", lib.kp_qk_norm_rope_kv_after, _ptr(qkv), _rows_2d(qkv, "qkv"), _ptr(q_w), _ptr(k_w), ctypes.c_float(eps),
                                   _ptr(cos_tab), _ptr(sin_tab), rotary_dim, int(interleaved), _ptr(positions),
                                   _ptr(slot_map), _ptr(q_out), 0 if q_out is None else _rows_2d(q_out, "q_out"), _ptr(cache),
                                   page_size,
                                   n, H, G, hd, int(write_kv), int(v_col), nd, ctypes.c_float(coef), ctypes.c_float(every),
-                                  dtype_code(qkv.dtype), STREAM)
+                                  int(bool(norm_after)), dtype_code(qkv.dtype), STREAM)
     return q_out
 
 
@@ -1117,6 +1170,48 @@ def qk_rownorm_kv(qkv: torch.Tensor, k_col: int, v_col: int, q_w: torch.Tensor, 
     return q_out
 
 
+def pool_blocks(cache: torch.Tensor, block_table: torch.Tensor, row_seg: torch.Tensor, positions: torch.Tensor,
+                pool_slot_map: torch.Tensor, pool_cache: torch.Tensor, pool: int, page_size: int, G: int, hd: int) -> None:
+    """The means of the blocks of ``pool`` positions that this step's rows complete, from the keys and values in ``cache``
+    (this step's already in it) to the entries ``pool_slot_map`` names (-1: the row completes no block)."""
+    _need(cache, "cache"); _need(pool_cache, "pool_cache", cache.dtype)
+    for t, nm in ((block_table, "block_table"), (row_seg, "row_seg"), (positions, "positions"), (pool_slot_map, "pool_slot_map")):
+        _need(t, nm, torch.int32)
+    n = positions.numel()
+    for c in (cache, pool_cache):
+        if tuple(c.shape[1:]) != (2, G, page_size, hd):
+            raise KernelError(f"pool_blocks: cache layout {tuple(c.shape)}")
+    if row_seg.numel() != n or pool_slot_map.numel() != n or pool < 1:
+        raise KernelError("pool_blocks: shape mismatch")
+    _run("pool_blocks", load_library("qkrope").kp_pool_blocks, _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(row_seg),
+         _ptr(positions), _ptr(pool_slot_map), _ptr(pool_cache), int(pool), page_size, n, G, hd, dtype_code(cache.dtype), STREAM)
+
+
+class Pooled:
+    """What the attention kernels need to read the means of blocks of positions behind a window: the positions a block
+    (``pool``), the layer's cache of the means and the requests' block tables into it."""
+
+    def __init__(self, pool: int, cache: torch.Tensor, block_table: torch.Tensor):
+        self.pool, self.cache, self.block_table = int(pool), cache, block_table
+
+    def check(self, cache: torch.Tensor, window, keep_first, block, what: str) -> None:
+        _need(self.cache, "pooled cache", cache.dtype); _need(self.block_table, "pooled block table", torch.int32)
+        if self.pool < 1 or not window or keep_first or block:
+            raise KernelError(f"{what}: pooled blocks go with a window, and not with kept first keys or blocks of positions")
+        if self.cache.shape[1:] != cache.shape[1:]:
+            raise KernelError(f"{what}: the pooled cache is laid out like the cache")
+
+    def chunks(self, n_chunks: int) -> int:
+        """Chunks of SPLIT_CHUNK entries that a context of ``n_chunks`` chunks of keys can have."""
+        return -(-(n_chunks * SPLIT_CHUNK // self.pool) // SPLIT_CHUNK) or 1
+
+
+def _pool_args(pooled: Optional[Pooled]):
+    if pooled is None:
+        return 0, _ptr(None), _ptr(None), 0
+    return pooled.pool, _ptr(pooled.cache), _ptr(pooled.block_table), pooled.block_table.shape[1]
+
+
 def _check_sink(sink: Optional[torch.Tensor], H: int, keep_first: int, window: Optional[int], block: Optional[int], what: str) -> None:
     if sink is not None:
         _need(sink, "sink", torch.float32)
@@ -1129,10 +1224,13 @@ def _check_sink(sink: Optional[torch.Tensor], H: int, keep_first: int, window: O
 def attention_rows(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, row_seg: torch.Tensor,
                    positions: torch.Tensor, out: torch.Tensor, scale: float, window: Optional[int],
                    page_size: int, H: int, G: int, hd: int, block: Optional[int] = None, keep_first: int = 0,
-                   sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   sink: Optional[torch.Tensor] = None, cap: float = 0.0, out_scale: float = 1.0,
+                   pooled: Optional[Pooled] = None) -> torch.Tensor:
     """``block``: a row reads no key from before the start of its own block of that many positions.
     ``keep_first``: behind its window a row still reads the first that many keys of its sequence.  ``sink``
-    (float32 [H]): ``exp(sink_h)`` joins the softmax's denominator, a key with a score and no value."""
+    (float32 [H]): ``exp(sink_h)`` joins the softmax's denominator, a key with a score and no value.  ``cap`` (0: none)
+    bounds the scores, ``cap tanh(s / cap)``; ``out_scale`` multiplies the output; ``pooled``: behind its window a row also
+    reads the means of the blocks of positions that lie wholly before it."""
     _need(q, "q", contiguous=False); _need(cache, "cache", q.dtype); _need(out, "out", q.dtype, contiguous=False)
     _need(block_table, "block_table", torch.int32); _need(row_seg, "row_seg", torch.int32)
     _need(positions, "positions", torch.int32)
@@ -1140,10 +1238,13 @@ def attention_rows(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tens
     if q.shape[1] != H * hd or out.shape != (n, H * hd) or tuple(cache.shape[1:]) != (2, G, page_size, hd):
         raise KernelError("attention_rows: shape mismatch")
     _check_sink(sink, H, keep_first, window, block, "attention_rows")
+    if pooled is not None:
+        pooled.check(cache, window, keep_first, block, "attention_rows")
     lib = load_library("attention")
-    _run("attention_rows", lib.kp_attention_rows_sink, _ptr(q), _rows_2d(q, "q"), _ptr(cache), _ptr(block_table),
+    _run("attention_rows", lib.kp_attention_rows_pooled, _ptr(q), _rows_2d(q, "q"), _ptr(cache), _ptr(block_table),
          block_table.shape[1], _ptr(row_seg), _ptr(positions), _ptr(out), _rows_2d(out, "out"), ctypes.c_float(scale),
-         int(window or 0), int(block or 0), int(keep_first or 0), _ptr(sink), page_size, n, H, G, hd, dtype_code(q.dtype), STREAM)
+         int(window or 0), int(block or 0), int(keep_first or 0), _ptr(sink), ctypes.c_float(cap), ctypes.c_float(out_scale),
+         *_pool_args(pooled), page_size, n, H, G, hd, dtype_code(q.dtype), STREAM)
     return out
 
 
@@ -1152,10 +1253,13 @@ SPLIT_CHUNK_MMA = 256       # keys a chunk of its tensor-core form: 64, 128 or 2
 SPLIT_MAX_RATIO = 8        # query heads per kv head it takes
 
 
-def attention_split_scratch(n_rows: int, H: int, hd: int, n_chunks: int, keep_first: int = 0) -> int:
+def attention_split_scratch(n_rows: int, H: int, hd: int, n_chunks: int, keep_first: int = 0,
+                            pooled: Optional["Pooled"] = None) -> int:
     """Float elements of scratch that :func:`attention_split` needs (``keep_first``: with slots for the chunks of
-    that many kept first keys)."""
+    that many kept first keys; ``pooled``: for those of the pooled entries)."""
     slots = n_chunks * (SPLIT_CHUNK // min(SPLIT_CHUNK, SPLIT_CHUNK_MMA)) + -(-int(keep_first or 0) // SPLIT_CHUNK)
+    if pooled is not None:
+        slots += pooled.chunks(n_chunks) * (SPLIT_CHUNK // min(SPLIT_CHUNK, SPLIT_CHUNK_MMA))
     return n_rows * H * slots * (hd + 2)
 
 
@@ -1163,7 +1267,8 @@ def attention_split(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Ten
                     positions: torch.Tensor, out: torch.Tensor, scratch: torch.Tensor, n_chunks: int, scale: float,
                     window: Optional[int], page_size: int, H: int, G: int, hd: int,
                     block: Optional[int] = None, exact_weights: bool = False, keep_first: int = 0,
-                    sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sink: Optional[torch.Tensor] = None, cap: float = 0.0, out_scale: float = 1.0,
+                    pooled: Optional[Pooled] = None) -> torch.Tensor:
     """Split-KV attention (chunks of 256 keys, merged in order).  ``n_chunks``
     must cover the largest position of the batch; ``scratch`` is float32.
     ``block``: a row reads no key from before the start of its own block of that many positions.
@@ -1171,7 +1276,8 @@ def attention_split(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Ten
     tensor-core form then multiplies their three bfloat16 parts one after the other) instead of rounded to bfloat16.
     ``keep_first`` / ``sink``: as in :func:`attention_rows`; the sink enters in the merge, once a row; kept first
     keys behind a window are computed by a second small launch where the tensor-core form (which knows nothing of
-    them) computes the window's chunks."""
+    them) computes the window's chunks.  ``cap``, ``out_scale``, ``pooled``: as there too; the pooled entries' chunks are
+    computed by a launch of their own, the output's factor enters in the merge."""
     _need(q, "q", contiguous=False); _need(cache, "cache", q.dtype); _need(out, "out", q.dtype, contiguous=False)
     _need(block_table, "block_table", torch.int32); _need(row_seg, "row_seg", torch.int32)
     _need(positions, "positions", torch.int32); _need(scratch, "scratch", torch.float32)
@@ -1179,33 +1285,45 @@ def attention_split(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Ten
     if q.shape[1] != H * hd or out.shape != (n, H * hd) or tuple(cache.shape[1:]) != (2, G, page_size, hd):
         raise KernelError("attention_split: shape mismatch")
     keep_first = int(keep_first or 0) if window else 0
-    if scratch.numel() < attention_split_scratch(n, H, hd, n_chunks, keep_first):
+    if scratch.numel() < attention_split_scratch(n, H, hd, n_chunks, keep_first, pooled):
         raise KernelError("attention_split: scratch too small")
     _check_sink(sink, H, keep_first, window, block, "attention_split")
+    if pooled is not None:
+        pooled.check(cache, window, keep_first, block, "attention_split")
     lib = load_library("attention_decode")
     if USE_MMA_ATTENTION and q.dtype == torch.bfloat16 and hd in (64, 128) and q.stride(0) % 2 == 0:
         # tensor-core chunk pass over smaller chunks, then the same merge; kept first keys get slots behind the window's
         # chunks (for the chunk pass they are chunks beyond every position: it leaves them alone)
         front0 = n_chunks * (SPLIT_CHUNK // SPLIT_CHUNK_MMA)
-        parts = front0 + -(-keep_first // SPLIT_CHUNK)
+        pool_chunks = pooled.chunks(n_chunks) * (SPLIT_CHUNK // SPLIT_CHUNK_MMA) if pooled is not None else 0
+        parts = front0 + -(-keep_first // SPLIT_CHUNK) + pool_chunks
         if keep_first:
             _run("attention_front_chunks", lib.kp_attention_front_chunks, _ptr(q), _rows_2d(q, "q"), _ptr(cache), _ptr(block_table),
                  block_table.shape[1], _ptr(row_seg), _ptr(positions), _ptr(scratch), parts, front0, ctypes.c_float(scale),
                  int(window), keep_first, page_size, n, H, G, hd, dtype_code(q.dtype), STREAM)
-        _run("attention_split_mma", load_library("attention_mma").kp_attention_split_mma_masked,
+        mma = load_library("attention_mma").kp_attention_split_mma_pooled
+        _run("attention_split_mma", mma,
             _ptr(q), _rows_2d(q, "q"), _ptr(cache), ctypes.c_longlong(cache.shape[0] if USE_TMA_ATTENTION else 0),
             _ptr(block_table), block_table.shape[1], _ptr(row_seg),
-            _ptr(positions), _ptr(scratch), parts, SPLIT_CHUNK_MMA, ctypes.c_float(scale), int(window or 0), int(block or 0),
-            int(bool(exact_weights)), page_size, n, H, G, hd, STREAM)
-        _run("attention_merge", lib.kp_attention_merge_sink, _ptr(positions), _ptr(out), _rows_2d(out, "out"), _ptr(scratch),
-             parts, SPLIT_CHUNK_MMA, int(window or 0), int(block or 0), keep_first, _ptr(sink), front0 if keep_first else -1, n, H, hd,
-             dtype_code(q.dtype), STREAM)
+            _ptr(positions), _ptr(scratch), front0, parts, 0, SPLIT_CHUNK_MMA, ctypes.c_float(scale), int(window or 0), int(block or 0),
+            int(bool(exact_weights)), ctypes.c_float(cap), 0, page_size, n, H, G, hd, STREAM)
+        if pooled is not None:
+            _run("attention_split_pool", mma,
+                _ptr(q), _rows_2d(q, "q"), _ptr(pooled.cache), ctypes.c_longlong(pooled.cache.shape[0] if USE_TMA_ATTENTION else 0),
+                _ptr(pooled.block_table), pooled.block_table.shape[1], _ptr(row_seg),
+                _ptr(positions), _ptr(scratch), pool_chunks, parts, front0, SPLIT_CHUNK_MMA, ctypes.c_float(scale), int(window), 0,
+                int(bool(exact_weights)), ctypes.c_float(cap), pooled.pool, page_size, n, H, G, hd, STREAM)
+        _run("attention_merge", lib.kp_attention_merge_pooled, _ptr(positions), _ptr(out), _rows_2d(out, "out"), _ptr(scratch),
+             parts, SPLIT_CHUNK_MMA, int(window or 0), int(block or 0), keep_first, _ptr(sink),
+             front0 if keep_first or pooled is not None else -1, ctypes.c_float(out_scale), pooled.pool if pooled is not None else 0,
+             n, H, hd, dtype_code(q.dtype), STREAM)
         return out
-    _run("attention_split", lib.kp_attention_split_sink, _ptr(q), _rows_2d(q, "q"), _ptr(cache), _ptr(block_table),
+    _run("attention_split", lib.kp_attention_split_pooled, _ptr(q), _rows_2d(q, "q"), _ptr(cache), _ptr(block_table),
          block_table.shape[1], _ptr(row_seg), _ptr(positions), _ptr(out), _rows_2d(out, "out"), _ptr(scratch),
-         n_chunks, ctypes.c_float(scale), int(window or 0), int(block or 0), keep_first, _ptr(sink), page_size, n, H, G, hd,
+         n_chunks, ctypes.c_float(scale), int(window or 0), int(block or 0), keep_first, _ptr(sink), ctypes.c_float(cap),
+         ctypes.c_float(out_scale), *_pool_args(pooled), pooled.chunks(n_chunks) if pooled is not None else 0, page_size, n, H, G, hd,
          dtype_code(q.dtype), STREAM)
-    LAUNCHES[0] += 1
+    LAUNCHES[0] += 1 if pooled is None else 2
     return out
 
 
@@ -1235,15 +1353,16 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
                       scale: float, window: Optional[int], page_size: int, H: int, G: int, hd: int,
                       big_tile_seg: Optional[torch.Tensor] = None, big_tile_row0: Optional[torch.Tensor] = None,
                       block: Optional[int] = None, exact_weights: bool = False, keep_first: int = 0,
-                      sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      sink: Optional[torch.Tensor] = None, cap: float = 0.0, out_scale: float = 1.0,
+                      pooled: Optional[Pooled] = None) -> torch.Tensor:
     """Tensor-core causal attention for segments of many rows.  ``tile_seg`` / ``tile_row0`` list, for every
     tile of 64 consecutive rows of a segment, its segment and its first row; ``big_tile_seg`` /
     ``big_tile_row0`` the same for tiles of 128 rows, the tile that reads the most keys first (with them the
     tcgen05 kernel runs where it takes the sizes).  ``block``: a row reads no key from before the start of its own
     block of that many positions.  ``exact_weights``: the softmax weights enter the product with V whole, as three
     bfloat16 parts multiplied one after the other (the mma.sync kernel; the tcgen05 kernel, whose weights pass
-    through shared memory as one bfloat16 operand, is then not taken).  ``keep_first`` / ``sink``: as in
-    :func:`attention_rows` (the mma.sync kernel has them, the tcgen05 kernel is then not taken)."""
+    through shared memory as one bfloat16 operand, is then not taken).  ``keep_first`` / ``sink`` / ``cap`` / ``out_scale`` /
+    ``pooled``: as in :func:`attention_rows` (the mma.sync kernel has them, the tcgen05 kernel is then not taken)."""
     _need(q, "q", torch.bfloat16, contiguous=False); _need(cache, "cache", torch.bfloat16)
     _need(out, "out", torch.bfloat16, contiguous=False)
     for t_, nm in ((block_table, "block_table"), (cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (tile_seg, "tile_seg"),
@@ -1255,9 +1374,11 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
     if tile_seg.numel() != tile_row0.numel():
         raise KernelError("attention_prefill: tile lists differ in length")
     _check_sink(sink, H, keep_first, window, block, "attention_prefill")
+    if pooled is not None:
+        pooled.check(cache, window, keep_first, block, "attention_prefill")
     keep_first = int(keep_first or 0) if window else 0
-    if (big_tile_seg is not None and not exact_weights and not keep_first and sink is None
-            and attention_prefill_tc_ok(q, out, cache, page_size, hd)):
+    if (big_tile_seg is not None and not exact_weights and not keep_first and sink is None and not cap and out_scale == 1.0
+            and pooled is None and attention_prefill_tc_ok(q, out, cache, page_size, hd)):
         _need(big_tile_seg, "big_tile_seg", torch.int32); _need(big_tile_row0, "big_tile_row0", torch.int32)
         if big_tile_seg.numel() != big_tile_row0.numel():
             raise KernelError("attention_prefill: tile lists differ in length")
@@ -1268,10 +1389,128 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
             _ptr(out), _rows_2d(out, "out"), ctypes.c_float(scale), int(window or 0), int(block or 0), page_size, H, G, hd,
             STREAM)
         return out
-    _run("attention_prefill_mma", load_library("attention_mma").kp_attention_prefill_mma_sink,
+    _run("attention_prefill_mma", load_library("attention_mma").kp_attention_prefill_mma_pooled,
         _ptr(q), _rows_2d(q, "q"), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(cu_rows), _ptr(seg_pos),
         _ptr(tile_seg), _ptr(tile_row0), tile_seg.numel(), _ptr(out), _rows_2d(out, "out"), ctypes.c_float(scale),
-        int(window or 0), int(block or 0), keep_first, _ptr(sink), int(bool(exact_weights)), page_size, H, G, hd, STREAM)
+        int(window or 0), int(block or 0), keep_first, _ptr(sink), int(bool(exact_weights)), ctypes.c_float(cap),
+        ctypes.c_float(out_scale), *_pool_args(pooled), page_size, H, G, hd, STREAM)
+    return out
+
+
+# ------------------------------------------------------------------ attention over cached latents
+
+LATENT_CHUNK = 256             # keys a chunk of the absorbed pass
+LATENT_PREFILL_MAX = (256, 256)    # key and value columns a head that the expanded pass takes
+USE_MMA_LATENT = True          # the absorbed pass of bfloat16 rows runs on the tensor cores where the sizes allow it
+
+
+def latent_prep(p: torch.Tensor, q_col: int, c_col: int, H: int, dimp: int, rotp: int, rank: int, rankp: int, w: torch.Tensor,
+                eps: float, rotary, positions: torch.Tensor, slot_map: torch.Tensor, cache: Optional[torch.Tensor],
+                page_size: int, qa: Optional[torch.Tensor], n_absorbed: int) -> None:
+    """Rows ``p`` of the input product hold H query heads of (dimp | rotp) at ``q_col`` and the latent (rankp) with the
+    shared key part (rotp) at ``c_col``: norm the latent over its ``rank`` columns (weight ``w`` [rank]), rotate the key part
+    and store both in the row's cache page; rotate the heads' query parts in place, and copy those of the first
+    ``n_absorbed`` rows behind the absorbed queries in ``qa`` [n_absorbed, H, rankp + rotp].  ``rotary``: (cos, sin,
+    dimensions, interleaved) as a position part gives it."""
+    _need(p, "p", contiguous=False); _need(w, "w", torch.float32); _need(positions, "positions", torch.int32)
+    n, W = p.shape[0], rankp + rotp
+    if p.stride(1) != 1 or q_col + H * (dimp + rotp) > p.shape[1] or c_col + W > p.shape[1] or w.numel() != rank:
+        raise KernelError("latent_prep: shape mismatch")
+    if cache is not None:
+        _need(cache, "cache", p.dtype); _need(slot_map, "slot_map", torch.int32)
+        if tuple(cache.shape[1:]) != (1, 1, page_size, W):
+            raise KernelError(f"latent_prep: cache layout {tuple(cache.shape)}")
+    if n_absorbed:
+        _need(qa, "qa", p.dtype)
+        if tuple(qa.shape) != (n_absorbed, H, W):
+            raise KernelError("latent_prep: qa shape")
+    cos, sin, rot, inter = rotary
+    if cos is not None:
+        _need(cos, "cos", torch.float32); _need(sin, "sin", torch.float32)
+        if cos.shape[1] != rot // 2 or rot > rotp:
+            raise KernelError("latent_prep: table width")
+    _run("latent_prep", load_library("latent").kp_latent_prep, _ptr(p), p.stride(0), int(q_col), int(c_col), H, dimp, rotp, rank, rankp,
+         _ptr(w), ctypes.c_float(eps), _ptr(cos), _ptr(sin), int(rot), int(bool(inter)), _ptr(positions), _ptr(slot_map), _ptr(cache),
+         page_size, _ptr(qa), int(n_absorbed), n, dtype_code(p.dtype), STREAM)
+
+
+def head_gemm(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[m, h, :] = a[m, h, :] @ b[h].T, times ``sigmoid(gate[m, h, :])`` if given.  ``a`` [M, H, K], ``out`` and ``gate``
+    [M, H, N] may be strided views (last dimension dense); ``b`` [H, N, K]."""
+    M, H, K = a.shape
+    N = b.shape[1]
+    _need(a, "a", contiguous=False); _need(b, "b", a.dtype); _need(out, "out", a.dtype, contiguous=False)
+    if tuple(b.shape) != (H, N, K) or tuple(out.shape) != (M, H, N) or a.stride(2) != 1 or out.stride(2) != 1:
+        raise KernelError(f"head_gemm: shapes a{tuple(a.shape)} b{tuple(b.shape)} out{tuple(out.shape)}")
+    if gate is not None:
+        _need(gate, "gate", a.dtype, contiguous=False)
+        if tuple(gate.shape) != (M, H, N) or gate.stride(2) != 1:
+            raise KernelError("head_gemm: gate shape")
+    ll = ctypes.c_longlong
+    _run("head_gemm", load_library("latent").kp_head_gemm, _ptr(a), ll(a.stride(0)), a.stride(1), _ptr(b), _ptr(out), ll(out.stride(0)),
+         out.stride(1), _ptr(gate), ll(gate.stride(0) if gate is not None else 0), gate.stride(1) if gate is not None else 0, M, N, K, H,
+         dtype_code(a.dtype), STREAM, tag=f" {H}x{N}x{K}", work=(2 * M * H * N * K, (H * N * K + M * H * (N + K)) * a.element_size()))
+    return out
+
+
+def latent_split_scratch(n: int, H: int, rankp: int, n_chunks: int) -> int:
+    return n * H * n_chunks * (rankp + 2)
+
+
+def latent_split(qa: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, row_seg: torch.Tensor, positions: torch.Tensor,
+                 scratch: torch.Tensor, n_chunks: int, u: torch.Tensor, scale: float, page_size: int) -> torch.Tensor:
+    """Causal softmax attention of absorbed queries ``qa`` [n, H, W] over the cached rows (the latents are the values too):
+    ``u`` [n, H, rankp].  ``n_chunks`` chunks of 256 keys must cover the largest position; ``scratch`` is float32."""
+    n, H, W = qa.shape
+    rankp = u.shape[2]
+    _need(qa, "qa"); _need(cache, "cache", qa.dtype); _need(u, "u", qa.dtype); _need(scratch, "scratch", torch.float32)
+    for t, nm in ((block_table, "block_table"), (row_seg, "row_seg"), (positions, "positions")):
+        _need(t, nm, torch.int32)
+    if tuple(cache.shape[1:]) != (1, 1, page_size, W) or tuple(u.shape) != (n, H, rankp) or row_seg.numel() != n or positions.numel() != n:
+        raise KernelError("latent_split: shape mismatch")
+    if scratch.numel() < latent_split_scratch(n, H, rankp, n_chunks):
+        raise KernelError("latent_split: scratch too small")
+    _run("latent_split", load_library("latent").kp_latent_split, _ptr(qa), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(row_seg),
+         _ptr(positions), _ptr(scratch), n_chunks, _ptr(u), ctypes.c_float(scale), page_size, n, H, rankp, W - rankp, dtype_code(qa.dtype),
+         int(USE_MMA_LATENT), STREAM)
+    LAUNCHES[0] += 1
+    return u
+
+
+def latent_prefill_ok(q: torch.Tensor, key_cols: int, value_cols: int) -> bool:
+    return q.dtype == torch.bfloat16 and key_cols <= LATENT_PREFILL_MAX[0] and value_cols <= LATENT_PREFILL_MAX[1]
+
+
+def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, ctx_base: torch.Tensor, n_rows: int, page_size: int) -> torch.Tensor:
+    """The cache rows of whole contexts side by side: row ``ctx_base[i] + t`` is key t of segment i."""
+    _need(cache, "cache", torch.bfloat16); _need(block_table, "block_table", torch.int32); _need(ctx_base, "ctx_base", torch.int32)
+    W = cache.shape[-1]
+    n_seg = block_table.shape[0]
+    if tuple(cache.shape[1:]) != (1, 1, page_size, W) or ctx_base.numel() != n_seg + 1:
+        raise KernelError("latent_gather: shape mismatch")
+    out = torch.empty((n_rows, W), dtype=cache.dtype, device=cache.device)
+    _run("latent_gather", load_library("latent").kp_latent_gather, _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(ctx_base), n_seg,
+         _ptr(out), n_rows, page_size, W, STREAM)
+    return out
+
+
+def latent_prefill(q: torch.Tensor, ex: torch.Tensor, rows: torch.Tensor, rankp: int, dimp: int, rotp: int, vdimp: int,
+                   cu_rows: torch.Tensor, seg_pos: torch.Tensor, tile_seg: torch.Tensor, tile_row0: torch.Tensor, ctx_base: torch.Tensor,
+                   out: torch.Tensor, scale: float, H: int) -> torch.Tensor:
+    """Causal attention of prompt portions over expanded latents: ``q`` [n, H (dimp + rotp)] (rows may be strided), ``ex`` [T, H
+    dimp + H vdimp] the expanded keys and values and ``rows`` [T, rankp + rotp] the gathered cache rows (their last rotp
+    columns are the shared key part), T the contexts of ``ctx_base``; tiles of 64 rows as attention_prefill takes them."""
+    _need(q, "q", torch.bfloat16, contiguous=False); _need(ex, "ex", torch.bfloat16); _need(rows, "rows", torch.bfloat16)
+    _need(out, "out", torch.bfloat16, contiguous=False)
+    for t, nm in ((cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (tile_seg, "tile_seg"), (tile_row0, "tile_row0"), (ctx_base, "ctx_base")):
+        _need(t, nm, torch.int32)
+    n = q.shape[0]
+    if (q.shape[1] != H * (dimp + rotp) or tuple(out.shape) != (n, H * vdimp) or ex.shape[1] != H * (dimp + vdimp)
+            or rows.shape != (ex.shape[0], rankp + rotp) or tile_seg.numel() != tile_row0.numel()):
+        raise KernelError("latent_prefill: shape mismatch")
+    _run("latent_prefill", load_library("latent").kp_latent_prefill, _ptr(q), _rows_2d(q, "q"), _ptr(ex), ex.shape[1], H * dimp, _ptr(rows), rankp,
+         dimp, rotp, vdimp, _ptr(cu_rows), _ptr(seg_pos), _ptr(tile_seg), _ptr(tile_row0), _ptr(ctx_base), tile_seg.numel(), _ptr(out),
+         _rows_2d(out, "out"), ctypes.c_float(scale), H, STREAM)
     return out
 
 
@@ -1279,6 +1518,7 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
 
 SKINNY_MAX_M = 64
 EPI_SWIGLU = 3
+EPI_ACT = 6
 
 
 def skinny_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
@@ -1317,7 +1557,7 @@ def tc_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
             accumulate: bool = False, swiglu: bool = False, split: bool = True, activation: str = "silu",
-            glu: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
+            glu: Optional[Tuple[float, float, float]] = None, plain_activation: Optional[str] = None) -> torch.Tensor:
     """out = a @ w.T (+ bias) on the tcgen05 tensor cores (TMA-fed, accumulator in tensor memory); with
     ``swiglu`` ``w`` holds gate rows then up rows and out = silu(gate) * up (or ``activation``; with ``glu`` =
     (limit, alpha, shift) the gated unit with limits of :func:`glu_clamped`).  With ``split`` a product of 17 to
@@ -1342,6 +1582,8 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[
              work=_gemm_work(M, N, K, a, w, out))
         return out
     epi = _skinny_epilogue(out, accumulate, swiglu) | (_fused_activation(activation) << 8 if swiglu else 0)
+    if plain_activation is not None:
+        epi = _plain_epilogue(epi, plain_activation)
     _run("gemm_tc", lib.kp_gemm_tc_split, _ptr(a), _rows_2d(a, "a"), _ptr(w), _rows_2d(w, "w"), _ptr(bias), _ptr(out),
          _rows_2d(out, "out"), M, N, K, epi, 1 if split else 0, STREAM, tag=f" {N}x{K}",
          work=_gemm_work(M, N, K, a, w, out))
@@ -1421,6 +1663,12 @@ def _fused_activation(name: str) -> int:
     return activation_code(name)
 
 
+def _plain_epilogue(epi: int, activation: str) -> int:
+    if epi != EPI_STORE:
+        raise KernelError("an ungated activation goes with a product stored in bfloat16")
+    return EPI_ACT | (plain_activation_code(activation) << 8)
+
+
 def _skinny_epilogue(out: torch.Tensor, accumulate: bool, swiglu: bool) -> int:
     if swiglu:
         if out.dtype != torch.bfloat16:
@@ -1439,7 +1687,7 @@ def _skinny_epilogue(out: torch.Tensor, accumulate: bool, swiglu: bool) -> int:
 
 def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
                 accumulate: bool = False, swiglu: bool = False, activation: str = "silu",
-                glu: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
+                glu: Optional[Tuple[float, float, float]] = None, plain_activation: Optional[str] = None) -> torch.Tensor:
     """out = a @ w.T (+ bias) for up to 64 rows of bfloat16 ``a``.  With
     ``swiglu`` ``w`` holds gate rows then up rows and out = silu(gate) * up (or ``activation``; with ``glu`` =
     (limit, alpha, shift) the gated unit with limits of :func:`glu_clamped`)."""
@@ -1468,6 +1716,8 @@ def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optio
         epi = EPI_STORE_F32
     else:
         raise KernelError("gemm_skinny: output dtype")
+    if plain_activation is not None:
+        epi = _plain_epilogue(epi, plain_activation)
     consts = _glu_floats(glu) if swiglu and glu is not None else ()
     if USE_STREAM and stream_fits(K, swiglu) and stream_pays(N, K) and M <= STREAM_MAX_M:
         lib = load_library("gemm_stream")
@@ -1485,6 +1735,7 @@ def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optio
 # ------------------------------------------------------------------ mixture of experts
 
 MOE_MAX_TOP = 32           # experts a row can use
+MOE_MAX_GROUPS = 64        # groups of experts a choice can be made from
 MOE_MAX_EXPERTS = 1536     # experts the routing kernels hold in shared memory
 
 
@@ -1503,9 +1754,13 @@ def _moe_routing(routing: str) -> int:
         raise KernelError(f"moe: routing '{routing}' (expected one of {', '.join(MOE_ROUTINGS)})") from None
 
 
+def _moe_groups(groups):
+    return (0, 0) if groups is None else (int(groups[0]), int(groups[1]))
+
+
 def moe_route(logits: torch.Tensor, top: int, idx: torch.Tensor, weights: torch.Tensor, layout: torch.Tensor,
               bias: Optional[torch.Tensor] = None, routing: str = "top_logits", scale: float = 1.0,
-              n_identity: int = 0) -> None:
+              n_identity: int = 0, groups: Optional[Tuple[int, int]] = None, renormalise: bool = False) -> None:
     """Router logits [n, E] (float32) -> the ``top`` experts of every row (``idx`` int32 [n, top], largest
     first, the lower index on ties), their weights (float32 [n, top]) and the
     layout of the (row, choice) pairs by expert (``layout``, int32, :func:`moe_layout_ints` words), which the
@@ -1513,7 +1768,9 @@ def moe_route(logits: torch.Tensor, top: int, idx: torch.Tensor, weights: torch.
     weighted by the softmax over the chosen logits alone; ``softmax_all``: scores = softmax over all E outputs, the
     largest score + ``bias`` are chosen and weighted by their score times ``scale``; ``sigmoid``: the largest logits
     are chosen and each weighted by its own ``sigmoid(logit)`` times ``scale``.  The last ``n_identity``
-    outputs stand for experts without weights (places in the layout, no tiles)."""
+    outputs stand for experts without weights (places in the layout, no tiles).  With ``softmax_all``: ``groups`` =
+    (count, keep) lets only experts of the ``keep`` best of ``count`` equal groups of neighbours be chosen (a group is as
+    good as its best expert), ``renormalise`` divides the chosen scores by their sum before ``scale``."""
     _need(logits, "logits", torch.float32); _need(idx, "idx", torch.int32); _need(weights, "weights", torch.float32)
     _need(layout, "layout", torch.int32)
     n, E = logits.shape
@@ -1526,7 +1783,8 @@ def moe_route(logits: torch.Tensor, top: int, idx: torch.Tensor, weights: torch.
     if idx.numel() != n * top or weights.numel() != n * top or layout.numel() < moe_layout_ints(n, E, top):
         raise KernelError("moe_route: output sizes")
     _run("moe_route", load_library("moe").kp_moe_route, _ptr(logits), _ptr(bias), n, E, top, _moe_routing(routing),
-         ctypes.c_float(scale), int(n_identity), _ptr(idx), _ptr(weights), _ptr(layout), STREAM)
+         ctypes.c_float(scale), int(n_identity), *_moe_groups(groups), int(bool(renormalise)), _ptr(idx), _ptr(weights), _ptr(layout),
+         STREAM)
     LAUNCHES[0] += 1
 
 
@@ -1550,7 +1808,7 @@ def moe_router_ok(d: int, E: int) -> bool:
 
 def moe_router(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx: torch.Tensor,
                weights: torch.Tensor, layout: torch.Tensor, routing: str = "top_logits", scale: float = 1.0,
-               n_identity: int = 0) -> None:
+               n_identity: int = 0, groups: Optional[Tuple[int, int]] = None, renormalise: bool = False) -> None:
     """The router in one go: logits ``h w_router^T`` in float32 (``w_router`` [E, d] and ``bias`` are float32;
     ``h`` is widened from its storage type), the choice and the layout as :func:`moe_route` leaves them."""
     _need(h, "h", contiguous=False); _need(w_router, "w_router", torch.float32)
@@ -1566,7 +1824,8 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Ten
     if idx.numel() != n * top or weights.numel() != n * top or layout.numel() < moe_layout_ints(n, E, top):
         raise KernelError("moe_router: output sizes")
     _run("moe_router", load_library("moe").kp_moe_router, _ptr(h), _rows_2d(h, "h"), _ptr(w_router), _ptr(bias), n, E, d, top,
-         _moe_routing(routing), ctypes.c_float(scale), int(n_identity), _ptr(idx), _ptr(weights), _ptr(layout), dtype_code(h.dtype), STREAM,
+         _moe_routing(routing), ctypes.c_float(scale), int(n_identity), *_moe_groups(groups), int(bool(renormalise)), _ptr(idx), _ptr(weights), _ptr(layout),
+         dtype_code(h.dtype), STREAM,
          work=(2 * n * E * d, n * d * h.element_size() + E * d * 4))
     LAUNCHES[0] += 1
 

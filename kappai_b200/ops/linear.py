@@ -46,6 +46,20 @@ def linear(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     return K.gemm_nt_simt(a, w, out, bias, accumulate)
 
 
+def linear_act(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], activation: str) -> torch.Tensor:
+    """``act(a @ w.T + bias)``, ungated, the activation taken of the float32 sums: in the product's epilogue where a kernel
+    fits the shape, else by a row-wise kernel behind a float32 product."""
+    M, N = a.shape[0], w.shape[0]
+    out = torch.empty((M, N), dtype=a.dtype, device=a.device)
+    if a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
+        tc = K.tc_ok(a, w)
+        if K.skinny_ok(a, w) and not (tc and K.tc_pays_for_few_rows(M, N, False)):
+            return K.gemm_skinny(a, w, out, bias, plain_activation=activation)
+        if tc:
+            return K.gemm_tc(a, w, out, bias, plain_activation=activation)
+    return K.activate(linear(a, w, bias, out_dtype=torch.float32), out, activation)
+
+
 def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, bias: Optional[torch.Tensor] = None,
                   activation: str = "silu", glu: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
     """``act(a @ Wg.T) * (a @ Wu.T)`` with ``w_gate_up = [Wg; Wu]`` and act = silu (or ``activation``); with

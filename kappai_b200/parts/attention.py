@@ -46,15 +46,24 @@ sequence stay visible to every later row, at their true places, and their pages 
 ``conv_kernel`` (taps; default 0, none): q, k and v each pass a causal convolution a channel over time, right behind the
 projection and its bias and before the norm and the rotation (tensors ``q_conv.weight`` and so on, [channels, taps], the
 last tap on the current token, no bias); their last ``conv_kernel - 1`` projected values are state in the request's slot
-beside the paged keys and values.  ``out_scale`` (default 1) multiplies the mixer's output; the values' taps and the
-output bias carry it, so it goes with ``conv_kernel``.
+beside the paged keys and values.  ``out_scale`` (default 1) multiplies the mixer's output; the output bias and, with
+``conv_kernel``, the values' taps carry it, else the attention kernels' last step.
+
+``qk_norm`` = ``"after_rotation"``: q and k are divided by their root mean square a head behind the rotation (no weight;
+``qk_norm_eps`` in the root).  ``softcap`` (a bound c): scores become ``c tanh(s / c)``.  ``pool`` (a number of positions,
+with a ``window``): beside its window a row reads one key and one value for each block of ``pool`` positions (counted from
+position 0) that lies wholly before it: the means of the block's keys and values as the cache holds them, in the same
+softmax.  The means are kept in a page group of their own, an entry a block, made when the block's last position
+is written; the keys themselves are given back when both the window and their own block have passed them.  ``bias`` =
+``"qkv"``: biases on q, k and v, none on the output.
 
 Sizes and constants (params): hidden_size, num_heads, num_kv_heads, head_dim,
 value_dim, scale, qk_norm_eps (None: no q/k norm), qk_norm ("per_head" |
-"projection"), window (None: all keys), cache_window, block (None), values
+"projection" | "after_rotation"), window (None: all keys), cache_window, block (None), values
 ("projection" | "keys"), kv ("own" | "borrowed"), gate (None | "sigmoid" |
 "head_sigmoid"), softmax_weights ("operand" | "float32"), position (a
-``position`` PartSpec), bias, keep_first, sink (None | "zero" | "learned"), q_temp, conv_kernel, out_scale.
+``position`` PartSpec), bias (False | True | "qkv"), keep_first, sink (None | "zero" | "learned"), q_temp, conv_kernel, out_scale,
+softcap, pool.
 """
 from __future__ import annotations
 
@@ -119,10 +128,13 @@ def attention_tiles(segs, split_ok: bool = True):
 class PagedAttentionKernels:
     """The choice among the attention kernels over the paged cache, shared by the mixers that keep keys and values
     there.  The mixer has ``H``, ``G``, ``hd``, ``scale``, ``window``, ``block``, ``exact_weights``, ``split_ok``
-    and ``step_tables_key``; ``keep_first`` and ``sink_w`` (float32 [H] or None) if it has kept first keys or a sink."""
+    and ``step_tables_key``; ``keep_first`` and ``sink_w`` (float32 [H] or None) if it has kept first keys or a sink, ``cap``
+    and ``kernel_scale`` if its scores are bounded or its output is weighed."""
 
     keep_first = 0
     sink_w = None
+    cap = 0.0
+    kernel_scale = 1.0
 
     def _read_sink(self, what: str):
         """The parameters ``sink`` and ``keep_first`` (shared by the mixers over the paged cache)."""
@@ -155,24 +167,24 @@ class PagedAttentionKernels:
     def step_tables(self, segs):
         return attention_tiles(segs, self.split_ok)
 
-    def _attend(self, q, ctx, view, cache):
+    def _attend(self, q, ctx, view, cache, pooled=None):
         """Causal attention of the rows ``q`` [n, H hd] over the cache (this step's keys and values already in
-        it); returns the heads side by side."""
+        it; ``pooled``: the means of blocks behind the window); returns the heads side by side."""
         H, G, hd = self.H, self.G, self.hd
         o = torch.empty_like(q)
-        extra = dict(keep_first=self.keep_first, sink=self.sink_w)
+        extra = dict(keep_first=self.keep_first, sink=self.sink_w, cap=self.cap, out_scale=self.kernel_scale, pooled=pooled)
         tiles = ctx.tables.get(self.step_tables_key)
         if self.split_ok and (tiles is None or q.dtype == torch.float32):
             # rows that each read a long cache (decode): split the keys over many CTAs.  The 32-bit path
             # takes this kernel for every row, whatever the length of its segment: its chunks lie at absolute
             # multiples of 256 keys and are summed in order, so a row's bits do not depend on how the step was cut.
-            self._split(q, o, ctx, view, cache, ctx.n_rows)
+            self._split(q, o, ctx, view, cache, ctx.n_rows, extra)
         elif tiles is not None and K.attention_prefill_ok(q, hd):
             lead = tiles.n_short_rows
             if lead and self.split_ok:
                 # decoded tokens beside prompt portions: the decoded rows lead the batch and go to the split
                 # kernel (in a row tile each would walk its whole cache alone), the portions to the tiled one
-                self._split(q, o, ctx, view, cache, lead)
+                self._split(q, o, ctx, view, cache, lead, extra)
                 t0 = tiles.n_short_tiles
                 K.attention_prefill(q, cache.tensor, view.block_table, ctx.cu_rows, ctx.seg_pos, tiles.tile_seg[t0:],
                                     tiles.tile_row0[t0:], o, self.scale, self.window, view.page_size, H, G, hd,
@@ -187,18 +199,24 @@ class PagedAttentionKernels:
         else:
             lead = tiles.n_short_rows if tiles is not None else 0
             if lead and self.split_ok:
-                self._split(q, o, ctx, view, cache, lead)
+                self._split(q, o, ctx, view, cache, lead, extra)
             else:
                 lead = 0
             K.attention_rows(q[lead:], cache.tensor, view.block_table, ctx.row_seg[lead:], ctx.positions[lead:], o[lead:],
                              self.scale, self.window, view.page_size, H, G, hd, self.block, **extra)
         return o
 
-    def _split(self, q, o, ctx, view, cache, n_rows):
+    def _split(self, q, o, ctx, view, cache, n_rows, extra):
         """Split-key attention for the first ``n_rows`` rows of the step."""
         H, G, hd = self.H, self.G, self.hd
         n_chunks = -(-ctx.max_context // K.SPLIT_CHUNK)
-        need = K.attention_split_scratch(n_rows, H, hd, n_chunks, self.keep_first)
+        ws = self._scratch(K.attention_split_scratch(n_rows, H, hd, n_chunks, self.keep_first, extra["pooled"]), q.device)
+        K.attention_split(q[:n_rows], cache.tensor, view.block_table, ctx.row_seg[:n_rows], ctx.positions[:n_rows],
+                          o[:n_rows], ws, n_chunks, self.scale, self.window, view.page_size, H, G, hd, self.block,
+                          self.exact_weights, **extra)
+
+    def _scratch(self, need, device):
+        """At least ``need`` floats that the attention mixers of a model share."""
         ws = self.env.shared.get("attn_scratch")
         if ws is None or ws.numel() < need:
             # A captured decode step keeps the address of the scratch it was captured with, so a buffer that
@@ -207,11 +225,9 @@ class PagedAttentionKernels:
             if ws is not None:
                 self.env.shared.setdefault("attn_scratch_retired", []).append(ws)
             ws = torch.zeros(max(need, 2 * (ws.numel() if ws is not None else 0), 1 << 16), dtype=torch.float32,
-                             device=q.device)
+                             device=device)
             self.env.shared["attn_scratch"] = ws
-        K.attention_split(q[:n_rows], cache.tensor, view.block_table, ctx.row_seg[:n_rows], ctx.positions[:n_rows],
-                          o[:n_rows], ws, n_chunks, self.scale, self.window, view.page_size, H, G, hd, self.block,
-                          self.exact_weights, keep_first=self.keep_first, sink=self.sink_w)
+        return ws
 
 
 class Attention(PagedAttentionKernels, Part):
@@ -228,7 +244,8 @@ class Attention(PagedAttentionKernels, Part):
         eps = self._p("qk_norm_eps", None)
         self.qk_norm_eps: Optional[float] = None if eps is None else float(eps)
         self.window: Optional[int] = self._p("window", None)
-        self.bias = bool(self._p("bias", False))
+        bias = self._p("bias", False)
+        self.bias, self.out_bias = bool(bias), bool(bias) and bias != "qkv"
         self.block: Optional[int] = self._p("block", None)
         if self.block is not None and int(self.block) < 1:
             raise ConfigError(f"attention: block={self.block} must be a positive number of positions")
@@ -246,8 +263,9 @@ class Attention(PagedAttentionKernels, Part):
             raise ConfigError(f"attention: softmax_weights='{sw}' (expected 'operand' or 'float32')")
         self.exact_weights = sw == "float32"
         self.qk_norm = self._p("qk_norm", "per_head")
-        if self.qk_norm not in ("per_head", "projection"):
-            raise ConfigError(f"attention: qk_norm='{self.qk_norm}' (expected 'per_head' or 'projection')")
+        if self.qk_norm not in ("per_head", "projection", "after_rotation"):
+            raise ConfigError(f"attention: qk_norm='{self.qk_norm}' (expected 'per_head', 'projection' or 'after_rotation')")
+        self.norm_after = self.qk_norm == "after_rotation"
         kv = self._p("kv", "own")
         if kv not in ("own", "borrowed"):
             raise ConfigError(f"attention: kv='{kv}' (expected 'own' or 'borrowed')")
@@ -265,7 +283,7 @@ class Attention(PagedAttentionKernels, Part):
         self.vdim = int(self._p("value_dim", self.dim))
         pos = self._p("position", None)
         kind = None if pos is None else (pos["kind"] if isinstance(pos, dict) else pos.kind)
-        odd_ok = kind in (None, "none") or (kind == "rope" and self.qk_norm_eps is None)
+        odd_ok = kind in (None, "none") or (kind == "rope" and (self.qk_norm_eps is None or self.norm_after))
         if self.qk_norm == "projection" or self.vdim != self.dim or (self.dim % 2 and odd_ok):
             # (an odd head size is stored wider too: the kernels take even sizes, and rotate a head's first dimensions only)
             if self.values_are_keys or (self.bias and self.qk_norm == "projection"):
@@ -277,6 +295,8 @@ class Attention(PagedAttentionKernels, Part):
             raise ConfigError("attention: kv='borrowed' goes with qk_norm='projection', a value matrix elsewhere and no biases")
         if self.qk_norm == "projection" and self.qk_norm_eps is None:
             raise ConfigError("attention: qk_norm='projection' needs qk_norm_eps")
+        if self.norm_after and (self.qk_norm_eps is None or self.values_are_keys):
+            raise ConfigError("attention: qk_norm='after_rotation' needs qk_norm_eps and a value matrix")
         if self.hd % 2 or not (2 <= self.hd <= 256):
             raise ConfigError(f"attention: head_dim={self.dim} is not supported by the kernels "
                               "(an even number from 2 to 256)")
@@ -296,7 +316,9 @@ class Attention(PagedAttentionKernels, Part):
                 raise ConfigError(f"attention: q_temp.every={every} must be positive")
             if not hasattr(self.position, "fused_rotary") or self.qk_norm == "projection":
                 raise ConfigError("attention: q_temp runs in the fused q/k kernel (no position part of its own, per-head norm or none)")
-        if self.vdim != self.dim and self.qk_norm != "projection" and self.qk_norm_eps is not None:
+        if self.norm_after and not hasattr(self.position, "fused_rotary"):
+            raise ConfigError("attention: qk_norm='after_rotation' runs in the fused q/k kernel (no position part of its own)")
+        if self.vdim != self.dim and self.qk_norm == "per_head" and self.qk_norm_eps is not None:
             if not hasattr(self.position, "fused_rotary") or self.position.fused_rotary()[2]:
                 raise ConfigError("attention: a per-head q/k norm with value_dim != head_dim runs without a rotation")
         if self.values_are_keys and not hasattr(self.position, "fused_rotary"):
@@ -309,8 +331,15 @@ class Attention(PagedAttentionKernels, Part):
             raise ConfigError(f"attention: conv_kernel={self.taps} outside 0..{K.SSM_MAX_TAPS}")
         if self.taps and (self.values_are_keys or self.borrows):
             raise ConfigError("attention: conv_kernel wants key and value matrices of the mixer's own")
-        if self.out_scale != 1.0 and not self.taps:
-            raise ConfigError("attention: out_scale is carried by the values' convolution (conv_kernel)")
+        self.kernel_scale = 1.0 if self.taps else self.out_scale     # (a convolution's taps carry the factor)
+        self.cap = float(self._p("softcap", None) or 0.0)
+        if self.cap < 0:
+            raise ConfigError(f"attention: softcap={self.cap} must be positive")
+        pool = self._p("pool", None)
+        self.pool: Optional[int] = None if pool is None else int(pool)
+        if self.pool is not None and (self.pool < 1 or self.window is None or self.keep_first or self.block is not None or self.borrows):
+            raise ConfigError("attention: pool (a positive number of positions) goes with a window and keys of the mixer's own, "
+                              "and not with keep_first or blocks of positions")
         self._tile_setup()
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -326,14 +355,15 @@ class Attention(PagedAttentionKernels, Part):
             s["q_norm.weight"] = WeightSpec((H * self.dim,), "norm")
             if not self.borrows:
                 s["k_norm.weight"] = WeightSpec((G * self.dim,), "norm")
-        elif self.qk_norm_eps is not None:
+        elif self.qk_norm_eps is not None and not self.norm_after:
             s["q_norm.weight"] = WeightSpec((self.dim,), "norm")
             s["k_norm.weight"] = WeightSpec((self.dim,), "norm")
         if self.sink == "learned":
             s["sink"] = WeightSpec((H,), "bias")
         if self.bias:
             for n, sz in (("q_proj", H * self.dim), ("k_proj", G * self.dim), ("v_proj", G * self.vdim), ("out_proj", d)):
-                s[n + ".bias"] = WeightSpec((sz,), "bias")
+                if n != "out_proj" or self.out_bias:
+                    s[n + ".bias"] = WeightSpec((sz,), "bias")
         if self.taps:
             for n, sz in (("q", H * self.dim), ("k", G * self.dim), ("v", G * self.vdim)):
                 s[n + "_conv.weight"] = WeightSpec((sz, self.taps), "conv")
@@ -372,7 +402,8 @@ class Attention(PagedAttentionKernels, Part):
                  for n, heads, width in (("q_proj", H, self.dim), ("k_proj", G, self.dim), ("v_proj", G, self.vdim))]
             b.append(torch.zeros(self.w_qkv.shape[0] - sum(x.shape[0] for x in b), dtype=torch.float32, device=self.w_qkv.device))
             self.b_qkv = torch.cat(b).contiguous()
-            self.b_o = (w["out_proj.bias"].float() * self.out_scale).contiguous()
+            if self.out_bias:
+                self.b_o = (w["out_proj.bias"].float() * self.out_scale).contiguous()
         self.conv_w = None
         if self.taps:
             self.conv_w = torch.cat([self._pad_heads(w["q_conv.weight"].float(), H, self.dim),
@@ -383,7 +414,7 @@ class Attention(PagedAttentionKernels, Part):
             self.q_w = self._pad_heads(w["q_norm.weight"].float(), H, self.dim)
             if not self.borrows:
                 self.k_w = self._pad_heads(w["k_norm.weight"].float(), G, self.dim)
-        elif self.qk_norm_eps is not None:
+        elif self.qk_norm_eps is not None and not self.norm_after:
             # (a head stored wider than it is: zeros behind the weight's own columns, as behind the head's)
             self.q_w = self._pad_heads(w["q_norm.weight"].float(), 1, self.dim)
             self.k_w = self._pad_heads(w["k_norm.weight"].float(), 1, self.dim)
@@ -391,11 +422,15 @@ class Attention(PagedAttentionKernels, Part):
 
     def cache_spec(self):
         # (a borrower names what it reads, so that the engine can see that lender and borrower agree)
-        kv = PagedKVSpec(self.G, self.hd, self.cache_window, None if self.block is None else int(self.block),
-                         self.keep_first if self.cache_window is not None else 0)
-        if self.taps < 2:
-            return kv
-        return CompositeSpec((kv, StateSpec(((self.taps - 1) * (self.H + 2 * self.G) * self.hd,), "float32")))
+        # (a block's keys stay until its mean is made, also where the window is shorter than a block)
+        window = self.cache_window if self.pool is None or self.cache_window is None else max(self.cache_window, self.pool)
+        parts = [PagedKVSpec(self.G, self.hd, window, None if self.block is None else int(self.block),
+                             self.keep_first if self.cache_window is not None else 0)]
+        if self.pool is not None:
+            parts.append(PagedKVSpec(self.G, self.hd, every=self.pool))
+        if self.taps > 1:
+            parts.append(StateSpec(((self.taps - 1) * (self.H + 2 * self.G) * self.hd,), "float32"))
+        return parts[0] if len(parts) == 1 else CompositeSpec(tuple(parts))
 
     def input_product(self):
         return self.w_qkv, self.b_qkv
@@ -404,8 +439,8 @@ class Attention(PagedAttentionKernels, Part):
         self.w_qkv = self.b_qkv = None
 
     def forward(self, h, residual, ctx, cache):
-        """``cache``: a :class:`~kappai_b200.cache.storage.KVLayerView` (with a convolution of two taps or more, that and the
-        :class:`~kappai_b200.cache.storage.StateView` of its kept inputs)."""
+        """``cache``: a :class:`~kappai_b200.cache.storage.KVLayerView` (with pooled blocks, that and the one of their means; with
+        a convolution of two taps or more, also the :class:`~kappai_b200.cache.storage.StateView` of its kept inputs)."""
         self.forward_projected(linear(h, self.w_qkv, self.b_qkv), residual, ctx, cache)
 
     def _convolve(self, qkv, ctx, kept, keep):
@@ -418,8 +453,11 @@ class Attention(PagedAttentionKernels, Part):
         """``qkv``: the rows of the input product (``input_product``), possibly columns of a wider one."""
         H, G, hd = self.H, self.G, self.hd
         proj = qkv
+        parts = list(getattr(cache, "parts", (cache,)))
+        cache = parts.pop(0)
+        means = parts.pop(0) if self.pool is not None else None
         if self.taps > 1:
-            cache, conv = cache.parts
+            conv = parts.pop(0)
             qkv = self._convolve(qkv, ctx, conv.tensor, conv.writes)
         elif self.taps == 1:
             qkv = self._convolve(qkv, ctx, torch.empty((1, 1), dtype=torch.float32, device=qkv.device), False)
@@ -435,7 +473,7 @@ class Attention(PagedAttentionKernels, Part):
             cos, sin, rot, inter = self.position.fused_rotary()
             K.qk_norm_rope_kv(qkv, self.q_w, self.k_w, self.qk_norm_eps or 0.0, cos, sin, rot, inter,
                               ctx.positions, view.slot_map, q, kv_out, view.page_size, H, G, hd, self.v_col,
-                              norm_dim=self.dim, q_temp=self.q_temp)
+                              norm_dim=self.dim, q_temp=self.q_temp, norm_after=self.norm_after)
         else:
             # a position encoding of its own: norm in place, let it change q and k, then scatter
             if self.q_w is not None:
@@ -444,7 +482,13 @@ class Attention(PagedAttentionKernels, Part):
             self.position.apply(qkv[:, :H * hd], qkv[:, H * hd:(H + G) * hd], ctx)
             K.qk_norm_rope_kv(qkv, None, None, 0.0, None, None, 0, False, ctx.positions, view.slot_map, q, kv_out,
                               view.page_size, H, G, hd)
-        o = self._attend(q, ctx, view, cache)
+        pooled = None
+        if means is not None:
+            pv = ctx.paged[means.group]
+            K.pool_blocks(cache.tensor, view.block_table, ctx.row_seg, ctx.positions, pv.slot_map, means.tensor, self.pool,
+                          view.page_size, G, hd)
+            pooled = K.Pooled(self.pool, means.tensor, pv.block_table)
+        o = self._attend(q, ctx, view, cache, pooled)
         if self.head_gate:
             K.head_gate(o, proj[:, self.gate_col:self.gate_col + H], H, hd)
         elif self.gated:

@@ -151,4 +151,4 @@ def _ensure_builtin() -> None:
     global _builtin
     if not _builtin:
         _builtin = True
-        from . import norm, position, attention, shortconv, lightning, ssm, gated, parallel, ffn, block, embedding, side, streams  # noqa: F401
+        from . import norm, position, attention, shortconv, lightning, ssm, gated, parallel, ffn, block, embedding, side, streams, latent  # noqa: F401

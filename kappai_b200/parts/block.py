@@ -26,6 +26,15 @@ its next use and, where another norm follows at once (the feed-forward's, or
 the first norm of the layer that runs next), norms the new residual for it in
 the same pass.
 
+``gated_residual``: ``h = norm1(x); x += ls1 * sigmoid(h Wg1^T + b1) * mixer(h)``, the
+same with norm2, ls2, Wg2, b2 for the feed-forward: a sublayer's output is scaled
+a channel (``layer_scale``; tensors ``ls1``, ``ls2`` [hidden]) and gated element by
+element by its own input (``gate``; ``rg1.weight`` [hidden, hidden] and ``rg1.bias``,
+and so on), either of which may be off.  The sublayer adds into a zeroed
+float32 branch; one kernel scales and gates it into the residual, clears it and
+norms the residual for the sublayer that follows (of this layer or the one that
+runs next).  Where the mixer offers its first product, the gate's rows run in it.
+
 ``streams_residual``: the residual is several float32 streams a row (streams.py).
 A sublayer reads ``norm(sum_b in_b x_b)`` and its output y joins every stream
 while the streams are mixed, ``x'_b = out_b y + sum_a mix_ab x_a``; mixer
@@ -39,7 +48,9 @@ from __future__ import annotations
 
 import torch
 
+from ..config.schema import ConfigError
 from ..ops import kernels as K
+from ..ops.linear import linear
 from .base import Part, WeightSpec, register_part
 from .streams import stream_norm
 
@@ -250,6 +261,92 @@ class StreamsResidualBlock(Part):
             ctx.streams_carry = (x, nxt, h)
 
 
+class GatedResidualBlock(Part):
+    category = "block"
+    graph_safe = True
+
+    def __init__(self, params, env):
+        super().__init__(params, env)
+        self.d = int(self._p("hidden_size"))
+        self.sublayers = int(self._p("sublayers", 2))           # 1: a layer without a feed-forward
+        self.layer_scale = bool(self._p("layer_scale", True))
+        self.gate = bool(self._p("gate", True))
+
+    def weight_specs(self):
+        s = {}
+        for q in range(1, self.sublayers + 1):
+            if self.layer_scale:
+                s[f"ls{q}"] = WeightSpec((self.d,), "norm")
+            if self.gate:
+                s[f"rg{q}.weight"] = WeightSpec((self.d, self.d))
+                s[f"rg{q}.bias"] = WeightSpec((self.d,), "bias")
+        return s
+
+    def assemble(self, mixer, ffn, mixer_norm, ffn_norm, side=None):
+        if side is not None:
+            raise ConfigError("gated_residual: no side part in this arrangement")
+        if self.sublayers != (1 if ffn is None else 2):
+            raise ConfigError("gated_residual: tensors for every sublayer the layer has, and no more")
+        if any(type(n).__name__ != "RMSNorm" for n in (mixer_norm, ffn_norm)[:self.sublayers]):
+            raise ConfigError("gated_residual: every sublayer has an RMS norm in front")
+        self.mixer, self.ffn, self.mixer_norm, self.ffn_norm, self.side = mixer, ffn, mixer_norm, ffn_norm, None
+        return self
+
+    def bind(self, w):
+        # (the mixer's own weights are bound already: a layer's parts are bound in the order in which they are made)
+        n = self.sublayers
+        self.ls = [w[f"ls{q}"].float().contiguous() if self.layer_scale else None for q in range(1, n + 1)]
+        self.w_g = [w[f"rg{q}.weight"].contiguous() if self.gate else None for q in range(1, n + 1)]
+        self.b_g = [w[f"rg{q}.bias"].float().contiguous() if self.gate else None for q in range(1, n + 1)]
+        self.w_in = self.b_in = None
+        offered = self.mixer.input_product() if self.gate and hasattr(self.mixer, "input_product") else None
+        if offered is not None and offered[0].dtype == self.w_g[0].dtype:
+            w_m, b_m = offered
+            self.cols = w_m.shape[0]
+            b_m = b_m if b_m is not None else torch.zeros(self.cols, dtype=torch.float32, device=w_m.device)
+            self.w_in = torch.cat([w_m, self.w_g[0]], 0).contiguous()
+            self.b_in = torch.cat([b_m, self.b_g[0]]).contiguous()
+            self.mixer.drop_input_product()
+            self.w_g[0] = self.b_g[0] = None
+
+    def _close(self, x, y, gate, q, norm):
+        """Sublayer q's output y joins the residual; with ``norm`` the normed residual leaves."""
+        if norm is None:
+            K.gated_add_norm_rows(y, gate, self.ls[q], x)
+            return None
+        h = torch.empty(x.shape, dtype=self.env.dtype, device=x.device)
+        K.gated_add_norm_rows(y, gate, self.ls[q], x, norm.weight, norm.eps, h)
+        return h
+
+    def forward(self, x, ctx, cache):
+        y = branch_rows(x.shape[0], x.shape[1], ctx, x.device)
+        # the input of this layer's mixer: left by the layer before for this very residual, or made here
+        carry = getattr(ctx, "gated_carry", None)
+        ctx.gated_carry = None
+        h = carry[2] if carry is not None and carry[0] is x and carry[1] is self.mixer_norm else self.mixer_norm.forward(x)
+        gate = None
+        if self.w_in is not None:
+            p = linear(h, self.w_in, self.b_in)
+            gate = p[:, self.cols:]
+            self.mixer.forward_projected(p[:, :self.cols], y, ctx, cache)
+        else:
+            if self.gate:
+                gate = linear(h, self.w_g[0], self.b_g[0])
+            self.mixer.forward(h, y, ctx, cache)
+        q = 0
+        if self.ffn is not None:
+            h = self._close(x, y, gate, 0, self.ffn_norm)
+            gate = linear(h, self.w_g[1], self.b_g[1]) if self.gate else None
+            self.ffn.forward(h, y, ctx)
+            q = 1
+        nxt = getattr(ctx, "next_block", None)
+        follows = isinstance(nxt, GatedResidualBlock)
+        h = self._close(x, y, gate, q, nxt.mixer_norm if follows else None)
+        if follows:
+            ctx.gated_carry = (x, nxt.mixer_norm, h)
+
+
+register_part("block", "gated_residual", GatedResidualBlock)
 register_part("block", "streams_residual", StreamsResidualBlock)
 register_part("block", "sandwich_residual", SandwichResidualBlock)
 register_part("block", "prenorm_residual", PreNormResidualBlock)

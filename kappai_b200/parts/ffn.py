@@ -9,6 +9,10 @@ Params: hidden_size, intermediate_size, bias, activation (``silu`` by default;
 ``relu`` and ``gelu_tanh`` make the same unit with another function on the gate:
 kind ``glu``).
 
+``mlp``: an ungated unit of two matrices, ``f = act(h Wu^T) Wd^T``, act =
+``relu_squared`` (the square of relu) or one of the above.  Params: hidden_size,
+intermediate_size, activation.
+
 ``glu_clamped``: the same three matrices with another unit between them: the
 gate is bounded above and the other branch on both sides,
 ``g = min(h Wg^T + bg, limit)``, ``u = clamp(h Wu^T + bu, -limit, limit)``,
@@ -29,7 +33,11 @@ which every row uses beside its chosen experts, its output times
 ``sigmoid(w_sg . h)``, one gate a row (``shared_gate`` = ``"sigmoid"``) or
 ungated (None).  ``routing`` = ``"sigmoid"``: the ``top`` largest logits are
 chosen and a chosen expert's weight is ``sigmoid(z)`` of its own logit times
-``router_scale``, not renormalised.  ``weight_on`` = ``"input"``: the weight
+``router_scale``, not renormalised.  ``renormalise`` (with ``softmax_all``): the
+chosen scores are divided by their sum (+ 1e-20) before ``router_scale``; ``groups`` =
+{count, keep}: the experts form ``count`` equal groups of neighbours, a group
+is as good as its best expert, and only experts of the ``keep`` best groups can be
+chosen.  ``weight_on`` = ``"input"``: the weight
 multiplies what the expert reads, ``sum_j expert_j(w_j h)``, instead of what it
 returns (``"output"``, the default).
 """
@@ -40,7 +48,7 @@ from typing import Dict
 import torch
 
 from ..ops import kernels as K
-from ..ops.linear import linear, linear_swiglu
+from ..ops.linear import linear, linear_act, linear_swiglu
 from ..config.schema import ConfigError
 from .base import Part, WeightSpec, register_part
 
@@ -77,6 +85,29 @@ class SwiGLU(Part):
     def forward(self, h, residual, ctx):
         act = linear_swiglu(h, self.w_gu, self.b_gu, self.activation)
         linear(act, self.w_down, self.b_down, out=residual, accumulate=True)
+
+
+class UngatedUnit(Part):
+    """``mlp``: see the module's text.  The activation runs in the first product's epilogue, on its float32 sums."""
+
+    category = "feed_forward"
+    graph_safe = True
+
+    def __init__(self, params, env):
+        super().__init__(params, env)
+        self.d = int(self._p("hidden_size"))
+        self.ff = int(self._p("intermediate_size"))
+        self.activation = str(self._p("activation"))
+        K.plain_activation_code(self.activation)
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {"up_proj.weight": WeightSpec((self.ff, self.d)), "down_proj.weight": WeightSpec((self.d, self.ff))}
+
+    def bind(self, w):
+        self.w_up, self.w_down = w["up_proj.weight"].contiguous(), w["down_proj.weight"].contiguous()
+
+    def forward(self, h, residual, ctx):
+        linear(linear_act(h, self.w_up, None, self.activation), self.w_down, out=residual, accumulate=True)
 
 
 class ClampedGLU(SwiGLU):
@@ -116,6 +147,9 @@ class MixtureOfExperts(Part):
             raise ConfigError(f"moe: routing='{self.routing}' (expected one of {', '.join(K.MOE_ROUTINGS)})")
         self.router_bias = bool(self._p("router_bias", self.routing == "top_logits"))
         self.correction = bool(self._p("correction", self.routing == "softmax_all"))
+        self.renormalise = bool(self._p("renormalise", False))
+        groups = self._p("groups", None)
+        self.groups = None if groups is None else (int(groups["count"]), int(groups["keep"]))
         self.router_scale = float(self._p("router_scale", 1.0))
         self.n_identity = int(self._p("identity_experts", 0))
         self.weight_on = str(self._p("weight_on", "output"))
@@ -132,6 +166,14 @@ class MixtureOfExperts(Part):
             raise ConfigError(f"moe: top={self.top} must lie between 1 and the {self.E_all} router outputs")
         if self.top > K.MOE_MAX_TOP or self.E_all > K.MOE_MAX_EXPERTS:
             raise ConfigError(f"moe: the kernels take top <= {K.MOE_MAX_TOP} and at most {K.MOE_MAX_EXPERTS} router outputs")
+        if (self.renormalise or self.groups is not None) and self.routing != "softmax_all":
+            raise ConfigError("moe: renormalised weights and groups belong to routing='softmax_all'")
+        if self.groups is not None:
+            count, keep = self.groups
+            if not (1 <= count <= K.MOE_MAX_GROUPS and 1 <= keep <= count) or self.E_all % count:
+                raise ConfigError(f"moe: groups of count={count} (at most {K.MOE_MAX_GROUPS}, a divisor of {self.E_all}), keep={keep}")
+            if self.top > keep * (self.E_all // count):
+                raise ConfigError(f"moe: top={self.top} exceeds the experts of {keep} of {count} groups")
         if self.routing == "top_logits" and self.correction:
             raise ConfigError("moe: a correction of the choice belongs to routing='softmax_all'")
         if self.routing == "sigmoid" and (self.router_bias or self.correction):
@@ -182,7 +224,8 @@ class MixtureOfExperts(Part):
         idx = torch.empty((n, self.top), dtype=torch.int32, device=h.device)
         weights = torch.empty((n, self.top), dtype=torch.float32, device=h.device)
         layout = torch.empty(K.moe_layout_ints(n, self.E_all, self.top), dtype=torch.int32, device=h.device)
-        how = dict(routing=self.routing, scale=self.router_scale, n_identity=self.n_identity)
+        how = dict(routing=self.routing, scale=self.router_scale, n_identity=self.n_identity, groups=self.groups,
+                   renormalise=self.renormalise)
         if K.moe_router_ok(self.d, self.E_all) and h.stride(1) == 1:
             K.moe_router(h, self.w_router, self.b_router, self.top, idx, weights, layout, **how)
         elif self.routing == "top_logits":
@@ -204,5 +247,6 @@ class MixtureOfExperts(Part):
 
 register_part("feed_forward", "swiglu", SwiGLU)
 register_part("feed_forward", "glu", SwiGLU)
+register_part("feed_forward", "mlp", UngatedUnit)
 register_part("feed_forward", "glu_clamped", ClampedGLU)
 register_part("feed_forward", "moe", MixtureOfExperts)

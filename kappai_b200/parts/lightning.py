@@ -25,10 +25,11 @@ k by position as the kernels read them, in float32; ``k_scale`` multiplies k
 behind the rotation; ``norm`` = ``"per_head"`` divides every head's ``o`` by
 its own root mean square and has no weight (the default ``"all_heads"`` is the
 norm above); ``gate`` = ``"silu"`` multiplies by ``silu(h Wg^T)`` instead.
+``out_scale`` (default 1) multiplies the mixer's output (the norm carries it).
 
 Params: hidden_size, num_heads, head_dim, value_dim, decay (a list, one a
 head), norm_eps, activation ("silu" | None), gate ("sigmoid" | "silu"), norm
-("all_heads" | "per_head"), position (None | a rope PartSpec), k_scale.
+("all_heads" | "per_head"), position (None | a rope PartSpec), k_scale, out_scale.
 """
 from __future__ import annotations
 
@@ -99,6 +100,7 @@ class LightningAttention(Part):
         if self.norm not in ("all_heads", "per_head"):
             raise ConfigError(f"lightning: norm='{self.norm}' (expected 'all_heads' or 'per_head')")
         self.k_scale = float(self._p("k_scale", 1.0))
+        self.out_scale = float(self._p("out_scale", 1.0))
         pos = self._p("position", None)
         self.rotary = None
         if pos is not None:
@@ -133,9 +135,17 @@ class LightningAttention(Part):
         return s
 
     def bind(self, w):
-        self.w_in = torch.cat([w["q_proj.weight"], w["k_proj.weight"], w["v_proj.weight"], w["gate_proj.weight"]], 0).contiguous()
+        rows = [w["q_proj.weight"], w["k_proj.weight"], w["v_proj.weight"], w["gate_proj.weight"]]
+        n_rows = sum(r.shape[0] for r in rows)
+        if n_rows % 8:
+            # zero rows behind the last, so that a row of the product's output starts on a 16-byte boundary
+            rows.append(torch.zeros((8 - n_rows % 8, self.d), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_in = torch.cat(rows, 0).contiguous()
         self.w_o = w["out_proj.weight"].contiguous()
         self.norm_w = w["norm.weight"].float().contiguous() if self.norm == "all_heads" else None
+        if self.out_scale != 1.0:
+            one = torch.ones(self.H * self.vdim, dtype=torch.float32, device=self.w_in.device) if self.norm_w is None else self.norm_w
+            self.norm_w = (one * self.out_scale).contiguous()
         # a decay as a float32 pair: hi the nearest float32, lo what it leaves of the constant
         a = np.asarray(self.decay, dtype=np.float64)
         hi = a.astype(np.float32)
@@ -152,10 +162,20 @@ class LightningAttention(Part):
     def cache_spec(self):
         return StateSpec((self.H, self.dim, self.vdim), "float32")
 
+    # (a mixer whose first product can be run together with others': see parallel.py)
+    def input_product(self):
+        return self.w_in, None
+
+    def drop_input_product(self):
+        self.w_in = None
+
     def forward(self, h, residual, ctx, cache):
         """``cache``: a :class:`~kappai_b200.cache.storage.StateView` with tensor [n_slots, H, head_dim, value_dim]."""
+        self.forward_projected(linear(h, self.w_in), residual, ctx, cache)
+
+    def forward_projected(self, p, residual, ctx, cache):
+        """``p``: the rows of the input product, [q | k | v | gate], possibly columns of a wider one."""
         H, dim, vdim, n = self.H, self.dim, self.vdim, ctx.n_rows
-        p = linear(h, self.w_in)                                 # [q | k | v | gate]
         o = torch.empty((n, H * vdim), dtype=torch.float32, device=p.device)
         chunks = ctx.tables.get(self.step_tables_key) if self.chunked else None
         scan = lambda n_seg: K.lightning_scan(p, 0, H * dim, 2 * H * dim, self.decay_hi, self.decay_lo, cache.tensor, ctx.cu_rows,

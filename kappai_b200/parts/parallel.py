@@ -2,7 +2,8 @@
 
 Every mixer reads the layer's normed input and adds its output into the residual (a mixer that is weighed in the sum has a
 parameter of its own for that, ``out_scale``).  Mixers that offer their first product (``input_product`` -> weight and
-bias, ``forward_projected`` on its rows) have it run as one product with the others'; what the mixers keep is a
+bias, ``forward_projected`` on its rows) have it run as one product with the others' (and where all of them do, the whole
+offers that product in turn); what the mixers keep is a
 :class:`~kappai_b200.cache.spec.CompositeSpec` in their order.
 
 Params: mixers (a dict name -> ``mixer`` PartSpec; a mixer's tensors are known here as ``<name>.<its local name>``, its own
@@ -65,12 +66,24 @@ class ParallelMixers(Part):
             for n in self.joined:
                 self.mixers[n].drop_input_product()
 
+    def input_product(self):
+        """The joined product, or None where some mixer runs a product of its own."""
+        return (self.w_in, self.b_in) if len(self.joined) == len(self.mixers) else None
+
+    def drop_input_product(self):
+        self.w_in = self.b_in = None
+
     def cache_spec(self):
         return CompositeSpec(tuple(m.cache_spec() for m in self.mixers.values()))
 
     def forward(self, h, residual, ctx, cache):
         """``cache``: a :class:`~kappai_b200.cache.storage.CompositeView`, one view a mixer."""
-        p = linear(h, self.w_in, self.b_in) if self.joined else None
+        self._run(h, linear(h, self.w_in, self.b_in) if self.joined else None, residual, ctx, cache)
+
+    def forward_projected(self, p, residual, ctx, cache):
+        self._run(None, p, residual, ctx, cache)
+
+    def _run(self, h, p, residual, ctx, cache):
         for (n, m), view in zip(self.mixers.items(), cache.parts):
             if n in self.cols:
                 a, b = self.cols[n]

@@ -12,7 +12,12 @@ frequencies by their wavelength ``l = 2 pi / f``: a frequency with
 ``l < original / high`` is kept, one with ``l > original / low`` is divided by
 ``factor``, and between the two, with ``s = (original / l - low) / (high - low)``,
 it becomes ``(1 - s) f / factor + s f``.  With the key ``factor`` alone every
-frequency is divided by it.
+frequency is divided by it.  With the keys ``factor``, ``original``, ``fast`` and
+``slow`` (YaRN) the blend runs over the pairs instead: pair t(n) = dims ln(original
+/ (2 pi n)) / (2 ln theta) turns n times over the original length, the pairs up
+to floor(t(fast)) keep their frequency, those from ceil(t(slow)) on are divided
+by ``factor``, linearly in between; and the cosines and sines are multiplied by
+``0.1 ln(factor) + 1``.
 
 ``none``: no rotation.
 """
@@ -27,11 +32,18 @@ from .base import Part, register_part
 
 def scaled_frequencies(f: np.ndarray, scaling) -> np.ndarray:
     """Rotary frequencies rescaled by wavelength (see the module's text); ``scaling`` is
-    (factor, low, high, original), (factor,) or None."""
+    (factor, low, high, original), (factor,), ("yarn", factor, original, fast, slow, theta) or None."""
     if scaling is None:
         return f
     if len(scaling) == 1:
         return f / scaling[0]
+    if scaling[0] == "yarn":
+        _, factor, original, fast, slow, theta = scaling
+        dims = 2 * len(f)
+        pair = lambda turns: dims * np.log(original / (2.0 * np.pi * turns)) / (2.0 * np.log(theta))
+        lo, hi = max(np.floor(pair(fast)), 0.0), min(np.ceil(pair(slow)), dims - 1.0)
+        ramp = np.clip((np.arange(len(f)) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+        return f / factor * ramp + f * (1.0 - ramp)
     factor, low, high, original = scaling
     lam = 2.0 * np.pi / f
     s = (original / lam - low) / (high - low)
@@ -59,6 +71,10 @@ class RotaryEncoding(Part):
             self.scaling = (float(scaling["factor"]),)
             if not self.scaling[0] > 0:
                 raise ConfigError("rope: scaling wants factor > 0")
+        elif scaling and set(scaling) == {"factor", "original", "fast", "slow"}:
+            self.scaling = ("yarn",) + tuple(float(scaling[k]) for k in ("factor", "original", "fast", "slow")) + (self.theta,)
+            if min(self.scaling[1:5]) <= 0 or self.theta <= 0 or self.theta == 1.0:
+                raise ConfigError("rope: scaling wants factor, original, fast and slow > 0")
         elif scaling:
             try:
                 self.scaling = tuple(float(scaling[k]) for k in ("factor", "low", "high", "original"))
@@ -73,8 +89,9 @@ class RotaryEncoding(Part):
             inv = scaled_frequencies(
                 np.power(self.theta, -2.0 * np.arange(half, dtype=np.float64) / self.rotary_dim), self.scaling)
             ang = np.arange(env.max_positions, dtype=np.float64)[:, None] * inv[None, :]
-            env.shared[key] = (torch.from_numpy(np.cos(ang).astype(np.float32)).to(env.device),
-                               torch.from_numpy(np.sin(ang).astype(np.float32)).to(env.device))
+            m = 0.1 * np.log(self.scaling[1]) + 1.0 if self.scaling and self.scaling[0] == "yarn" else 1.0
+            env.shared[key] = (torch.from_numpy((np.cos(ang) * m).astype(np.float32)).to(env.device),
+                               torch.from_numpy((np.sin(ang) * m).astype(np.float32)).to(env.device))
         self.cos, self.sin = env.shared[key]
 
     def fused_rotary(self):
