@@ -58,6 +58,11 @@ linear attention, windowed attention with short convolutions side by side with a
 run twice) beside Tupalorn layers of the same sizes, the closest design the engine has (recurrent mixers with float32
 states and convolutions, windowed attention, gated units).
 
+``--design ladedra`` does the same for the Ladedra design (scaled and gated sublayers; attention over cached latents; windowed
+attention with pooled blocks, soft-capped scores and learned sinks side by side with retention; a square-of-relu unit and
+mixtures chosen from groups, with a shared unit) beside Vekuzen layers of the same sizes, the closest design the engine has
+(latent attention and lightning layers in turn, mixtures with a shared unit, whole softmax weights).
+
 Only one GPU is used; ``--gpus N`` with N > 1 prints a line that says so and
 exits with 2.
 """
@@ -504,6 +509,30 @@ def gosulorn_config(width, H, G, hd, ff):
             "layers": layers}
 
 
+LADEDRA_WINDOW = 1024
+LADEDRA_POOL = 16
+
+
+def ladedra_config(width, H, G, hd, ff, E, top, ff_e, layers):
+    """Layers of the sizes of the other designs' (``layers``: d = dense, m = mixture): latent attention (a latent of 512, a
+    rotated part of 64) and, in turn, windowed attention with pooled blocks beside retention; a dense layer's unit is the
+    square-of-relu one, mixtures choose from the better half of four groups."""
+    latent = {"heads": H, "dim": hd, "vdim": hd, "kv_rank": 512, "rot_dim": 64, "scale": (hd + 64) ** -0.5,
+              "rot": {"dims": 64, "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
+    left = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0,
+            "mask": {"size": LADEDRA_WINDOW, "pool": LADEDRA_POOL}, "rot": {"dims": hd, "base": 500000.0}}
+    right = {"heads": H, "dim": hd, "vdim": hd, "decay": [1.0 - 2.0 ** (-3 - 6 * h / max(1, H - 1)) for h in range(H)],
+             "rot": {"dims": hd, "base": 10000.0}}
+    both = {"left": left, "left_scale": 1.0, "right": right, "right_scale": 0.7}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff_e}, "shared": {"ff": ff_e},
+           "router": {"experts": E, "top": top, "scale": 2.0, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Ladedra", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5},
+            "max_positions": VEKUZEN_POSITIONS,
+            "layers": [{"type": "latent_attention" if i % 2 == 0 else "parallel", "mixer": dict(latent if i % 2 == 0 else both),
+                        "mlp": dict(dense if c == "d" else moe)} for i, c in enumerate(layers)]}
+
+
 def lfm2_like_config(width, H, G, hd, ff, n_layers):
     return dict(architectures=["Lfm2ForCausalLM"], vocab_size=DESIGN_VOCAB, hidden_size=width, num_hidden_layers=n_layers,
                 num_attention_heads=H, num_key_value_heads=G, head_dim=hd, layer_types=["full_attention"] * n_layers,
@@ -551,7 +580,8 @@ def run_design(a) -> int:
     import kappai_b200.models.vekuzen as vk
     import kappai_b200.models.vumotar as vm
     import kappai_b200.models.gosulorn as gs
-    tz.SOFTMAX_WEIGHTS = vk.SOFTMAX_WEIGHTS = vm.SOFTMAX_WEIGHTS = gs.SOFTMAX_WEIGHTS = a.softmax_weights
+    import kappai_b200.models.ladedra as ld
+    tz.SOFTMAX_WEIGHTS = vk.SOFTMAX_WEIGHTS = vm.SOFTMAX_WEIGHTS = gs.SOFTMAX_WEIGHTS = ld.SOFTMAX_WEIGHTS = a.softmax_weights
     pk = peaks()
     T, B, ctx_len = PROMPT_LEN, a.batch, PROMPT_LEN + 256
     warmup = max(a.warmup, 3)
@@ -560,8 +590,10 @@ def run_design(a) -> int:
     tupalorn = a.design == "tupalorn"
     vumotar = a.design == "vumotar"
     gosulorn = a.design == "gosulorn"
+    ladedra = a.design == "ladedra"
     out = {"design": a.design.capitalize(),
-           "beside": ("Tupalorn layers of the same sizes" if gosulorn else
+           "beside": ("Vekuzen layers of the same sizes" if ladedra else
+                      "Tupalorn layers of the same sizes" if gosulorn else
                       "Tizusun mixture layers of the same sizes" if vumotar else
                       "dense Vekuzen layers of the same sizes" if tupalorn else "Tizusun layers of the same sizes" if vekuzen
                       else "LFM2 attention layers of the same sizes"), "dtype": "bf16",
@@ -578,7 +610,9 @@ def run_design(a) -> int:
             layers = "dddd"
         if vumotar:
             layers = "mmm"
-        pair = ((("gosulorn", gosulorn_config(width, H, G, hd, ff)), ("tupalorn", tupalorn_config(width, H, G, hd, ff))) if gosulorn else
+        pair = ((("ladedra", ladedra_config(width, H, G, hd, ff, E, top, ff_e, layers)),
+                 ("vekuzen", vekuzen_config(width, H, G, hd, ff, E, top, ff_e, layers))) if ladedra else
+                (("gosulorn", gosulorn_config(width, H, G, hd, ff)), ("tupalorn", tupalorn_config(width, H, G, hd, ff))) if gosulorn else
                 (("vumotar", vumotar_config(width, H, G, hd, E, top, ff_e)),
                  ("tizusun", tizusun_config(width, H, G, hd, ff, E, top, ff_e, layers))) if vumotar else
                 (("tupalorn", tupalorn_config(width, H, G, hd, ff)),
@@ -730,7 +764,7 @@ def main() -> int:
                     help="with --workload: launch every kernel on its own between CUDA events and print the device "
                          "time by kernel class (the run's throughput is then not the engine's)")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="prompt length of --probe")
-    ap.add_argument("--design", choices=["tizusun", "vekuzen", "tupalorn", "vumotar", "gosulorn"], default=None,
+    ap.add_argument("--design", choices=["tizusun", "vekuzen", "tupalorn", "vumotar", "gosulorn", "ladedra"], default=None,
                     help="time another design at a few layer sizes beside the closest existing model of the same sizes "
                          "(tizusun beside LFM2 attention layers, vekuzen beside tizusun, tupalorn beside dense vekuzen layers) "
                          "(prefill, decode, device time by kernel class) instead of the default line")

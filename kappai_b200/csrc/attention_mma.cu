@@ -109,6 +109,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __res
                       const int* __restrict__ positions, float* __restrict__ part_acc, float* __restrict__ part_ml,
                       int n_slots, int slot0, float scale, int window, int page_size, int H, int G, int block, float cap, int pool) {
     constexpr bool exact_p = MODE >= 1;                           // the softmax weights enter the product with V whole
+    const float two_over_cap = MODE == 2 && cap > 0.f ? 2.0f / cap : 0.f;
     kp_pdl_begin_early_if(gridDim.z > 1);
     extern __shared__ unsigned char smem_dyn[];
     unsigned char* smem_raw = reinterpret_cast<unsigned char*>(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023);
@@ -206,7 +207,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __res
 #pragma unroll
         for (int i = 0; i < 2; i++) {
             const int key = t0 + nt * 8 + 2 * t + i;
-            const float sv = MODE == 2 ? kp_capped(s[nt][i] * scale, cap) : s[nt][i] * scale;
+            const float sv = MODE == 2 ? kp_capped_fast(s[nt][i] * scale, cap, two_over_cap) : s[nt][i] * scale;
             const float v = (key >= k_lo && key <= k_hi) ? sv : -INFINITY;
             s[nt][i] = v;
             m = fmaxf(m, v);
@@ -312,6 +313,7 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
                        int n_chunks, int n_slots, int slot0, float scale, int window, int page_size, int H, int G, int n_rows,
                        int block, float cap, int pool) {
     constexpr bool exact_p = MODE >= 1;
+    const float two_over_cap = MODE == 2 && cap > 0.f ? 2.0f / cap : 0.f;
     kp_pdl_begin_early_if(n_rows > 1);
     extern __shared__ unsigned char smem_dyn[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_dyn + 1023) & ~(uintptr_t)1023);
@@ -467,7 +469,7 @@ attn_split_ring_kernel(const __grid_constant__ CUtensorMap tmC, const bf16* __re
 #pragma unroll
             for (int i = 0; i < 2; i++) {
                 const int key = t0 + nt * 8 + 2 * t + i;
-                const float sv = MODE == 2 ? kp_capped(sc[nt][i] * scale, cap) : sc[nt][i] * scale;
+                const float sv = MODE == 2 ? kp_capped_fast(sc[nt][i] * scale, cap, two_over_cap) : sc[nt][i] * scale;
                 const float v = (key >= k_lo && key <= k_hi) ? sv : -INFINITY;
                 sc[nt][i] = v;
                 m = fmaxf(m, v);
@@ -562,6 +564,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
                         float out_scale, int pool, const bf16* __restrict__ pool_cache, const int* __restrict__ pool_table,
                         int max_pool_blocks) {
     constexpr bool exact_p = MODE >= 1;
+    const float two_over_cap = MODE == 2 && cap > 0.f ? 2.0f / cap : 0.f;
     kp_pdl_begin();
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* Ks = reinterpret_cast<bf16*>(smem_raw);                 // [2][64][HD]
@@ -656,8 +659,8 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, int ldq, const bf16* __restr
                     const int key = t0 + nt * 8 + 2 * t + i;
                     const bool in_a = front ? key < cnt_a : key <= pos_a && (key >= lo_a || key < keep_first);
                     const bool in_b = front ? key < cnt_b : key <= pos_b && (key >= lo_b || key < keep_first);
-                    const float ca_ = MODE == 2 ? kp_capped(s[nt][i] * scale, cap) : s[nt][i] * scale;
-                    const float cb_ = MODE == 2 ? kp_capped(s[nt][2 + i] * scale, cap) : s[nt][2 + i] * scale;
+                    const float ca_ = MODE == 2 ? kp_capped_fast(s[nt][i] * scale, cap, two_over_cap) : s[nt][i] * scale;
+                    const float cb_ = MODE == 2 ? kp_capped_fast(s[nt][2 + i] * scale, cap, two_over_cap) : s[nt][2 + i] * scale;
                     const float va = has_a && in_a ? ca_ : -INFINITY;
                     const float vb = has_b && in_b ? cb_ : -INFINITY;
                     s[nt][i] = va; s[nt][2 + i] = vb;

@@ -88,6 +88,11 @@ __device__ __forceinline__ int kp_key_lo(int pos, int window, int block) {
 __device__ __forceinline__ int kp_pooled_count(int pos, int window, int pool) { return max(0, pos - window + 1) / pool; }
 // A score bounded smoothly by `cap` (0: as it is).
 __device__ __forceinline__ float kp_capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
+// The same from one exponential and one division, tanh(x) = 1 - 2 / (e^2x + 1), in float32 throughout; off by an absolute
+// 1e-7 cap or so.  For the tensor-core kernels, whose scores are sums of products of bfloat16 operands.
+__device__ __forceinline__ float kp_capped_fast(float s, float cap, float two_over_cap) {
+    return cap > 0.f ? cap - __fdividef(2.0f * cap, __expf(s * two_over_cap) + 1.0f) : s;
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -304,8 +304,10 @@ class GatedResidualBlock(Part):
             w_m, b_m = offered
             self.cols = w_m.shape[0]
             b_m = b_m if b_m is not None else torch.zeros(self.cols, dtype=torch.float32, device=w_m.device)
-            self.w_in = torch.cat([w_m, self.w_g[0]], 0).contiguous()
-            self.b_in = torch.cat([b_m, self.b_g[0]]).contiguous()
+            # (zero rows behind the last, so that a row of the product's output starts on a 16-byte boundary)
+            pad = -(self.cols + self.d) % 8
+            self.w_in = torch.cat([w_m, self.w_g[0], w_m.new_zeros((pad, self.d))], 0).contiguous()
+            self.b_in = torch.cat([b_m, self.b_g[0], b_m.new_zeros(pad)]).contiguous()
             self.mixer.drop_input_product()
             self.w_g[0] = self.b_g[0] = None
 
@@ -327,7 +329,7 @@ class GatedResidualBlock(Part):
         gate = None
         if self.w_in is not None:
             p = linear(h, self.w_in, self.b_in)
-            gate = p[:, self.cols:]
+            gate = p[:, self.cols:self.cols + self.d]
             self.mixer.forward_projected(p[:, :self.cols], y, ctx, cache)
         else:
             if self.gate:

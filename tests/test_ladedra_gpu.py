@@ -1,0 +1,818 @@
+"""Ladedra on the GPU: every new mechanism's kernel against the plain functions, the mixers, the feed-forwards and the
+layer arrangement as parts in batches cut in two, then whole models through the step function, the trace runner and
+the engine in every way of cutting the work."""
+import copy
+import math
+
+import numpy as np
+import pytest
+import torch
+
+import plain_ladedra as P
+import replay_util as R
+from ladedra_configs import CONFIGS, make_model_dir, make_weights, write_model_dir
+from test_kernels_gpu import i32, paged_setup, rt
+from tolerances import tol_for
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda:0"
+DTYPES = [torch.float32, torch.bfloat16]
+BF = torch.bfloat16
+
+
+def dev(a, dtype=torch.float32):
+    return torch.as_tensor(np.asarray(a), dtype=torch.float32).to(DEV).to(dtype).contiguous()
+
+
+def host(t):
+    return t.detach().double().cpu().numpy()
+
+
+def close(got, want, dtype, tol16=0.02, tol32=3e-5):
+    tol = tol32 if dtype == torch.float32 else tol16
+    err = np.abs(got - want).max() / max(1.0, np.abs(want).max())
+    assert err <= tol, err
+
+
+@pytest.fixture(scope="module")
+def lad_dirs(tmp_path_factory):
+    root = tmp_path_factory.mktemp("ladedra")
+    return {n: make_model_dir(n, str(root)) for n in CONFIGS}
+
+
+@pytest.fixture(scope="module")
+def lad_plain(lad_dirs):
+    return {n: P.PlainLadedra(d) for n, d in lad_dirs.items()}
+
+
+# ------------------------------------------------------------------------------------- pooled attention kernels
+
+def _pooled_setup(rng, seq_lens, page, G, hd, dtype, window, pool):
+    """Keys and values on scrambled pages, whose pages behind the window (and behind the unfinished block) are released, and
+    the means of every whole block on pages of their own, in the storage type: (cache, bt, pool cache, pool bt, ks, vs,
+    means of the keys and of the values as stored)."""
+    cache, bt, ks, vs = paged_setup(rng, seq_lens, page, G, hd, dtype)
+    bt = bt.copy()
+    keep = max(window, pool)
+    for i, L in enumerate(seq_lens):
+        for b in range(max(0, L - 1 - keep + 1) // page):
+            bt[i, b] = -1
+    n_ent = [L // pool for L in seq_lens]
+    blocks = [max(1, -(-n // page)) for n in n_ent]
+    pcache = rt(rng.standard_normal((sum(blocks) + 2, 2, G, page, hd)) * 5, dtype)
+    perm = rng.permutation(sum(blocks) + 2)
+    pbt = np.full((len(seq_lens), max(blocks)), -1, np.int32)
+    kms, vms, o = [], [], 0
+    for i, (n, nb) in enumerate(zip(n_ent, blocks)):
+        pbt[i, :nb] = perm[o:o + nb]
+        o += nb
+        km, vm = rt(P.block_means(ks[i], pool), dtype), rt(P.block_means(vs[i], pool), dtype)
+        for e in range(n):
+            pcache[pbt[i, e // page], 0, :, e % page] = km[e]
+            pcache[pbt[i, e // page], 1, :, e % page] = vm[e]
+        kms.append(km)
+        vms.append(vm)
+    return cache, bt, pcache, pbt, ks, vs, kms, vms
+
+
+def _plain_pooled(q, k, v, km, vm, scale, window, pool, cap, sink, out_scale=1.0):
+    """As plain_ladedra.pooled_attention, with the blocks' means given: q [L, H, hd] -> [L, H, hd]."""
+    L, H, _ = q.shape
+    G = k.shape[1]
+    tok, blk = P.pooled_window_masks(L, window, pool)
+    mask = np.concatenate([blk, tok], axis=1)
+    out = np.zeros((L, H, v.shape[2]))
+    for h in range(H):
+        g = h // (H // G)
+        s = P.softcap((q[:, h] @ np.concatenate([km[:, g], k[:, g]]).T) * scale, cap)
+        out[:, h] = P.softmax_with_sink(s, mask, None if sink is None else sink[h]) @ np.concatenate([vm[:, g], v[:, g]])
+    return out * out_scale
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,hd,page,window,pool,cap,sink,out_scale", [
+    (4, 2, 16, 16, 20, 5, 4.0, True, 1.3), (5, 1, 48, 32, 7, 9, 0.0, True, 1.0), (6, 3, 112, 8, 50, 3, 30.0, False, 0.7),
+    (8, 2, 64, 64, 128, 24, 30.0, True, 0.5), (4, 4, 128, 16, 40, 7, 2.0, True, 1.0), (2, 2, 64, 8, 1, 2, 5.0, False, 1.0),
+    (8, 1, 64, 32, 33, 1, 0.0, True, 2.0), (16, 1, 32, 16, 30, 8, 10.0, True, 1.1), (3, 3, 64, 16, 64, 64, 3.0, True, 1.0)])
+def test_decoded_rows_with_pooled_blocks(dtype, H, G, hd, page, window, pool, cap, sink, out_scale):
+    """The last row of requests whose lengths put the window's edge and the last pooled block on both sides of page, tile and
+    chunk borders, through the split-key kernels (where they take the shape) and the general kernel."""
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(H + hd + window + pool)
+    seq_lens = [1, 4, window, window + 1, window + pool - 1, window + pool, window + 2 * pool, 255, 256, 257, 700, 513]
+    cache, bt, pc, pbt, ks, vs, kms, vms = _pooled_setup(rng, seq_lens, page, G, hd, dtype, window, pool)
+    scale = 1.0 / math.sqrt(hd)
+    sk = rt(rng.uniform(-1, 3, H), torch.float32) if sink else None
+    qs = [rt(rng.standard_normal((L, H, hd)) * 2, dtype) for L in seq_lens]
+    n = len(seq_lens)
+    want = np.stack([_plain_pooled(q, k, v, km, vm, scale, window, pool, cap, sk, out_scale)[-1]
+                     for q, k, v, km, vm in zip(qs, ks, vs, kms, vms)])
+    args = (dev(np.stack([q[-1] for q in qs]).reshape(n, H * hd), dtype), dev(cache, dtype), i32(bt), i32(range(n)), i32([L - 1 for L in seq_lens]))
+    extra = dict(sink=dev(sk) if sink else None, cap=cap, out_scale=out_scale, pooled=Kn.Pooled(pool, dev(pc, dtype), i32(pbt)))
+    gen = torch.empty((n, H * hd), dtype=dtype, device=DEV)
+    Kn.attention_rows(*args, gen, scale, window, page, H, G, hd, **extra)
+    close(host(gen).reshape(want.shape), want, dtype)
+    if H // G <= Kn.SPLIT_MAX_RATIO and hd % 16 == 0:
+        for n_chunks in (-(-max(seq_lens) // Kn.SPLIT_CHUNK), 7):
+            ws = torch.full((Kn.attention_split_scratch(n, H, hd, n_chunks, 0, extra["pooled"]),), float("nan"), device=DEV)
+            out = torch.empty_like(gen)
+            Kn.attention_split(*args, out, ws, n_chunks, scale, window, page, H, G, hd, exact_weights=True, **extra)
+            close(host(out).reshape(want.shape), want, dtype)
+    assert Kn.attention_mma_status() == 0
+
+
+def _portions(seq_lens, q_from, tile=64):
+    cu, seg_pos, tile_seg, tile_row0, row_seg, positions = [0], [], [], [], [], []
+    for i, (L, a) in enumerate(zip(seq_lens, q_from)):
+        for r0 in range(cu[-1], cu[-1] + L - a, tile):
+            tile_seg.append(i)
+            tile_row0.append(r0)
+        cu.append(cu[-1] + L - a)
+        seg_pos.append(a)
+        row_seg += [i] * (L - a)
+        positions += list(range(a, L))
+    return cu, seg_pos, tile_seg, tile_row0, row_seg, positions
+
+
+@pytest.mark.parametrize("H,G,hd,page,window,pool,cap,out_scale", [
+    (8, 2, 64, 64, 128, 24, 30.0, 0.5), (4, 4, 128, 16, 40, 7, 2.0, 1.3), (2, 2, 64, 8, 300, 9, 0.0, 1.0), (8, 1, 64, 32, 33, 1, 5.0, 1.0),
+    (4, 2, 64, 16, 1, 2, 4.0, 1.0), (6, 3, 128, 32, 64, 64, 10.0, 2.0), (4, 1, 64, 16, 5, 70, 20.0, 1.0)])
+def test_prompt_portions_with_pooled_blocks(H, G, hd, page, window, pool, cap, out_scale):
+    """The tensor-core prompt kernel over whole prompts and late portions, against whole-sequence attention and the general
+    kernel."""
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(hd + window + pool)
+    seq_lens, q_from = [130, 700, 257, 64, 420], [0, 391, 255, 1, 70]
+    cache, bt, pc, pbt, ks, vs, kms, vms = _pooled_setup(rng, seq_lens, page, G, hd, BF, 10 ** 6, pool)     # (nothing released)
+    scale = 1.0 / math.sqrt(hd)
+    sk = rt(rng.uniform(-1, 3, H), torch.float32)
+    qs = [rt(rng.standard_normal((L, H, hd)) * 2, BF) for L in seq_lens]
+    cu, seg_pos, tile_seg, tile_row0, row_seg, positions = _portions(seq_lens, q_from)
+    want = np.concatenate([_plain_pooled(qs[i], ks[i], vs[i], kms[i], vms[i], scale, window, pool, cap, sk, out_scale)[a:]
+                           for i, a in enumerate(q_from)], 0)
+    q_rows = dev(np.concatenate([q[a:] for q, a in zip(qs, q_from)], 0).reshape(cu[-1], H * hd), BF)
+    extra = dict(sink=dev(sk), cap=cap, out_scale=out_scale, pooled=Kn.Pooled(pool, dev(pc, BF), i32(pbt)))
+    out = torch.empty((cu[-1], H * hd), dtype=BF, device=DEV)
+    Kn.attention_prefill(q_rows, dev(cache, BF), i32(bt), i32(cu), i32(seg_pos), i32(tile_seg), i32(tile_row0), out, scale,
+                         window, page, H, G, hd, exact_weights=True, **extra)
+    close(host(out).reshape(want.shape), want, BF)
+    gen = torch.empty_like(out)
+    Kn.attention_rows(q_rows, dev(cache, BF), i32(bt), i32(row_seg), i32(positions), gen, scale, window, page, H, G, hd, **extra)
+    assert (gen.float() - out.float()).abs().max().item() <= 2.5e-2 * max(1.0, out_scale)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("which", ["window_in", "window_out", "block_in", "block_out", "sink"])
+def test_one_score_stands_out_at_every_edge(which, dtype):
+    """Among hundreds of keys one has a score 12 above the rest: the window's last key (it carries the row), the first one
+    behind it (it must not count, nor its block, which is not wholly behind), the last block that is wholly behind the
+    window (its mean carries the row), the one after it (it must not), or the sink.  Decoded row and prompt portion."""
+    from kappai_b200.ops import kernels as Kn
+    H, G, hd, page, window, pool, L = 4, 2, 64, 16, 100, 12, 600
+    rng = np.random.default_rng(5)
+    i = L - 1
+    last_block = (i - window + 1) // pool - 1                                  # the last block that row i sees
+    target = {"window_in": i - window + 1, "window_out": i - window, "sink": None}.get(which)
+    block = {"block_in": last_block, "block_out": last_block + 1}.get(which)
+    assert (i - window) // pool == last_block + 1                              # the key behind the window lies in an unseen block
+    cache, bt, ks, vs = paged_setup(rng, [L], page, G, hd, dtype)
+    if block is not None:
+        # a block whose keys all point the same way, so that their mean is as long as they are
+        for p in range(block * pool, block * pool + pool):
+            ks[0][p] = rt(ks[0][block * pool], dtype)
+            cache[bt[0, p // page], 0, :, p % page] = ks[0][p]
+        target = block * pool
+    km, vm = rt(P.block_means(ks[0], pool), dtype), rt(P.block_means(vs[0], pool), dtype)
+    pc, pbt = np.zeros((5, 2, G, page, hd)), np.array([[3, 1, 4, 0]], np.int32)
+    for e in range(L // pool):
+        pc[pbt[0, e // page], 0, :, e % page], pc[pbt[0, e // page], 1, :, e % page] = km[e], vm[e]
+    q = rt(rng.standard_normal((L, H, hd)) * 0.1, dtype)
+    sk = np.zeros(H)
+    if target is not None:
+        q[-1] = rt(np.repeat(ks[0][target], H // G, axis=0) * (12.0 / (ks[0][target] ** 2).sum(-1)).repeat(H // G)[:, None], dtype)
+    else:
+        sk = np.full(H, 12.0)
+    want = _plain_pooled(q, ks[0], vs[0], km, vm, 1.0, window, pool, 50.0, sk)[-1]
+    if which == "window_in":
+        assert np.abs(want - np.repeat(vs[0][target], H // G, axis=0)).max() < 0.15
+    if which == "block_in":
+        assert np.abs(want - np.repeat(vm[block], H // G, axis=0)).max() < 0.15
+    if which == "window_out":
+        assert np.abs(want - np.repeat(vs[0][target], H // G, axis=0)).min() < 2 and np.abs(want).max() < 1.0
+    if which == "sink":
+        assert np.abs(want).max() < 0.01
+    qr = dev(q.reshape(L, H * hd), dtype)
+    extra = dict(sink=dev(sk), cap=50.0, pooled=Kn.Pooled(pool, dev(pc, dtype), i32(pbt)))
+    gen = torch.empty((1, H * hd), dtype=dtype, device=DEV)
+    Kn.attention_rows(qr[-1:], dev(cache, dtype), i32(bt), i32([0]), i32([i]), gen, 1.0, window, page, H, G, hd, **extra)
+    close(host(gen).reshape(H, hd), want, dtype)
+    ws = torch.zeros(Kn.attention_split_scratch(1, H, hd, 3, 0, extra["pooled"]), device=DEV)
+    out = torch.empty_like(gen)
+    Kn.attention_split(qr[-1:], dev(cache, dtype), i32(bt), i32([0]), i32([i]), out, ws, 3, 1.0, window, page, H, G, hd,
+                       exact_weights=True, **extra)
+    close(host(out).reshape(H, hd), want, dtype)
+    if dtype == BF:
+        a = L - 70
+        tiles = list(range(0, 70, Kn.PREFILL_TILE))
+        pre = torch.empty((70, H * hd), dtype=dtype, device=DEV)
+        Kn.attention_prefill(qr[a:].contiguous(), dev(cache, dtype), i32(bt), i32([0, 70]), i32([a]), i32([0] * len(tiles)), i32(tiles), pre,
+                             1.0, window, page, H, G, hd, exact_weights=True, **extra)
+        close(host(pre)[-1].reshape(H, hd), want, dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("G,hd,page,pool", [(2, 16, 16, 5), (1, 64, 8, 24), (3, 112, 64, 1), (2, 128, 16, 16), (1, 6, 4, 3)])
+def test_means_of_the_blocks_that_a_step_completes(G, hd, page, pool, dtype):
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(hd + pool)
+    L, n_pages = 5 * pool + 3, -(-(5 * pool + 3) // page) + 2
+    cache, bt, ks, vs = paged_setup(rng, [L, 2 * pool], page, G, hd, dtype)
+    before = rt(rng.standard_normal((n_pages, 2, G, page, hd)), dtype)
+    pc = dev(before, dtype)
+    pos = list(range(pool + 1, L)) + [2 * pool - 1]                           # a late portion and one decoded token
+    seg = [0] * (L - pool - 1) + [1]
+    slots = rng.permutation(n_pages * page)
+    sm, want = [], before.copy()
+    for i, p in zip(seg, pos):
+        s = int(slots[len(sm)]) if (p + 1) % pool == 0 else -1
+        sm.append(s)
+        if s >= 0:
+            want[s // page, 0, :, s % page] = P.block_means(ks[i], pool)[p // pool]
+            want[s // page, 1, :, s % page] = P.block_means(vs[i], pool)[p // pool]
+    assert sum(s >= 0 for s in sm) == L // pool - (pool + 1) // pool + 1
+    Kn.pool_blocks(dev(cache, dtype), i32(bt), i32(seg), i32(pos), i32(sm), pc, pool, page, G, hd)
+    close(host(pc), want, dtype, tol16=0.005, tol32=1e-6)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dim,hd,page,rot", [(4, 2, 16, 32, 16, 8), (5, 1, 8, 16, 8, 8), (8, 2, 64, 64, 64, 64), (4, 2, 48, 64, 16, 48),
+                                                 (3, 3, 128, 128, 32, 128), (2, 1, 64, 64, 16, 32), (2, 1, 7, 16, 8, 6), (2, 2, 64, 64, 16, 0)])
+def test_norm_behind_the_rotation(H, G, dim, hd, page, rot, dtype):
+    from kappai_b200.config.schema import PartSpec
+    from kappai_b200.ops import kernels as Kn
+    from kappai_b200.parts import make_part
+    from test_parts_gpu import env_for
+    rng = np.random.default_rng(H * hd + rot)
+    n, eps = 37, 1e-2
+    pos = rng.integers(0, 400, n)
+    heads = np.zeros((n, H + 2 * G, hd))
+    heads[:, :H + G, :dim] = rng.standard_normal((n, H + G, dim)) * 0.3
+    heads[:, H + G:] = rng.standard_normal((n, G, hd))
+    heads = rt(heads, dtype)
+    # (YaRN frequencies: their cosines and sines carry a factor, which a norm in front of the rotation would keep)
+    sc = {"factor": 16.0, "original": 64, "fast": 8.0, "slow": 1.0}
+    enc = make_part("position", PartSpec("rope", {"rotary_dim": rot, "theta": 300.0, "scaling": sc}), env_for(dtype)) if rot else None
+    n_pages = -(-n // page) + 1
+    slots = rng.permutation(n_pages * page)[:n]
+    cache = torch.zeros((n_pages, 2, G, page, hd), dtype=dtype, device=DEV)
+    q_out = torch.empty((n, H * hd), dtype=dtype, device=DEV)
+    Kn.qk_norm_rope_kv(dev(heads.reshape(n, -1), dtype), None, None, eps, enc.cos if rot else None, enc.sin if rot else None, rot, False,
+                       i32(pos), i32(slots), q_out, cache, page, H, G, hd, norm_dim=dim, norm_after=True)
+    want = np.concatenate([P.rms(P.rotate(heads[j:j + 1, :H + G, :dim], {"dims": rot, "base": 300.0, "scaling": sc} if rot else None, False, int(pos[j])), eps)
+                           for j in range(n)])
+    got_q = host(q_out).reshape(n, H, hd)
+    close(got_q[:, :, :dim], want[:, :H], dtype)
+    assert np.all(got_q[:, :, dim:] == 0)
+    c = host(cache)
+    close(np.stack([c[s // page, 0, :, s % page, :dim] for s in slots]), want[:, H:], dtype)
+    assert np.array_equal(np.stack([c[s // page, 1, :, s % page] for s in slots]), heads[:, H + G:])
+
+
+# ------------------------------------------------------------------------------------- the latent kernels
+
+def _latent_rows(rng, seq_lens, page, rankp, rotp, dtype):
+    """Cache rows on scrambled pages: (cache, bt, rows of every request)."""
+    blocks = [-(-L // page) for L in seq_lens]
+    perm = rng.permutation(sum(blocks) + 2)
+    cache = rt(rng.standard_normal((sum(blocks) + 2, 1, 1, page, rankp + rotp)) * 5, dtype)
+    bt = np.full((len(seq_lens), max(blocks)), -1, np.int32)
+    rows, o = [], 0
+    for i, (L, nb) in enumerate(zip(seq_lens, blocks)):
+        bt[i, :nb] = perm[o:o + nb]
+        o += nb
+        r = rt(rng.standard_normal((L, rankp + rotp)), dtype)
+        for p in range(L):
+            cache[bt[i, p // page], 0, 0, p % page] = r[p]
+        rows.append(r)
+    return cache, bt, rows
+
+
+LENS = [1, 2, 31, 32, 33, 127, 128, 129, 255, 256, 257, 700]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,rankp,rotp,page", [(3, 32, 16, 16), (1, 16, 16, 8), (4, 128, 64, 64), (16, 112, 32, 32), (17, 208, 16, 16), (20, 272, 16, 64),
+                                               (33, 512, 64, 64), (2, 528, 32, 16), (40, 96, 48, 128), (64, 256, 64, 64), (8, 64, 16, 4)])
+def test_absorbed_pass_over_cached_latents(dtype, H, rankp, rotp, page):
+    """Rows whose contexts end on both sides of tile, chunk and page borders, through the tensor-core form (bfloat16, where it
+    takes the sizes) and the scalar form; one key of the first half stands out so that a lost or doubled key shows."""
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(H + rankp)
+    cache, bt, rows = _latent_rows(rng, LENS, page, rankp, rotp, dtype)
+    W, n = rankp + rotp, len(LENS)
+    qa = rng.standard_normal((n, H, W))
+    for i, L in enumerate(LENS):
+        t = L // 3
+        qa[i, 0] = rows[i][t] * 3.0                                               # head 0 looks at key L // 3
+    qa = rt(qa, dtype)
+    scale = 3.0 / W
+    want = np.stack([P.softmax_with_sink(qa[i] @ rows[i].T * scale, np.ones((H, L), bool)) @ rows[i][:, :rankp] for i, L in enumerate(LENS)])
+    perm = rng.permutation(n)
+    for use_mma in ((True, False) if dtype == BF else (False,)):
+        for n_chunks in (-(-max(LENS) // Kn.LATENT_CHUNK), 9):
+            Kn.USE_MMA_LATENT = use_mma
+            try:
+                ws = torch.full((Kn.latent_split_scratch(n, H, rankp, n_chunks),), float("nan"), device=DEV)
+                u = torch.empty((n, H, rankp), dtype=dtype, device=DEV)
+                Kn.latent_split(dev(qa[perm], dtype), dev(cache, dtype), i32(bt), i32(perm), i32([LENS[i] - 1 for i in perm]), ws, n_chunks, u,
+                                scale, page)
+            finally:
+                Kn.USE_MMA_LATENT = True
+            close(host(u), want[perm], dtype, tol16=0.01)
+    assert Kn.read_status().get("latent", 0) == 0
+
+
+def test_what_lies_behind_a_rows_keys_does_not_matter():
+    """NaN in the page places behind a row's last key and in pages of nobody: the tensor-core forms must not multiply them."""
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(0)
+    H, rankp, rotp, page, lens = 5, 64, 32, 16, [3, 70, 129]
+    cache, bt, rows = _latent_rows(rng, lens, page, rankp, rotp, BF)
+    used = np.zeros(cache.shape[:1] + (page,), bool)
+    for i, L in enumerate(lens):
+        for p in range(L):
+            used[bt[i, p // page], p % page] = True
+    cache[:, 0, 0][~used] = np.nan
+    qa = rt(rng.standard_normal((3, H, rankp + rotp)), BF)
+    u = torch.empty((3, H, rankp), dtype=BF, device=DEV)
+    ws = torch.zeros(Kn.latent_split_scratch(3, H, rankp, 1), device=DEV)
+    Kn.latent_split(dev(qa, BF), dev(cache, BF), i32(bt), i32([0, 1, 2]), i32([L - 1 for L in lens]), ws, 1, u, 0.1, page)
+    want = np.stack([P.softmax_with_sink(qa[i] @ rows[i].T * 0.1, np.ones((H, L), bool)) @ rows[i][:, :rankp] for i, L in enumerate(lens)])
+    close(host(u), want, BF, tol16=0.01)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("M,H,N,K,gate", [(1, 3, 32, 16, False), (8, 16, 512, 64, False), (16, 5, 48, 272, True), (17, 2, 64, 80, True), (33, 4, 16, 128, False),
+                                          (100, 3, 208, 32, True), (64, 1, 96, 96, False)])
+def test_per_head_products(M, H, N, K, gate, dtype):
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(M + N)
+    wide = rt(rng.standard_normal((M, H * (K + 16) + 8)), dtype)                  # heads inside a wider row
+    a = wide[:, :H * (K + 16)].reshape(M, H, K + 16)[:, :, :K]
+    b = rt(rng.standard_normal((H, N, K)) / math.sqrt(K), dtype)
+    g = rt(rng.standard_normal((M, H * N)), dtype)
+    want = np.einsum("mhk,hnk->mhn", a, b)
+    if gate:
+        want = want * P.sigmoid(g.reshape(M, H, N))
+    at = dev(wide, dtype)[:, :H * (K + 16)].unflatten(1, (H, K + 16))[:, :, :K]
+    out = torch.zeros((M, H, N + 16), dtype=dtype, device=DEV)
+    Kn.head_gemm(at, dev(b, dtype), out[:, :, :N], dev(g, dtype).unflatten(1, (H, N)) if gate else None)
+    close(host(out[:, :, :N]), want, dtype)
+    assert not out[:, :, N:].any()
+
+
+@pytest.mark.parametrize("H,dimp,rotp,vdimp,rankp,page", [(3, 32, 16, 16, 32, 16), (4, 64, 64, 64, 128, 64), (2, 128, 64, 128, 112, 32), (5, 16, 16, 80, 48, 8),
+                                                          (2, 192, 64, 160, 64, 16), (1, 96, 32, 256, 32, 64)])
+def test_expanded_pass_over_gathered_latents(H, dimp, rotp, vdimp, rankp, page):
+    """Whole prompts and late portions behind a lead of short segments that another pass takes; the gathered rows too."""
+    from kappai_b200.ops import kernels as Kn
+    rng = np.random.default_rng(H + dimp)
+    lens, q_from = [40, 130, 300, 64, 257, 200], [39, 0, 191, 1, 255, 70]                    # the first segment is a decoded token
+    cache, bt, rows = _latent_rows(rng, lens, page, rankp, rotp, BF)
+    ctx = [0] + lens[1:]
+    base = np.concatenate([[0], np.cumsum(ctx)])
+    got_rows = Kn.latent_gather(dev(cache, BF), i32(bt), i32(base), int(base[-1]), page)
+    all_rows = np.concatenate(rows[1:], 0)
+    assert np.array_equal(host(got_rows), all_rows)
+    ex = rt(rng.standard_normal((len(all_rows), H * (dimp + vdimp))), BF)
+    cu, seg_pos, tile_seg, tile_row0, _, _ = _portions(lens, q_from)
+    q = rt(rng.standard_normal((cu[-1], H * (dimp + rotp) + 8)), BF)
+    scale = 2.0 / math.sqrt(dimp + rotp)
+    out = torch.full((cu[-1], H * vdimp), 7.0, dtype=BF, device=DEV)
+    Kn.latent_prefill(dev(q, BF)[:, :H * (dimp + rotp)], dev(ex, BF), got_rows, rankp, dimp, rotp, vdimp, i32(cu), i32(seg_pos), i32(tile_seg)[1:],
+                      i32(tile_row0)[1:], i32(base), out, scale, H)
+    got = host(out)
+    assert np.all(got[0] == 7.0)
+    for i in range(1, len(lens)):
+        e, r = ex[base[i]:base[i + 1]], rows[i]
+        L, a = lens[i], q_from[i]
+        causal = np.arange(L)[a:, None] >= np.arange(L)[None, :]
+        for h in range(H):
+            qh = q[cu[i]:cu[i + 1], h * (dimp + rotp):(h + 1) * (dimp + rotp)]
+            s = (qh[:, :dimp] @ e[:, h * dimp:(h + 1) * dimp].T + qh[:, dimp:] @ r[:, rankp:].T) * scale
+            v = e[:, H * dimp + h * vdimp:H * dimp + (h + 1) * vdimp]
+            close(got[cu[i]:cu[i + 1], h * vdimp:(h + 1) * vdimp], P.softmax_with_sink(s, causal) @ v, BF, tol16=0.02)
+
+
+# ------------------------------------------------------------------------------------- router, units, residual
+
+@pytest.mark.parametrize("n,E,top,d,groups,scale", [(7, 6, 2, 64, (3, 2), 1.5), (130, 8, 3, 128, (4, 2), 2.5), (3, 3, 3, 36, None, 1.0), (40, 64, 6, 48, (8, 3), 0.7),
+                                                    (9, 40, 6, 50, (5, 1), 1.0), (5, 12, 1, 160, (2, 2), 3.0), (11, 128, 4, 64, (64, 5), 1.0)])
+def test_router_with_groups(n, E, top, d, groups, scale):
+    from kappai_b200.ops import kernels as K
+    rng = np.random.default_rng(n + E)
+    h = rt(rng.normal(0, 1, (n, d)), BF)
+    wr = rt(rng.normal(0, 3 / math.sqrt(d), (E, d)), BF)
+    r = {"experts": E, "top": top, "scale": scale}
+    if groups:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    idx_w, wts_w = P.route(h, wr, r)
+    for form in ("fused", "product"):
+        idx = torch.empty((n, top), dtype=torch.int32, device=DEV)
+        wts = torch.empty((n, top), device=DEV)
+        layout = torch.empty(K.moe_layout_ints(n, E, top), dtype=torch.int32, device=DEV)
+        how = dict(routing="softmax_all", scale=scale, groups=groups, renormalise=True)
+        if form == "fused":
+            if not K.moe_router_ok(d, E):
+                continue
+            K.moe_router(dev(h, BF), dev(wr), None, top, idx, wts, layout, **how)
+        else:
+            K.moe_route(dev(h @ wr.T), top, idx, wts, layout, **how)
+        assert np.array_equal(idx.cpu().numpy(), idx_w), form
+        assert np.abs(wts.cpu().numpy() - wts_w).max() <= 5e-6 * max(1.0, scale), form
+        assert np.array_equal(np.diff(layout.cpu().numpy()[:E + 1]), np.bincount(idx_w.reshape(-1), minlength=E))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,d,ff", [(1, 512, 256), (5, 64, 40), (8, 96, 104), (24, 512, 1024), (64, 160, 72), (130, 512, 1024), (300, 64, 50), (7, 37, 28)])
+def test_square_of_relu_unit(n, d, ff, dtype):
+    """The ungated unit through every product kernel (weight streaming, few rows, tcgen05 and its split form, and the CUDA
+    cores with the activation behind them)."""
+    from kappai_b200.config import PartSpec
+    from kappai_b200.parts import make_part
+    from test_parts_gpu import bind_random, env_for
+    rng = np.random.default_rng(n + d)
+    part = make_part("feed_forward", PartSpec("mlp", {"hidden_size": d, "intermediate_size": ff, "activation": "relu_squared"}), env_for(dtype))
+    w = bind_random(part, rng, dtype)
+    h = rt(rng.normal(0, 1, (n, d)), dtype)
+    res = torch.ones((n, d), device=DEV)
+    part.forward(dev(h, dtype), res, None)
+    close(host(res) - 1.0, P.squared_relu_unit(h, {"up": w["up_proj.weight"], "down": w["down_proj.weight"]}), dtype, tol16=0.02)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n,d", [(5, 36), (40, 64), (3, 512), (70, 4100), (9, 160), (2, 9000), (6, 37)])
+def test_scaled_and_gated_sum_with_the_next_norm(n, d, dtype):
+    from kappai_b200.ops import kernels as K
+    rng = np.random.default_rng(n + d)
+    y, x, ls, wn = (rt(a, torch.float32) for a in (rng.normal(0, 3, (n, d)), rng.normal(0, 1, (n, d)), 1 + 0.2 * rng.standard_normal(d),
+                                                   1 + 0.2 * rng.standard_normal(d)))
+    g = rt(rng.normal(0, 2, (n, d + 8)), dtype)                                    # the gate as columns of a wider row
+    for scaled, gated, with_next in ((True, True, True), (False, True, True), (True, False, True), (True, True, False)):
+        x_want = x + (ls if scaled else 1.0) * (P.sigmoid(g[:, 8:]) if gated else 1.0) * y
+        yt, xt = dev(y), dev(x)
+        h = torch.empty((n, d), dtype=dtype, device=DEV) if with_next else None
+        K.gated_add_norm_rows(yt, dev(g, dtype)[:, 8:] if gated else None, dev(ls) if scaled else None, xt, dev(wn) if with_next else None, 1e-3, h)
+        assert np.abs(host(xt) - x_want).max() <= 1e-5 * max(1.0, np.abs(x_want).max())
+        assert torch.count_nonzero(yt).item() == 0
+        if with_next:
+            close(host(h), P.rms(x_want, 1e-3) * wn, dtype, tol16=0.01)
+
+
+# ------------------------------------------------------------------------------------- the mixers as parts
+
+def _bind(part, rng, dtype):
+    ws, vals = {}, {}
+    for name, spec in part.weight_specs().items():
+        if name.endswith("sink"):
+            a = rng.uniform(-1.0, 3.0, spec.shape)
+        elif spec.role == "norm":
+            a = 1 + 0.2 * rng.standard_normal(spec.shape)
+        elif spec.role == "bias":
+            a = 0.5 * rng.standard_normal(spec.shape)
+        else:
+            a = rng.standard_normal(spec.shape) / math.sqrt(spec.shape[-1])
+        store = dtype if spec.role in ("matrix", "embedding") else torch.float32
+        t = torch.as_tensor(a.astype(np.float32)).to(store)
+        ws[name] = t.cuda()
+        vals[name] = t.double().numpy()
+    part.bind(ws)
+    return vals
+
+
+def _config_of(mixer, width, eps=1e-5):
+    from kappai_b200.config.registry import config_from_dict
+    from kappai_b200.models import ladedra
+    c = {"architecture": "Ladedra", "vocab": 8, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": eps}, "layers": [dict(mixer, mlp=None)]}
+    _, typed = config_from_dict(c)
+    return ladedra._mixer_spec(typed, c["layers"][0], "")
+
+
+def _run_part(mixer, width, plain_fn, dtype, page, tol16, lens=(300, 70, 33, 5), cuts=(1, 64, 31, 3)):
+    """Four requests, each in two steps (all in one batch), with and without the tables of the kernels for portions; once
+    more in another order and cut elsewhere."""
+    from kappai_b200.parts import make_part
+    from test_parts_gpu import env_for, run_mixer_two_steps
+    rng = np.random.default_rng(width + page)
+    spec = _config_of(mixer, width)
+    part = make_part("mixer", spec, env_for(dtype, 1024))
+    w = _bind(part, rng, dtype)
+    local = {spec.rename.get(k, k): v for k, v in w.items()}
+    hs = [rt(rng.normal(0, 1, (L, width)), dtype) for L in lens]
+    for order, cut, tables in (((0, 1, 2, 3), cuts, True), ((3, 0, 2, 1), (5, 130, 2, 33), True), ((0, 1, 2, 3), cuts, False)):
+        outs = run_mixer_two_steps(part, [hs[i] for i in order], [lens[i] for i in order], list(cut), page, dtype, tables=tables)
+        for i, got in zip(order, outs):
+            close(got, plain_fn(hs[i], local), dtype, tol16=tol16)
+    return part
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("cfg,layer,page", [("A", 0, 16), ("A", 2, 8), ("C", 0, 32), ("D", 0, 64), ("D", 2, 16), ("E", 0, 64), ("E", 2, 16), ("F", 1, 8)])
+def test_latent_attention_part(cfg, layer, page, dtype):
+    c = CONFIGS[cfg][0]
+    m = copy.deepcopy(c["layers"][layer])
+    m["mixer"]["scale"] *= 2
+    # (the part's own norm constant, an odd one)
+    _run_part(m, c["width"], lambda h, w: P.latent_attention(h, w, m["mixer"], 1e-5), dtype, page, 0.06)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("cfg,layer,page", [("A", 1, 16), ("A", 3, 8), ("B", 0, 16), ("B", 2, 32), ("C", 1, 16), ("C", 2, 8), ("D", 1, 64), ("D", 3, 16), ("E", 1, 8),
+                                            ("F", 0, 16)])
+def test_parallel_part_of_pooled_attention_and_retention(cfg, layer, page, dtype):
+    c = CONFIGS[cfg][0]
+    m = c["layers"][layer]
+    part = _run_part(m, c["width"], lambda h, w: P.parallel(h, w, m["mixer"], 1e-5), dtype, page, 0.06)
+    assert len(part.joined) == 2 and part.w_in is not None                          # one product for both mixers
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("edge", ["size", "pool", "no_pool", "sink", "cap", "scale"])
+def test_a_mask_one_token_off_shows_in_the_part(edge, dtype):
+    """With scores so peaked that a row sits on one or two keys, the plain mixer with its window or blocks one token
+    longer, without blocks or sink, another cap or other weights of the sum is far away; the part is not."""
+    m = copy.deepcopy(CONFIGS["A"][0]["layers"][1])
+    m["mixer"]["left"].update(scale=0.2 if edge == "sink" else 3.0, softcap=12.0)
+    other = copy.deepcopy(m)
+    lo = other["mixer"]["left"]
+    if edge == "size":
+        lo["mask"]["size"] += 1
+    elif edge == "pool":
+        lo["mask"]["pool"] += 1
+    elif edge == "no_pool":
+        lo["mask"].pop("pool")
+    elif edge == "cap":
+        lo["softcap"] = None
+    elif edge == "scale":
+        other["mixer"]["left_scale"], other["mixer"]["right_scale"] = 1.0, 1.0
+    rng = np.random.default_rng(0)
+    far = []
+
+    def plain(h, w):
+        want = P.parallel(h, w, m["mixer"], 1e-5)
+        w2 = dict(w, **{"left.sink": w["left.sink"] - 30.0}) if edge == "sink" else w
+        d = np.abs(P.parallel(h, w2, other["mixer"], 1e-5) - want).max(1) / np.abs(want).max()
+        far.append(int((d > 0.08).sum()))
+        return want
+
+    _run_part(m, 64, plain, dtype, 16, 0.05)
+    assert max(far) >= 10, far
+
+
+# ------------------------------------------------------------------------------------- whole models
+
+# The smallest gap between two router outcomes that a request's tokens may have (see plain_ladedra.choice_margin): in 16
+# bits a row's router logits (spread: about 3) differ from the plain ones by a hundredth or two, so a closer call may
+# fall the other way, and the token that took another expert stays in the caches behind it.
+MARGIN = 0.05
+_PLAIN = {}
+_REQS = {}
+
+
+def _requests(plain, name, lengths, seed):
+    """Random requests whose router choices all have a margin (four tokens that bring a closer call are drawn again)."""
+    key = (name, tuple(lengths), seed)
+    if key in _REQS:
+        return _REQS[key]
+    rng = np.random.default_rng(seed)
+    reqs = {}
+    for i, n in enumerate(lengths):
+        toks = []
+        while len(toks) < n:
+            new = rng.integers(0, plain.cfg["vocab"], min(4, n - len(toks))).tolist()
+            m = []
+            plain.forward(toks + new, margins=m)
+            if m and min(float(x[len(toks):].min()) for x in m) < MARGIN:
+                continue
+            toks += new
+        reqs[f"r{i}"] = toks
+    _REQS[key] = reqs
+    return reqs
+
+
+def _expect(plain, name, toks):
+    """(the plain logits [T, vocab], every position's smallest router margin [T]) of a sequence."""
+    key = (name, tuple(toks))
+    if key not in _PLAIN:
+        m = []
+        lg = plain.forward(toks, margins=m)
+        _PLAIN[key] = (lg, np.min(m, axis=0) if m else np.full(len(toks), np.inf))
+    return _PLAIN[key]
+
+
+# lengths above every window and its first pooled blocks (A: 20 + 5, B: 33 + 1, C: 7, D: 128 + 24, E: 30 + 8) plus the decoded
+# tail, requests of two or three tokens, and lengths that end on and one behind a page's last token
+LENGTHS = {"A": [150, 3, 64, 49], "B": [130, 41, 2, 97], "C": [77, 20, 101], "D": [290, 65, 201], "E": [180, 64, 140], "F": [90, 33, 2]}
+PROMPTS = {"A": [30, 1, 60, 48], "B": [50, 40, 1, 80], "C": [40, 19, 60], "D": [100, 3, 128], "E": [150, 63, 30], "F": [40, 32, 1]}
+N_LAST = {"A": 110, "B": 60, "C": 40, "D": 170, "E": 70, "F": 30}      # windows and blocks pass over decoded tokens only
+BF16_REL_RMS = 0.04    # a row's 16-bit error (rms over the vocabulary / the row's spread): 95 % of the rows; 99 % twice that
+BF16_BETWEEN_CUTS = 0.06
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,page_size", [("A", 16), ("B", None), ("C", 32), ("D", None), ("E", 8), ("F", 16)])
+def test_every_cut_agrees_with_plain(name, page_size, dtype, lad_dirs, lad_plain, tmp_path):
+    """Whole prompts, the last tokens decoded one by one, portions down to two tokens, and up to four requests mixed in a
+    pool so small that pages and slots go round."""
+    plain = lad_plain[name]
+    reqs = _requests(plain, name, LENGTHS[name], 31)
+    prompt_len = dict(zip(reqs, PROMPTS[name]))
+    expected = {rid: _expect(plain, name, t)[0] for rid, t in reqs.items()}
+    page = page_size or 64
+    rounded = sorted(-(-len(t) // page) * page for t in reqs.values())
+    max_tokens = rounded[-1] + rounded[0] + 2 * page          # the longest request and the shortest fit together, not all
+    tr = R.Trace()
+    R.whole(tr, reqs)
+    R.last_decoded(tr, reqs, n_last=N_LAST[name])
+    R.portions(tr, reqs)
+    b = len(tr.steps)
+    R.mixed(tr, reqs, prompt_len, seed=5, max_live=4, page=page, max_tokens=max_tokens)
+    assert max(len(s["entries"]) for s in tr.steps[b:]) >= 2
+    out = R.run_trace(lad_dirs[name], dtype, tr, str(tmp_path / "out"), max_tokens, page_size)
+    rel = []
+    for st, rows in zip(tr.steps, tr.rows):
+        for j, (rid, pos) in enumerate(rows):
+            e = expected[rid][pos]
+            rel.append((float(np.sqrt(np.mean((out[st["step"]][j] - e) ** 2)) / e.std()), st["step"], rid, pos))
+    r = np.array([x[0] for x in rel])
+    print(f"{name} {dtype}: {len(r)} rows, relative rms error median {np.median(r):.2e}, 95 % {np.quantile(r, 0.95):.2e}, worst {r.max():.2e}")
+    if dtype == "bfloat16":
+        assert np.quantile(r, 0.95) <= BF16_REL_RMS and np.quantile(r, 0.99) <= 2 * BF16_REL_RMS, max(rel)
+        apart = []
+        for place, rows in R.rows_by_place(tr, out).items():
+            e = expected[place[0]][place[1]]
+            apart.append(max(float(np.sqrt(np.mean((x - rows[0]) ** 2)) / e.std()) for x in rows[1:]))
+        assert np.quantile(apart, 0.99) <= BF16_BETWEEN_CUTS, max(apart)
+    else:
+        assert r.max() <= 1e-4, max(rel)
+        for place, rows in R.rows_by_place(tr, out).items():
+            assert len(rows) >= 2, place
+            for x in rows[1:]:
+                assert np.array_equal(rows[0], x), f"{name}: float32 logits of {place} differ between cuts"
+    stats = R.cache_stats(str(tmp_path / "out"))
+    assert stats and all(g["reused"] > 0 for g in stats.values()), stats
+
+
+@pytest.mark.parametrize("name", ["A", "B", "C", "D", "E", "F"])
+def test_residual_after_every_layer(name, lad_dirs, lad_plain):
+    from kappai_b200 import ModelRunner, StepEntry
+    plain = lad_plain[name]
+    toks = _requests(plain, name, [57], 8)["r0"]
+    want = []
+    plain.forward(toks, want)
+    r = ModelRunner(lad_dirs[name], dtype="float32", max_tokens=256, max_requests=2, cuda_graphs=False)
+    got = []
+    r.observer = lambda i, x: got.append(x.detach().cpu().numpy().copy())
+    r.step([StepEntry("a", toks, [0])])
+    assert len(got) == len(want) + 1
+    for i, w in enumerate(want):
+        assert np.abs(got[i + 1] - w).max() < 1e-4 * max(1.0, np.abs(w).max()), (i, np.abs(got[i + 1] - w).max())
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_batched_requests_equal_each_alone_and_captured_steps_equal_eager(dtype, lad_dirs, lad_plain):
+    """Unequal requests decode together for many steps (the steps are captured into CUDA graphs on the way); every row
+    equals the row of the request run alone without graphs."""
+    from kappai_b200 import ModelRunner, StepEntry
+    n_dec = 40
+    reqs = _requests(lad_plain["A"], "A", [61 + n_dec, 9 + n_dec, 30 + n_dec], 12)
+
+    def run(runner, group):
+        out = {rid: [] for rid in group}
+        lg = runner.step([StepEntry(rid, reqs[rid][:len(reqs[rid]) - n_dec], [len(reqs[rid]) - n_dec - 1]) for rid in group])
+        for j, rid in enumerate(group):
+            out[rid].append(lg[j].cpu().numpy().copy())
+        for s in range(n_dec):
+            lg = runner.step([StepEntry(rid, [reqs[rid][len(reqs[rid]) - n_dec + s]], [0]) for rid in group])
+            for j, rid in enumerate(group):
+                out[rid].append(lg[j].cpu().numpy().copy())
+        for rid in group:
+            runner.end(rid)
+        return out
+
+    r1 = ModelRunner(lad_dirs["A"], dtype=dtype, max_tokens=512, max_requests=4, page_size=16)
+    together = run(r1, list(reqs))
+    assert r1.model.graph_safe and r1.graphs is not None and len(r1.graphs.graphs) >= 1
+    alone_runner = ModelRunner(lad_dirs["A"], dtype=dtype, max_tokens=512, max_requests=4, page_size=16, cuda_graphs=False)
+    for rid in reqs:
+        for a, b in zip(run(alone_runner, [rid])[rid], together[rid]):
+            if dtype == "float32":
+                assert np.array_equal(a, b)
+            else:
+                assert np.abs(a - b).max() <= 2 * tol_for(dtype, a)
+
+
+@pytest.mark.parametrize("name", ["A", "B", "D"])
+def test_a_slot_and_pages_used_again_start_empty(name, lad_dirs):
+    """One slot and just enough pages for one request: a second request takes the slot and the pages of the first (also
+    the pages that held its pooled blocks) and gives what it gives alone."""
+    from kappai_b200 import ModelRunner, StepEntry
+    rng = np.random.default_rng(2)
+    V = CONFIGS[name][0]["vocab"]
+    a, b = rng.integers(0, V, 60).tolist(), rng.integers(0, V, 45).tolist()
+    mk = lambda: ModelRunner(lad_dirs[name], dtype="float32", max_tokens=64, max_requests=1, page_size=16, cuda_graphs=False)
+    r = mk()
+    r.step([StepEntry("a", a, [len(a) - 1])])
+    r.end("a")
+    second = r.step([StepEntry("b", b[:7], [6])]).cpu().numpy().copy()
+    second2 = r.step([StepEntry("b", b[7:], [len(b) - 8])]).cpu().numpy().copy()
+    r.end("b")
+    fresh = mk()
+    assert np.array_equal(second, fresh.step([StepEntry("x", b[:7], [6])]).cpu().numpy())
+    assert np.array_equal(second2, fresh.step([StepEntry("x", b[7:], [len(b) - 8])]).cpu().numpy())
+
+
+def test_token_pages_go_back_while_pooled_entries_stay(lad_dirs):
+    """Model A: a window of 20 with blocks of 5.  After 150 tokens the token group holds the window's pages only, the pooled
+    group an entry for each of 30 blocks, and the latent group one row a token."""
+    from kappai_b200 import ModelRunner, StepEntry
+    from kappai_b200.cache.manager import RELEASED
+    r = ModelRunner(lad_dirs["A"], dtype="float32", max_tokens=256, max_requests=2, page_size=8, cuda_graphs=False)
+    toks = np.random.default_rng(4).integers(0, CONFIGS["A"][0]["vocab"], 150).tolist()
+    r.step([StepEntry("a", toks[:100], [])])
+    r.step([StepEntry("a", toks[100:], [])])
+    pools = r.cache.pools
+    token = [gk for gk in pools if gk[1:4] == (2, 32, 20)][0]
+    pooled = [gk for gk in pools if ("every", 5) in gk][0]
+    t = r.cache.block_table("a", token)
+    assert sum(p != RELEASED for p in t) == 3 and all(p == RELEASED for p in t[:(150 - 20 + 1) // 8])
+    t = r.cache.block_table("a", pooled)
+    assert len(t) == -(-30 // 8) and all(p != RELEASED for p in t)
+    assert r.storage.bytes_per_token([gk for gk in pools if ("planes", 1) in gk][0]) == 4 * (32 + 16)
+    assert pools[pooled].n_pages < pools[token].n_pages
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "B", "D"])
+def test_greedy_generation_through_the_engine(name, dtype, lad_dirs, lad_plain):
+    from kappai_b200 import Engine, EngineArgs, SamplingParams
+    plain = lad_plain[name]
+    prompts = list(_requests(plain, name, [5, 26, 60], 21).values())
+    n_new = 50
+    eng = Engine(EngineArgs(model=lad_dirs[name], dtype=dtype, max_batch=4, max_step_tokens=16, page_size=16, kv_tokens=1024))
+    outs = eng.generate(prompts, SamplingParams(temperature=0.0, n_predict=n_new))
+    assert [len(o) for o in outs] == [n_new] * len(prompts)
+    for p, o in zip(prompts, outs):
+        lg, margin = _expect(plain, name, p + o)
+        lg, margin = lg[len(p) - 1:-1], margin[len(p) - 1:-1]
+        for j, t in enumerate(o):
+            if dtype == "bfloat16" and margin[:j + 1].min() < MARGIN:
+                break                      # a router call too close for 16 bits: from here on the sequences may part
+            best = int(np.argmax(lg[j]))
+            assert t == best or lg[j][best] - lg[j][t] <= 4 * tol_for(dtype, lg[j]), (j, t, best)
+    assert eng.runner.cache.slots.n_free == 4 and all(p.n_free == p.n_pages for p in eng.runner.cache.pools.values())
+
+
+def test_long_decoding_past_many_blocks(lad_dirs, lad_plain):
+    """Three hundred tokens decoded one by one from a short prompt, in a pool without room to spare, equal the whole sequence."""
+    from kappai_b200 import ModelRunner, StepEntry
+    plain = lad_plain["A"]
+    toks = _requests(plain, "A", [312], 5)["r0"]
+    want = plain.forward(toks)
+    r = ModelRunner(lad_dirs["A"], dtype="float32", max_tokens=320, max_requests=1, page_size=16)
+    got = [r.step([StepEntry("a", toks[:12], list(range(12)))]).cpu().numpy().copy()]
+    got += [r.step([StepEntry("a", [t], [0])]).cpu().numpy().copy() for t in toks[12:]]
+    got = np.concatenate(got, 0)
+    err = np.sqrt(((got - want) ** 2).mean(1)) / want.std(1)
+    assert err.max() < 1e-4, (int(err.argmax()), err.max())
+
+
+def test_command_line_and_random_weights(lad_dirs, lad_plain, tmp_path):
+    """The command line runs the design like any other: greedy tokens equal the plain model's, --time names the design's
+    kernels, and --random-weights writes a loadable model folder from a Ladedra config.json."""
+    import json
+    import os
+    import subprocess
+    import sys
+    plain = lad_plain["A"]
+    prompt = _requests(plain, "A", [30], 77)["r0"]
+    cmd = [sys.executable, "-m", "kappai_b200.cli", "-m", lad_dirs["A"], "-p", ",".join(map(str, prompt)), "-n", "12", "-t", "0",
+           "--fp32", "--time"]
+    p = subprocess.run(cmd, cwd=R.ROOT, capture_output=True, text=True, timeout=600)
+    assert p.returncode == 0, p.stderr[-2000:]
+    out = [int(t) for t in p.stdout.split()]
+    assert len(out) == 12
+    lg = plain.forward(prompt + out)[len(prompt) - 1:-1]
+    for j, t in enumerate(out):
+        best = int(np.argmax(lg[j]))
+        assert t == best or lg[j][best] - lg[j][t] <= 1e-4, (j, t, best)
+    for name in ("gated_add_norm_rows", "latent_prep", "latent_split", "head_gemm", "pool_blocks", "qk_norm_rope_kv", "lightning_scan", "moe_router"):
+        assert name in p.stderr, (name, p.stderr[-3000:])
+    cfgp = tmp_path / "c.json"
+    cfgp.write_text(json.dumps(CONFIGS["B"][0]))
+    made = tmp_path / "rw"
+    cmd = [os.path.join(R.ROOT, "bin", "kappai-cli"), "--random-weights", str(cfgp), "-s", "5", "-m", str(made), "-t", "0", "-n", "5",
+           "1 2 3"]
+    p = subprocess.run(cmd, cwd=str(tmp_path), capture_output=True, text=True, timeout=600)
+    assert p.returncode == 0, p.stderr[-2000:]
+    assert len(p.stdout.split()) == 5 and os.path.isfile(made / "model.safetensors")

@@ -50,18 +50,20 @@ class Batch:
         from kappai_b200.cache import CacheManager, PagedKVSpec, leaf_specs
         from kappai_b200.cache.storage import CacheStorage
         self.lens, self.cuts, self.page = lens, cuts, page
+        self.builders = {}                          # step tables key -> the part that builds the tables
         gks = {s.group_key: s for spec in specs for s in leaf_specs(spec) if isinstance(s, PagedKVSpec)}
         n_pages = sum(-(-L // page) for L in lens) + 2
         self.storage = CacheStorage(specs, [None] * len(specs), {g: n_pages for g in gks}, page, len(lens) + 1,
                                     dtype, torch.device("cuda:0"))
-        self.cache = CacheManager({g: (n_pages, page, s.window, s.block, s.keep_first if s.window is not None else 0)
+        self.cache = CacheManager({g: (n_pages, page, s.window, s.block, s.keep_first if s.window is not None else 0, s.every)
                                    for g, s in gks.items()}, len(lens) + 1)
         self.groups = {g: page for g in gks}
+        self.every = {g: s.every for g, s in gks.items()}
         for i in range(len(lens)):
             self.cache.admit(i)
 
     def context(self, step):
-        from kappai_b200.engine.batch import Segment, build_step_context
+        from kappai_b200.engine.batch import Segment, lay_out_step, upload_step
         segs = []
         for i, (L, c) in enumerate(zip(self.lens, self.cuts)):
             a, b = (0, c) if step == 0 else (c, L)
@@ -72,18 +74,23 @@ class Batch:
             segs.append(Segment(i, [0] * (b - a), a, [], rc.slot,
                                 {g: self.cache.block_table(i, g) for g in self.groups},
                                 {g: self.cache.token_slots(i, g, a, b - a) for g in self.groups}))
-        ctx = build_step_context(segs, self.groups, torch.device("cuda:0"), 10, 4096)
+        ctx = upload_step(lay_out_step(segs, self.groups, 10, 4096, self.builders, every=self.every), torch.device("cuda:0"))
         rows = [(s.req, s.pos_start, len(s.tokens)) for s in segs]
         for s in segs:
             self.cache.advance(s.req, s.pos_start + len(s.tokens))
         return ctx, rows
 
 
-def run_mixer_two_steps(mixer, h_all, lens, cuts, page, dtype):
+def run_mixer_two_steps(mixer, h_all, lens, cuts, page, dtype, tables=False):
     """Run each request's rows 0..cut in step 0 and cut..len in step 1 (all requests in one batch);
-    returns the mixer's output (what it adds to a zero residual) per request."""
+    returns the mixer's output (what it adds to a zero residual) per request.  ``tables``: with the step tables
+    that the mixer's kernels for portions read (without them a mixer takes its kernels for single rows)."""
     d = h_all[0].shape[1]
     b = Batch([mixer.cache_spec()], lens, cuts, page, dtype)
+    if tables:
+        for m in (mixer,) + tuple(mixer.inner_parts):
+            if m.step_tables_key is not None:
+                b.builders[m.step_tables_key] = m
     outs = [np.zeros((L, d)) for L in lens]
     for step in (0, 1):
         ctx, rows = b.context(step)
