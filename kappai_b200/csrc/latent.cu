@@ -1,32 +1,43 @@
 // Attention over a cache of latents: keys and values are expanded from one low-rank latent a token, k_h = Wuk_h c and
 // v_h = Wuv_h c, beside a rotated key part that all heads share, and only the latent c and that part are kept.
 //
-//   cache row of a token: [ c (rank, normed; zeros up to rankp) | rotated key part (rot_dim; zeros up to rotp) ]
+//   cache row of a token: [ c (rank, normed; zeros up to rankp) | rotated key part (rot_dim; zeros up to rotp) | zeros up to W ]
 //   s_h(t) = (q_h . Wuk_h c_t + qr_h . kr_t) scale ,  o_h = sum_t softmax(s_h)_t Wuv_h c_t        (causal)
 //
-// rankp and rotp are rank and rot_dim rounded up to 16; a row has W = rankp + rotp elements and lies in pages
+// rankp and rotp are rank and rot_dim rounded up to 16, the row's W = rankp + rotp to 64; rows lie in pages
 // [page][1][1][page_size][W].  Two ways of computing the same:
 //
 //  * absorbed (decoded tokens, short portions, the 32-bit mode): the expanding matrices move to the other side of the
 //    sums, q'_h = Wuk_h^T q_h once a row, s_h(t) = ([q'_h | qr_h] . row_t) scale, u_h = sum_t softmax(s_h)_t c_t and
 //    o_h = Wuv_h u_h.  All heads read the same rows, so a cache row is fetched once for up to 16 heads.  Per-head
-//    products (head_gemm), a pass over chunks of 256 keys (latent_split: bfloat16 on the tensor cores, or scalar) that
+//    products (head_gemm), a pass over chunks of keys (latent_split: bfloat16 on the tcgen05 tensor cores, or scalar) that
 //    leaves each chunk's maximum, sum and unnormalised latent, and a merge in chunk order.
 //  * expanded (prompt portions): the latents of the request's whole context are gathered from its pages, one product
 //    expands them, and latent_prefill runs tiles of 64 query rows over the expanded rows.
 //
-// The softmax statistics are float32; its weights enter the products whole, as three bfloat16 parts.  Chunks lie at
-// multiples of 256 of the absolute key index and tiles at multiples of 32 or 64, so the order of a row's sums does not
-// depend on how its prompt was cut or on what else is in the batch.
+// The softmax statistics are float32; its weights enter the products whole, as three bfloat16 parts.  The
+// scalar form's chunks lie at multiples of 256 keys, so in the 32-bit mode the order of a row's sums does not depend on how its
+// prompt was cut or on what else is in the batch; the tensor-core form makes its chunks as long as the step's rows allow
+// (a few rows of short contexts still fill the device, and long ones are not cut finer than that needs), which
+// moves the order of the float32 sums, nothing else.
 #include "mma.cuh"
+#include "tcgen05.cuh"
 
-#define LA_CHUNK 256               // keys a chunk of the absorbed pass
-#define LA_TILE 32                 // keys a tile of its tensor-core form
-#define LA_MAX_STAGES 4
+#define LA_CHUNK 256               // keys a chunk of the absorbed pass's scalar form
 #define LA_SCALAR_HEADS 4          // heads a CTA of its scalar form
 #define LP_TILE 64                 // query rows and keys a tile of the expanded form
 
 KP_STATUS_WORD(g_latent_status, latent)          // 0 ok; 1: a bounded wait gave up
+
+// Keys a chunk of the tensor-core form: so many tiles that n_chunks chunks reach the longest of the step's rows.  (Every
+// CTA works it out from the rows' positions, one warp at a time; n_chunks is the host's choice.)
+#define LT_TILE 64
+__device__ __forceinline__ int lt_chunk_keys(const int* __restrict__ positions, int n_rows, int n_chunks) {
+    int hi = 0;
+    for (int i = threadIdx.x & 31; i < n_rows; i += 32) hi = max(hi, positions[i]);
+    hi = __reduce_max_sync(0xffffffffu, hi);
+    return (hi / LT_TILE + n_chunks) / n_chunks * LT_TILE;
+}
 
 // ------------------------------------------------------------------------------------------------ preparation
 // One block a row of the input product p = [.. q: H heads of (dimp unrotated | rotp rotated) .. | latent (rankp) and key
@@ -37,12 +48,12 @@ KP_STATUS_WORD(g_latent_status, latent)          // 0 ok; 1: a bounded wait gave
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(T* __restrict__ p, int ld, int q_col, int c_col, int H, int dimp, int rotp, int rank, int rankp,
-                   const float* __restrict__ w, float eps, const float* __restrict__ cos_tab, const float* __restrict__ sin_tab,
+                   int W, const float* __restrict__ w, float eps, const float* __restrict__ cos_tab, const float* __restrict__ sin_tab,
                    int rot, int interleaved, const int* __restrict__ positions, const int* __restrict__ slot_map,
                    T* __restrict__ cache, int page_size, T* __restrict__ qa, int n_absorbed) {
     kp_pdl_begin_early_if(gridDim.x > 1);
     __shared__ float red[32];
-    const int row = blockIdx.x, tid = threadIdx.x, W = rankp + rotp;
+    const int row = blockIdx.x, tid = threadIdx.x;
     T* pr = p + (size_t)row * ld;
     const T* c = pr + c_col;
     const int pos = positions[row];
@@ -68,6 +79,7 @@ latent_prep_kernel(T* __restrict__ p, int ld, int q_col, int c_col, int H, int d
             }
             dst[rankp + i] = from_f32<T>(v);
         }
+        for (int i = rankp + rotp + tid; i < W; i += 256) dst[i] = from_f32<T>(0.f);
     }
     const int Dq = dimp + rotp;
     for (int i = tid; i < H * half; i += 256) {
@@ -84,11 +96,11 @@ latent_prep_kernel(T* __restrict__ p, int ld, int q_col, int c_col, int H, int d
             d[ib] = rb;
         }
     }
-    if (row < n_absorbed && rotp > 2 * half) {                     // what is not rotated passes on as it is
-        const int rest = rotp - 2 * half;
+    if (row < n_absorbed && W - rankp > 2 * half) {                // what is not rotated passes on as it is, and zeros behind
+        const int rest = W - rankp - 2 * half;
         for (int i = tid; i < H * rest; i += 256) {
             const int h = i / rest, j = 2 * half + i % rest;
-            qa[((size_t)row * H + h) * W + rankp + j] = pr[q_col + (size_t)h * Dq + dimp + j];
+            qa[((size_t)row * H + h) * W + rankp + j] = j < rotp ? pr[q_col + (size_t)h * Dq + dimp + j] : from_f32<T>(0.f);
         }
     }
 }
@@ -212,166 +224,331 @@ head_gemm_simt_kernel(const HeadGemmArgs p) {
 }
 
 // --------------------------------------------------------------------------------- absorbed pass, tensor cores
-// One CTA: one chunk of 256 keys, up to 16 heads, one row.  Tiles of 32 cache rows come by bulk copies (one a key,
-// issued by the lanes of warp 0) into a ring; S = Q K^T by all 8 warps (8 keys x half of W each), the softmax of the
-// 16 x 32 scores by half-warps (a head each), then every warp sums its own columns of the latent, P V with V = the
-// latent columns of the same tile.  PT: pairs of 8-column tiles a warp (rank <= 128 PT).
-template <int PT>
-__global__ void __launch_bounds__(256, 2)
-latent_split_mma_kernel(const bf16* __restrict__ qa, const bf16* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
-                        const int* __restrict__ row_seg, const int* __restrict__ positions, float* __restrict__ part_acc,
-                        float* __restrict__ part_ml, int n_chunks, float scale, int page_size, int H, int rankp, int W, int n_stages) {
-    kp_pdl_begin_early_if(gridDim.z > 1);
-    extern __shared__ __align__(128) unsigned char la_smem[];
-    const int pitch = W + 8;                                       // (an odd number of 16-byte pieces: ldmatrix rows do not collide)
-    bf16* Ks = reinterpret_cast<bf16*>(la_smem);                   // [n_stages][LA_TILE][pitch]
-    bf16* Qs = Ks + (size_t)n_stages * LA_TILE * pitch;            // [16][pitch]
-    bf16* Ps = Qs + (size_t)16 * pitch;                            // [3][16][40]
-    float* Sp = reinterpret_cast<float*>(Ps + 3 * 16 * 40);        // [2][16][36]
-    float* corr_s = Sp + 2 * 16 * 36;                              // [16]
-    uint64_t* bars = reinterpret_cast<uint64_t*>(corr_s + 16);     // [n_stages]
+// One CTA: one chunk of one row's keys, NH (16 or 32) heads, on the 5th-generation tensor cores.  The keys stand where
+// the tensor core wants many rows and the heads where it can do with few, so nothing is padded but the head count:
+//
+//   S^T = rows Q'^T    [keys x heads]: 64 cache rows a tile (K-major, as TMA brings them: boxes of 64 columns, 128-byte
+//                      swizzle) times the absorbed queries, in MMAs of 64 x NH x 16.  Such an MMA leaves its rows in the lower
+//                      half of every lane quarter; the odd boxes' sums go to the upper half, so that two chains run side
+//                      by side and every lane has a part in what follows;
+//   U^T = rows^T P^T   [latent columns x heads]: the same tile in shared memory, read as the MN-major operand in blocks of
+//                      128 columns, times the softmax weights as 3 NH rows of bfloat16: the three parts of every
+//                      head's float32 weights side by side, so that they enter whole for a few more columns.
+//
+// Roles by warp: 0 TMA (the queries once, a ring of tiles), 1 tensor memory and MMA of S, 2 - 9 two groups of four warps, a
+// lane quarter each, 10 the MMA of U.  In the softmax of a tile a group has half of the heads, a lane 16 q + i of a quarter and its partner
+// 16 lanes on the same key, half of those heads each; then all eight warps add U^T's columns (blocks shared among the
+// groups) to their registers, rescaled by the heads' change of maximum, so that no pass over tensor memory rescales anything.  S and the weights are double-buffered:
+// a tile's softmax runs while the tile before it is multiplied.
+// Every wait is bounded; one that gives up sets the status word and an abort flag, and the CTA frees its tensor memory
+// and returns.
+#define LT_BOX_BYTES (LT_TILE * 128)                               // 64 rows x 64 columns of bfloat16
+#define LT_MAX_STAGES 4
+#define LT_THREADS 352
 
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    const int chunk = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
-    const int k_hi = positions[row], c0 = chunk * LA_CHUNK;
-    if (c0 > k_hi) return;
-    const int n_keys = min(k_hi + 1 - c0, LA_CHUNK), n_tiles = (n_keys + LA_TILE - 1) / LA_TILE;
-    const int* bt = block_table + (size_t)row_seg[row] * max_blocks;
-    const int nh = min(16, H - h0);
+struct LatentSplitArgs {
+    const int* block_table; const int* row_seg; const int* positions;
+    float* part_acc; float* part_ml;
+    int max_blocks, n_chunks, page_size, H, rankp, n_box, n_stages;
+    float scale;
+};
 
-    if (tid == 0) {
-        for (int s = 0; s < n_stages; s++) kp_mbar_init(&bars[s], 1);
+__device__ __forceinline__ float la_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+template <int NH>
+__global__ void __launch_bounds__(LT_THREADS, 1)
+latent_split_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmQ, const LatentSplitArgs p) {
+    constexpr int HH = NH / 2, HQ = NH / 4;                        // heads a group has in the softmax, and a thread
+    constexpr int NP = 3 * NH;                                     // columns of U^T in tensor memory, a block
+    constexpr uint32_t TMEM_COLS = NH == 16 ? 256 : 512;           // S twice, four blocks of U^T
+    extern __shared__ unsigned char lt_raw[];
+    unsigned char* sm = reinterpret_cast<unsigned char*>(((uintptr_t)lt_raw + 1023) & ~(uintptr_t)1023);
+    const uint32_t tile_bytes = (uint32_t)p.n_box * LT_BOX_BYTES;
+    unsigned char* Ks = sm;                                        // [n_stages][n_box][64 rows x 128 bytes]
+    unsigned char* Qs = Ks + (size_t)p.n_stages * tile_bytes;      // [n_box][NH rows x 128 bytes]
+    unsigned char* Ps = Qs + (size_t)p.n_box * NH * 128;           // [2][NP rows x 128 bytes]
+    float* max_s = reinterpret_cast<float*>(Ps + 2 * NP * 128);    // [2 tiles][NH][4 quarters]
+    float* sum_s = max_s + 8 * NH;                                 // [NH][4 quarters]
+    float* corr_s = sum_s + 4 * NH;                                // [4 tiles][NH]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(corr_s + 4 * NH);
+    uint64_t* q_full = bars;
+    uint64_t* k_full = bars + 1;                                   // [LT_MAX_STAGES]
+    uint64_t* k_empty = k_full + LT_MAX_STAGES;                    // [LT_MAX_STAGES]
+    uint64_t* s_full = k_empty + LT_MAX_STAGES;                    // [2]
+    uint64_t* p_full = s_full + 2;                                 // [2]
+    uint64_t* u_full = p_full + 2;
+    uint64_t* u_empty = u_full + 1;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(u_empty + 1);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (threadIdx.x == 0) {
+        kp_mbar_init(q_full, 1);
+        for (int s = 0; s < LT_MAX_STAGES; s++) { kp_mbar_init(&k_full[s], 1); kp_mbar_init(&k_empty[s], 1); }
+        for (int b = 0; b < 2; b++) { kp_mbar_init(&s_full[b], 1); kp_mbar_init(&p_full[b], 256); }
+        kp_mbar_init(u_full, 1);
+        kp_mbar_init(u_empty, 8);
+        *abort_flag = 0;
         kp_mbar_init_fence();
     }
+    kp_pdl_begin_early_if(gridDim.z > 1);
+    // (the whole CTA leaves here or stays: tensor memory is taken only by one that stays)
+    const int chunk = blockIdx.x, h0 = blockIdx.y * NH, row = blockIdx.z;
+    const int k_hi = p.positions[row], seg = p.row_seg[row], ck = lt_chunk_keys(p.positions, gridDim.z, p.n_chunks), c0 = chunk * ck;
+    if (c0 > k_hi) return;
+    const int n_keys = min(k_hi + 1 - c0, ck), n_tiles = (n_keys + LT_TILE - 1) / LT_TILE;
+    if (warp == 1) kp_tmem_alloc(tmem_slot, TMEM_COLS);
+    kp_tc_fence_before();
     __syncthreads();
-    auto load = [&](int it) {                                      // warp 0: tile it into its stage
-        const int s = it % n_stages, r = it * LA_TILE + lane;
-        if (lane == 0) kp_mbar_expect_tx(&bars[s], (uint32_t)min(LA_TILE, n_keys - it * LA_TILE) * W * 2);
-        __syncwarp();
-        if (r < n_keys) {
-            const int key = c0 + r;
-            kp_bulk_g2s(Ks + ((size_t)s * LA_TILE + lane) * pitch,
-                        cache + ((size_t)bt[key / page_size] * page_size + key % page_size) * W, (uint32_t)W * 2, &bars[s]);
-        }
-    };
-    if (warp == 0)
-        for (int it = 0; it < min(n_stages, n_tiles); it++) load(it);
-    {
-        const int per = W >> 3;                                    // 16-byte pieces a row
-        const bf16* src = qa + ((size_t)row * H + h0) * W;
-        for (int i = tid; i < 16 * per; i += 256) {
-            const int r = i / per, c = (i - r * per) * 8;
-            *reinterpret_cast<uint4*>(Qs + (size_t)r * pitch + c) =
-                r < nh ? *reinterpret_cast<const uint4*>(src + (size_t)r * W + c) : make_uint4(0, 0, 0, 0);
-        }
-    }
-    float o[PT][2][4];
-#pragma unroll
-    for (int j = 0; j < PT; j++)
-#pragma unroll
-        for (int i = 0; i < 4; i++) o[j][0][i] = o[j][1][i] = 0.f;
-    float m_run = -INFINITY, l_run = 0.f;                          // of head tid / 16, the same in its 16 lanes
-    const int KS = W >> 4, nt = warp & 3, kh = warp >> 2;
-    const int ks_lo = kh ? KS / 2 : 0, ks_hi = kh ? KS : KS / 2;
-    __syncthreads();                                               // Q is there
+    kp_tc_fence_after();
+    const uint32_t tmem_s = *tmem_slot, tmem_u = tmem_s + 2 * NH;
+    const int n_blk = (p.rankp + 127) / 128;
 
-    bool ok = true;
-    for (int it = 0; it < n_tiles; it++) {
-        const int s = it % n_stages;
-        const bf16* Kt = Ks + (size_t)s * LA_TILE * pitch;
-        const int valid = min(LA_TILE, n_keys - it * LA_TILE);
-        ok = kp_mbar_wait_bounded(&bars[s], (it / n_stages) & 1);
-        if (valid < LA_TILE) {                                     // the chunk's last tile: rows that no copy filled
-            const int per = W >> 3;
-            for (int i = tid; i < (LA_TILE - valid) * per; i += 256) {
-                const int r = i / per;
-                *reinterpret_cast<uint4*>(const_cast<bf16*>(Kt) + (size_t)(valid + r) * pitch + (i - r * per) * 8) = make_uint4(0, 0, 0, 0);
-            }
-            __syncthreads();
-        }
-        float sa[4] = {0.f, 0.f, 0.f, 0.f}, sb[4] = {0.f, 0.f, 0.f, 0.f};
-        for (int ks = ks_lo; ks < ks_hi; ks++) {
-            uint32_t a[4], b[2];
-            ldmatrix_x4(a, Qs + (size_t)(lane & 15) * pitch + ks * 16 + (lane >> 4) * 8);
-            ldmatrix_x2(b, Kt + (size_t)(nt * 8 + (lane & 7)) * pitch + ks * 16 + ((lane >> 3) & 1) * 8);
-            if ((ks - ks_lo) & 1) mma_bf16(sb, a[0], a[1], a[2], a[3], b[0], b[1]);
-            else mma_bf16(sa, a[0], a[1], a[2], a[3], b[0], b[1]);
-        }
-        {
-            float* d = Sp + (size_t)kh * 16 * 36 + nt * 8 + 2 * t;
-            *reinterpret_cast<float2*>(d + g * 36) = make_float2(sa[0] + sb[0], sa[1] + sb[1]);
-            *reinterpret_cast<float2*>(d + (g + 8) * 36) = make_float2(sa[2] + sb[2], sa[3] + sb[3]);
-        }
-        if (!__syncthreads_and(ok)) { ok = false; break; }         // (all threads leave together)
-        {
-            const int hr = tid >> 4, kk = (tid & 15) * 2;
-            const float2 x = *reinterpret_cast<const float2*>(Sp + hr * 36 + kk), y = *reinterpret_cast<const float2*>(Sp + 16 * 36 + hr * 36 + kk);
-            float p0 = kk < valid ? (x.x + y.x) * scale : -INFINITY, p1 = kk + 1 < valid ? (x.y + y.y) * scale : -INFINITY;
-            float mx = fmaxf(p0, p1);
-#pragma unroll
-            for (int d = 8; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-            const float m_new = fmaxf(m_run, mx);                  // (finite: the first key of every tile is the row's)
-            const float corr = m_run == -INFINITY ? 0.f : expf(m_run - m_new);
-            p0 = kk < valid ? expf(p0 - m_new) : 0.f;
-            p1 = kk + 1 < valid ? expf(p1 - m_new) : 0.f;
-            float sum = p0 + p1;
-#pragma unroll
-            for (int d = 8; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
-            l_run = l_run * corr + sum;
-            m_run = m_new;
-#pragma unroll
-            for (int part = 0; part < 3; part++)
-                *reinterpret_cast<uint32_t*>(Ps + (size_t)(part * 16 + hr) * 40 + kk) = pack_bf16_part(p0, p1);
-            if ((tid & 15) == 0) corr_s[hr] = corr;
-        }
-        __syncthreads();
-        const float ca = corr_s[g], cb = corr_s[g + 8];
-        uint32_t pf[3][2][4];
-#pragma unroll
-        for (int part = 0; part < 3; part++)
-#pragma unroll
-            for (int ks = 0; ks < 2; ks++) ldmatrix_x4(pf[part][ks], Ps + (size_t)(part * 16 + (lane & 15)) * 40 + ks * 16 + (lane >> 4) * 8);
-#pragma unroll
-        for (int j = 0; j < PT; j++) {
-            const int c = (warp + 8 * j) * 16;                     // this warp's j-th stretch of 16 columns
-            if (c < rankp) {
-#pragma unroll
-                for (int i = 0; i < 2; i++) { o[j][i][0] *= ca; o[j][i][1] *= ca; o[j][i][2] *= cb; o[j][i][3] *= cb; }
-#pragma unroll
-                for (int ks = 0; ks < 2; ks++) {
-                    uint32_t b[4];
-                    ldmatrix_x4_trans(b, Kt + (size_t)(ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * pitch + c + (lane >> 4) * 8);
-#pragma unroll
-                    for (int part = 0; part < 3; part++) {
-                        mma_bf16(o[j][0], pf[part][ks][0], pf[part][ks][1], pf[part][ks][2], pf[part][ks][3], b[0], b[1]);
-                        mma_bf16(o[j][1], pf[part][ks][0], pf[part][ks][1], pf[part][ks][2], pf[part][ks][3], b[2], b[3]);
-                    }
+    if (warp == 0) {
+        if (lane == 0) {
+            const int* bt = p.block_table + (size_t)seg * p.max_blocks;
+            const int box = min(p.page_size, LT_TILE);             // rows a load
+            for (int it = 0; it < n_tiles; it++) {
+                const int s = it % p.n_stages;
+                if (*abort_flag || !kp_mbar_wait_bounded(&k_empty[s], ((it / p.n_stages) & 1) ^ 1)) { *abort_flag = 1; break; }
+                const int t0 = it * LT_TILE;                       // first key of the tile, counted from the chunk's
+                const int n_boxes = (min(LT_TILE, n_keys - t0) + box - 1) / box;
+                kp_mbar_expect_tx(&k_full[s], (uint32_t)(n_boxes * box * 128 * p.n_box));
+                for (int b = 0; b < n_boxes; b++) {
+                    const int key = c0 + t0 + b * box;
+                    const int y = bt[key / p.page_size] * p.page_size + key % p.page_size;
+                    unsigned char* dst = Ks + (size_t)s * tile_bytes + (size_t)b * box * 128;
+                    if (box == LT_TILE) kp_tma_load_3d(dst, &tmC, 0, y, 0, &k_full[s]);      // the whole tile
+                    else                                           // (smaller pages: a load a group of columns, which lie a tile apart)
+                        for (int j = 0; j < p.n_box; j++) kp_tma_load_3d(dst + (size_t)j * LT_BOX_BYTES, &tmC, 0, y, j, &k_full[s]);
+                }
+                if (it == 0) {                                     // (behind the first tile, which takes longer to come)
+                    kp_mbar_expect_tx(q_full, (uint32_t)p.n_box * NH * 128);
+                    kp_tma_load_3d(Qs, &tmQ, 0, row * p.H + h0, 0, q_full);
                 }
             }
         }
-        __syncthreads();                                           // the stage, the scores and the weights are free
-        if (warp == 0 && it + n_stages < n_tiles) load(it + n_stages);
-    }
-    if (!ok) {
-        if (tid == 0) atomicExch(&g_latent_status, 1);
-        kp_linger_after_failure();
-        return;
-    }
+    } else if (warp == 1) {
+        // ---- S^T of tile it: the tile has come, and the softmax has read what stood in its columns (all lanes in step, an
+        // elected one issues)
+        constexpr uint32_t idesc_s = kp_umma_idesc(64, NH);
+        const uint64_t k_desc = kp_umma_desc(kp_smem_u32(Ks)), q_desc = kp_umma_desc(kp_smem_u32(Qs));
+        bool ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(q_full, 0));
+        for (int it = 0; it < n_tiles && ok; it++) {
+            const int s = it % p.n_stages;
+            ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&k_full[s], (it / p.n_stages) & 1));
+            if (ok && it > 1) ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&p_full[it & 1], ((it - 2) >> 1) & 1));
+            if (!ok || __any_sync(0xffffffffu, *abort_flag)) { ok = false; break; }
+            kp_tc_fence_after();
+            const uint64_t kd = k_desc + s * (tile_bytes >> 4);    // (the address is the descriptor's low field, in 16 bytes)
+            const uint32_t d = tmem_s + (it & 1) * NH;
+            for (int j = 0; j < p.n_box; j++)
+                kp_umma_bf16_box(d + ((uint32_t)(j & 1) << 20), kd + j * (LT_BOX_BYTES >> 4), q_desc + j * (NH * 128 >> 4), idesc_s, j > 1);
+            kp_umma_commit_warp(&s_full[it & 1]);
+        }
+        if (!ok) *abort_flag = 1;
+    } else if (warp == 10) {
+        // ---- U^T of tile it: its weights are there, and U of the tile before has been read
+        constexpr uint32_t idesc_u = kp_umma_idesc(128, NP, false, true);
+        const uint64_t v_desc = kp_umma_desc_mn(kp_smem_u32(Ks), LT_BOX_BYTES), p_desc = kp_umma_desc(kp_smem_u32(Ps));
+        bool ok = true;
+        for (int it = 0; it < n_tiles && ok; it++) {
+            const int s = it % p.n_stages;
+            ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&p_full[it & 1], (it >> 1) & 1));
+            if (ok && it > 0) ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(u_empty, (it - 1) & 1));
+            if (!ok || __any_sync(0xffffffffu, *abort_flag)) { ok = false; break; }
+            kp_tc_fence_after();
+            const uint64_t vd = v_desc + s * (tile_bytes >> 4), pd = p_desc + (it & 1) * (NP * 128 >> 4);
+            for (int m = 0; m < n_blk; m++) {
 #pragma unroll
-    for (int j = 0; j < PT; j++) {
-        const int c = (warp + 8 * j) * 16;
-        if (c >= rankp) continue;
+                for (int kk = 0; kk < LT_TILE / 16; kk++)
+                    kp_umma_bf16_warp(tmem_u + m * NP, vd + m * (2 * LT_BOX_BYTES >> 4) + kk * (2048 >> 4), pd + 2 * kk, idesc_u, kk ? 1u : 0u);
+            }
+            kp_umma_commit_warp(u_full);
+            kp_umma_commit_warp(&k_empty[s]);
+        }
+        if (!ok) *abort_flag = 1;
+    } else {
+        const int grp = (warp - 2) >> 2, q4 = warp & 3;            // (a warp reads lanes 32 (warp % 4) .. of tensor memory)
+        const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
+        const bool upper = lane >= 16;
+        const int key = q4 * 16 + (lane & 15);                     // of the tile
+        const int head0 = grp * HH + (upper ? HQ : 0);             // this thread's heads in the softmax: HQ from here on
+        const float sl2 = p.scale * 1.4426950408889634f;           // scores in units of log2
+        float m_run[HQ], l_run[HQ];
 #pragma unroll
-        for (int i = 0; i < 2; i++) {
-            const int col = c + i * 8 + 2 * t;
-            if (g < nh)
-                *reinterpret_cast<float2*>(part_acc + (((size_t)row * H + h0 + g) * n_chunks + chunk) * rankp + col) = make_float2(o[j][i][0], o[j][i][1]);
-            if (g + 8 < nh)
-                *reinterpret_cast<float2*>(part_acc + (((size_t)row * H + h0 + g + 8) * n_chunks + chunk) * rankp + col) = make_float2(o[j][i][2], o[j][i][3]);
+        for (int h = 0; h < HQ; h++) { m_run[h] = -INFINITY; l_run[h] = 0.f; }
+        float acc[2][NH];
+#pragma unroll
+        for (int b = 0; b < 2; b++)
+#pragma unroll
+            for (int h = 0; h < NH; h++) acc[b][h] = 0.f;
+        bool ok = true;
+        // The warps of a group meet at a barrier in every tile, so they go on or leave together: a wait that gave up is
+        // only noted (`ok`), and the barrier tells all (its result: do all say ok?).
+        auto agree = [&](bool mine) {
+            uint32_t r;
+            asm volatile("{\n .reg .pred a, b;\n setp.ne.u32 a, %1, 0;\n barrier.cta.red.and.pred b, %2, 128, a;\n selp.u32 %0, 1, 0, b;\n}"
+                         : "=r"(r) : "r"(mine ? 1u : 0u), "r"(1 + grp) : "memory");
+            return r != 0;
+        };
+        auto softmax = [&](int it) {                               // false: the warps of the group leave
+            const int b = it & 1, s = it % p.n_stages;
+            if (ok && (!kp_mbar_wait_bounded(&s_full[b], (it >> 1) & 1) || *abort_flag)) ok = false;
+            kp_tc_fence_after();
+            const int valid = min(LT_TILE, n_keys - it * LT_TILE);
+            float v[HQ];
+            {
+                uint32_t raw[HH];
+                if constexpr (HH == 8) kp_tmem_ld8_issue(tmem_s + b * NH + grp * HH + lane_off, raw);
+                else kp_tmem_ld16_issue(tmem_s + b * NH + grp * HH + lane_off, raw);
+                kp_tmem_ld_wait();
+                // the even boxes' sums are in the lower lanes, the odd boxes' in the upper ones (if there are any)
+#pragma unroll
+                for (int h = 0; h < HQ; h++) {
+                    const float lo = __uint_as_float(raw[h]), hi = __uint_as_float(raw[HQ + h]);
+                    const float other = __shfl_xor_sync(0xffffffffu, upper ? lo : hi, 16);
+                    const float sum = p.n_box > 1 ? (upper ? hi : lo) + other : (upper ? other : lo);
+                    v[h] = key < valid ? sum * sl2 : -INFINITY;
+                }
+            }
+            if (valid < LT_TILE) {
+                // the chunk's last tile: rows that no copy of this tile filled, or that hold another request's keys, meet
+                // weights of 0 below and are cleared (0 times NaN is not 0); S has read them already
+                unsigned char* kt = Ks + (size_t)s * tile_bytes;
+                const int n = (LT_TILE - valid) * 2 * n_blk;       // (row, box) pairs
+                const int n_real = min(2 * n_blk, p.n_box);
+                for (int i = threadIdx.x - 64; i < n; i += 256) {
+                    const int r = valid + i / (2 * n_blk), j = i % (2 * n_blk);
+                    if (j >= n_real) continue;
+                    uint4* d = reinterpret_cast<uint4*>(kt + (size_t)j * LT_BOX_BYTES + r * 128);
+#pragma unroll
+                    for (int c = 0; c < 8; c++) d[c] = make_uint4(0, 0, 0, 0);
+                }
+            }
+            // the tile's maximum of every head: over the half warp's keys, then over the four warps of the group
+            float* mx = max_s + b * 4 * NH;
+            float mine = 0.f;
+#pragma unroll
+            for (int h = 0; h < HQ; h++) {
+                float w = v[h];
+#pragma unroll
+                for (int o = 8; o > 0; o >>= 1) w = fmaxf(w, __shfl_xor_sync(0xffffffffu, w, o));
+                if ((lane & 15) == h) mine = w;
+            }
+            if ((lane & 15) < HQ) mx[(head0 + (lane & 15)) * 4 + q4] = mine;
+            if (!agree(ok)) { ok = false; return false; }
+            unsigned char* pr = Ps + (size_t)b * (NP * 128) + (key & 7) * 2;
+#pragma unroll
+            for (int h = 0; h < HQ; h++) {
+                const int hh = head0 + h;
+                const float4 m4 = *reinterpret_cast<const float4*>(mx + hh * 4);
+                const float m_new = fmaxf(fmaxf(m_run[h], fmaxf(m4.x, m4.y)), fmaxf(m4.z, m4.w));   // (finite: a tile's first key is the row's)
+                const float corr = la_exp2(m_run[h] - m_new);      // (2^-inf = 0 for the first tile)
+                float w = la_exp2(v[h] - m_new);
+                m_run[h] = m_new;
+                l_run[h] = fmaf(l_run[h], corr, w);
+                if (key == 0) corr_s[(it & 3) * NH + hh] = corr;
+#pragma unroll
+                for (int part = 0; part < 3; part++) {
+                    const bf16 x = __float2bfloat16_rn(w);
+                    w -= __bfloat162float(x);
+                    const int n = part * NH + hh;
+                    *reinterpret_cast<bf16*>(pr + n * 128 + (((key >> 3) ^ (n & 7)) << 4)) = x;
+                }
+            }
+            kp_tc_fence_before();                                  // the reads of S are done
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the weights and cleared rows are read by the tensor core
+            kp_mbar_arrive(&p_full[b]);
+            return true;
+        };
+        auto gather = [&](int it) {
+            if (!kp_mbar_wait_bounded(u_full, it & 1) || *abort_flag) { ok = false; return; }
+            kp_tc_fence_after();
+            const float* corr = corr_s + (it & 3) * NH;
+#pragma unroll
+            for (int b = 0; b < 2; b++) {
+                const int m = grp + 2 * b;                         // the group's blocks of 128 columns
+                if (m < n_blk) {
+                    const uint32_t ta = tmem_u + m * NP + lane_off;
+                    if constexpr (NH == 16) {
+                        uint32_t u[3][16];
+#pragma unroll
+                        for (int part = 0; part < 3; part++) kp_tmem_ld16_issue(ta + part * NH, u[part]);
+                        kp_tmem_ld_wait();
+#pragma unroll
+                        for (int h = 0; h < 16; h++)
+                            acc[b][h] = fmaf(acc[b][h], corr[h], __uint_as_float(u[0][h]) + (__uint_as_float(u[1][h]) + __uint_as_float(u[2][h])));
+                    } else {
+#pragma unroll
+                        for (int half = 0; half < 2; half++) {
+                            uint32_t u[3][16];
+#pragma unroll
+                            for (int part = 0; part < 3; part++) kp_tmem_ld16_issue(ta + part * NH + half * 16, u[part]);
+                            kp_tmem_ld_wait();
+#pragma unroll
+                            for (int h = 0; h < 16; h++)
+                                acc[b][half * 16 + h] = fmaf(acc[b][half * 16 + h], corr[half * 16 + h],
+                                                             __uint_as_float(u[0][h]) + (__uint_as_float(u[1][h]) + __uint_as_float(u[2][h])));
+                        }
+                    }
+                }
+            }
+            kp_tc_fence_before();
+            __syncwarp();
+            if (lane == 0) kp_mbar_arrive(u_empty);
+        };
+        bool together = softmax(0);
+        for (int it = 0; it < n_tiles && together; it++) {
+            if (it + 1 < n_tiles) together = softmax(it + 1);
+            if (ok) gather(it);
+        }
+        if (together) {
+            // the tiles' sums of weights: over the half warp, then over the four warps of the group
+#pragma unroll
+            for (int h = 0; h < HQ; h++) {
+                float l = l_run[h];
+#pragma unroll
+                for (int o = 8; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+                if ((lane & 15) == 0) sum_s[(head0 + h) * 4 + q4] = l;
+            }
+            ok = agree(ok);
+        }
+        if (!ok) *abort_flag = 1;
+        if (ok) {
+            const int nh = min(NH, p.H - h0);
+#pragma unroll
+            for (int b = 0; b < 2; b++) {
+                const int col = (grp + 2 * b) * 128 + q4 * 32 + lane;
+                if (col < p.rankp) {
+#pragma unroll
+                    for (int h = 0; h < NH; h++)
+                        if (h < nh) p.part_acc[(((size_t)row * p.H + h0 + h) * p.n_chunks + chunk) * p.rankp + col] = acc[b][h];
+                }
+            }
+            if (key == 0) {
+#pragma unroll
+                for (int h = 0; h < HQ; h++) {
+                    const int hh = head0 + h;
+                    const float4 l4 = *reinterpret_cast<const float4*>(sum_s + hh * 4);
+                    if (hh < nh)
+                        *reinterpret_cast<float2*>(p.part_ml + (((size_t)row * p.H + h0 + hh) * p.n_chunks + chunk) * 2) =
+                            make_float2(m_run[h] * 0.6931471805599453f, (l4.x + l4.y) + (l4.z + l4.w));
+                }
+            }
         }
     }
-    if ((tid & 15) == 0 && (tid >> 4) < nh)
-        *reinterpret_cast<float2*>(part_ml + (((size_t)row * H + h0 + (tid >> 4)) * n_chunks + chunk) * 2) = make_float2(m_run, l_run);
+    kp_tc_fence_before();
+    __syncthreads();
+    if (*abort_flag) {
+        if (threadIdx.x == 0) atomicExch(&g_latent_status, 1);
+        kp_linger_after_failure();
+    }
+    if (warp == 1) kp_tmem_dealloc(tmem_s, TMEM_COLS);
 }
 
 // ------------------------------------------------------------------------------------- absorbed pass, CUDA cores
@@ -449,12 +626,13 @@ latent_split_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, const int* __restrict__ positions,
-                    T* __restrict__ out, int n_chunks, int H, int rankp) {
+                    T* __restrict__ out, int n_chunks, int H, int rankp, int fixed_chunk) {
     kp_pdl_begin_early_if(gridDim.y > 1);
     extern __shared__ float lm_w[];                                // [n_chunks] weights, [32]
     float* red = lm_w + n_chunks;
     const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x;
-    const int n = min(positions[row] / LA_CHUNK + 1, n_chunks);
+    const int pos = positions[row];
+    const int n = min(pos / (fixed_chunk ? LA_CHUNK : lt_chunk_keys(positions, gridDim.y, n_chunks)) + 1, n_chunks);
     const float* ml = part_ml + ((size_t)row * H + h) * n_chunks * 2;
     float m = -INFINITY;
     for (int c = tid; c < n; c += 128) { const float v = ml[2 * c]; lm_w[c] = v; m = fmaxf(m, v); }
@@ -667,9 +845,18 @@ latent_prefill_kernel(const LatentPrefillArgs p) {
     }
 }
 
-static size_t la_fixed_bytes(int W) { return (size_t)16 * (W + 8) * 2 + 3 * 16 * 40 * 2 + 2 * 16 * 36 * 4 + 16 * 4 + LA_MAX_STAGES * 8; }
-static size_t la_tile_bytes(int W) { return (size_t)LA_TILE * (W + 8) * 2; }
-#define LA_SMEM_BUDGET (112 * 1024)                                // two CTAs an SM
+static size_t lt_fixed_bytes(int n_box, int nh) {
+    return 1024 + (size_t)n_box * nh * 128 + 2 * 3 * nh * 128 + 16 * nh * sizeof(float) + (2 * LT_MAX_STAGES + 7) * 8 + 16;
+}
+#define LT_SMEM_MAX (226 * 1024)
+
+// Can the tensor-core form of the absorbed pass take these sizes (two tiles in shared memory, the latent's blocks in tensor
+// memory, pages that boxes of rows divide)?
+static bool lt_fits(int rankp, int W, int H, int page_size) {
+    const int n_box = W / 64;
+    return rankp <= 512 && W % 64 == 0 && page_size % 8 == 0 && (page_size % LT_TILE == 0 || LT_TILE % page_size == 0) &&
+           lt_fixed_bytes(n_box, H > 16 ? 32 : 16) + (size_t)2 * n_box * LT_BOX_BYTES <= LT_SMEM_MAX;
+}
 
 template <typename F>
 static int la_set_smem(F kern, size_t sm) {
@@ -679,15 +866,15 @@ static int la_set_smem(F kern, size_t sm) {
 
 extern "C" {
 
-int kp_latent_prep(void* p, int ld, int q_col, int c_col, int H, int dimp, int rotp, int rank, int rankp, const float* w, float eps,
+int kp_latent_prep(void* p, int ld, int q_col, int c_col, int H, int dimp, int rotp, int rank, int rankp, int W, const float* w, float eps,
                    const float* cos_tab, const float* sin_tab, int rot, int interleaved, const int* positions, const int* slot_map,
                    void* cache, int page_size, void* qa, int n_absorbed, int n, int dtype, void* stream) {
     if (n <= 0) return 0;
-    if (H < 1 || rank < 1 || rank > rankp || (rankp & 15) || (rotp & 15) || rotp < 0 || page_size < 1 || (cos_tab && (rot < 2 || (rot & 1) || rot > rotp)) ||
+    if (H < 1 || rank < 1 || rank > rankp || (rankp & 15) || (rotp & 15) || rotp < 0 || W < rankp + rotp || page_size < 1 || (cos_tab && (rot < 2 || (rot & 1) || rot > rotp)) ||
         n_absorbed < 0 || n_absorbed > n || (n_absorbed > 0 && !qa))
         return KP_ERR_BAD_ARG;
     KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(latent_prep_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, (T*)p, ld, q_col, c_col, H,
-                                               dimp, rotp, rank, rankp, w, eps, cos_tab, sin_tab, rot, interleaved, positions,
+                                               dimp, rotp, rank, rankp, W, w, eps, cos_tab, sin_tab, rot, interleaved, positions,
                                                slot_map, (T*)cache, page_size, (T*)qa, n_absorbed)));
     return kp_launch_status();
 }
@@ -711,36 +898,53 @@ int kp_head_gemm(const void* a, long long a_row, int a_head, const void* b, void
     return kp_launch_status();
 }
 
-long long kp_latent_split_scratch(int n, int H, int rankp, int n_chunks) { return (long long)n * H * n_chunks * (rankp + 2); }
+// The chunks a row has at most in kp_latent_split with these sizes (its scratch: n H chunks (rankp + 2) floats).  The tensor-core
+// form: as many as give the fewest rounds of CTAs over the SMs (one an SM) times the tiles of a CTA, what a CTA
+// costs beside its tiles (launch, the first tile's way, the last one's products: about two and a half tiles) counted in.
+int kp_latent_chunks(int n, int max_context, int rankp, int W, int H, int page_size, int dtype, int tensor_cores) {
+    if (!(tensor_cores && dtype == KP_DTYPE_BF16 && lt_fits(rankp, W, H, page_size))) return (max_context + LA_CHUNK - 1) / LA_CHUNK;
+    const long long ctas = (long long)n * ((H + (H > 16 ? 31 : 15)) / (H > 16 ? 32 : 16));
+    const int tiles = (max_context + LT_TILE - 1) / LT_TILE, sms = 148;
+    int best_c = 1;
+    double best = 1e30;
+    for (int c = 1; c <= tiles && c <= 512; c++) {
+        const double cost = (double)((ctas * c + sms - 1) / sms) * ((tiles + c - 1) / c + 2.5);
+        if (cost < best) { best = cost; best_c = c; }
+    }
+    return best_c;
+}
 
-// qa [n][H][W] -> u [n][H][rankp]; scratch: kp_latent_split_scratch floats; n_chunks chunks of 256 keys must reach the
-// largest position.
-int kp_latent_split(const void* qa, const void* cache, const int* block_table, int max_blocks, const int* row_seg, const int* positions,
-                    float* scratch, int n_chunks, void* u, float scale, int page_size, int n, int H, int rankp, int rotp, int dtype,
-                    int tensor_cores, void* stream) {
+// qa [n][H][W] -> u [n][H][rankp]; max_context: beyond the largest position of the rows; n_pages: pages of the cache.
+int kp_latent_split(const void* qa, const void* cache, long long n_pages, const int* block_table, int max_blocks, const int* row_seg,
+                    const int* positions, float* scratch, int max_context, void* u, float scale, int page_size, int n, int H, int rankp,
+                    int W, int dtype, int tensor_cores, void* stream) {
     if (n <= 0) return 0;
-    if (n > 65535 || H < 1 || n_chunks < 1 || page_size < 1 || (rankp & 15) || (rotp & 15) || rankp < 16) return KP_ERR_BAD_ARG;
-    const int W = rankp + rotp;
+    if (n > 65535 || H < 1 || max_context < 1 || page_size < 1 || (rankp & 15) || (W & 15) || rankp < 16 || W < rankp)
+        return KP_ERR_BAD_ARG;
+    const int n_chunks = kp_latent_chunks(n, max_context, rankp, W, H, page_size, dtype, tensor_cores);
     float* part_acc = scratch;
     float* part_ml = scratch + (size_t)n * H * n_chunks * rankp;
     cudaStream_t s = (cudaStream_t)stream;
     int st = 0;
-    const size_t fixed = la_fixed_bytes(W), tile = la_tile_bytes(W);
-    if (tensor_cores && dtype == KP_DTYPE_BF16 && rankp <= 512 && fixed + 2 * tile <= 2 * LA_SMEM_BUDGET && !(((uintptr_t)qa | (uintptr_t)cache) & 15)) {
-        const size_t budget = fixed + 2 * tile <= LA_SMEM_BUDGET ? LA_SMEM_BUDGET : 2 * LA_SMEM_BUDGET;
-        int stages = (int)((budget - fixed) / tile);
-        if (stages > LA_MAX_STAGES) stages = LA_MAX_STAGES;
+    const bool tc = tensor_cores && dtype == KP_DTYPE_BF16 && lt_fits(rankp, W, H, page_size);
+    if (tc) {
+        if (((uintptr_t)qa | (uintptr_t)cache) & 15 || n_pages * page_size >= 2147483647LL || (long long)n * H >= 2147483647LL) return KP_ERR_UNSUPPORTED;
+        const int nh = H > 16 ? 32 : 16, n_box = W / 64;
+        const size_t fixed = lt_fixed_bytes(n_box, nh), tile = (size_t)n_box * LT_BOX_BYTES;
+        int stages = (int)((LT_SMEM_MAX - fixed) / tile);
+        if (stages > LT_MAX_STAGES) stages = LT_MAX_STAGES;
         const size_t sm = fixed + stages * tile;
-        dim3 grid(n_chunks, (H + 15) / 16, n);
-#define LA_MMA(PT)                                                                                                        \
-    do {                                                                                                                  \
-        st = la_set_smem(latent_split_mma_kernel<PT>, sm);                                                                \
-        if (st) return st;                                                                                                \
-        kp_launch_pdl(latent_split_mma_kernel<PT>, grid, dim3(256), sm, s, (const bf16*)qa, (const bf16*)cache, block_table, max_blocks, \
-                      row_seg, positions, part_acc, part_ml, n_chunks, scale, page_size, H, rankp, W, stages);            \
-    } while (0)
-        if (rankp <= 128) LA_MMA(1); else if (rankp <= 256) LA_MMA(2); else LA_MMA(4);
-#undef LA_MMA
+        alignas(64) CUtensorMap tc_map, tq_map;
+        st = page_size < LT_TILE ? kp_make_map_bf16_groups(&tc_map, cache, (unsigned long long)n_pages * page_size, n_box, W, page_size, 1)
+                                 : kp_make_map_bf16_groups(&tc_map, cache, (unsigned long long)n_pages * page_size, n_box, W, LT_TILE);
+        if (!st) st = kp_make_map_bf16_groups(&tq_map, qa, (unsigned long long)n * H, n_box, W, nh);
+        if (st) return st;
+        LatentSplitArgs a = {block_table, row_seg, positions, part_acc, part_ml, max_blocks, n_chunks, page_size, H, rankp, n_box, stages, scale};
+        dim3 grid(n_chunks, (H + nh - 1) / nh, n);
+        auto kern = nh == 16 ? latent_split_tc_kernel<16> : latent_split_tc_kernel<32>;
+        st = la_set_smem(kern, sm);
+        if (st) return st;
+        kp_launch_pdl(kern, grid, dim3(LT_THREADS), sm, s, tc_map, tq_map, a);
     } else {
         const size_t sm = ((size_t)LA_SCALAR_HEADS * (W + LA_CHUNK) + 32 + LA_CHUNK) * sizeof(float);
         if (sm > 200 * 1024) return KP_ERR_UNSUPPORTED;
@@ -759,7 +963,8 @@ int kp_latent_split(const void* qa, const void* cache, const int* block_table, i
     KP_DISPATCH_DTYPE(dtype, T, {
         st = la_set_smem(latent_merge_kernel<T>, msm);
         if (st) return st;
-        kp_launch_pdl(latent_merge_kernel<T>, dim3(H, n), dim3(128), msm, s, part_acc, part_ml, positions, (T*)u, n_chunks, H, rankp);
+        kp_launch_pdl(latent_merge_kernel<T>, dim3(H, n), dim3(128), msm, s, part_acc, part_ml, positions, (T*)u, n_chunks, H, rankp,
+                      tc ? 0 : 1);
     });
     return kp_launch_status();
 }
@@ -775,15 +980,15 @@ int kp_latent_gather(const void* cache, const int* block_table, int max_blocks, 
 
 // q: rows of H heads of dimp + rotp; ex [T][ld_ex]: the expanded keys (H heads of dimp) and, from v_col on, values (H
 // heads of vdimp); rows [T][W]: the gathered cache rows; tile_seg / tile_row0: n_tiles tiles of 64 rows.
-int kp_latent_prefill(const void* q, int ldq, const void* ex, int ld_ex, int v_col, const void* rows, int rankp, int dimp, int rotp,
+int kp_latent_prefill(const void* q, int ldq, const void* ex, int ld_ex, int v_col, const void* rows, int W, int rankp, int dimp, int rotp,
                       int vdimp, const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0, const int* ctx_base,
                       int n_tiles, void* out, int ldo, float scale, int H, void* stream) {
     if (n_tiles <= 0) return 0;
-    if ((dimp & 15) || (rotp & 15) || (vdimp & 15) || (rankp & 15) || H < 1 || H > 65535) return KP_ERR_BAD_ARG;
+    if ((dimp & 15) || (rotp & 15) || (vdimp & 15) || (rankp & 15) || (W & 7) || W < rankp + rotp || H < 1 || H > 65535) return KP_ERR_BAD_ARG;
     if ((ldq & 1) || (ldo & 1) || (ld_ex & 7) || (v_col & 7) || (((uintptr_t)ex | (uintptr_t)rows) & 15)) return KP_ERR_UNSUPPORTED;
     const int Dq = dimp + rotp;
     LatentPrefillArgs a = {(const bf16*)q, (const bf16*)ex, (const bf16*)rows, (bf16*)out, cu_rows, seg_pos, tile_seg, tile_row0, ctx_base,
-                           ldq, ldo, ld_ex, rankp + rotp, rankp, dimp, rotp, vdimp, v_col, n_tiles, scale};
+                           ldq, ldo, ld_ex, W, rankp, dimp, rotp, vdimp, v_col, n_tiles, scale};
     const size_t sm = (size_t)2 * LP_TILE * (Dq + 8 + vdimp + 8) * 2;
     if (sm > 200 * 1024) return KP_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;

@@ -20,6 +20,30 @@ __device__ __forceinline__ void kp_umma_bf16(uint32_t tmem_d, uint64_t adesc, ui
                  " tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n}"
                  ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(0u) : "memory");
 }
+// The same for a whole warp in step, whose operands are the same in every lane: one elected lane issues it.  (From inside a
+// branch that one lane took, the operands pass through general registers: 94 cycles an MMA against 30.)
+__device__ __forceinline__ void kp_umma_bf16_warp(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile("{\n .reg .pred p, e;\n elect.sync _|e, 0xffffffff;\n setp.ne.b32 p, %4, 0;\n"
+                 " @e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n}"
+                 ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(0u) : "memory");
+}
+// Four MMAs along K over one 128-byte box of a K-major A and B (64 elements), by an elected lane; `accumulate` is that of
+// the first.
+__device__ __forceinline__ void kp_umma_bf16_box(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, bool accumulate) {
+    asm volatile("{\n .reg .pred p, e;\n .reg .b64 a, b;\n elect.sync _|e, 0xffffffff;\n setp.ne.b32 p, %4, 0;\n"
+                 " @e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n"
+                 " add.s64 a, %1, 2;\n add.s64 b, %2, 2;\n setp.eq.b32 p, 0, 0;\n"
+                 " @e tcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, {%5, %5, %5, %5}, p;\n"
+                 " add.s64 a, %1, 4;\n add.s64 b, %2, 4;\n"
+                 " @e tcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, {%5, %5, %5, %5}, p;\n"
+                 " add.s64 a, %1, 6;\n add.s64 b, %2, 6;\n"
+                 " @e tcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, {%5, %5, %5, %5}, p;\n}"
+                 ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate ? 1u : 0u), "r"(0u) : "memory");
+}
+__device__ __forceinline__ void kp_umma_commit_warp(uint64_t* bar) {
+    asm volatile("{\n .reg .pred e;\n elect.sync _|e, 0xffffffff;\n"
+                 " @e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n}" ::"r"(kp_smem_u32(bar)) : "memory");
+}
 // the mbarrier gets one arrival when every MMA issued so far by this thread has completed
 __device__ __forceinline__ void kp_umma_commit(uint64_t* bar) {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(kp_smem_u32(bar)) : "memory");
@@ -49,6 +73,18 @@ __device__ __forceinline__ void kp_tmem_ld32_issue(uint32_t taddr, uint32_t (&r)
                    "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
                  : "r"(taddr));
 }
+// 16 and 8 columns, without the wait
+__device__ __forceinline__ void kp_tmem_ld16_issue(uint32_t taddr, uint32_t (&r)[16]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+                 "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
+                   "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+                 : "r"(taddr));
+}
+__device__ __forceinline__ void kp_tmem_ld8_issue(uint32_t taddr, uint32_t (&r)[8]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]) : "r"(taddr));
+}
 __device__ __forceinline__ void kp_tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 // 32 consecutive columns of this thread's lane written back to tensor memory (complete after kp_tmem_st_wait())
 __device__ __forceinline__ void kp_tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
@@ -77,9 +113,13 @@ __device__ __forceinline__ uint64_t kp_umma_desc(uint32_t smem_addr) {
     d |= (uint64_t)2 << 61;
     return d;
 }
-// Instruction descriptor: float32 accumulator, bfloat16 A and B, A K-major, B K-major or (b_mn) MN-major,
+// The same for an MN-major operand of more than 64 elements along MN: its stretches of 64 lie lead_bytes apart.
+__device__ __forceinline__ uint64_t kp_umma_desc_mn(uint32_t smem_addr, uint32_t lead_bytes) {
+    return (kp_umma_desc(smem_addr) & ~((uint64_t)0x3FFF << 16)) | ((uint64_t)((lead_bytes >> 4) & 0x3FFF) << 16);
+}
+// Instruction descriptor: float32 accumulator, bfloat16 A and B, each K-major or (a_mn, b_mn) MN-major,
 // N and M of the MMA.
-__host__ __device__ constexpr uint32_t kp_umma_idesc(int M, int N, bool b_mn = false) {
-    return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((uint32_t)(N >> 3) << 17) |
+__host__ __device__ constexpr uint32_t kp_umma_idesc(int M, int N, bool b_mn = false, bool a_mn = false) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | (a_mn ? (1u << 15) : 0u) | (b_mn ? (1u << 16) : 0u) | ((uint32_t)(N >> 3) << 17) |
            ((uint32_t)(M >> 4) << 24);
 }

@@ -74,6 +74,12 @@ __device__ __forceinline__ void kp_tma_load_2d(void* dst, const CUtensorMap* map
                  ::"r"(kp_smem_u32(dst)), "l"(map), "r"(x), "r"(y), "r"(kp_smem_u32(bar)) : "memory");
 }
 
+// box of a 3-D tensor at (x, y, z)
+__device__ __forceinline__ void kp_tma_load_3d(void* dst, const CUtensorMap* map, int x, int y, int z, uint64_t* bar) {
+    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
+                 ::"r"(kp_smem_u32(dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(kp_smem_u32(bar)) : "memory");
+}
+
 typedef CUresult (*KpEncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
                                     const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
                                     CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -101,6 +107,23 @@ static inline int kp_make_map_bf16_2d(CUtensorMap* map, const void* base, unsign
     cuuint32_t box[2] = {(cuuint32_t)box_cols, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? 0 : KP_ERR_UNSUPPORTED;
+}
+
+// rows x (64 groups) bf16 with row stride ld elements, seen as (64 columns, rows, groups): a box of box_rows rows takes all
+// groups at once (or box_groups of them) and lies in shared memory as `groups` tiles of box_rows rows of 128 bytes (128-byte swizzle), the layout
+// that `groups` loads through the map above would give
+static inline int kp_make_map_bf16_groups(CUtensorMap* map, const void* base, unsigned long long rows, int groups, long long ld, int box_rows,
+                                          int box_groups = 0) {
+    KpEncodeTiledFn fn = kp_encode_tiled_fn();
+    if (!fn) return KP_ERR_UNSUPPORTED;
+    cuuint64_t dims[3] = {64, (cuuint64_t)rows, (cuuint64_t)groups};
+    cuuint64_t strides[2] = {(cuuint64_t)ld * 2, 128};
+    cuuint32_t box[3] = {64, (cuuint32_t)box_rows, (cuuint32_t)(box_groups ? box_groups : groups)};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                     CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS ? 0 : KP_ERR_UNSUPPORTED;

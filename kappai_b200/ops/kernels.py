@@ -1399,22 +1399,23 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
 
 # ------------------------------------------------------------------ attention over cached latents
 
-LATENT_CHUNK = 256             # keys a chunk of the absorbed pass
 LATENT_PREFILL_MAX = (256, 256)    # key and value columns a head that the expanded pass takes
-USE_MMA_LATENT = True          # the absorbed pass of bfloat16 rows runs on the tensor cores where the sizes allow it
+USE_TC_LATENT = True           # the absorbed pass of bfloat16 rows runs on the tcgen05 tensor cores where the sizes allow it
 
 
-def latent_prep(p: torch.Tensor, q_col: int, c_col: int, H: int, dimp: int, rotp: int, rank: int, rankp: int, w: torch.Tensor,
+def latent_prep(p: torch.Tensor, q_col: int, c_col: int, H: int, dimp: int, rotp: int, rank: int, rankp: int, W: int, w: torch.Tensor,
                 eps: float, rotary, positions: torch.Tensor, slot_map: torch.Tensor, cache: Optional[torch.Tensor],
                 page_size: int, qa: Optional[torch.Tensor], n_absorbed: int) -> None:
     """Rows ``p`` of the input product hold H query heads of (dimp | rotp) at ``q_col`` and the latent (rankp) with the
     shared key part (rotp) at ``c_col``: norm the latent over its ``rank`` columns (weight ``w`` [rank]), rotate the key part
     and store both in the row's cache page; rotate the heads' query parts in place, and copy those of the first
-    ``n_absorbed`` rows behind the absorbed queries in ``qa`` [n_absorbed, H, rankp + rotp].  ``rotary``: (cos, sin,
+    ``n_absorbed`` rows behind the absorbed queries in ``qa`` [n_absorbed, H, W].  A cache row and an absorbed query have ``W``
+    elements, zeros behind their rankp + rotp.  ``rotary``: (cos, sin,
     dimensions, interleaved) as a position part gives it."""
     _need(p, "p", contiguous=False); _need(w, "w", torch.float32); _need(positions, "positions", torch.int32)
-    n, W = p.shape[0], rankp + rotp
-    if p.stride(1) != 1 or q_col + H * (dimp + rotp) > p.shape[1] or c_col + W > p.shape[1] or w.numel() != rank:
+    n = p.shape[0]
+    if (p.stride(1) != 1 or q_col + H * (dimp + rotp) > p.shape[1] or c_col + rankp + rotp > p.shape[1] or w.numel() != rank
+            or W < rankp + rotp):
         raise KernelError("latent_prep: shape mismatch")
     if cache is not None:
         _need(cache, "cache", p.dtype); _need(slot_map, "slot_map", torch.int32)
@@ -1430,7 +1431,7 @@ def latent_prep(p: torch.Tensor, q_col: int, c_col: int, H: int, dimp: int, rotp
         if cos.shape[1] != rot // 2 or rot > rotp:
             raise KernelError("latent_prep: table width")
     _run("latent_prep", load_library("latent").kp_latent_prep, _ptr(p), p.stride(0), int(q_col), int(c_col), H, dimp, rotp, rank, rankp,
-         _ptr(w), ctypes.c_float(eps), _ptr(cos), _ptr(sin), int(rot), int(bool(inter)), _ptr(positions), _ptr(slot_map), _ptr(cache),
+         int(W), _ptr(w), ctypes.c_float(eps), _ptr(cos), _ptr(sin), int(rot), int(bool(inter)), _ptr(positions), _ptr(slot_map), _ptr(cache),
          page_size, _ptr(qa), int(n_absorbed), n, dtype_code(p.dtype), STREAM)
 
 
@@ -1453,14 +1454,21 @@ def head_gemm(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, gate: Optiona
     return out
 
 
-def latent_split_scratch(n: int, H: int, rankp: int, n_chunks: int) -> int:
-    return n * H * n_chunks * (rankp + 2)
+def latent_chunks(n: int, max_context: int, H: int, rankp: int, W: int, page_size: int, dtype: torch.dtype) -> int:
+    """Chunks that :func:`latent_split` cuts a context of ``max_context`` keys into at most, for these sizes and ``n`` rows."""
+    return int(load_library("latent").kp_latent_chunks(int(n), int(max_context), rankp, W, H, page_size, dtype_code(dtype), int(USE_TC_LATENT)))
+
+
+def latent_split_scratch(n: int, H: int, rankp: int, W: int, max_context: int, page_size: int, dtype: torch.dtype) -> int:
+    """Float elements of scratch that :func:`latent_split` needs."""
+    return n * H * latent_chunks(n, max_context, H, rankp, W, page_size, dtype) * (rankp + 2)
 
 
 def latent_split(qa: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, row_seg: torch.Tensor, positions: torch.Tensor,
-                 scratch: torch.Tensor, n_chunks: int, u: torch.Tensor, scale: float, page_size: int) -> torch.Tensor:
+                 scratch: torch.Tensor, max_context: int, u: torch.Tensor, scale: float, page_size: int) -> torch.Tensor:
     """Causal softmax attention of absorbed queries ``qa`` [n, H, W] over the cached rows (the latents are the values too):
-    ``u`` [n, H, rankp].  ``n_chunks`` chunks of 256 keys must cover the largest position; ``scratch`` is float32."""
+    ``u`` [n, H, rankp].  ``max_context`` lies beyond the largest position; ``scratch`` is float32.  bfloat16 rows run
+    on the tcgen05 tensor cores where the sizes allow it."""
     n, H, W = qa.shape
     rankp = u.shape[2]
     _need(qa, "qa"); _need(cache, "cache", qa.dtype); _need(u, "u", qa.dtype); _need(scratch, "scratch", torch.float32)
@@ -1468,11 +1476,11 @@ def latent_split(qa: torch.Tensor, cache: torch.Tensor, block_table: torch.Tenso
         _need(t, nm, torch.int32)
     if tuple(cache.shape[1:]) != (1, 1, page_size, W) or tuple(u.shape) != (n, H, rankp) or row_seg.numel() != n or positions.numel() != n:
         raise KernelError("latent_split: shape mismatch")
-    if scratch.numel() < latent_split_scratch(n, H, rankp, n_chunks):
+    if scratch.numel() < latent_split_scratch(n, H, rankp, W, max_context, page_size, qa.dtype):
         raise KernelError("latent_split: scratch too small")
-    _run("latent_split", load_library("latent").kp_latent_split, _ptr(qa), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(row_seg),
-         _ptr(positions), _ptr(scratch), n_chunks, _ptr(u), ctypes.c_float(scale), page_size, n, H, rankp, W - rankp, dtype_code(qa.dtype),
-         int(USE_MMA_LATENT), STREAM)
+    _run("latent_split", load_library("latent").kp_latent_split, _ptr(qa), _ptr(cache), ctypes.c_longlong(cache.shape[0]), _ptr(block_table),
+         block_table.shape[1], _ptr(row_seg), _ptr(positions), _ptr(scratch), int(max_context), _ptr(u), ctypes.c_float(scale), page_size, n, H,
+         rankp, W, dtype_code(qa.dtype), int(USE_TC_LATENT), STREAM)
     LAUNCHES[0] += 1
     return u
 
@@ -1498,18 +1506,18 @@ def latent_prefill(q: torch.Tensor, ex: torch.Tensor, rows: torch.Tensor, rankp:
                    cu_rows: torch.Tensor, seg_pos: torch.Tensor, tile_seg: torch.Tensor, tile_row0: torch.Tensor, ctx_base: torch.Tensor,
                    out: torch.Tensor, scale: float, H: int) -> torch.Tensor:
     """Causal attention of prompt portions over expanded latents: ``q`` [n, H (dimp + rotp)] (rows may be strided), ``ex`` [T, H
-    dimp + H vdimp] the expanded keys and values and ``rows`` [T, rankp + rotp] the gathered cache rows (their last rotp
-    columns are the shared key part), T the contexts of ``ctx_base``; tiles of 64 rows as attention_prefill takes them."""
+    dimp + H vdimp] the expanded keys and values and ``rows`` [T, W] the gathered cache rows (the rotp columns behind the first
+    rankp are the shared key part), T the contexts of ``ctx_base``; tiles of 64 rows as attention_prefill takes them."""
     _need(q, "q", torch.bfloat16, contiguous=False); _need(ex, "ex", torch.bfloat16); _need(rows, "rows", torch.bfloat16)
     _need(out, "out", torch.bfloat16, contiguous=False)
     for t, nm in ((cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (tile_seg, "tile_seg"), (tile_row0, "tile_row0"), (ctx_base, "ctx_base")):
         _need(t, nm, torch.int32)
     n = q.shape[0]
     if (q.shape[1] != H * (dimp + rotp) or tuple(out.shape) != (n, H * vdimp) or ex.shape[1] != H * (dimp + vdimp)
-            or rows.shape != (ex.shape[0], rankp + rotp) or tile_seg.numel() != tile_row0.numel()):
+            or rows.shape[0] != ex.shape[0] or rows.shape[1] < rankp + rotp or tile_seg.numel() != tile_row0.numel()):
         raise KernelError("latent_prefill: shape mismatch")
-    _run("latent_prefill", load_library("latent").kp_latent_prefill, _ptr(q), _rows_2d(q, "q"), _ptr(ex), ex.shape[1], H * dimp, _ptr(rows), rankp,
-         dimp, rotp, vdimp, _ptr(cu_rows), _ptr(seg_pos), _ptr(tile_seg), _ptr(tile_row0), _ptr(ctx_base), tile_seg.numel(), _ptr(out),
+    _run("latent_prefill", load_library("latent").kp_latent_prefill, _ptr(q), _rows_2d(q, "q"), _ptr(ex), ex.shape[1], H * dimp, _ptr(rows),
+         rows.shape[1], rankp, dimp, rotp, vdimp, _ptr(cu_rows), _ptr(seg_pos), _ptr(tile_seg), _ptr(tile_row0), _ptr(ctx_base), tile_seg.numel(), _ptr(out),
          _rows_2d(out, "out"), ctypes.c_float(scale), H, STREAM)
     return out
 

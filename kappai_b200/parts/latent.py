@@ -7,7 +7,7 @@
     s_h(t) = (q_h . k_h(t) + qr_h . r(t)) scale ,  causal softmax,  o_h = sum_t softmax(s_h)_t v_h(t)
 
 and the concatenated heads, times ``sigmoid(h Wg^T)`` (``gate`` = ``"sigmoid"``), go through the output matrix.  Only c and
-r are cached: one row a token in a page group of one plane, padded to multiples of 16.  (:class:`~.attention.LatentAttention`
+r are cached: one row a token in a page group of one plane, padded to a multiple of 64.  (:class:`~.attention.LatentAttention`
 is the kind that expands the latents before it caches them.)
 
 Decoded tokens, short portions and every row of the 32-bit mode run *absorbed*: the expanding matrices are applied to the
@@ -79,7 +79,7 @@ class LatentCacheAttention(PagedAttentionKernels, Part):
             raise ConfigError("latent_cache_attention: heads, head sizes and the rank must be positive")
         # the sizes as the kernels see them: zero rows and columns behind every part up to a multiple of 16
         self.dimp, self.rotp, self.vdimp, self.rankp = _up16(self.dim), _up16(self.rdim), _up16(self.vdim), _up16(self.rank)
-        self.row = self.rankp + self.rotp
+        self.row = -(-(self.rankp + self.rotp) // 64) * 64                             # elements of a cache row and an absorbed query
         pos = self._p("position", None)
         pos = PartSpec("none") if pos is None else (PartSpec(**pos) if isinstance(pos, dict) else pos)
         self.position = make_part("position", pos, env)
@@ -121,7 +121,7 @@ class LatentCacheAttention(PagedAttentionKernels, Part):
         kv = w["kv_down.weight"]
         rows = [q, padded(kv[:self.rank], self.rankp, d), padded(kv[self.rank:], self.rotp, d)]
         self.c_col = q.shape[0]
-        self.g_col = self.c_col + self.row
+        self.g_col = self.c_col + self.rankp + self.rotp
         if self.gated:
             rows.append(padded(w["gate_proj.weight"].reshape(H, self.vdim, d), H, self.vdimp, d).reshape(-1, d))
         self.w_in = torch.cat(rows, 0).contiguous()                                    # (a multiple of 16 rows)
@@ -154,7 +154,7 @@ class LatentCacheAttention(PagedAttentionKernels, Part):
         tiles = ctx.tables.get(self.step_tables_key) if self.expands else None
         na = n if tiles is None else tiles.n_short_rows                                # rows that run absorbed: the first na
         qa = torch.empty((na, H, self.row), dtype=p.dtype, device=p.device) if na else None
-        K.latent_prep(p, 0, self.c_col, H, self.dimp, self.rotp, self.rank, self.rankp, self.norm_w, self.eps, self.rotary,
+        K.latent_prep(p, 0, self.c_col, H, self.dimp, self.rotp, self.rank, self.rankp, self.row, self.norm_w, self.eps, self.rotary,
                       ctx.positions, view.slot_map, cache.tensor if cache.writes else None, view.page_size, qa, na)
         o = torch.empty((n, H * self.vdimp), dtype=p.dtype, device=p.device)
         gate = p[:, self.g_col:self.g_col + H * self.vdimp] if self.gated else None
@@ -170,10 +170,9 @@ class LatentCacheAttention(PagedAttentionKernels, Part):
         H, n = self.H, p.shape[0]
         heads = lambda x, width: x.unflatten(1, (H, width))
         K.head_gemm(heads(p[:, :H * (self.dimp + self.rotp)], self.dimp + self.rotp)[:, :, :self.dimp], self.w_uk_t, qa[:, :, :self.rankp])
-        n_chunks = -(-ctx.max_context // K.LATENT_CHUNK)
-        ws = self._scratch(K.latent_split_scratch(n, H, self.rankp, n_chunks), p.device)
+        ws = self._scratch(K.latent_split_scratch(n, H, self.rankp, self.row, ctx.max_context, view.page_size, p.dtype), p.device)
         u = torch.empty((n, H, self.rankp), dtype=p.dtype, device=p.device)
-        K.latent_split(qa, cache.tensor, view.block_table, ctx.row_seg[:n], ctx.positions[:n], ws, n_chunks, u, self.scale, view.page_size)
+        K.latent_split(qa, cache.tensor, view.block_table, ctx.row_seg[:n], ctx.positions[:n], ws, ctx.max_context, u, self.scale, view.page_size)
         K.head_gemm(u, self.w_uv, heads(o, self.vdimp), None if gate is None else heads(gate, self.vdimp))
 
     def _expanded(self, p, o, ctx, view, cache, tiles):

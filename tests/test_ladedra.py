@@ -44,7 +44,7 @@ def test_what_every_layer_keeps(name):
         up = lambda n: -(-n // 16) * 16
         if layer["type"] == "latent_attention":
             # one row a token: the latent and the shared key part, nothing a head
-            assert leaves == [PagedKVSpec(1, up(m["kv_rank"]) + up(m["rot_dim"]), planes=1)]
+            assert leaves == [PagedKVSpec(1, -(-(up(m["kv_rank"]) + up(m["rot_dim"])) // 64) * 64, planes=1)]
             continue
         left, right = m["left"], m["right"]
         mask = left.get("mask") or {}

@@ -308,8 +308,8 @@ def test_absorbed_pass_over_cached_latents(dtype, H, rankp, rotp, page):
     takes the sizes) and the scalar form; one key of the first half stands out so that a lost or doubled key shows."""
     from kappai_b200.ops import kernels as Kn
     rng = np.random.default_rng(H + rankp)
-    cache, bt, rows = _latent_rows(rng, LENS, page, rankp, rotp, dtype)
-    W, n = rankp + rotp, len(LENS)
+    W, n = -(-(rankp + rotp) // 64) * 64, len(LENS)
+    cache, bt, rows = _latent_rows(rng, LENS, page, rankp, W - rankp, dtype)
     qa = rng.standard_normal((n, H, W))
     for i, L in enumerate(LENS):
         t = L // 3
@@ -318,16 +318,16 @@ def test_absorbed_pass_over_cached_latents(dtype, H, rankp, rotp, page):
     scale = 3.0 / W
     want = np.stack([P.softmax_with_sink(qa[i] @ rows[i].T * scale, np.ones((H, L), bool)) @ rows[i][:, :rankp] for i, L in enumerate(LENS)])
     perm = rng.permutation(n)
-    for use_mma in ((True, False) if dtype == BF else (False,)):
-        for n_chunks in (-(-max(LENS) // Kn.LATENT_CHUNK), 9):
-            Kn.USE_MMA_LATENT = use_mma
+    for use_tc in ((True, False) if dtype == BF else (False,)):
+        for max_ctx in (max(LENS), 5000):
+            Kn.USE_TC_LATENT = use_tc
             try:
-                ws = torch.full((Kn.latent_split_scratch(n, H, rankp, n_chunks),), float("nan"), device=DEV)
+                ws = torch.full((Kn.latent_split_scratch(n, H, rankp, W, max_ctx, page, dtype),), float("nan"), device=DEV)
                 u = torch.empty((n, H, rankp), dtype=dtype, device=DEV)
-                Kn.latent_split(dev(qa[perm], dtype), dev(cache, dtype), i32(bt), i32(perm), i32([LENS[i] - 1 for i in perm]), ws, n_chunks, u,
+                Kn.latent_split(dev(qa[perm], dtype), dev(cache, dtype), i32(bt), i32(perm), i32([LENS[i] - 1 for i in perm]), ws, max_ctx, u,
                                 scale, page)
             finally:
-                Kn.USE_MMA_LATENT = True
+                Kn.USE_TC_LATENT = True
             close(host(u), want[perm], dtype, tol16=0.01)
     assert Kn.read_status().get("latent", 0) == 0
 
@@ -345,8 +345,8 @@ def test_what_lies_behind_a_rows_keys_does_not_matter():
     cache[:, 0, 0][~used] = np.nan
     qa = rt(rng.standard_normal((3, H, rankp + rotp)), BF)
     u = torch.empty((3, H, rankp), dtype=BF, device=DEV)
-    ws = torch.zeros(Kn.latent_split_scratch(3, H, rankp, 1), device=DEV)
-    Kn.latent_split(dev(qa, BF), dev(cache, BF), i32(bt), i32([0, 1, 2]), i32([L - 1 for L in lens]), ws, 1, u, 0.1, page)
+    ws = torch.zeros(Kn.latent_split_scratch(3, H, rankp, rankp + rotp, 129, page, BF), device=DEV)
+    Kn.latent_split(dev(qa, BF), dev(cache, BF), i32(bt), i32([0, 1, 2]), i32([L - 1 for L in lens]), ws, 129, u, 0.1, page)
     want = np.stack([P.softmax_with_sink(qa[i] @ rows[i].T * 0.1, np.ones((H, L), bool)) @ rows[i][:, :rankp] for i, L in enumerate(lens)])
     close(host(u), want, BF, tol16=0.01)
 
@@ -748,7 +748,7 @@ def test_token_pages_go_back_while_pooled_entries_stay(lad_dirs):
     assert sum(p != RELEASED for p in t) == 3 and all(p == RELEASED for p in t[:(150 - 20 + 1) // 8])
     t = r.cache.block_table("a", pooled)
     assert len(t) == -(-30 // 8) and all(p != RELEASED for p in t)
-    assert r.storage.bytes_per_token([gk for gk in pools if ("planes", 1) in gk][0]) == 4 * (32 + 16)
+    assert r.storage.bytes_per_token([gk for gk in pools if ("planes", 1) in gk][0]) == 2 * 64 * 4
     assert pools[pooled].n_pages < pools[token].n_pages
 
 
