@@ -105,6 +105,94 @@ latent_prep_kernel(T* __restrict__ p, int ld, int q_col, int c_col, int H, int d
     }
 }
 
+// The same for bfloat16 rows on 16-byte boundaries and interleaved pairs, four of them (eight elements) a thread: the row's
+// query parts are fetched before the latent's sum is waited for.  Whole groups of four pairs are rotated (rot % 8 == 0, or
+// nothing is).  PER: groups of eight query elements a thread at most.
+template <int PER>
+__global__ void __launch_bounds__(256)
+latent_prep_vec_kernel(bf16* __restrict__ p, int ld, int q_col, int c_col, int H, int dimp, int rotp, int rank, int rankp, int W,
+                       const float* __restrict__ w, float eps, const float* __restrict__ cos_tab, const float* __restrict__ sin_tab,
+                       int rot, const int* __restrict__ positions, const int* __restrict__ slot_map, bf16* __restrict__ cache,
+                       int page_size, bf16* __restrict__ qa, int n_absorbed) {
+    kp_pdl_begin_early_if(gridDim.x > 1);
+    __shared__ float red[32];
+    const int row = blockIdx.x, tid = threadIdx.x;
+    bf16* pr = p + (size_t)row * ld;
+    const int pos = positions[row], half = rot >> 1;
+    const float* ct = cos_tab ? cos_tab + (size_t)pos * half : nullptr;
+    const float* st = cos_tab ? sin_tab + (size_t)pos * half : nullptr;
+    const int Dq = dimp + rotp, gh = rotp >> 3, n_g = H * gh;      // groups a head, groups a row
+    uint4 q[PER];
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+        const int i = tid + k * 256;
+        if (i < n_g) q[k] = *reinterpret_cast<const uint4*>(pr + q_col + (size_t)(i / gh) * Dq + dimp + (i % gh) * 8);
+    }
+    // the latent: rank / 8 groups and the key part behind it, one a thread (W <= 2048)
+    const int ng = (rankp + rotp) >> 3;
+    uint4 c = make_uint4(0, 0, 0, 0);
+    float f[8];
+    float ss = 0.f;
+    if (tid < ng) c = *reinterpret_cast<const uint4*>(pr + c_col + tid * 8);
+    {
+        const __nv_bfloat162* c2 = reinterpret_cast<const __nv_bfloat162*>(&c);
+#pragma unroll
+        for (int j = 0; j < 4; j++) { const float2 x = __bfloat1622float2(c2[j]); f[2 * j] = x.x; f[2 * j + 1] = x.y; }
+        if (tid * 8 < rankp) {                                     // (columns behind the rank are zero in the product)
+#pragma unroll
+            for (int j = 0; j < 8; j++) ss = fmaf(f[j], f[j], ss);
+        }
+    }
+    ss = block_sum(ss, red);
+    const float scale = 1.0f / sqrtf(ss / (float)rank + eps);
+    auto rotate = [&](uint4 v, int g) {                            // group g of a rotated part
+        if (ct == nullptr || g * 8 >= rot) return v;
+        const float4 cc = __ldg(reinterpret_cast<const float4*>(ct + g * 4)), sn = __ldg(reinterpret_cast<const float4*>(st + g * 4));
+        const float cs[4] = {cc.x, cc.y, cc.z, cc.w}, si[4] = {sn.x, sn.y, sn.z, sn.w};
+        __nv_bfloat162* v2 = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const float2 x = __bfloat1622float2(v2[j]);
+            v2[j] = __floats2bfloat162_rn(x.x * cs[j] - x.y * si[j], x.x * si[j] + x.y * cs[j]);
+        }
+        return v;
+    };
+    const int slot = cache ? slot_map[row] : -1;
+    if (slot >= 0) {
+        bf16* dst = cache + ((size_t)(slot / page_size) * page_size + slot % page_size) * W;
+        if (tid * 8 < W) {
+            uint4 o = make_uint4(0, 0, 0, 0);
+            if (tid * 8 < rankp) {
+                __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    const int e = tid * 8 + 2 * j;
+                    const float w0 = e < rank ? w[e] : 0.f, w1 = e + 1 < rank ? w[e + 1] : 0.f;
+                    o2[j] = __floats2bfloat162_rn((f[2 * j] * scale) * w0, (f[2 * j + 1] * scale) * w1);
+                }
+            } else if (tid < ng) {
+                o = rotate(c, tid - (rankp >> 3));
+            }
+            *reinterpret_cast<uint4*>(dst + tid * 8) = o;
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < PER; k++) {
+        const int i = tid + k * 256;
+        if (i < n_g) {
+            const int h = i / gh, g = i % gh;
+            const uint4 v = rotate(q[k], g);
+            if (ct != nullptr) *reinterpret_cast<uint4*>(pr + q_col + (size_t)h * Dq + dimp + g * 8) = v;
+            if (row < n_absorbed) *reinterpret_cast<uint4*>(qa + ((size_t)row * H + h) * W + rankp + g * 8) = v;
+        }
+    }
+    if (row < n_absorbed && W > rankp + rotp) {
+        const int gz = (W - rankp - rotp) >> 3;
+        for (int i = tid; i < H * gz; i += 256)
+            *reinterpret_cast<uint4*>(qa + ((size_t)row * H + i / gz) * W + rankp + rotp + (i % gz) * 8) = make_uint4(0, 0, 0, 0);
+    }
+}
+
 // ------------------------------------------------------------------------------------------- per-head products
 // out[m, h, n] = sum_k a[m, h, k] b[h][n][k]   (times sigmoid(gate[m, h, n]) if gate).  Row and head strides are given.
 // One CTA: 16 MT rows x 32 columns of one head, four warps of 8 columns; k in stretches of 64, double-buffered.
@@ -266,7 +354,7 @@ latent_split_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_con
     constexpr int NP = 3 * NH;                                     // columns of U^T in tensor memory, a block
     constexpr uint32_t TMEM_COLS = NH == 16 ? 256 : 512;           // S twice, four blocks of U^T
     extern __shared__ unsigned char lt_raw[];
-    unsigned char* sm = reinterpret_cast<unsigned char*>(((uintptr_t)lt_raw + 1023) & ~(uintptr_t)1023);
+    unsigned char* sm = lt_raw + ((1024u - (kp_smem_u32(lt_raw) & 1023u)) & 1023u);      // (by offset: it stays known as shared memory)
     const uint32_t tile_bytes = (uint32_t)p.n_box * LT_BOX_BYTES;
     unsigned char* Ks = sm;                                        // [n_stages][n_box][64 rows x 128 bytes]
     unsigned char* Qs = Ks + (size_t)p.n_stages * tile_bytes;      // [n_box][NH rows x 128 bytes]
@@ -873,6 +961,16 @@ int kp_latent_prep(void* p, int ld, int q_col, int c_col, int H, int dimp, int r
     if (H < 1 || rank < 1 || rank > rankp || (rankp & 15) || (rotp & 15) || rotp < 0 || W < rankp + rotp || page_size < 1 || (cos_tab && (rot < 2 || (rot & 1) || rot > rotp)) ||
         n_absorbed < 0 || n_absorbed > n || (n_absorbed > 0 && !qa))
         return KP_ERR_BAD_ARG;
+    const int groups = H * (rotp >> 3);
+    if (dtype == KP_DTYPE_BF16 && (!cos_tab || (interleaved && (rot & 7) == 0)) && !(ld & 7) && !(q_col & 7) && !(c_col & 7) && !(W & 7) && W <= 2048 &&
+        groups <= 8 * 256 && !(((uintptr_t)p | (uintptr_t)cache | (uintptr_t)qa | (uintptr_t)cos_tab | (uintptr_t)sin_tab) & 15)) {
+#define PREP_VEC(PER)                                                                                                     \
+    kp_launch_pdl(latent_prep_vec_kernel<PER>, dim3(n), dim3(256), 0, (cudaStream_t)stream, (bf16*)p, ld, q_col, c_col, H, dimp, rotp, rank, \
+                  rankp, W, w, eps, cos_tab, sin_tab, rot, positions, slot_map, (bf16*)cache, page_size, (bf16*)qa, n_absorbed)
+        if (groups <= 256) PREP_VEC(1); else if (groups <= 512) PREP_VEC(2); else if (groups <= 1024) PREP_VEC(4); else PREP_VEC(8);
+#undef PREP_VEC
+        return kp_launch_status();
+    }
     KP_DISPATCH_DTYPE(dtype, T, (kp_launch_pdl(latent_prep_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, (T*)p, ld, q_col, c_col, H,
                                                dimp, rotp, rank, rankp, W, w, eps, cos_tab, sin_tab, rot, interleaved, positions,
                                                slot_map, (T*)cache, page_size, (T*)qa, n_absorbed)));

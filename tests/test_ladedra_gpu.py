@@ -352,6 +352,53 @@ def test_what_lies_behind_a_rows_keys_does_not_matter():
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,dim,rdim,rank,rot,interleaved,page", [(3, 24, 8, 20, 8, True, 16), (16, 64, 64, 512, 64, True, 64), (5, 7, 2, 11, 2, True, 8),
+                                                                  (2, 16, 32, 96, 16, True, 32), (4, 32, 16, 48, 16, False, 16), (33, 16, 64, 272, 0, True, 8),
+                                                                  (100, 16, 64, 128, 64, True, 64), (1, 128, 24, 208, 24, True, 4)])
+def test_what_stands_in_front_of_the_latent_passes(H, dim, rdim, rank, rot, interleaved, page, dtype):
+    """The latent's norm, the rotations, the cache rows and the absorbed rows' query parts, in both forms of the kernel."""
+    from kappai_b200.config.schema import PartSpec
+    from kappai_b200.ops import kernels as Kn
+    from kappai_b200.parts import make_part
+    from test_parts_gpu import env_for
+    up = lambda n, m=16: -(-n // m) * m
+    dimp, rotp, rankp = up(dim), up(rdim), up(rank)
+    W, n, na, eps = up(rankp + rotp, 64), 21, 13, 1e-3
+    rng = np.random.default_rng(H + rank)
+    pos = rng.integers(0, 400, n)
+    q, c = np.zeros((n, H, dimp + rotp)), np.zeros((n, rankp + rotp))
+    q[:, :, :dim], q[:, :, dimp:dimp + rdim] = rng.standard_normal((n, H, dim)), rng.standard_normal((n, H, rdim))
+    c[:, :rank], c[:, rankp:rankp + rdim] = rng.standard_normal((n, rank)) * 0.4, rng.standard_normal((n, rdim))
+    q, c, w = rt(q, dtype), rt(c, dtype), rt(1 + 0.2 * rng.standard_normal(rank), torch.float32)
+    wide = dev(np.concatenate([q.reshape(n, -1), c, np.ones((n, 8))], 1), dtype)
+    sc = {"factor": 16.0, "original": 64, "fast": 8.0, "slow": 1.0}
+    rc = {"dims": rot, "base": 300.0, "scaling": sc} if rot else None
+    spec = PartSpec("rope", {"rotary_dim": rot, "theta": 300.0, "scaling": sc, "pairing": "interleaved" if interleaved else "neox"}) if rot else PartSpec("none")
+    n_pages = -(-n // page) + 2
+    slots = rng.permutation(n_pages * page)[:n]
+    cache = torch.full((n_pages, 1, 1, page, W), 7.0, dtype=dtype, device=DEV)
+    qa = torch.full((na, H, W), 9.0, dtype=dtype, device=DEV)
+    Kn.latent_prep(wide, 0, H * (dimp + rotp), H, dimp, rotp, rank, rankp, W, dev(w), eps, make_part("position", spec, env_for(dtype)).fused_rotary(), i32(pos),
+                   i32(slots), cache, page, qa, na)
+    turn = lambda x: np.concatenate([P.rotate(x[j:j + 1], rc, interleaved, int(pos[j])) for j in range(n)])
+    got = host(cache)
+    rows = np.stack([got[s // page, 0, 0, s % page] for s in slots])
+    want = np.zeros((n, W))
+    want[:, :rank] = P.rms(c[:, :rank], eps) * w
+    want[:, rankp:rankp + rdim] = turn(c[:, None, rankp:rankp + rdim])[:, 0]
+    close(rows, want, dtype)
+    assert np.all(rows[:, rank:rankp] == 0) and np.all(rows[:, rankp + rdim:] == 0) and (got == 7.0).sum() == (n_pages * page - n) * W
+    qr = turn(q[:, :, dimp:dimp + rdim])
+    out = host(wide)
+    got_q = out[:, :H * (dimp + rotp)].reshape(n, H, -1)
+    close(got_q[:, :, dimp:dimp + rdim], qr, dtype)
+    assert np.array_equal(got_q[:, :, :dimp], q[:, :, :dimp]) and np.all(out[:, -8:] == 1.0)
+    a = host(qa)
+    close(a[:, :, rankp:rankp + rdim], qr[:na], dtype)
+    assert np.all(a[:, :, :rankp] == 9.0) and np.all(a[:, :, rankp + rdim:] == 0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("M,H,N,K,gate", [(1, 3, 32, 16, False), (8, 16, 512, 64, False), (16, 5, 48, 272, True), (17, 2, 64, 80, True), (33, 4, 16, 128, False),
                                           (100, 3, 208, 32, True), (64, 1, 96, 96, False)])
 def test_per_head_products(M, H, N, K, gate, dtype):
