@@ -13,7 +13,8 @@
 //    products (head_gemm), a pass over chunks of keys (latent_split: bfloat16 on the tcgen05 tensor cores, or scalar) that
 //    leaves each chunk's maximum, sum and unnormalised latent, and a merge in chunk order.
 //  * expanded (prompt portions): the latents of the request's whole context are gathered from its pages, one product
-//    expands them, and latent_prefill runs tiles of 64 query rows over the expanded rows.
+//    expands them, and latent_prefill runs tiles of query rows over the expanded rows (128 rows on the tcgen05 tensor cores,
+//    or 64 with mma.sync where the sizes are none of theirs).
 //
 // The softmax statistics are float32; its weights enter the products whole, as three bfloat16 parts.  The
 // scalar form's chunks lie at multiples of 256 keys, so in the 32-bit mode the order of a row's sums does not depend on how its
@@ -933,6 +934,280 @@ latent_prefill_kernel(const LatentPrefillArgs p) {
     }
 }
 
+// The expanded pass on the 5th-generation tensor cores: one CTA takes 128 query rows of a segment and one head, over tiles of
+// 64 keys.
+//
+//   S  = Q K^T     128 x 64: Q and the tile's key parts K-major, by TMA (boxes of 64 columns, 128-byte swizzle): the expanded
+//                  unrotated part and the shared rotated part stand in boxes of their own, and only the steps of 16
+//                  columns that the parts have are multiplied;
+//   PV = P V       128 x vdimp: the float32 weights as three bfloat16 parts, multiplied one after the other into the same
+//                  columns, so that they enter whole; V as it lies (keys x columns: the MN-major operand).
+//
+// Roles by warp: 0 TMA (Q once, a ring of two tiles), 1 tensor memory and MMA of S, 2 - 9 the rows, 10 MMA of PV.  A row has
+// two threads (two groups of four warps, a lane quarter each): both take the maximum of its 64 scores, each the exponentials
+// of half of its keys and the sums of half of its value columns, which stay in registers and are rescaled there, so
+// nothing rescales tensor memory.  S and the weights are double-buffered: a tile's softmax runs while the tile before it is
+// multiplied.  `gate` (or null): the output is multiplied by sigmoid(gate) on its way out.
+// Every wait is bounded; one that gives up sets the status word and an abort flag, and the CTA frees its tensor memory
+// and returns.
+#define LE_ROWS 128
+#define LE_KEYS 64
+#define LE_STAGES 2
+#define LE_THREADS 352
+#define LE_Q_BOX (LE_ROWS * 128)
+#define LE_K_BOX (LE_KEYS * 128)
+#define LE_TMEM 256                                                // S twice (64 columns each), PV (at most 128)
+
+struct LatentExpandedArgs {
+    const bf16* gate; bf16* out;
+    const int* cu_rows; const int* seg_pos; const int* tile_seg; const int* tile_row0; const int* ctx_base;
+    int ldo, ldg, rankp, dimp, rotp, vdimp, v_col;
+    float scale;
+};
+
+__global__ void __launch_bounds__(LE_THREADS, 1)
+latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmE, const __grid_constant__ CUtensorMap tmR,
+                         const LatentExpandedArgs p) {
+    extern __shared__ unsigned char le_raw[];
+    unsigned char* sm = le_raw + ((1024u - (kp_smem_u32(le_raw) & 1023u)) & 1023u);
+    const int nb = (p.dimp + 63) >> 6, rb = (p.rotp + 63) >> 6, vb = (p.vdimp + 63) >> 6;      // boxes of the three parts
+    const uint32_t stage_bytes = (uint32_t)(nb + rb + vb) * LE_K_BOX;
+    unsigned char* Qs = sm;                                        // [nb + rb][128 rows x 128 bytes]
+    unsigned char* St = Qs + (size_t)(nb + rb) * LE_Q_BOX;         // [LE_STAGES][nb + rb + vb][64 rows x 128 bytes]
+    unsigned char* Ps = St + LE_STAGES * stage_bytes;              // [2][3 parts][128 rows x 128 bytes]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(Ps + 2 * 3 * LE_Q_BOX);
+    uint64_t* q_full = bars;
+    uint64_t* k_full = bars + 1;                                   // [LE_STAGES]
+    uint64_t* k_empty = k_full + LE_STAGES;                        // [LE_STAGES]
+    uint64_t* s_full = k_empty + LE_STAGES;                        // [2]
+    uint64_t* p_full = s_full + 2;                                 // [2]
+    uint64_t* o_full = p_full + 2;
+    uint64_t* o_empty = o_full + 1;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_empty + 1);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (threadIdx.x == 0) {
+        kp_mbar_init(q_full, 1);
+        for (int s = 0; s < LE_STAGES; s++) { kp_mbar_init(&k_full[s], 1); kp_mbar_init(&k_empty[s], 1); }
+        for (int b = 0; b < 2; b++) { kp_mbar_init(&s_full[b], 1); kp_mbar_init(&p_full[b], 256); }
+        kp_mbar_init(o_full, 1);
+        kp_mbar_init(o_empty, 8);
+        *abort_flag = 0;
+        kp_mbar_init_fence();
+    }
+    if (warp == 1) kp_tmem_alloc(tmem_slot, LE_TMEM);
+    kp_tc_fence_before();
+    __syncthreads();
+    kp_tc_fence_after();
+    const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 2 * LE_KEYS;
+    kp_pdl_begin();
+    const int h = blockIdx.y, seg = p.tile_seg[blockIdx.x], row0 = p.tile_row0[blockIdx.x];
+    const int n_rows = min(LE_ROWS, p.cu_rows[seg + 1] - row0);
+    const int pos0 = p.seg_pos[seg] + (row0 - p.cu_rows[seg]);
+    const int k_hi = pos0 + n_rows - 1, n_kt = k_hi / LE_KEYS + 1;
+    const int Dq = p.dimp + p.rotp;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            const int base = p.ctx_base[seg];
+            kp_mbar_expect_tx(q_full, (uint32_t)(nb + rb) * LE_Q_BOX);
+            for (int j = 0; j < nb; j++) kp_tma_load_2d(Qs + (size_t)j * LE_Q_BOX, &tmQ, h * Dq + j * 64, row0, q_full);
+            for (int j = 0; j < rb; j++) kp_tma_load_2d(Qs + (size_t)(nb + j) * LE_Q_BOX, &tmQ, h * Dq + p.dimp + j * 64, row0, q_full);
+            for (int kt = 0; kt < n_kt; kt++) {
+                const int s = kt % LE_STAGES;
+                if (*abort_flag || !kp_mbar_wait_bounded(&k_empty[s], ((kt / LE_STAGES) & 1) ^ 1)) { *abort_flag = 1; break; }
+                unsigned char* st = St + (size_t)s * stage_bytes;
+                const int y = base + kt * LE_KEYS;
+                kp_mbar_expect_tx(&k_full[s], stage_bytes);
+                for (int j = 0; j < nb; j++) kp_tma_load_2d(st + (size_t)j * LE_K_BOX, &tmE, h * p.dimp + j * 64, y, &k_full[s]);
+                for (int j = 0; j < rb; j++) kp_tma_load_2d(st + (size_t)(nb + j) * LE_K_BOX, &tmR, p.rankp + j * 64, y, &k_full[s]);
+                for (int j = 0; j < vb; j++)
+                    kp_tma_load_2d(st + (size_t)(nb + rb + j) * LE_K_BOX, &tmE, p.v_col + h * p.vdimp + j * 64, y, &k_full[s]);
+            }
+        }
+    } else if (warp == 1) {
+        constexpr uint32_t idesc = kp_umma_idesc(LE_ROWS, LE_KEYS);
+        const uint64_t q_desc = kp_umma_desc(kp_smem_u32(Qs)), k_desc = kp_umma_desc(kp_smem_u32(St));
+        const int n_d = p.dimp >> 4, n_r = p.rotp >> 4;            // steps of 16 columns
+        bool ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(q_full, 0));
+        for (int kt = 0; kt < n_kt && ok; kt++) {
+            const int s = kt % LE_STAGES;
+            ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&k_full[s], (kt / LE_STAGES) & 1));
+            if (ok && kt > 1) ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&p_full[kt & 1], ((kt - 2) >> 1) & 1));
+            if (!ok || __any_sync(0xffffffffu, *abort_flag)) { ok = false; break; }
+            kp_tc_fence_after();
+            const uint64_t kd = k_desc + s * (stage_bytes >> 4);
+            const uint32_t d = tmem_s + (kt & 1) * LE_KEYS;
+            for (int k = 0; k < n_d; k++)
+                kp_umma_bf16_warp(d, q_desc + (k >> 2) * (LE_Q_BOX >> 4) + 2 * (k & 3), kd + (k >> 2) * (LE_K_BOX >> 4) + 2 * (k & 3), idesc, k ? 1u : 0u);
+            for (int k = 0; k < n_r; k++)
+                kp_umma_bf16_warp(d, q_desc + (nb + (k >> 2)) * (LE_Q_BOX >> 4) + 2 * (k & 3), kd + (nb + (k >> 2)) * (LE_K_BOX >> 4) + 2 * (k & 3),
+                                  idesc, 1u);
+            kp_umma_commit_warp(&s_full[kt & 1]);
+        }
+        if (!ok) *abort_flag = 1;
+    } else if (warp == 10) {
+        const uint32_t idesc = kp_umma_idesc(LE_ROWS, p.vdimp, true);
+        const uint64_t p_desc = kp_umma_desc(kp_smem_u32(Ps)), v_desc = kp_umma_desc_mn(kp_smem_u32(St) + (nb + rb) * LE_K_BOX, LE_K_BOX);
+        bool ok = true;
+        for (int kt = 0; kt < n_kt && ok; kt++) {
+            const int s = kt % LE_STAGES;
+            ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&p_full[kt & 1], (kt >> 1) & 1));
+            if (ok && kt > 0) ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(o_empty, (kt - 1) & 1));
+            if (!ok || __any_sync(0xffffffffu, *abort_flag)) { ok = false; break; }
+            kp_tc_fence_after();
+            const uint64_t pd = p_desc + (kt & 1) * (3 * LE_Q_BOX >> 4), vd = v_desc + s * (stage_bytes >> 4);
+            for (int part = 0; part < 3; part++) {
+#pragma unroll
+                for (int kk = 0; kk < LE_KEYS / 16; kk++)
+                    kp_umma_bf16_warp(tmem_o, pd + part * (LE_Q_BOX >> 4) + 2 * kk, vd + kk * (2048 >> 4), idesc, (part | kk) ? 1u : 0u);
+            }
+            kp_umma_commit_warp(o_full);
+            kp_umma_commit_warp(&k_empty[s]);
+        }
+        if (!ok) *abort_flag = 1;
+    } else {
+        const int grp = (warp - 2) >> 2, q4 = warp & 3, r = q4 * 32 + lane;            // r: this thread's row
+        const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
+        const int pos = pos0 + r, vh = p.vdimp >> 1;               // the thread's value columns: vh from grp * vh on
+        const float sl2 = p.scale * 1.4426950408889634f;
+        float acc[64];
+#pragma unroll
+        for (int i = 0; i < 64; i++) acc[i] = 0.f;
+        float m = -INFINITY, l = 0.f, corr_next = 0.f;
+        bool ok = true;
+        auto softmax = [&](int kt) {
+            const int b = kt & 1;
+            if (ok) ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(&s_full[b], (kt >> 1) & 1) && !*abort_flag);    // (a warp gives up as one)
+            if (!ok) return;
+            kp_tc_fence_after();
+            const uint32_t ts = tmem_s + b * LE_KEYS + lane_off;
+            const int k0 = kt * LE_KEYS;
+            uint32_t mine[32];
+            float mx = -INFINITY;
+            {
+                uint32_t other[32];
+                kp_tmem_ld32_issue(ts + (grp ^ 1) * 32, other);
+                kp_tmem_ld32_issue(ts + grp * 32, mine);
+                kp_tmem_ld_wait();
+                if (k0 + LE_KEYS - 1 > pos0) {                     // the tile reaches beyond the first row's position
+#pragma unroll
+                    for (int j = 0; j < 32; j++) {
+                        if (k0 + (grp ^ 1) * 32 + j <= pos) mx = fmaxf(mx, __uint_as_float(other[j]));
+                        if (k0 + grp * 32 + j > pos) mine[j] = 0xff800000u;                 // -inf
+                        mx = fmaxf(mx, __uint_as_float(mine[j]));
+                    }
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 32; j++) mx = fmaxf(mx, fmaxf(__uint_as_float(other[j]), __uint_as_float(mine[j])));
+                }
+            }
+            if (kt == n_kt - 1 && k_hi + 1 - k0 < LE_KEYS) {
+                // the last tile: values of keys behind the context (another request's, or nobody's) meet weights of 0 and are
+                // cleared (0 times NaN is not 0)
+                const int first = k_hi + 1 - k0;
+                unsigned char* vt = St + (size_t)(kt % LE_STAGES) * stage_bytes + (size_t)(nb + rb) * LE_K_BOX;
+                for (int i = threadIdx.x - 64; i < (LE_KEYS - first) * vb * 8; i += 256)
+                    *reinterpret_cast<uint4*>(vt + (size_t)((i >> 3) % vb) * LE_K_BOX + (first + (i >> 3) / vb) * 128 + (i & 7) * 16) = make_uint4(0, 0, 0, 0);
+            }
+            const float m_new = fmaxf(m, mx * sl2);                // (finite: every row sees key 0)
+            corr_next = la_exp2(m - m_new);
+            m = m_new;
+            unsigned char* pr = Ps + (size_t)b * 3 * LE_Q_BOX + r * 128;
+            float sum = 0.f;
+#pragma unroll
+            for (int c = 0; c < 4; c++) {                          // eight keys: a 16-byte piece of the row in each part
+                float w[8];
+#pragma unroll
+                for (int j = 0; j < 8; j++) { w[j] = la_exp2(fmaf(__uint_as_float(mine[c * 8 + j]), sl2, -m_new)); sum += w[j]; }
+                const int piece = ((grp * 4 + c) ^ (r & 7)) << 4;
+#pragma unroll
+                for (int part = 0; part < 3; part++) {
+                    uint4 o;
+                    o.x = pack_bf16_part(w[0], w[1]); o.y = pack_bf16_part(w[2], w[3]);
+                    o.z = pack_bf16_part(w[4], w[5]); o.w = pack_bf16_part(w[6], w[7]);
+                    *reinterpret_cast<uint4*>(pr + (size_t)part * LE_Q_BOX + piece) = o;
+                }
+            }
+            l = fmaf(l, corr_next, sum);
+            kp_tc_fence_before();                                  // the reads of S are done
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the weights are read by the tensor core
+            kp_mbar_arrive(&p_full[b]);
+        };
+        softmax(0);
+        for (int kt = 0; kt < n_kt && ok; kt++) {
+            const float corr = corr_next;
+            if (kt + 1 < n_kt) softmax(kt + 1);
+            if (ok) ok = __all_sync(0xffffffffu, kp_mbar_wait_bounded(o_full, kt & 1) && !*abort_flag);
+            if (!ok) break;
+            kp_tc_fence_after();
+#pragma unroll
+            for (int c = 0; c < 4; c += 2) {
+                if (c * 16 < vh) {
+                    uint32_t u[2][16];
+                    kp_tmem_ld16_issue(tmem_o + lane_off + grp * vh + c * 16, u[0]);
+                    if ((c + 1) * 16 < vh) kp_tmem_ld16_issue(tmem_o + lane_off + grp * vh + (c + 1) * 16, u[1]);
+                    kp_tmem_ld_wait();
+#pragma unroll
+                    for (int i = 0; i < 16; i++) acc[c * 16 + i] = fmaf(acc[c * 16 + i], corr, __uint_as_float(u[0][i]));
+                    if ((c + 1) * 16 < vh) {
+#pragma unroll
+                        for (int i = 0; i < 16; i++) acc[c * 16 + 16 + i] = fmaf(acc[c * 16 + 16 + i], corr, __uint_as_float(u[1][i]));
+                    }
+                }
+            }
+            kp_tc_fence_before();
+            __syncwarp();
+            if (lane == 0) kp_mbar_arrive(o_empty);
+        }
+        if (!ok) *abort_flag = 1;
+        // the two threads of a row put their sums together (every product has read Q by now: its place takes them)
+        float* sums = reinterpret_cast<float*>(Qs);
+        sums[grp * LE_ROWS + r] = l;
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (ok && r < n_rows) {
+            const float inv = 1.0f / (sums[r] + sums[LE_ROWS + r]);
+            const size_t col = (size_t)h * p.vdimp + grp * vh;
+            bf16* dst = p.out + (size_t)(row0 + r) * p.ldo + col;
+            const bf16* g = p.gate ? p.gate + (size_t)(row0 + r) * p.ldg + col : nullptr;
+#pragma unroll
+            for (int c = 0; c < 64; c += 8) {
+                if (c < vh) {
+                    float f[8];
+#pragma unroll
+                    for (int i = 0; i < 8; i++) f[i] = acc[c + i] * inv;
+                    if (g) {
+                        const uint4 raw = *reinterpret_cast<const uint4*>(g + c);
+                        const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                        for (int i = 0; i < 4; i++) {
+                            const float2 z = __bfloat1622float2(z2[i]);
+                            f[2 * i] /= 1.0f + expf(-z.x);
+                            f[2 * i + 1] /= 1.0f + expf(-z.y);
+                        }
+                    }
+                    uint4 o;
+                    o.x = pack_bf16(f[0], f[1]); o.y = pack_bf16(f[2], f[3]); o.z = pack_bf16(f[4], f[5]); o.w = pack_bf16(f[6], f[7]);
+                    *reinterpret_cast<uint4*>(dst + c) = o;
+                }
+            }
+        }
+    }
+    kp_tc_fence_before();
+    __syncthreads();
+    if (*abort_flag) {
+        if (threadIdx.x == 0) atomicExch(&g_latent_status, 1);
+        kp_linger_after_failure();
+    }
+    if (warp == 1) kp_tmem_dealloc(tmem_s, LE_TMEM);
+}
+
+static size_t le_smem(int dimp, int rotp, int vdimp) {
+    const int nb = (dimp + 63) / 64, rb = (rotp + 63) / 64, vb = (vdimp + 63) / 64;
+    return 1024 + (size_t)(nb + rb) * LE_Q_BOX + (size_t)LE_STAGES * (nb + rb + vb) * LE_K_BOX + 6 * LE_Q_BOX + (2 * LE_STAGES + 7) * 8 + 16;
+}
+
 static size_t lt_fixed_bytes(int n_box, int nh) {
     return 1024 + (size_t)n_box * nh * 128 + 2 * 3 * nh * 128 + 16 * nh * sizeof(float) + (2 * LT_MAX_STAGES + 7) * 8 + 16;
 }
@@ -1073,6 +1348,36 @@ int kp_latent_gather(const void* cache, const int* block_table, int max_blocks, 
     if (n_seg < 1 || page_size < 1 || (W & 7)) return KP_ERR_BAD_ARG;
     kp_launch_pdl(latent_gather_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, (cudaStream_t)stream, (const bf16*)cache, block_table, max_blocks,
                   ctx_base, n_seg, (bf16*)out, n_rows, page_size, W);
+    return kp_launch_status();
+}
+
+// 1 if the tcgen05 form of the expanded pass takes these sizes.
+int kp_latent_prefill_tc_ok(int dimp, int rotp, int vdimp) {
+    return !(dimp & 15) && !(rotp & 15) && dimp >= 16 && rotp >= 16 && vdimp >= 32 && vdimp % 32 == 0 && vdimp <= 128 &&
+           le_smem(dimp, rotp, vdimp) <= LT_SMEM_MAX;
+}
+
+// As kp_latent_prefill, with tiles of 128 rows, on the tcgen05 tensor cores; n_rows rows of q, n_ctx rows of ex and `rows`; gate
+// (rows ldg apart, H heads of vdimp) or null: the output times sigmoid(gate).
+int kp_latent_prefill_tc(const void* q, int ldq, int n_rows, const void* ex, int ld_ex, int v_col, const void* rows, int n_ctx, int W, int rankp,
+                         int dimp, int rotp, int vdimp, const int* cu_rows, const int* seg_pos, const int* tile_seg, const int* tile_row0,
+                         const int* ctx_base, int n_tiles, const void* gate, int ldg, void* out, int ldo, float scale, int H, void* stream) {
+    if (n_tiles <= 0) return 0;
+    if (!kp_latent_prefill_tc_ok(dimp, rotp, vdimp) || (rankp & 15) || W < rankp + rotp || H < 1 || H > 65535 || n_rows < 1 || n_ctx < 1)
+        return KP_ERR_BAD_ARG;
+    if ((ldq & 7) || (ldo & 7) || (ld_ex & 7) || (v_col & 7) || (W & 7) || (gate && (ldg & 7)) ||
+        (((uintptr_t)q | (uintptr_t)ex | (uintptr_t)rows | (uintptr_t)out | (uintptr_t)gate) & 15))
+        return KP_ERR_UNSUPPORTED;
+    alignas(64) CUtensorMap tq, te, tr;
+    int st = kp_make_map_bf16_2d(&tq, q, (unsigned long long)n_rows, H * (dimp + rotp), ldq, 64, LE_ROWS);
+    if (!st) st = kp_make_map_bf16_2d(&te, ex, (unsigned long long)n_ctx, v_col + H * vdimp, ld_ex, 64, LE_KEYS);
+    if (!st) st = kp_make_map_bf16_2d(&tr, rows, (unsigned long long)n_ctx, W, W, 64, LE_KEYS);
+    if (st) return st;
+    const size_t sm = le_smem(dimp, rotp, vdimp);
+    st = la_set_smem(latent_prefill_tc_kernel, sm);
+    if (st) return st;
+    LatentExpandedArgs a = {(const bf16*)gate, (bf16*)out, cu_rows, seg_pos, tile_seg, tile_row0, ctx_base, ldo, ldg, rankp, dimp, rotp, vdimp, v_col, scale};
+    kp_launch_pdl(latent_prefill_tc_kernel, dim3(n_tiles, H), dim3(LE_THREADS), sm, (cudaStream_t)stream, tq, te, tr, a);
     return kp_launch_status();
 }
 

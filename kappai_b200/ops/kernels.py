@@ -1400,7 +1400,7 @@ def attention_prefill(q: torch.Tensor, cache: torch.Tensor, block_table: torch.T
 # ------------------------------------------------------------------ attention over cached latents
 
 LATENT_PREFILL_MAX = (256, 256)    # key and value columns a head that the expanded pass takes
-USE_TC_LATENT = True           # the absorbed pass of bfloat16 rows runs on the tcgen05 tensor cores where the sizes allow it
+USE_TC_LATENT = True           # both latent passes of bfloat16 rows run on the tcgen05 tensor cores where the sizes allow it
 
 
 def latent_prep(p: torch.Tensor, q_col: int, c_col: int, H: int, dimp: int, rotp: int, rank: int, rankp: int, W: int, w: torch.Tensor,
@@ -1499,6 +1499,36 @@ def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, ctx_base: torc
     out = torch.empty((n_rows, W), dtype=cache.dtype, device=cache.device)
     _run("latent_gather", load_library("latent").kp_latent_gather, _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(ctx_base), n_seg,
          _ptr(out), n_rows, page_size, W, STREAM)
+    return out
+
+
+def latent_prefill_tc_ok(q: torch.Tensor, ex: torch.Tensor, dimp: int, rotp: int, vdimp: int) -> bool:
+    """Can the tcgen05 form of the expanded pass take this call?"""
+    return (USE_TC_LATENT and q.dtype == torch.bfloat16 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and ex.stride(0) % 8 == 0
+            and bool(load_library("latent").kp_latent_prefill_tc_ok(dimp, rotp, vdimp)))
+
+
+def latent_prefill_tc(q: torch.Tensor, ex: torch.Tensor, rows: torch.Tensor, rankp: int, dimp: int, rotp: int, vdimp: int,
+                      cu_rows: torch.Tensor, seg_pos: torch.Tensor, big_tile_seg: torch.Tensor, big_tile_row0: torch.Tensor,
+                      ctx_base: torch.Tensor, out: torch.Tensor, scale: float, H: int, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """As :func:`latent_prefill`, over tiles of 128 rows, on the tcgen05 tensor cores; ``gate`` [n, H vdimp] (rows may be strided):
+    the output leaves times ``sigmoid(gate)``."""
+    _need(q, "q", torch.bfloat16, contiguous=False); _need(ex, "ex", torch.bfloat16); _need(rows, "rows", torch.bfloat16)
+    _need(out, "out", torch.bfloat16, contiguous=False)
+    for t, nm in ((cu_rows, "cu_rows"), (seg_pos, "seg_pos"), (big_tile_seg, "tile_seg"), (big_tile_row0, "tile_row0"), (ctx_base, "ctx_base")):
+        _need(t, nm, torch.int32)
+    n = q.shape[0]
+    if (q.shape[1] != H * (dimp + rotp) or tuple(out.shape) != (n, H * vdimp) or ex.shape[1] != H * (dimp + vdimp)
+            or rows.shape[0] != ex.shape[0] or rows.shape[1] < rankp + rotp or big_tile_seg.numel() != big_tile_row0.numel()):
+        raise KernelError("latent_prefill_tc: shape mismatch")
+    if gate is not None:
+        _need(gate, "gate", torch.bfloat16, contiguous=False)
+        if gate.shape != out.shape:
+            raise KernelError("latent_prefill_tc: gate shape")
+    _run("latent_prefill_tc", load_library("latent").kp_latent_prefill_tc, _ptr(q), _rows_2d(q, "q"), n, _ptr(ex), ex.shape[1], H * dimp, _ptr(rows),
+         rows.shape[0], rows.shape[1], rankp, dimp, rotp, vdimp, _ptr(cu_rows), _ptr(seg_pos), _ptr(big_tile_seg), _ptr(big_tile_row0), _ptr(ctx_base),
+         big_tile_seg.numel(), _ptr(gate), _rows_2d(gate, "gate") if gate is not None else 0, _ptr(out), _rows_2d(out, "out"), ctypes.c_float(scale), H,
+         STREAM)
     return out
 
 

@@ -13,10 +13,12 @@ is the kind that expands the latents before it caches them.)
 Decoded tokens, short portions and every row of the 32-bit mode run *absorbed*: the expanding matrices are applied to the
 query and to the weighted sum of latents, and all heads read the cached rows as they are.  Longer portions (16-bit mode)
 run *expanded*: the latents of the request's whole context are gathered from its pages, one product makes the heads'
-keys and values of them, and a tiled kernel reads those.  csrc/latent.cu has the kernels and how they sum.
+keys and values of them, and a tiled kernel reads those (on the tcgen05 tensor cores for value heads of up to 128 columns).
+csrc/latent.cu has the kernels and how they sum.
 
 The query, the latent, the key part and the gate read the layer's input in one product; one kernel norms and rotates
-what comes out of it and writes the cache row.  The gate of absorbed rows runs in the epilogue of their last product.
+what comes out of it and writes the cache row.  The gate of absorbed rows runs in the epilogue of their last product, that
+of expanded rows in the attention kernel's last store.
 
 Params: hidden_size, num_heads, head_dim, rot_dim, value_dim, kv_rank, scale, norm_eps, gate (None | "sigmoid"), position (None
 | a rope PartSpec over at most rot_dim dimensions).
@@ -50,8 +52,6 @@ def latent_tiles(segs):
     lead = tables.scalars["n_short_tiles"]
     ctx = [0 if i < lead else int(segs.seg_pos[i]) + segs.seg_len[i] for i in range(segs.n_seg)]
     base = np.concatenate([[0], np.cumsum(ctx)]).astype(np.int32)
-    for name in ("big_tile_seg", "big_tile_row0"):
-        del tables.arrays[name]
     tables.arrays["ctx_base"] = base
     tables.scalars["n_ctx"] = int(base[-1])
     return tables
@@ -161,9 +161,7 @@ class LatentCacheAttention(PagedAttentionKernels, Part):
         if na:
             self._absorbed(p[:na], qa, o[:na], gate[:na] if self.gated else None, ctx, view, cache)
         if na < n:
-            self._expanded(p, o, ctx, view, cache, tiles)
-            if self.gated:
-                K.sigmoid_gate(o[na:], gate[na:])
+            self._expanded(p, o, gate, ctx, view, cache, tiles)
         linear(o, self.w_o, out=residual, accumulate=True)
 
     def _absorbed(self, p, qa, o, gate, ctx, view, cache):
@@ -175,12 +173,19 @@ class LatentCacheAttention(PagedAttentionKernels, Part):
         K.latent_split(qa, cache.tensor, view.block_table, ctx.row_seg[:n], ctx.positions[:n], ws, ctx.max_context, u, self.scale, view.page_size)
         K.head_gemm(u, self.w_uv, heads(o, self.vdimp), None if gate is None else heads(gate, self.vdimp))
 
-    def _expanded(self, p, o, ctx, view, cache, tiles):
-        H, t0 = self.H, tiles.n_short_tiles
+    def _expanded(self, p, o, gate, ctx, view, cache, tiles):
+        H, t0, na = self.H, tiles.n_short_tiles, tiles.n_short_rows
         rows = K.latent_gather(cache.tensor, view.block_table, tiles.ctx_base, tiles.n_ctx, view.page_size)
         ex = linear(rows[:, :self.rankp], self.w_ex)
-        K.latent_prefill(p[:, :H * (self.dimp + self.rotp)], ex, rows, self.rankp, self.dimp, self.rotp, self.vdimp, ctx.cu_rows, ctx.seg_pos,
-                         tiles.tile_seg[t0:], tiles.tile_row0[t0:], tiles.ctx_base, o, self.scale, H)
+        q, sizes = p[:, :H * (self.dimp + self.rotp)], (self.rankp, self.dimp, self.rotp, self.vdimp)
+        if K.latent_prefill_tc_ok(q, ex, self.dimp, self.rotp, self.vdimp):
+            K.latent_prefill_tc(q, ex, rows, *sizes, ctx.cu_rows, ctx.seg_pos, tiles.big_tile_seg, tiles.big_tile_row0, tiles.ctx_base, o,
+                                self.scale, H, gate)
+            return
+        K.latent_prefill(q, ex, rows, *sizes, ctx.cu_rows, ctx.seg_pos, tiles.tile_seg[t0:], tiles.tile_row0[t0:], tiles.ctx_base, o,
+                         self.scale, H)
+        if gate is not None:
+            K.sigmoid_gate(o[na:], gate[na:])
 
 
 register_part("mixer", "latent_cache_attention", LatentCacheAttention)

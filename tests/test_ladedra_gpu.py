@@ -419,7 +419,8 @@ def test_per_head_products(M, H, N, K, gate, dtype):
 
 
 @pytest.mark.parametrize("H,dimp,rotp,vdimp,rankp,page", [(3, 32, 16, 16, 32, 16), (4, 64, 64, 64, 128, 64), (2, 128, 64, 128, 112, 32), (5, 16, 16, 80, 48, 8),
-                                                          (2, 192, 64, 160, 64, 16), (1, 96, 32, 256, 32, 64)])
+                                                          (2, 192, 64, 160, 64, 16), (1, 96, 32, 256, 32, 64), (3, 48, 80, 96, 64, 16), (2, 16, 16, 32, 16, 8),
+                                                          (1, 16, 16, 32, 16, 8)])
 def test_expanded_pass_over_gathered_latents(H, dimp, rotp, vdimp, rankp, page):
     """Whole prompts and late portions behind a lead of short segments that another pass takes; the gathered rows too."""
     from kappai_b200.ops import kernels as Kn
@@ -434,12 +435,26 @@ def test_expanded_pass_over_gathered_latents(H, dimp, rotp, vdimp, rankp, page):
     ex = rt(rng.standard_normal((len(all_rows), H * (dimp + vdimp))), BF)
     cu, seg_pos, tile_seg, tile_row0, _, _ = _portions(lens, q_from)
     q = rt(rng.standard_normal((cu[-1], H * (dimp + rotp) + 8)), BF)
+    gate = rt(rng.standard_normal((cu[-1], H * vdimp + 16)) * 2, BF)
     scale = 2.0 / math.sqrt(dimp + rotp)
     out = torch.full((cu[-1], H * vdimp), 7.0, dtype=BF, device=DEV)
-    Kn.latent_prefill(dev(q, BF)[:, :H * (dimp + rotp)], dev(ex, BF), got_rows, rankp, dimp, rotp, vdimp, i32(cu), i32(seg_pos), i32(tile_seg)[1:],
+    qt = dev(q, BF)[:, :H * (dimp + rotp)]
+    Kn.latent_prefill(qt, dev(ex, BF), got_rows, rankp, dimp, rotp, vdimp, i32(cu), i32(seg_pos), i32(tile_seg)[1:],
                       i32(tile_row0)[1:], i32(base), out, scale, H)
     got = host(out)
     assert np.all(got[0] == 7.0)
+    tc = Kn.latent_prefill_tc_ok(qt, dev(ex, BF), dimp, rotp, vdimp)
+    assert tc == (vdimp <= 128 and vdimp % 32 == 0 and dimp + rotp <= 192)
+    if tc:
+        # the tcgen05 form: tiles of 128 rows in any order, with and without the gate
+        _, _, ts, t0, _, _ = _portions(lens, q_from, 128)
+        for g in (None, dev(gate, BF)[:, 16:]):
+            big = torch.full_like(out, 7.0)
+            Kn.latent_prefill_tc(qt, dev(ex, BF), got_rows, rankp, dimp, rotp, vdimp, i32(cu), i32(seg_pos), i32(ts[1:][::-1]), i32(t0[1:][::-1]),
+                                 i32(base), big, scale, H, g)
+            b = host(big)
+            assert np.all(b[0] == 7.0) and Kn.read_status().get("latent", 0) == 0
+            close(b[1:], got[1:] * (1.0 if g is None else P.sigmoid(gate[1:, 16:])), BF, tol16=0.01)
     for i in range(1, len(lens)):
         e, r = ex[base[i]:base[i + 1]], rows[i]
         L, a = lens[i], q_from[i]
