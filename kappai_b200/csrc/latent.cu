@@ -325,10 +325,10 @@ head_gemm_simt_kernel(const HeadGemmArgs p) {
 //                      head's float32 weights side by side, so that they enter whole for a few more columns.
 //
 // Roles by warp: 0 TMA (the queries once, a ring of tiles), 1 tensor memory and MMA of S, 2 - 9 two groups of four warps, a
-// lane quarter each, 10 the MMA of U.  In the softmax of a tile a group has half of the heads, a lane 16 q + i of a quarter and its partner
-// 16 lanes on the same key, half of those heads each; then all eight warps add U^T's columns (blocks shared among the
-// groups) to their registers, rescaled by the heads' change of maximum, so that no pass over tensor memory rescales anything.  S and the weights are double-buffered:
-// a tile's softmax runs while the tile before it is multiplied.
+// lane quarter each, 10 the MMA of U.  In the softmax of a tile a group has half of the heads, a lane 16 q + i of a quarter
+// and its partner 16 lanes on the same key, half of those heads each; then all eight warps add U^T's columns (blocks shared
+// among the groups) to their registers, rescaled by the heads' change of maximum, so that no pass over tensor memory
+// rescales anything.  S and the weights are double-buffered: a tile's softmax runs while the tile before it is multiplied.
 // Every wait is bounded; one that gives up sets the status word and an abort flag, and the CTA frees its tensor memory
 // and returns.
 #define LT_BOX_BYTES (LT_TILE * 128)                               // 64 rows x 64 columns of bfloat16
